@@ -72,9 +72,20 @@ enum {
     SPK_STATUS_TABLE_FULL = 1u << 4,    /* a row needs more than max_blocks blocks          */
     SPK_STATUS_FREE_LIST_OVERFLOW = 1u << 5, /* a release would push past the list's capacity    */
     SPK_STATUS_ROW_BUSY = 1u << 6,      /* admit into a row that still holds a sequence      */
-    SPK_STATUS_DEVICE_WAIT_EXPIRED = 1u << 7 /* a kernel gave up waiting for its own tensor-core work;
+    SPK_STATUS_DEVICE_WAIT_EXPIRED = 1u << 7, /* a kernel gave up waiting for its own tensor-core work;
                                             the affected rows of the output are zero           */
+    SPK_STATUS_BAD_TOKEN = 1u << 8    /* a token id outside the embedding table               */
 };
+
+/* ---- what a batch row is doing (the `active` array of the metadata builder) ---- */
+enum {
+    SPK_ROW_FREE = 0,       /* no sequence                                                       */
+    SPK_ROW_DECODING = 1,   /* takes part in every decode step                                   */
+    SPK_ROW_HELD = 2        /* holds a sequence (between portions of its prompt) and sits out    */
+};
+
+/* ---- place of a token in its portion ---- */
+enum { SPK_EDGE_FIRST = 1, SPK_EDGE_LAST = 2 };
 
 /* Library version, (major << 16) | (minor << 8) | patch. */
 int spk_version(void);
@@ -332,7 +343,7 @@ int spk_gather_kv_unpacked_batch(const int32_t* cache, int64_t s_t, int64_t s_h,
  *   free_list  int32 [num_alloc_blocks]  stack; entries [0, *free_count) are free and the
  *                                        next block handed out is free_list[*free_count-1]
  *   free_count int32 [1]
- *   active     int32 [max_rows]          1 = row holds a running sequence
+ *   active     int32 [max_rows]          SPK_ROW_*
  *   seq_lens   int32 [max_rows]          cached length (after advance: including the new token)
  *   positions  int64 [max_rows]
  *   slot_mapping int64 [max_rows]
@@ -375,6 +386,17 @@ int spk_meta_admit(int32_t row, const int32_t* src_table, int32_t seq_len, int64
 int spk_meta_take(int32_t* free_list, int32_t* free_count, int32_t count, int32_t* dst_table,
                   uint32_t* status, void* stream);
 
+/* Append n tokens to the sequence of `row` (a free row starts a new sequence): pops the blocks the longer sequence needs,
+ * in allocation order, sets seq_lens[row] and leaves the row held (it sits out decode steps until active[row] is set to
+ * SPK_ROW_DECODING).  Fills the portion's per-token arrays: tok_positions / tok_slots (int64 [n]), tok_rows (int32 [n],
+ * the row) and tok_edges (int32 [n], SPK_EDGE_FIRST / SPK_EDGE_LAST).  If the pool or the table is too small nothing changes,
+ * a status bit is set and the tokens point at the pad slot with row -1. */
+int spk_meta_extend(int32_t row, int32_t n, int32_t* free_list, int32_t* free_count, int32_t* active,
+                    int32_t* seq_lens, int64_t* positions, int64_t* slot_mapping, int32_t* block_tables,
+                    int64_t* tok_positions, int64_t* tok_slots, int32_t* tok_rows, int32_t* tok_edges,
+                    int32_t max_rows, int32_t max_blocks, int32_t pad_block, int32_t block_size,
+                    uint32_t* status, void* stream);
+
 /* Finish `row`: push its ceil(seq_len / bs) blocks back in table order
  * (block_manager.py:63-66), reset the row to the pad state.  num_alloc_blocks is the capacity of
  * free_list: a push that would pass it is skipped and SPK_STATUS_FREE_LIST_OVERFLOW is set. */
@@ -383,6 +405,183 @@ int spk_meta_release(int32_t row, int32_t* free_list, int32_t* free_count, int32
                      int32_t* block_tables, int32_t max_rows, int32_t max_blocks,
                      int32_t pad_block, int32_t block_size, int32_t num_alloc_blocks,
                      uint32_t* status, void* stream);
+
+/* ---------------------------------------------------------------------------
+ * Dense (non-spiking) decoder operators: post-norm residual stream in 32 bits, paged attention with element-wise
+ * key weights, linear attention with a decaying state.  No counterpart in the reference.  Storage type `dtype` is
+ * SPK_F32 or SPK_BF16; arithmetic is 32-bit (the tensor-core forms take 16-bit operands and add up in 32 bits).
+ *
+ * "Decode" form of an operator: token t of the call is batch row t, gated by active[t] == SPK_ROW_DECODING (active may be
+ * NULL: all rows run).  "Prefill" form: the tokens of one or more portions, one after the other, described by the
+ * per-token arrays of spk_meta_extend and by small int32[4] tables.
+ * ------------------------------------------------------------------------- */
+
+/* One sublayer boundary.  y = embed[ids[t]] when ids != NULL, else y = layernorm(alpha * x + delta) * w (mean removed, no
+ * bias, eps inside the root).  x_out (32-bit, may be NULL) <- y.  out (dtype) <-
+ *   mix != NULL: y + (y' - y) * mix, y' = the previous token's y; for the first token of a portion y' is prev[row]
+ *                (zeros at position 0);
+ *   w2 != NULL:  layernorm(y) * w2;
+ *   otherwise y.
+ * commit != NULL: for the last token of a portion commit[row] <- x[t] (the OLD x), so that the launch that ends a sublayer
+ * saves what the next portion's first token needs.  In the prefill form with mix, x_out must not alias x.
+ * prev and commit are [state_rows, width] contiguous. */
+typedef struct spk_residual_norm_args {
+    const float* x;
+    float* x_out;
+    const void* delta;          /* [n, width] in delta_dtype */
+    const void* embed;          /* [vocab, width] in dtype   */
+    const int64_t* ids;
+    int64_t vocab;
+    const float* w;
+    const float* w2;
+    const float* mix;
+    const float* prev;
+    float* commit;
+    int64_t state_rows;
+    const int64_t* positions;
+    const int32_t* token_rows;  /* NULL: decode form */
+    const int32_t* token_edges;
+    const int32_t* active;
+    void* out;
+    int64_t n;
+    int64_t width;
+    float alpha;
+    float eps;
+    int32_t dtype;
+    int32_t delta_dtype;
+    uint32_t* status;
+} spk_residual_norm_args;
+int spk_residual_norm(const spk_residual_norm_args* args, void* stream);
+
+/* out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 per row, N(y) = y / sqrt(mean(y^2) + eps); out may alias z. */
+int spk_poly_norm(const void* z, const float* coef, float eps, void* out, int64_t rows, int64_t width, int dtype, void* stream);
+
+/* A dense K or V pool is [num_blocks][kv_heads][block_size][pad] elements; pad >= the head size, channels beyond it stay
+ * zero.  tiled != 0 (pad % 64 == 0, block_size % 8 == 0): a page is stored as 64-channel column tiles of
+ * block_size x 128 bytes whose 16-byte groups are XOR-swizzled with the row (see csrc/spk_dense.cuh).
+ *
+ * Rotary embedding on the first rot_dims channels of q and k (channel i with channel i + rot_dims / 2; rot_table float2
+ * (cos, sin) [rot_positions, rot_dims / 2]; NULL = none), then, when unit_norm, division by the head's root mean
+ * square; q to q_out [n, heads, k_pad] (padding zeroed), k and v to the page of slot_mapping[t]. */
+typedef struct spk_qk_prepare_args {
+    const void* q;              /* row t, head h at q + t * ld + h * dim */
+    const void* k;
+    const void* v;
+    int64_t ld;
+    void* q_out;
+    void* k_pool;
+    void* v_pool;
+    const float* rot_table;
+    const int64_t* positions;
+    const int64_t* slot_mapping;
+    int64_t rot_positions;
+    int64_t n;
+    int64_t num_blocks;
+    int32_t heads, kv_heads, dim, vdim;
+    int32_t k_pad, v_pad, k_tiled, v_tiled;
+    int32_t block_size;
+    int32_t rot_dims;
+    int32_t unit_norm;
+    int32_t dtype;
+    float eps;
+    float _pad;
+    uint32_t* status;
+} spk_qk_prepare_args;
+int spk_qk_prepare(const spk_qk_prepare_args* args, void* stream);
+
+/* out[t, h, :] = out_scale * sum_j sigmoid(scale * q[t,h].k_j + head_bias[h]) v_j over the keys 0 .. position of token t,
+ * k_j, v_j of KV head h / (heads / kv_heads) read through the block table of the token's row.
+ * Prefill form: tiles int32 [n_tiles][4] = (first token, tokens <= spk_sigmoid_attn_tile_tokens(), row, position of the
+ * first).  Decode form (tiles NULL): token t = row t, position seq_lens[t] - 1; inactive rows give zeros. */
+typedef struct spk_sigmoid_attn_args {
+    const void* q;              /* [n, heads, k_pad] */
+    const void* k_pool;
+    const void* v_pool;
+    const int32_t* tables;      /* [table_rows, max_blocks], row stride table_stride */
+    const int32_t* seq_lens;
+    const int32_t* active;
+    const int32_t* tiles;
+    const float* head_bias;
+    void* out;                  /* row t, head h at out + t * out_stride + h * vdim */
+    int64_t out_stride;
+    int64_t table_stride;
+    int64_t table_rows;
+    int64_t max_blocks;
+    int64_t n;
+    int64_t num_blocks;
+    int32_t n_tiles;
+    int32_t heads, kv_heads, dim, vdim;
+    int32_t k_pad, v_pad, k_tiled, v_tiled;
+    int32_t block_size;
+    int32_t dtype;
+    float scale;
+    float out_scale;
+    float _pad;
+    uint32_t* status;
+} spk_sigmoid_attn_args;
+int spk_sigmoid_attn_tile_tokens(void);
+int spk_sigmoid_attn(const spk_sigmoid_attn_args* args, void* stream);
+
+/* S_t = decay_h S_{t-1} + k_t v_t^T, out_t = S_t^T q_t, with silu applied to q, k and v first when silu != 0.
+ * state: 32-bit, row r, head h at state + r * state_stride + h * dim * vdim, [dim][vdim].  decay_pow [heads][chunk + 1]: the
+ * powers 0 .. spk_decay_chunk_tokens() of every head's decay.  out 32-bit [n, heads * vdim].
+ * _step: decode form.  _chunks: prefill form; chunks int32 [n_chunks][4] = (first token, tokens, sequence, index in the
+ * sequence), seqs int32 [n_seqs][4] = (first chunk, chunks, state row, tokens before this portion: 0 starts from a zero
+ * state whatever the slot holds); workspace of spk_decay_attn_workspace_bytes. */
+typedef struct spk_decay_attn_args {
+    const void* q;
+    const void* k;
+    const void* v;
+    int64_t ld;
+    float* state;
+    int64_t state_stride;
+    int64_t state_rows;
+    const float* decay_pow;
+    float* out;
+    const int32_t* active;
+    const int32_t* chunks;
+    const int32_t* seqs;
+    float* workspace;
+    int64_t workspace_bytes;
+    int64_t n;
+    int32_t n_chunks, n_seqs;
+    int32_t heads, dim, vdim;
+    int32_t silu;
+    int32_t dtype;
+    int32_t _pad;
+    uint32_t* status;
+} spk_decay_attn_args;
+int spk_decay_chunk_tokens(void);
+int64_t spk_decay_attn_workspace_bytes(int n_chunks, int heads, int dim, int vdim);
+int spk_decay_attn_step(const spk_decay_attn_args* args, void* stream);
+int spk_decay_attn_chunks(const spk_decay_attn_args* args, void* stream);
+
+/* out[t, out_offset + c] = scale * (x / sqrt(mean(x^2) + eps) * w)[c] * sigmoid(gate[t, c]) over the `width` columns of x (32-bit).
+ * partials != NULL (decode form): out[t, c] = left_scale * sum of the partial sums [n][splits][left_width] whose key range
+ * (keys_per_split each) begins below seq_lens[t], for c < left_width <= out_offset. */
+typedef struct spk_gated_norm_args {
+    const float* x;             /* [n, width] */
+    const float* w;
+    const void* gate;
+    int64_t gate_stride;
+    void* out;
+    int64_t out_stride;
+    const float* partials;
+    const int32_t* seq_lens;
+    const int32_t* active;
+    int64_t n;
+    int32_t width;
+    int32_t out_offset;
+    int32_t splits;
+    int32_t keys_per_split;
+    int32_t left_width;
+    int32_t dtype;
+    float eps;
+    float scale;
+    float left_scale;
+    float _pad;
+} spk_gated_norm_args;
+int spk_gated_norm(const spk_gated_norm_args* args, void* stream);
 
 #ifdef __cplusplus
 }

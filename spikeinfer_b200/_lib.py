@@ -25,6 +25,9 @@ STATUS_TABLE_FULL = 1 << 4
 STATUS_FREE_LIST_OVERFLOW = 1 << 5
 STATUS_ROW_BUSY = 1 << 6
 STATUS_DEVICE_WAIT_EXPIRED = 1 << 7
+STATUS_BAD_TOKEN = 1 << 8
+
+ROW_FREE, ROW_DECODING, ROW_HELD = 0, 1, 2
 
 MAX_LIF_SITES = 4
 
@@ -84,6 +87,52 @@ class LifSite(Structure):
     ]
 
 
+def _fields(spec: str):
+    """ctypes fields from ``"kind name name ...; ..."`` with p = pointer, l = int64, i = int32, f = float."""
+    kinds = {"p": c_void_p, "l": c_int64, "i": c_int32, "f": c_float}
+    out = []
+    for group in spec.split(";"):
+        kind, *names = group.split()
+        out += [(n, kinds[kind]) for n in names]
+    return out
+
+
+class ResidualNormArgs(Structure):
+    """Mirror of ``spk_residual_norm_args``."""
+
+    _fields_ = _fields("p x x_out delta embed ids; l vocab; p w w2 mix prev commit; l state_rows; p positions token_rows "
+                       "token_edges active out; l n width; f alpha eps; i dtype delta_dtype; p status")
+
+
+class QkPrepareArgs(Structure):
+    """Mirror of ``spk_qk_prepare_args``."""
+
+    _fields_ = _fields("p q k v; l ld; p q_out k_pool v_pool rot_table positions slot_mapping; l rot_positions n num_blocks; "
+                       "i heads kv_heads dim vdim k_pad v_pad k_tiled v_tiled block_size rot_dims unit_norm dtype; f eps _pad; p status")
+
+
+class SigmoidAttnArgs(Structure):
+    """Mirror of ``spk_sigmoid_attn_args``."""
+
+    _fields_ = _fields("p q k_pool v_pool tables seq_lens active tiles head_bias out; l out_stride table_stride table_rows "
+                       "max_blocks n num_blocks; i n_tiles heads kv_heads dim vdim k_pad v_pad k_tiled v_tiled block_size dtype; "
+                       "f scale out_scale _pad; p status")
+
+
+class DecayAttnArgs(Structure):
+    """Mirror of ``spk_decay_attn_args``."""
+
+    _fields_ = _fields("p q k v; l ld; p state; l state_stride state_rows; p decay_pow out active chunks seqs workspace; "
+                       "l workspace_bytes n; i n_chunks n_seqs heads dim vdim silu dtype _pad; p status")
+
+
+class GatedNormArgs(Structure):
+    """Mirror of ``spk_gated_norm_args``."""
+
+    _fields_ = _fields("p x w gate; l gate_stride; p out; l out_stride; p partials seq_lens active; l n; i width out_offset splits "
+                       "keys_per_split left_width dtype; f eps scale left_scale _pad")
+
+
 # name -> (restype, argtypes); every symbol include/spikeinfer_b200.h declares
 I64P = POINTER(c_int64)
 SIGNATURES = {
@@ -141,11 +190,34 @@ SIGNATURES = {
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                c_int32, c_void_p, c_void_p]),
     "spk_meta_take": (c_int, [c_void_p, c_void_p, c_int32, c_void_p, c_void_p, c_void_p]),
+    "spk_meta_extend": (c_int, [c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
+    "spk_residual_norm": (c_int, [POINTER(ResidualNormArgs), c_void_p]),
+    "spk_poly_norm": (c_int, [c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int64, c_int, c_void_p]),
+    "spk_qk_prepare": (c_int, [POINTER(QkPrepareArgs), c_void_p]),
+    "spk_sigmoid_attn_tile_tokens": (c_int, []),
+    "spk_sigmoid_attn": (c_int, [POINTER(SigmoidAttnArgs), c_void_p]),
+    "spk_decay_chunk_tokens": (c_int, []),
+    "spk_decay_attn_workspace_bytes": (c_int64, [c_int, c_int, c_int, c_int]),
+    "spk_decay_attn_step": (c_int, [POINTER(DecayAttnArgs), c_void_p]),
+    "spk_decay_attn_chunks": (c_int, [POINTER(DecayAttnArgs), c_void_p]),
+    "spk_gated_norm": (c_int, [POINTER(GatedNormArgs), c_void_p]),
     "spk_meta_release": (c_int, [c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
 }
 
 _lib = None
+_lib_path = LIB_PATH
+
+
+def use_library(path: Path) -> None:
+    """Load ``path`` (a library of some components, :func:`spikeinfer_b200.build.build_components`) instead of the full
+    library.  No effect on a library that is loaded already, provided it is that one or the full one."""
+    global _lib_path
+    if _lib is not None and _lib_path not in (path, LIB_PATH):
+        raise SpkError(f"{_lib_path.name} is loaded already and does not hold what {path.name} holds")
+    if _lib is None:
+        _lib_path = path
 
 
 def load() -> ctypes.CDLL:
@@ -153,14 +225,19 @@ def load() -> ctypes.CDLL:
     global _lib
     if _lib is not None:
         return _lib
-    if not LIB_PATH.exists():
+    if not _lib_path.exists():
         raise SpkError(
-            f"{LIB_PATH} is missing: build it with `python -m spikeinfer_b200.build` "
+            f"{_lib_path} is missing: build it with `python -m spikeinfer_b200.build` "
             "(there is no fallback path)"
         )
-    lib = ctypes.CDLL(str(LIB_PATH))
+    lib = ctypes.CDLL(str(_lib_path))
     for name, (restype, argtypes) in SIGNATURES.items():
-        fn = getattr(lib, name)
+        try:
+            fn = getattr(lib, name)
+        except AttributeError:
+            if _lib_path == LIB_PATH:
+                raise
+            continue  # a component this library was built without
         fn.restype = restype
         fn.argtypes = argtypes
     _lib = lib

@@ -47,6 +47,25 @@ class AttentionMetadata:
     decode attention on the stream began (they are written at the head of the step).  The attention launch of
     :func:`fused_qkv_attention` may then overlap the tail of the LIF launch before it."""
 
+    row_active: torch.Tensor | None = None
+    """int32 ``[n_dec]``: 1 for the rows that take part in this decode step (recurrent state of the others must stay)."""
+    prefill_rows: list[int] = field(default_factory=list)
+    """Batch row (= state slot) of every prefill chunk."""
+    token_rows: torch.Tensor | None = None
+    """int32 ``[n_prefill_tok]``: batch row of every prefill token."""
+    token_edges: torch.Tensor | None = None
+    """int32 ``[n_prefill_tok]``: bit 0 = first, bit 1 = last token of its chunk."""
+    row_tables: torch.Tensor | None = None
+    """int32 ``[max_rows, max_blocks]``: block tables of all batch rows."""
+    plan: "PrefillPlan | None" = None
+    """Work lists of the dense prefill kernels, built on first use (:meth:`prefill_plan`)."""
+
+    def prefill_plan(self) -> "PrefillPlan":
+        if self.plan is None:
+            self.plan = PrefillPlan(self.prefill_query_starts, self.prefill_query_lens, self.prefill_context_lens,
+                                    self.prefill_rows, self.slot_mapping.device)
+        return self.plan
+
     @property
     def num_prefills(self) -> int:
         return len(self.prefill_query_lens)
@@ -63,7 +82,46 @@ class AttentionMetadata:
             prefill_query_lens=self.prefill_query_lens, prefill_context_lens=self.prefill_context_lens,
             prefill_block_tables=[mv(t) for t in self.prefill_block_tables], status=mv(self.status),
             prefill_row_tables=mv(self.prefill_row_tables), prefill_row_lens=mv(self.prefill_row_lens),
-            tables_settled=self.tables_settled)
+            tables_settled=self.tables_settled, row_active=mv(self.row_active), prefill_rows=self.prefill_rows,
+            token_rows=mv(self.token_rows), token_edges=mv(self.token_edges), row_tables=mv(self.row_tables))
+
+
+class PrefillPlan:
+    """Work lists of the dense prefill kernels for one batch of portions: attention query tiles and recurrence chunks.
+
+    Portions are cut from their own first token, so a tile or chunk never spans two sequences.  The lists are small int32
+    tables, built on the host and copied once per batch; all layers share them."""
+
+    def __init__(self, starts, lens, contexts, rows, device: torch.device) -> None:
+        self.starts, self.lens, self.contexts, self.rows = list(starts), list(lens), list(contexts), list(rows)
+        if len(self.rows) != len(self.lens):
+            raise ValueError("every prefill portion needs its batch row")
+        self.device = device
+        self._tiles: dict[int, torch.Tensor] = {}
+        self._chunks: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+
+    def _table(self, entries: list[tuple[int, int, int, int]]) -> torch.Tensor:
+        return torch.tensor(entries, dtype=torch.int32).to(self.device)
+
+    def tiles(self, tokens: int) -> torch.Tensor:
+        """int32 ``[n, 4]``: (first token, tokens, row, position of the first token), longest context first."""
+        if tokens not in self._tiles:
+            out = [(s + lo, min(tokens, n - lo), row, ctx + lo)
+                   for s, n, ctx, row in zip(self.starts, self.lens, self.contexts, self.rows) for lo in range(0, n, tokens)]
+            out.sort(key=lambda e: -e[3])  # the tiles that see the most keys start first
+            self._tiles[tokens] = self._table(out)
+        return self._tiles[tokens]
+
+    def chunks(self, tokens: int) -> tuple[torch.Tensor, torch.Tensor]:
+        """``(chunks, seqs)``: int32 ``[n, 4]`` (first token, tokens, portion, index in the portion) and ``[portions, 4]``
+        (first chunk, chunks, row, tokens before this portion)."""
+        if tokens not in self._chunks:
+            chunks, seqs = [], []
+            for i, (s, n, ctx, row) in enumerate(zip(self.starts, self.lens, self.contexts, self.rows)):
+                seqs.append((len(chunks), -(-n // tokens), row, ctx))
+                chunks += [(s + lo, min(tokens, n - lo), i, lo // tokens) for lo in range(0, n, tokens)]
+            self._chunks[tokens] = (self._table(chunks), self._table(seqs))
+        return self._chunks[tokens]
 
 
 def build_prefill_rows(meta: AttentionMetadata, pad_block: int = 0) -> AttentionMetadata:

@@ -3,7 +3,8 @@
 ``python -m spikeinfer_b200.build`` compiles ``csrc/*.cu`` into
 ``spikeinfer_b200/libspikeinfer_b200.so``.  nvcc cross-compiles without a GPU, so this
 also runs on a CPU-only build machine.  The library is rebuilt only when a source or
-header is newer than it (``force=True`` overrides).
+header is newer than it (``force=True`` overrides).  :func:`build_components` builds a library of some of
+the translation units only, for a process that serves one kind of model from a fresh checkout.
 """
 from __future__ import annotations
 
@@ -27,6 +28,13 @@ NVCC_FLAGS = [
 # recurrence (every product and sum is rounded on its own, as the reference does) and the RMSNorm's mean + eps.
 NO_FMA_CONTRACTION = {"spk_lif.cu", "spk_norm.cu"}
 
+# Groups of translation units a model may need; "core" (C ABI basics, batch metadata, sampling) is part of every library.
+COMPONENTS = {
+    "core": ("spk_capi.cu", "spk_meta.cu", "spk_sample.cu"),
+    "spike": ("spk_attn.cu", "spk_attn_stream.cu", "spk_lif.cu", "spk_norm.cu", "spk_pack.cu"),
+    "dense": ("spk_postnorm.cu", "spk_paged_attn.cu", "spk_decay.cu"),
+}
+
 
 def _nvcc() -> str:
     exe = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
@@ -35,27 +43,46 @@ def _nvcc() -> str:
     return exe
 
 
-def sources() -> list[Path]:
-    return sorted(CSRC.glob("*.cu"))
+def sources(components=None) -> list[Path]:
+    if components is None:
+        return sorted(CSRC.glob("*.cu"))
+    names = {n for c in {"core", *components} for n in COMPONENTS[c]}
+    return sorted(CSRC / n for n in names)
 
 
-def is_stale() -> bool:
-    if not LIB_PATH.exists():
+def library_path(components=None) -> Path:
+    if components is None:
+        return LIB_PATH
+    return PKG_DIR / f"libspikeinfer_b200.{'-'.join(sorted({'core', *components}))}.so"
+
+
+def is_stale(components=None) -> bool:
+    lib = library_path(components)
+    if not lib.exists():
         return True
-    built = LIB_PATH.stat().st_mtime
-    deps = list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh")) + list(INCLUDE.glob("*.h"))
+    built = lib.stat().st_mtime
+    deps = sources(components) + list(CSRC.glob("*.cuh")) + list(INCLUDE.glob("*.h"))
     return any(p.stat().st_mtime > built for p in deps)
 
 
-def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
-    if not force and not is_stale():
+def build_components(components) -> Path:
+    """The library to load for these components: the full one when it is there and current, else one of their
+    translation units alone, compiled on first use."""
+    if not is_stale():
         return LIB_PATH
+    return build(components=tuple(components))
+
+
+def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False, components=None) -> Path:
+    lib_path = library_path(components)
+    if not force and not is_stale(components):
+        return lib_path
     obj_dir = PKG_DIR / "build"
     obj_dir.mkdir(exist_ok=True)
     nvcc = _nvcc()
     objs = []
     procs = []
-    for src in sources():
+    for src in sources(components):
         obj = obj_dir / (src.stem + ".o")
         cmd = [nvcc, *NVCC_FLAGS, "-I", str(INCLUDE), "-c", str(src), "-o", str(obj)]
         if src.name in NO_FMA_CONTRACTION:
@@ -75,14 +102,14 @@ def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) 
             print(f"--- {src.name} ---\n{out}", flush=True)
     if failed:
         raise RuntimeError("nvcc failed:\n" + "\n".join(failed))
-    tmp = LIB_PATH.with_suffix(".so.tmp")
+    tmp = lib_path.with_suffix(".so.tmp")
     link = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", str(tmp),
             *map(str, objs), "-lcudart", "-ldl"]
     if verbose:
         print(" ".join(link), flush=True)
     subprocess.run(link, check=True)
-    os.replace(tmp, LIB_PATH)
-    return LIB_PATH
+    os.replace(tmp, lib_path)
+    return lib_path
 
 
 if __name__ == "__main__":

@@ -46,7 +46,8 @@ meta_advance_kernel(int32_t* free_list, int32_t* free_count, const int32_t* acti
     const int lane = row & 31;
     const int wid = row >> 5;
     const bool in_range = row < max_rows;
-    const bool act = in_range && active[row] != 0;
+    const int32_t mode = in_range ? active[row] : SPK_ROW_FREE;
+    const bool act = mode == SPK_ROW_DECODING;
     int pos = 0;
     bool need = false;
     bool full = false;
@@ -93,11 +94,11 @@ meta_advance_kernel(int32_t* free_list, int32_t* free_count, const int32_t* acti
                 slot_mapping[row] = static_cast<int64_t>(pad_block) * block_size;
             }
             if (next_tokens != nullptr) input_ids[row] = next_tokens[row];
-        } else if (!act) {
+        } else if (mode == SPK_ROW_FREE) {
             seq_lens[row] = 1;
             positions[row] = 0;
             slot_mapping[row] = static_cast<int64_t>(pad_block) * block_size;
-        } else {
+        } else {  // a held row (its sequence stays as it is), or a full table
             slot_mapping[row] = static_cast<int64_t>(pad_block) * block_size;
         }
     }
@@ -138,6 +139,43 @@ __global__ void meta_admit_kernel(int32_t row, const int32_t* src_table, int32_t
         slot_mapping[row] = static_cast<int64_t>(pad_block) * block_size;
         input_ids[row] = last_token;
         if (next_tokens != nullptr) next_tokens[row] = last_token;
+    }
+}
+
+// Append n tokens to the sequence of `row` (a free row starts a new one) and hold the row: blocks are popped in
+// order, the portion's per-token arrays are filled in.  One CTA.
+__global__ void meta_extend_kernel(int32_t row, int32_t n, int32_t* free_list, int32_t* free_count, int32_t* active,
+                                   int32_t* seq_lens, int64_t* positions, int64_t* slot_mapping, int32_t* tables,
+                                   int64_t* tok_positions, int64_t* tok_slots, int32_t* tok_rows, int32_t* tok_edges,
+                                   int32_t max_blocks, int32_t pad_block, int32_t block_size, uint32_t* status) {
+    const int64_t pad_slot = static_cast<int64_t>(pad_block) * block_size;
+    const int start = active[row] != SPK_ROW_FREE ? seq_lens[row] : 0;
+    const int fc = *free_count;
+    const int64_t end = static_cast<int64_t>(start) + n;
+    const int have = (start + block_size - 1) / block_size;
+    const int64_t want = (end + block_size - 1) / block_size;
+    const int64_t add = want - have;
+    const bool full = want > max_blocks;
+    const bool ok = !full && add <= fc;
+    int32_t* table = tables + static_cast<int64_t>(row) * max_blocks;
+    __syncthreads();  // every thread has read the state before it changes
+    if (!ok && threadIdx.x == 0) spk_flag(status, full ? SPK_STATUS_TABLE_FULL : SPK_STATUS_POOL_EXHAUSTED);
+    if (ok)
+        for (int i = threadIdx.x; i < add; i += blockDim.x) table[have + i] = free_list[fc - 1 - i];
+    __syncthreads();
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int pos = start + i;
+        tok_positions[i] = ok ? pos : 0;
+        tok_slots[i] = ok ? static_cast<int64_t>(table[pos / block_size]) * block_size + pos % block_size : pad_slot;
+        tok_rows[i] = ok ? row : -1;
+        tok_edges[i] = (i == 0 ? SPK_EDGE_FIRST : 0) | (i == n - 1 ? SPK_EDGE_LAST : 0);
+    }
+    if (ok && threadIdx.x == 0) {
+        *free_count = fc - static_cast<int>(add);
+        active[row] = SPK_ROW_HELD;
+        seq_lens[row] = static_cast<int32_t>(end);
+        positions[row] = end - 1;
+        slot_mapping[row] = pad_slot;
     }
 }
 
@@ -233,6 +271,24 @@ extern "C" int spk_meta_admit(int32_t row, const int32_t* src_table, int32_t seq
     meta_admit_kernel<<<1, 256, 0, spk_stream(stream)>>>(row, src_table, seq_len, last_token, active, seq_lens,
                                                          positions, slot_mapping, block_tables, input_ids,
                                                          next_tokens, max_blocks, pad_block, block_size, status);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+extern "C" int spk_meta_extend(int32_t row, int32_t n, int32_t* free_list, int32_t* free_count, int32_t* active,
+                               int32_t* seq_lens, int64_t* positions, int64_t* slot_mapping, int32_t* block_tables,
+                               int64_t* tok_positions, int64_t* tok_slots, int32_t* tok_rows, int32_t* tok_edges,
+                               int32_t max_rows, int32_t max_blocks, int32_t pad_block, int32_t block_size,
+                               uint32_t* status, void* stream) {
+    SpkRange nvtx_range("spk_meta_extend");
+    if (row < 0 || row >= max_rows || n < 1 || max_blocks < 1 || block_size < 1) return SPK_ERR_BAD_SHAPE;
+    if (free_list == nullptr || free_count == nullptr || active == nullptr || seq_lens == nullptr ||
+        positions == nullptr || slot_mapping == nullptr || block_tables == nullptr || tok_positions == nullptr ||
+        tok_slots == nullptr || tok_rows == nullptr || tok_edges == nullptr)
+        return SPK_ERR_NULL_POINTER;
+    meta_extend_kernel<<<1, 256, 0, spk_stream(stream)>>>(row, n, free_list, free_count, active, seq_lens, positions,
+                                                          slot_mapping, block_tables, tok_positions, tok_slots, tok_rows,
+                                                          tok_edges, max_blocks, pad_block, block_size, status);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }

@@ -1,0 +1,239 @@
+// Dense paged attention with element-wise (sigmoid) key weights: the K/V write and the 32-bit form of the product.
+//
+//  * qk_prepare_kernel: per (token, head) rotary embedding on the first channels, division by the head's root mean square,
+//    q to a dense buffer, k and v into the sequence's pages.  One launch for q, k and v.
+//  * sigmoid_attn_simt_kernel: out = sum_j sigmoid(scale q.k_j + bias_h) v_j over the visible keys, every product in
+//    32 bits; any head sizes, prefill tiles and decode rows alike.
+// A weight depends on its own key alone, so there is no running maximum and no denominator, and sums over
+// different key ranges simply add up.
+#include "spk_dense.cuh"
+
+namespace {
+
+constexpr int kWarps = 8;
+constexpr int kThreads = 32 * kWarps;
+
+// ---- rotary embedding, unit norm, page write ---------------------------------------------------------------
+// One warp per (token, head slot); slots are the query heads, then the key heads, then the value heads.
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+qk_prepare_kernel(const spk_qk_prepare_args a) {
+    extern __shared__ float sm[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int slots = a.heads + 2 * a.kv_heads;
+    const int64_t item = static_cast<int64_t>(blockIdx.x) * kWarps + warp;
+    const int64_t t = item / slots;
+    if (t >= a.n) return;
+    const int s = static_cast<int>(item % slots);
+    const bool is_q = s < a.heads;
+    const bool is_v = s >= a.heads + a.kv_heads;
+    const int width = is_v ? a.vdim : a.dim;
+    const T* src;
+    if (is_q) src = static_cast<const T*>(a.q) + t * a.ld + static_cast<int64_t>(s) * a.dim;
+    else if (!is_v) src = static_cast<const T*>(a.k) + t * a.ld + static_cast<int64_t>(s - a.heads) * a.dim;
+    else src = static_cast<const T*>(a.v) + t * a.ld + static_cast<int64_t>(s - a.heads - a.kv_heads) * a.vdim;
+
+    T* page = nullptr;
+    int r = 0;
+    SpkPageLayout lay{a.kv_heads, a.block_size, is_v ? a.v_pad : a.k_pad, is_v ? a.v_tiled : a.k_tiled};
+    if (!is_q) {
+        const int64_t slot = a.slot_mapping[t];
+        const int64_t block = slot / a.block_size;
+        if (slot < 0 || block >= a.num_blocks) {
+            if (lane == 0) spk_flag(a.status, SPK_STATUS_BAD_SLOT);
+            return;
+        }
+        r = static_cast<int>(slot % a.block_size);
+        const int g = is_v ? s - a.heads - a.kv_heads : s - a.heads;
+        page = static_cast<T*>(is_v ? a.v_pool : a.k_pool) + spk_page_base(lay, block, g);
+    }
+    if (is_v) {
+        for (int c = lane; c < width; c += 32) page[spk_page_channel(lay, r, c)] = src[c];
+        return;
+    }
+    float* x = sm + warp * a.dim;
+    for (int c = lane; c < width; c += 32) x[c] = spk_to_float<T>(src[c]);
+    __syncwarp();
+    const int half = a.rot_table != nullptr ? a.rot_dims / 2 : 0;
+    if (half > 0) {
+        int64_t pos = a.positions[t];
+        if (pos < 0 || pos >= a.rot_positions) {
+            if (lane == 0) spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+            pos = 0;
+        }
+        const float2* cs = reinterpret_cast<const float2*>(a.rot_table) + pos * half;
+        for (int i = lane; i < half; i += 32) {
+            const float2 f = cs[i];
+            const float u = x[i], w = x[i + half];
+            x[i] = u * f.x - w * f.y;
+            x[i + half] = w * f.x + u * f.y;
+        }
+        __syncwarp();
+    }
+    float ss = 0.0f;
+    for (int c = lane; c < width; c += 32) ss = fmaf(x[c], x[c], ss);
+    ss = spk_warp_sum(ss);
+    const float inv = a.unit_norm ? 1.0f / sqrtf(ss / static_cast<float>(width) + a.eps) : 1.0f;
+    if (is_q) {
+        T* o = static_cast<T*>(a.q_out) + (t * a.heads + s) * a.k_pad;
+        for (int c = lane; c < a.k_pad; c += 32) o[c] = spk_from_float<T>(c < width ? x[c] * inv : 0.0f);
+    } else {
+        for (int c = lane; c < width; c += 32) page[spk_page_channel(lay, r, c)] = spk_from_float<T>(x[c] * inv);
+    }
+}
+
+// ---- attention, 32-bit -----------------------------------------------------------------------------------------
+constexpr int kTileQ = 16;
+constexpr int kTileK = 32;
+constexpr int kMaxCols = 16;  // output columns per thread and query tile: vdim <= 16 * kThreads / kTileQ = 256
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+sigmoid_attn_simt_kernel(const spk_sigmoid_attn_args a) {
+    extern __shared__ float sm[];
+    const int h = blockIdx.y;
+    const int g = h / (a.heads / a.kv_heads);
+    int64_t t0;
+    int nq, row;
+    int64_t pos0;
+    if (a.tiles != nullptr) {
+        const int4 e = reinterpret_cast<const int4*>(a.tiles)[blockIdx.x];  // first token, tokens, row, position of the first
+        t0 = e.x; nq = e.y; row = e.z; pos0 = e.w;
+    } else {
+        t0 = row = blockIdx.x;
+        nq = 1;
+        pos0 = static_cast<int64_t>(a.seq_lens[row]) - 1;
+    }
+    const int dim = a.dim, vdim = a.vdim;
+    T* out = static_cast<T*>(a.out) + t0 * a.out_stride + static_cast<int64_t>(h) * vdim;
+    bool live = a.tiles != nullptr || a.active == nullptr || a.active[row] == 1;
+    if (live && (pos0 < 0 || pos0 + nq > a.max_blocks * a.block_size || row < 0 || row >= a.table_rows)) {
+        if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+        live = false;
+    }
+    if (!live) {
+        for (int i = threadIdx.x; i < nq * vdim; i += kThreads) out[(i / vdim) * a.out_stride + i % vdim] = spk_from_float<T>(0.0f);
+        return;
+    }
+    float* q = sm;                         // [kTileQ][dim]
+    float* k = q + kTileQ * dim;           // [kTileK][dim + 1]
+    float* v = k + kTileK * (dim + 1);     // [kTileK][vdim]
+    float* p = v + kTileK * vdim;          // [kTileQ][kTileK]
+    for (int i = threadIdx.x; i < kTileQ * dim; i += kThreads) {
+        const int r = i / dim, c = i % dim;
+        q[i] = r < nq ? spk_to_float<T>(static_cast<const T*>(a.q)[((t0 + r) * a.heads + h) * a.k_pad + c]) : 0.0f;
+    }
+    const SpkPageLayout kl{a.kv_heads, a.block_size, a.k_pad, a.k_tiled}, vl{a.kv_heads, a.block_size, a.v_pad, a.v_tiled};
+    const int32_t* table = a.tables + static_cast<int64_t>(row) * a.table_stride;
+    const float bias = a.head_bias[h];
+    const int cols = kTileQ * vdim;
+    float acc[kMaxCols];
+#pragma unroll
+    for (int i = 0; i < kMaxCols; ++i) acc[i] = 0.0f;
+    const int64_t keys = pos0 + nq;
+    for (int64_t j0 = 0; j0 < keys; j0 += kTileK) {
+        __syncthreads();
+        for (int i = threadIdx.x; i < kTileK * (dim + vdim); i += kThreads) {
+            const int r = i / (dim + vdim), c = i % (dim + vdim);
+            const int64_t j = j0 + r;
+            float val = 0.0f;
+            if (j < keys) {
+                const int64_t block = table[j / a.block_size];
+                const int slot = static_cast<int>(j % a.block_size);
+                if (block >= 0 && block < a.num_blocks) {
+                    val = c < dim ? spk_to_float<T>(static_cast<const T*>(a.k_pool)[spk_page_base(kl, block, g) + spk_page_channel(kl, slot, c)])
+                                  : spk_to_float<T>(static_cast<const T*>(a.v_pool)[spk_page_base(vl, block, g) + spk_page_channel(vl, slot, c - dim)]);
+                } else if (c == 0) {
+                    spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
+                }
+            }
+            if (c < dim) k[r * (dim + 1) + c] = val;
+            else v[r * vdim + c - dim] = val;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < kTileQ * kTileK; i += kThreads) {
+            const int r = i / kTileK, c = i % kTileK;
+            float s = 0.0f;
+            for (int d = 0; d < dim; ++d) s = fmaf(q[r * dim + d], k[c * (dim + 1) + d], s);
+            p[i] = r < nq && j0 + c <= pos0 + r ? spk_sigmoid(fmaf(s, a.scale, bias)) : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kMaxCols; ++i) {
+            const int e = threadIdx.x + i * kThreads;
+            if (e < cols) {
+                const int r = e / vdim, c = e % vdim;
+                float s = 0.0f;
+                for (int j = 0; j < kTileK; ++j) s = fmaf(p[r * kTileK + j], v[j * vdim + c], s);
+                acc[i] += s;
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < kMaxCols; ++i) {
+        const int e = threadIdx.x + i * kThreads;
+        if (e < cols && e / vdim < nq) out[(e / vdim) * a.out_stride + e % vdim] = spk_from_float<T>(acc[i] * a.out_scale);
+    }
+}
+
+template <typename T>
+int launch_simt(const spk_sigmoid_attn_args& a, cudaStream_t s) {
+    if (kTileQ * a.vdim > kMaxCols * kThreads) return SPK_ERR_UNSUPPORTED;
+    const size_t bytes = sizeof(float) * (static_cast<size_t>(kTileQ) * a.dim + kTileK * (a.dim + 1) + kTileK * a.vdim + kTileQ * kTileK);
+    if (bytes > 227 * 1024) return SPK_ERR_UNSUPPORTED;
+    if (bytes > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(sigmoid_attn_simt_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+        if (e != cudaSuccess) return spk_set_cuda_error(e);
+    }
+    const dim3 grid(a.tiles != nullptr ? a.n_tiles : static_cast<int>(a.n), a.heads);
+    sigmoid_attn_simt_kernel<T><<<grid, kThreads, bytes, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+}  // namespace
+
+extern "C" int spk_qk_prepare(const spk_qk_prepare_args* a, void* stream) {
+    SpkRange nvtx_range("spk_qk_prepare");
+    if (a == nullptr) return SPK_ERR_NULL_POINTER;
+    if (a->n < 0 || a->heads < 1 || a->kv_heads < 1 || a->dim < 1 || a->vdim < 1 || a->block_size < 1 || a->num_blocks < 1 ||
+        a->k_pad < a->dim || a->v_pad < a->vdim || a->heads % a->kv_heads != 0)
+        return SPK_ERR_BAD_SHAPE;
+    if (a->dtype != SPK_F32 && a->dtype != SPK_BF16) return SPK_ERR_BAD_DTYPE;
+    if (((a->k_tiled && (a->k_pad % 64 != 0 || a->block_size % 8 != 0)) || (a->v_tiled && (a->v_pad % 64 != 0 || a->block_size % 8 != 0))))
+        return SPK_ERR_UNSUPPORTED;
+    if (a->rot_table != nullptr && (a->rot_dims < 2 || a->rot_dims % 2 != 0 || a->rot_dims > a->dim || a->rot_positions < 1 || a->positions == nullptr))
+        return SPK_ERR_BAD_SHAPE;
+    if (a->n == 0) return SPK_OK;
+    if (a->q == nullptr || a->k == nullptr || a->v == nullptr || a->q_out == nullptr || a->k_pool == nullptr || a->v_pool == nullptr ||
+        a->slot_mapping == nullptr)
+        return SPK_ERR_NULL_POINTER;
+    const int64_t items = a->n * (a->heads + 2 * static_cast<int64_t>(a->kv_heads));
+    const int64_t grid = (items + kWarps - 1) / kWarps;
+    const size_t bytes = sizeof(float) * kWarps * a->dim;
+    if (grid > 0x7fffffffLL || bytes > 48 * 1024) return SPK_ERR_TOO_LARGE;
+    cudaStream_t s = spk_stream(stream);
+    if (a->dtype == SPK_F32) qk_prepare_kernel<float><<<static_cast<unsigned>(grid), kThreads, bytes, s>>>(*a);
+    else qk_prepare_kernel<__nv_bfloat16><<<static_cast<unsigned>(grid), kThreads, bytes, s>>>(*a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+extern "C" int spk_sigmoid_attn_tile_tokens(void) { return kTileQ; }
+
+extern "C" int spk_sigmoid_attn(const spk_sigmoid_attn_args* a, void* stream) {
+    SpkRange nvtx_range("spk_sigmoid_attn");
+    if (a == nullptr) return SPK_ERR_NULL_POINTER;
+    if (a->n < 0 || a->heads < 1 || a->kv_heads < 1 || a->dim < 1 || a->vdim < 1 || a->block_size < 1 || a->num_blocks < 1 ||
+        a->max_blocks < 1 || a->k_pad < a->dim || a->v_pad < a->vdim || a->heads % a->kv_heads != 0 || a->heads > 65535)
+        return SPK_ERR_BAD_SHAPE;
+    if (a->dtype != SPK_F32 && a->dtype != SPK_BF16) return SPK_ERR_BAD_DTYPE;
+    if (a->n == 0) return SPK_OK;
+    if (a->q == nullptr || a->k_pool == nullptr || a->v_pool == nullptr || a->tables == nullptr || a->head_bias == nullptr || a->out == nullptr)
+        return SPK_ERR_NULL_POINTER;
+    if (a->tiles == nullptr && a->seq_lens == nullptr) return SPK_ERR_NULL_POINTER;
+    if (a->tiles != nullptr && (a->n_tiles < 1 || reinterpret_cast<uintptr_t>(a->tiles) % 16 != 0)) return SPK_ERR_BAD_SHAPE;
+    if (a->tiles == nullptr && a->n > a->table_rows) return SPK_ERR_BAD_SHAPE;
+    cudaStream_t s = spk_stream(stream);
+    return a->dtype == SPK_F32 ? launch_simt<float>(*a, s) : launch_simt<__nv_bfloat16>(*a, s);
+}

@@ -1,14 +1,15 @@
-"""Decode-side engine pieces: the paged spike pool, the on-GPU batch state and its host-side block ledger."""
+"""Decode-side engine pieces: the paged pools, the on-GPU batch state and its host-side block ledger."""
 from .batch_state import DecodeBatchState
 from .block_ledger import BlockLedger
+from .kv_state_cache import PagedKVStateCache
 from .spike_cache import PagedSpikeCache
 
-__all__ = ["DecodeBatchState", "BlockLedger", "PagedSpikeCache", "SpikeDecodeEngine"]
+__all__ = ["DecodeBatchState", "BlockLedger", "PagedSpikeCache", "PagedKVStateCache", "PagedDecodeEngine", "SpikeDecodeEngine"]
 
 
 def __getattr__(name):
-    if name == "SpikeDecodeEngine":  # imported lazily: it pulls in the model
-        from .decode_engine import SpikeDecodeEngine
+    if name in ("PagedDecodeEngine", "SpikeDecodeEngine"):  # imported lazily: they pull in the attention operators
+        from . import decode_engine
 
-        return SpikeDecodeEngine
+        return getattr(decode_engine, name)
     raise AttributeError(name)

@@ -90,6 +90,28 @@ class DecodeBatchState:
                 self.pad_block, self.block_size, self.status.data_ptr(), self._stream())
         _lib.check(rc, "spk_meta_admit")
 
+    def extend(self, row: int, n: int, positions: torch.Tensor, slots: torch.Tensor, rows: torch.Tensor,
+               edges: torch.Tensor) -> None:
+        """Append ``n`` tokens to the sequence of ``row`` (a free row starts one) and hold the row.  The portion's per-token
+        arrays (int64 positions and slots, int32 rows and edges, ``n`` entries each) are filled in on the device."""
+        with torch.cuda.device(self.device):
+            rc = self._lib.spk_meta_extend(
+                row, n, self.free_list.data_ptr(), self._free_count.data_ptr(), self.active.data_ptr(),
+                self.seq_lens.data_ptr(), self.positions.data_ptr(), self.slot_mapping.data_ptr(),
+                self.block_tables.data_ptr(), positions.data_ptr(), slots.data_ptr(), rows.data_ptr(), edges.data_ptr(),
+                self.max_rows, self.max_blocks, self.pad_block, self.block_size, self.status.data_ptr(), self._stream())
+        _lib.check(rc, "spk_meta_extend")
+
+    def resume(self, rows: torch.Tensor, tokens: torch.Tensor) -> None:
+        """Let held rows (int64 device indices) take part in decode steps again, ``tokens`` (int64) being fed next."""
+        self.active[rows] = _lib.ROW_DECODING
+        self.next_tokens[rows] = tokens
+        self.input_ids[rows] = tokens
+
+    def hold(self, rows: torch.Tensor) -> None:
+        """Make rows that hold a sequence sit out the next decode steps."""
+        self.active[rows] = _lib.ROW_HELD
+
     def release(self, row: int) -> None:
         """Retire ``row``: its blocks return to the free list in table order."""
         with torch.cuda.device(self.device):
@@ -114,5 +136,6 @@ class DecodeBatchState:
                                     ("block table full", _lib.STATUS_TABLE_FULL),
                                     ("free list overflow", _lib.STATUS_FREE_LIST_OVERFLOW),
                                     ("row busy", _lib.STATUS_ROW_BUSY),
-                                    ("device wait expired", _lib.STATUS_DEVICE_WAIT_EXPIRED)) if bits & b]
+                                    ("device wait expired", _lib.STATUS_DEVICE_WAIT_EXPIRED),
+                                    ("bad token id", _lib.STATUS_BAD_TOKEN)) if bits & b]
             raise _lib.SpkError("device status: " + ", ".join(names))

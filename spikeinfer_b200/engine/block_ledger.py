@@ -19,7 +19,8 @@ class BlockLedger:
         self.block_size = block_size
         self.max_blocks_per_seq = max_blocks_per_seq
         self.free = num_alloc_blocks
-        self.seq_lens: dict[int, int] = {}  # active row -> cached length
+        self.seq_lens: dict[int, int] = {}  # row that holds a sequence -> cached length
+        self.held: set[int] = set()  # rows among them that sit out decode steps
 
     def blocks_for(self, num_tokens: int) -> int:
         return -(-num_tokens // self.block_size)
@@ -46,17 +47,40 @@ class BlockLedger:
         self.free -= self.blocks_for(seq_len)
         self.seq_lens[row] = seq_len
 
+    def extend_error(self, portions: list[tuple[int, int]]) -> str | None:
+        """Why these ``(row, tokens)`` portions cannot be appended right now, or None if they can."""
+        need = 0
+        for row, n in portions:
+            if n < 1:
+                return "empty portion"
+            have = self.seq_lens.get(row, 0)
+            if have + n > self.max_seq_len:
+                return f"sequence of {have + n} tokens exceeds max_model_len {self.max_seq_len}"
+            need += self.blocks_for(have + n) - self.blocks_for(have)
+        if need > self.free:
+            return f"portions need {need} blocks, {self.free} are free"
+        return None
+
+    def extend(self, row: int, n: int) -> None:
+        """Mirror of ``DecodeBatchState.extend``: the row is held afterwards."""
+        have = self.seq_lens.get(row, 0)
+        self.free -= self.blocks_for(have + n) - self.blocks_for(have)
+        self.seq_lens[row] = have + n
+        self.held.add(row)
+
     def blocks_next_step(self) -> int:
-        """Blocks the next ``advance`` will pop: one per active row whose length sits on a page boundary
+        """Blocks the next ``advance`` will pop: one per decoding row whose length sits on a page boundary
         and whose table still has room."""
         bs = self.block_size
-        return sum(1 for n in self.seq_lens.values() if n % bs == 0 and n // bs < self.max_blocks_per_seq)
+        return sum(1 for row, n in self.seq_lens.items() if row not in self.held and n % bs == 0 and n // bs < self.max_blocks_per_seq)
 
     def advance(self) -> None:
         """Mirror of one ``DecodeBatchState.advance``: rows are served in row order; a row that finds the list
         empty, or whose table is full, stays where it is."""
         bs = self.block_size
         for row in sorted(self.seq_lens):
+            if row in self.held:
+                continue
             n = self.seq_lens[row]
             if n // bs >= self.max_blocks_per_seq:
                 continue
@@ -68,6 +92,7 @@ class BlockLedger:
 
     def release(self, row: int) -> None:
         n = self.seq_lens.pop(row)
+        self.held.discard(row)
         self.free += min(self.blocks_for(n), self.max_blocks_per_seq)
 
 
@@ -87,3 +112,22 @@ def covering_bucket(buckets: list[int], rows_in_use) -> int:
         if b >= top:
             return b
     return buckets[-1]
+
+
+def cut_portions(lengths: list[int], budget: int | None) -> list[list[tuple[int, int, int]]]:
+    """Cut prompts into prefill calls of at most ``budget`` tokens, in order: each call is a list of
+    ``(prompt, start, stop)`` with at most one portion per prompt.  ``None``: everything in one call."""
+    if budget is None:
+        return [[(i, 0, n) for i, n in enumerate(lengths)]] if lengths else []
+    calls, call, left = [], [], budget
+    for i, n in enumerate(lengths):
+        lo = 0
+        while lo < n:
+            take = min(left, n - lo)
+            call.append((i, lo, lo + take))
+            lo += take
+            left -= take
+            if left == 0:
+                calls.append(call)
+                call, left = [], budget
+    return calls + [call] if call else calls

@@ -93,6 +93,10 @@ class PagedSpikeCache:
         T, H, nb, bs, W = pool.shape
         return pool.reshape(T, H, nb * bs, W)
 
+    def recurrent_tensors(self) -> tuple:
+        """State that a replayed step would not rewrite by itself: none."""
+        return ()
+
     def reset(self) -> None:
         for t in self._buffers:
             t.zero_()

@@ -21,13 +21,14 @@ Dense GEMMs stay PyTorch (cuBLAS), as do the embedding lookup, the final mean ov
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, fields
 
 import torch
 import torch.nn.functional as F
 
 from . import _lib
 from .attention import AttentionMetadata, fused_qkv_attention
+from .engine.spike_cache import PagedSpikeCache
 from .kernels import add_rms_norm, lif_gate_mul
 
 
@@ -44,6 +45,14 @@ class SpikingQwenConfig:
     rms_norm_eps: float = 1e-6
     rope_theta: float = 1e6
     tie_word_embeddings: bool = True
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "SpikingQwenConfig":
+        """From the parsed ``config.json`` of a model folder (Qwen2's key names, plus ``T``)."""
+        names = {f.name for f in fields(cls)}
+        known = {k: v for k, v in d.items() if k in names}
+        known.setdefault("head_dim", d["hidden_size"] // d["num_attention_heads"])
+        return cls(**known)
 
     @classmethod
     def qwen2_5_0p5b(cls) -> "SpikingQwenConfig":
@@ -135,6 +144,17 @@ class SpikingQwenModel:
         gets bit-identical factors.  Positions beyond the table must not be fed afterwards."""
         cos, sin = self._rope_direct(torch.arange(max_positions, device=self.device))
         self.rope_table = torch.stack((cos, sin), dim=1).contiguous()  # [max_positions, 2, head_dim]
+
+    def prepare(self, max_positions: int) -> None:
+        """Engine hook: positions ``0 .. max_positions - 1`` may be fed."""
+        if self.rope_table is None or self.rope_table.shape[0] < max_positions:
+            self.build_rope_table(max_positions)
+
+    def new_cache(self, num_blocks: int, block_size: int, max_rows: int) -> PagedSpikeCache:
+        """Engine hook: the paged pool this model's layers write (``max_rows`` is for models with per-row state)."""
+        c = self.config
+        return PagedSpikeCache(c.num_hidden_layers, c.T, c.num_key_value_heads, c.head_dim, num_blocks, block_size,
+                               device=self.device)
 
     def rope(self, positions: torch.Tensor):
         """``(cos, sin)``, each ``[n_tok, head_dim]`` in the model dtype (rows may be strided)."""
