@@ -491,8 +491,11 @@ int spk_qk_prepare(const spk_qk_prepare_args* args, void* stream);
 
 /* out[t, h, :] = out_scale * sum_j sigmoid(scale * q[t,h].k_j + head_bias[h]) v_j over the keys 0 .. position of token t,
  * k_j, v_j of KV head h / (heads / kv_heads) read through the block table of the token's row.
- * Prefill form: tiles int32 [n_tiles][4] = (first token, tokens <= spk_sigmoid_attn_tile_tokens(), row, position of the
- * first).  Decode form (tiles NULL): token t = row t, position seq_lens[t] - 1; inactive rows give zeros. */
+ * Prefill form: tiles int32 [n_tiles][4] = (first token, tokens <= spk_sigmoid_attn_tile_tokens(...), row, position of the
+ * first).  Decode form (tiles NULL): token t = row t, position seq_lens[t] - 1; inactive rows give zeros.
+ * Decode form with partials != NULL (where spk_sigmoid_attn_splits(...) > 0): a row's keys are cut into `splits` ranges and
+ * the ranges' unscaled sums go to partials [n][splits][heads * vdim]; out is not written, ranges without keys are left as
+ * they are, and spk_gated_norm adds the rest. */
 typedef struct spk_sigmoid_attn_args {
     const void* q;              /* [n, heads, k_pad] */
     const void* k_pool;
@@ -509,7 +512,9 @@ typedef struct spk_sigmoid_attn_args {
     int64_t max_blocks;
     int64_t n;
     int64_t num_blocks;
+    float* partials;
     int32_t n_tiles;
+    int32_t splits;
     int32_t heads, kv_heads, dim, vdim;
     int32_t k_pad, v_pad, k_tiled, v_tiled;
     int32_t block_size;
@@ -519,12 +524,16 @@ typedef struct spk_sigmoid_attn_args {
     float _pad;
     uint32_t* status;
 } spk_sigmoid_attn_args;
-int spk_sigmoid_attn_tile_tokens(void);
+int spk_sigmoid_attn_tile_tokens(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size);
+/* Key ranges the decode form should be cut into for n rows of at most max_keys keys; 0: there is no partial form for these
+ * sizes. */
+int spk_sigmoid_attn_splits(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size, int64_t n, int heads,
+                            int kv_heads, int64_t max_keys);
 int spk_sigmoid_attn(const spk_sigmoid_attn_args* args, void* stream);
 
 /* S_t = decay_h S_{t-1} + k_t v_t^T, out_t = S_t^T q_t, with silu applied to q, k and v first when silu != 0.
- * state: 32-bit, row r, head h at state + r * state_stride + h * dim * vdim, [dim][vdim].  decay_pow [heads][chunk + 1]: the
- * powers 0 .. spk_decay_chunk_tokens() of every head's decay.  out 32-bit [n, heads * vdim].
+ * state: 32-bit, row r, head h at state + r * state_stride + h * dim * vdim, [dim][vdim].  decay_pow [heads][
+ * spk_decay_powers()]: the powers 0, 1, 2 ... of every head's decay.  out 32-bit [n, heads * vdim].
  * _step: decode form.  _chunks: prefill form; chunks int32 [n_chunks][4] = (first token, tokens, sequence, index in the
  * sequence), seqs int32 [n_seqs][4] = (first chunk, chunks, state row, tokens before this portion: 0 starts from a zero
  * state whatever the slot holds); workspace of spk_decay_attn_workspace_bytes. */
@@ -551,14 +560,16 @@ typedef struct spk_decay_attn_args {
     int32_t _pad;
     uint32_t* status;
 } spk_decay_attn_args;
-int spk_decay_chunk_tokens(void);
+int spk_decay_powers(void);
+/* Tokens per chunk of the prefill form for a call of n tokens: chunks may not be longer. */
+int spk_decay_chunk_tokens(int dtype, int dim, int vdim, int64_t n, int heads);
 int64_t spk_decay_attn_workspace_bytes(int n_chunks, int heads, int dim, int vdim);
 int spk_decay_attn_step(const spk_decay_attn_args* args, void* stream);
 int spk_decay_attn_chunks(const spk_decay_attn_args* args, void* stream);
 
 /* out[t, out_offset + c] = scale * (x / sqrt(mean(x^2) + eps) * w)[c] * sigmoid(gate[t, c]) over the `width` columns of x (32-bit).
- * partials != NULL (decode form): out[t, c] = left_scale * sum of the partial sums [n][splits][left_width] whose key range
- * (keys_per_split each) begins below seq_lens[t], for c < left_width <= out_offset. */
+ * partials != NULL (decode form): out[t, c] = left_scale * sum of spk_sigmoid_attn's partial sums [n][splits][left_width] of
+ * the key ranges that seq_lens[t] keys fill, for c < left_width <= out_offset; the same splits as there. */
 typedef struct spk_gated_norm_args {
     const float* x;             /* [n, width] */
     const float* w;
@@ -573,13 +584,11 @@ typedef struct spk_gated_norm_args {
     int32_t width;
     int32_t out_offset;
     int32_t splits;
-    int32_t keys_per_split;
     int32_t left_width;
     int32_t dtype;
     float eps;
     float scale;
     float left_scale;
-    float _pad;
 } spk_gated_norm_args;
 int spk_gated_norm(const spk_gated_norm_args* args, void* stream);
 

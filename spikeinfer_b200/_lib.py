@@ -115,7 +115,7 @@ class SigmoidAttnArgs(Structure):
     """Mirror of ``spk_sigmoid_attn_args``."""
 
     _fields_ = _fields("p q k_pool v_pool tables seq_lens active tiles head_bias out; l out_stride table_stride table_rows "
-                       "max_blocks n num_blocks; i n_tiles heads kv_heads dim vdim k_pad v_pad k_tiled v_tiled block_size dtype; "
+                       "max_blocks n num_blocks; p partials; i n_tiles splits heads kv_heads dim vdim k_pad v_pad k_tiled v_tiled block_size dtype; "
                        "f scale out_scale _pad; p status")
 
 
@@ -130,7 +130,7 @@ class GatedNormArgs(Structure):
     """Mirror of ``spk_gated_norm_args``."""
 
     _fields_ = _fields("p x w gate; l gate_stride; p out; l out_stride; p partials seq_lens active; l n; i width out_offset splits "
-                       "keys_per_split left_width dtype; f eps scale left_scale _pad")
+                       "left_width dtype; f eps scale left_scale")
 
 
 # name -> (restype, argtypes); every symbol include/spikeinfer_b200.h declares
@@ -195,9 +195,11 @@ SIGNATURES = {
     "spk_residual_norm": (c_int, [POINTER(ResidualNormArgs), c_void_p]),
     "spk_poly_norm": (c_int, [c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int64, c_int, c_void_p]),
     "spk_qk_prepare": (c_int, [POINTER(QkPrepareArgs), c_void_p]),
-    "spk_sigmoid_attn_tile_tokens": (c_int, []),
+    "spk_sigmoid_attn_tile_tokens": (c_int, [c_int] * 6),
+    "spk_sigmoid_attn_splits": (c_int, [c_int] * 6 + [c_int64, c_int, c_int, c_int64]),
     "spk_sigmoid_attn": (c_int, [POINTER(SigmoidAttnArgs), c_void_p]),
-    "spk_decay_chunk_tokens": (c_int, []),
+    "spk_decay_powers": (c_int, []),
+    "spk_decay_chunk_tokens": (c_int, [c_int, c_int, c_int, c_int64, c_int]),
     "spk_decay_attn_workspace_bytes": (c_int64, [c_int, c_int, c_int, c_int]),
     "spk_decay_attn_step": (c_int, [POINTER(DecayAttnArgs), c_void_p]),
     "spk_decay_attn_chunks": (c_int, [POINTER(DecayAttnArgs), c_void_p]),

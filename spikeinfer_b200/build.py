@@ -32,7 +32,8 @@ NO_FMA_CONTRACTION = {"spk_lif.cu", "spk_norm.cu"}
 COMPONENTS = {
     "core": ("spk_capi.cu", "spk_meta.cu", "spk_sample.cu"),
     "spike": ("spk_attn.cu", "spk_attn_stream.cu", "spk_lif.cu", "spk_norm.cu", "spk_pack.cu"),
-    "dense": ("spk_postnorm.cu", "spk_paged_attn.cu", "spk_decay.cu"),
+    "dense": ("spk_postnorm.cu", "spk_paged_attn.cu", "spk_sigmoid_prefill.cu", "spk_sigmoid_decode.cu", "spk_decay.cu",
+              "spk_decay_mma.cu"),
 }
 
 

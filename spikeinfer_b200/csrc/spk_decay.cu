@@ -3,19 +3,21 @@
 //   S_t = decay_h S_{t-1} + k_t v_t^T        o_t = S_t^T q_t        (S in 32 bits, one state per sequence and head)
 //
 //  * decay_step_kernel: one token per row (decode), state read and written once.
-//  * prefill cuts a portion into chunks of 64 tokens: every chunk's own sum of k v^T (decay_chunk_sum_kernel), a scan
-//    over the chunks that leaves each chunk the state it starts from (decay_scan_kernel), and the outputs, a decayed
-//    masked product inside the chunk plus the incoming state (decay_chunk_out_kernel).  All chunks of all sequences of the
-//    call run at once; only the scan walks them in order.
+//  * prefill cuts a portion into chunks: every chunk's own sum of k v^T (decay_chunk_sum_kernel), a scan over the chunks that
+//    leaves each chunk the state it starts from (decay_scan_kernel), and the outputs, a decayed masked product inside the
+//    chunk plus the incoming state (decay_chunk_out_kernel).  All chunks of all sequences of the call run at once; only the
+//    scan walks them in order.  The two outer kernels here are the 32-bit form (any sizes, chunks of 64 tokens); bf16
+//    projections with heads of up to 128 channels take the tensor-core form of spk_decay_mma.cu.
 //  * gated_norm_kernel: the heads' outputs under one RMS norm, times sigmoid(gate), scaled into one half of the operand
 //    of the output projection; in decode steps it also adds up the attention's partial sums into the other half.
 //
-// Decay powers come from a host table [head][0 .. 64] (evaluated in double precision), never from repeated products.
-#include "spk_dense.cuh"
+// Decay powers come from a host table [head][0 .. 512] (evaluated in double precision), never from repeated products.
+#include "spk_decay.cuh"
 
 namespace {
 
-constexpr int kChunk = 64;
+constexpr int kChunk = kDecayChunk;
+constexpr int kPow = kDecayMaxSpan + 1;  // tabulated powers per head
 constexpr int kThreads = 256;
 
 __device__ __forceinline__ float act(float x, int silu) { return silu ? spk_silu(x) : x; }
@@ -47,7 +49,7 @@ decay_step_kernel(const spk_decay_attn_args a) {
     }
     for (int e = threadIdx.x; e < vdim; e += kThreads) v[e] = act(spk_to_float<T>(vr[e]), a.silu);
     __syncthreads();
-    const float decay = a.decay_pow[h * (kChunk + 1) + 1];
+    const float decay = a.decay_pow[h * kPow + 1];
     float* S = a.state + row * a.state_stride + static_cast<int64_t>(h) * dim * vdim;
     const int cols = vdim / W;
     const int slices = cols < kThreads ? kThreads / cols : 1;
@@ -118,29 +120,19 @@ __device__ __forceinline__ void stage_rows(float* dst, const T* src, int64_t ld,
     }
 }
 
-struct ChunkInfo {
-    int64_t start;
-    int len, seq, index;
-};
-
-__device__ __forceinline__ ChunkInfo chunk_info(const spk_decay_attn_args& a, int c) {
-    const int4 e = reinterpret_cast<const int4*>(a.chunks)[c];
-    return {e.x, e.y, e.z, e.w};
-}
-
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 decay_chunk_sum_kernel(const spk_decay_attn_args a) {
     extern __shared__ float sm[];
     const int c = blockIdx.x, h = blockIdx.y;
-    const ChunkInfo ci = chunk_info(a, c);
+    const SpkChunk ci = spk_chunk(a, c);
     const int dp = pad4(a.dim), ep = pad4(a.vdim);
     float* k = sm;
     float* v = k + kChunk * dp;
     stage_rows<T>(k, static_cast<const T*>(a.k) + ci.start * a.ld + static_cast<int64_t>(h) * a.dim, a.ld, ci.len, a.dim, a.silu);
     stage_rows<T>(v, static_cast<const T*>(a.v) + ci.start * a.ld + static_cast<int64_t>(h) * a.vdim, a.ld, ci.len, a.vdim, a.silu);
     __syncthreads();
-    const float* pw = a.decay_pow + h * (kChunk + 1);
+    const float* pw = a.decay_pow + h * kPow;
     float* U = a.workspace + (static_cast<int64_t>(c) * a.heads + h) * a.dim * a.vdim;
     const int te = ep / 4, tiles = (dp / 4) * te;
     for (int t = threadIdx.x; t < tiles; t += kThreads) {
@@ -178,7 +170,7 @@ decay_scan_kernel(const spk_decay_attn_args a) {
         if (i == 0) spk_flag(a.status, SPK_STATUS_BAD_SLOT);
         return;
     }
-    const float* pw = a.decay_pow + (i / per_head) * (kChunk + 1);
+    const float* pw = a.decay_pow + (i / per_head) * kPow;
     float* slot = a.state + sq.z * a.state_stride + i;
     float S = sq.w > 0 ? *slot : 0.0f;
     float* w = a.workspace + sq.x * per_chunk + i;
@@ -195,7 +187,7 @@ __global__ void __launch_bounds__(kThreads)
 decay_chunk_out_kernel(const spk_decay_attn_args a) {
     extern __shared__ float sm[];
     const int c = blockIdx.x, h = blockIdx.y;
-    const ChunkInfo ci = chunk_info(a, c);
+    const SpkChunk ci = spk_chunk(a, c);
     const int dp = pad4(a.dim), ep = pad4(a.vdim);
     constexpr int AP = kChunk + 1;
     float* q = sm;
@@ -206,7 +198,7 @@ decay_chunk_out_kernel(const spk_decay_attn_args a) {
     stage_rows<T>(k, static_cast<const T*>(a.k) + ci.start * a.ld + static_cast<int64_t>(h) * a.dim, a.ld, ci.len, a.dim, a.silu);
     stage_rows<T>(v, static_cast<const T*>(a.v) + ci.start * a.ld + static_cast<int64_t>(h) * a.vdim, a.ld, ci.len, a.vdim, a.silu);
     __syncthreads();
-    const float* pw = a.decay_pow + h * (kChunk + 1);
+    const float* pw = a.decay_pow + h * kPow;
     {
         const int i0 = threadIdx.x / 16, j0 = threadIdx.x % 16;  // rows i0 + 16 x, columns j0 + 16 y
         float acc[4][4] = {};
@@ -280,8 +272,8 @@ gated_norm_kernel(const spk_gated_norm_args a) {
     const bool live = a.active == nullptr || a.active[t] == 1;
     if (a.partials != nullptr) {
         const int len = live ? a.seq_lens[t] : 0;
-        int valid = (len + a.keys_per_split - 1) / a.keys_per_split;
-        if (valid > a.splits) valid = a.splits;
+        const int per = spk_split_keys(len, a.splits);
+        const int valid = (len + per - 1) / per;
         const float* p = a.partials + t * a.splits * a.left_width;
         for (int c = threadIdx.x; c < a.left_width; c += kThreads) {
             float s = 0.0f;
@@ -336,6 +328,13 @@ int launch_step(const spk_decay_attn_args& a, cudaStream_t s) {
     return SPK_OK;
 }
 
+int launch_scan(const spk_decay_attn_args& a, cudaStream_t s) {
+    const int64_t per = static_cast<int64_t>(a.heads) * a.dim * a.vdim;
+    decay_scan_kernel<<<dim3(static_cast<unsigned>((per + kThreads - 1) / kThreads), a.n_seqs), kThreads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
 template <typename T>
 int launch_chunks(const spk_decay_attn_args& a, cudaStream_t s) {
     const size_t dp = pad4(a.dim), ep = pad4(a.vdim);
@@ -345,9 +344,7 @@ int launch_chunks(const spk_decay_attn_args& a, cudaStream_t s) {
     const dim3 grid(a.n_chunks, a.heads);
     decay_chunk_sum_kernel<T><<<grid, kThreads, b1, s>>>(a);
     SPK_CHECK_LAUNCH();
-    const int64_t per = static_cast<int64_t>(a.heads) * a.dim * a.vdim;
-    decay_scan_kernel<<<dim3(static_cast<unsigned>((per + kThreads - 1) / kThreads), a.n_seqs), kThreads, 0, s>>>(a);
-    SPK_CHECK_LAUNCH();
+    if (const int rc = launch_scan(a, s)) return rc;
     decay_chunk_out_kernel<T><<<grid, kThreads, b3, s>>>(a);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
@@ -355,7 +352,14 @@ int launch_chunks(const spk_decay_attn_args& a, cudaStream_t s) {
 
 }  // namespace
 
-extern "C" int spk_decay_chunk_tokens(void) { return kChunk; }
+extern "C" int spk_decay_powers(void) { return kPow; }
+
+extern "C" int spk_decay_chunk_tokens(int dtype, int dim, int vdim, int64_t n, int heads) {
+    if (!spk_decay_tensor_form(dtype, dim, vdim) || n < 1 || heads < 1) return kChunk;
+    int span = kDecayMaxSpan;  // as long as two CTAs per SM remain
+    while (span > kChunk && n * heads < static_cast<int64_t>(span) * 2 * 148) span /= 2;
+    return span;
+}
 
 extern "C" int64_t spk_decay_attn_workspace_bytes(int n_chunks, int heads, int dim, int vdim) {
     if (n_chunks < 1 || heads < 1 || dim < 1 || vdim < 1) return 0;
@@ -382,6 +386,11 @@ extern "C" int spk_decay_attn_chunks(const spk_decay_attn_args* a, void* stream)
     if (a->workspace == nullptr || a->workspace_bytes < spk_decay_attn_workspace_bytes(a->n_chunks, a->heads, a->dim, a->vdim))
         return SPK_ERR_WORKSPACE_TOO_SMALL;
     cudaStream_t s = spk_stream(stream);
+    if (spk_decay_tensor_form(a->dtype, a->dim, a->vdim)) {
+        if (const int e = spk_decay_mma_sums(*a, s)) return e;
+        if (const int e = launch_scan(*a, s)) return e;
+        return spk_decay_mma_outputs(*a, s);
+    }
     return a->dtype == SPK_F32 ? launch_chunks<float>(*a, s) : launch_chunks<__nv_bfloat16>(*a, s);
 }
 
@@ -393,7 +402,7 @@ extern "C" int spk_gated_norm(const spk_gated_norm_args* a, void* stream) {
     if (a->n == 0) return SPK_OK;
     if (a->n > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
     if (a->x == nullptr || a->w == nullptr || a->gate == nullptr || a->out == nullptr) return SPK_ERR_NULL_POINTER;
-    if (a->partials != nullptr && (a->seq_lens == nullptr || a->splits < 1 || a->keys_per_split < 1 || a->left_width < 1 ||
+    if (a->partials != nullptr && (a->seq_lens == nullptr || a->splits < 1 || a->left_width < 1 ||
                                    a->left_width > a->out_offset))
         return SPK_ERR_BAD_SHAPE;
     cudaStream_t s = spk_stream(stream);

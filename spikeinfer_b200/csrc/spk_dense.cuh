@@ -102,3 +102,9 @@ __device__ __forceinline__ int spk_page_channel(const SpkPageLayout& p, int r, i
 __device__ __forceinline__ int64_t spk_page_base(const SpkPageLayout& p, int64_t block, int head) {
     return (block * p.heads + head) * static_cast<int64_t>(p.block_size) * p.dim_pad;
 }
+
+// Keys per range when a row of `len` keys is cut into at most `splits` ranges: whole groups of 64 keys.
+__host__ __device__ __forceinline__ int spk_split_keys(int len, int splits) {
+    const int per = (len + splits - 1) / splits;
+    return per <= 64 ? 64 : (per + 63) & ~63;
+}

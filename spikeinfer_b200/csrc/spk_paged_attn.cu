@@ -6,6 +6,7 @@
 //    32 bits; any head sizes, prefill tiles and decode rows alike.
 // A weight depends on its own key alone, so there is no running maximum and no denominator, and sums over
 // different key ranges simply add up.
+#include "spk_paged_attn.cuh"
 #include "spk_dense.cuh"
 
 namespace {
@@ -219,7 +220,18 @@ extern "C" int spk_qk_prepare(const spk_qk_prepare_args* a, void* stream) {
     return SPK_OK;
 }
 
-extern "C" int spk_sigmoid_attn_tile_tokens(void) { return kTileQ; }
+extern "C" int spk_sigmoid_attn_tile_tokens(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size) {
+    return spk_attn_tensor_form(dtype, k_pad, v_pad, k_tiled, v_tiled, block_size) ? 128 : kTileQ;
+}
+
+extern "C" int spk_sigmoid_attn_splits(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size, int64_t n, int heads,
+                                       int kv_heads, int64_t max_keys) {
+    if (n < 1 || heads < 1 || kv_heads < 1 || max_keys < 1 || !spk_attn_tensor_form(dtype, k_pad, v_pad, k_tiled, v_tiled, block_size)) return 0;
+    const int64_t ctas = n * kv_heads * ((heads / kv_heads + 15) / 16);
+    const int64_t want = (3 * 148 + ctas - 1) / ctas, most = (max_keys + 255) / 256;
+    const int64_t splits = want < most ? want : most;
+    return static_cast<int>(splits < 1 ? 1 : splits > 64 ? 64 : splits);
+}
 
 extern "C" int spk_sigmoid_attn(const spk_sigmoid_attn_args* a, void* stream) {
     SpkRange nvtx_range("spk_sigmoid_attn");
@@ -229,11 +241,22 @@ extern "C" int spk_sigmoid_attn(const spk_sigmoid_attn_args* a, void* stream) {
         return SPK_ERR_BAD_SHAPE;
     if (a->dtype != SPK_F32 && a->dtype != SPK_BF16) return SPK_ERR_BAD_DTYPE;
     if (a->n == 0) return SPK_OK;
-    if (a->q == nullptr || a->k_pool == nullptr || a->v_pool == nullptr || a->tables == nullptr || a->head_bias == nullptr || a->out == nullptr)
+    if (a->q == nullptr || a->k_pool == nullptr || a->v_pool == nullptr || a->tables == nullptr || a->head_bias == nullptr ||
+        (a->out == nullptr && (a->partials == nullptr || a->tiles != nullptr)))
         return SPK_ERR_NULL_POINTER;
     if (a->tiles == nullptr && a->seq_lens == nullptr) return SPK_ERR_NULL_POINTER;
     if (a->tiles != nullptr && (a->n_tiles < 1 || reinterpret_cast<uintptr_t>(a->tiles) % 16 != 0)) return SPK_ERR_BAD_SHAPE;
     if (a->tiles == nullptr && a->n > a->table_rows) return SPK_ERR_BAD_SHAPE;
     cudaStream_t s = spk_stream(stream);
+    if (spk_attn_tensor_form(a->dtype, a->k_pad, a->v_pad, a->k_tiled, a->v_tiled, a->block_size)) {
+        // tiles of the tensor-core form's own size; q rows and pages are read 16 bytes at a time
+        if (reinterpret_cast<uintptr_t>(a->q) % 16 != 0 || reinterpret_cast<uintptr_t>(a->k_pool) % 16 != 0 ||
+            reinterpret_cast<uintptr_t>(a->v_pool) % 16 != 0)
+            return SPK_ERR_BAD_STRIDE;
+        if (a->tiles != nullptr) return spk_sigmoid_prefill_launch(*a, s);
+        if (a->partials != nullptr) return a->splits < 1 ? SPK_ERR_BAD_SHAPE : spk_sigmoid_decode_launch(*a, s);
+    } else if (a->partials != nullptr) {
+        return SPK_ERR_UNSUPPORTED;
+    }
     return a->dtype == SPK_F32 ? launch_simt<float>(*a, s) : launch_simt<__nv_bfloat16>(*a, s);
 }

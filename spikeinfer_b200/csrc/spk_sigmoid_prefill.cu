@@ -1,0 +1,292 @@
+// Prefill attention with sigmoid key weights on the fifth-generation tensor cores (tcgen05), bf16, head sizes up to 128.
+//
+// CTA = (128 query tokens of one portion, query head).  Ten warps:
+//  * warp 8 copies K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
+//    handful of plain bulk copies (cp.async.bulk), no tensor map, whatever pages the block table names;
+//  * warp 9 (one thread) issues the MMAs: S = Q K^T into one of two TMEM buffers, O += P V with P read from TMEM;
+//  * warps 0-3 and 4-7 turn the even and the odd tiles' scores into weights (one thread per query row).
+// A weight is sigmoid(score) of its own key: no running maximum, no rescaling of O, no denominator.  Weights are computed in
+// 32 bits and enter the product as a bf16 pair (hi + lo: 16 significant bits), so O is a 32-bit sum of them to 2^-17.
+// Visible keys are those up to the query's own position; the last tile's rows of V beyond the portion's end are cleared in
+// shared memory (a page's unwritten rows may hold anything, and 0 * NaN is NaN).
+#include "spk_paged_attn.cuh"
+#include "spk_tensor.cuh"
+
+namespace {
+
+using namespace spk_tc;
+
+constexpr int kTile = 128;            // query rows, and keys per step
+constexpr int kColTile = kTile * 128; // bytes of a 64-channel column tile
+constexpr int kSigmoidThreads = 256;
+constexpr int kThreads = kSigmoidThreads + 64;
+constexpr uint32_t kTmemS = 0, kTmemLo = 256, kTmemO = 384;  // S/P-hi buffers 2 x 128, P-lo 2 x 64, O up to 128
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <int CK, int CV>
+struct Shape {
+    static constexpr int NS = CK + CV <= 2 ? 4 : 2;  // stages of K and of V
+    static constexpr int kK = CK * kColTile, kV = CV * kColTile;
+    static constexpr int kBytes = kK + NS * (kK + kV) + 1024 + 256;
+};
+
+struct Bars {
+    uint64_t k_full[4], k_free[4], v_full[4], v_free[4], s_full[2], p_full[2], p_free[2], o_full;
+    int abort;
+    uint32_t tmem;
+};
+
+template <int CK, int CV>
+__global__ void __launch_bounds__(kThreads, 1)
+sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
+    using Sh = Shape<CK, CV>;
+    constexpr int NS = Sh::NS;
+    extern __shared__ uint8_t raw[];
+    uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
+    uint8_t* q_s = base;
+    uint8_t* k_s = q_s + Sh::kK;
+    uint8_t* v_s = k_s + NS * Sh::kK;
+    Bars* bars = reinterpret_cast<Bars*>(v_s + NS * Sh::kV);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+    const int h = blockIdx.x;
+    const int g = h / (a.heads / a.kv_heads);
+    const int4 tile = reinterpret_cast<const int4*>(a.tiles)[blockIdx.y];
+    const int64_t t0 = tile.x;
+    const int nq = tile.y, row = tile.z, pos0 = tile.w;
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + t0 * a.out_stride + static_cast<int64_t>(h) * a.vdim;
+    // uniform over the CTA: nothing has been set up yet
+    if (row < 0 || row >= a.table_rows || pos0 < 0 || nq < 1 || nq > kTile ||
+        static_cast<int64_t>(pos0) + nq > a.max_blocks * a.block_size) {
+        if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+        for (int i = threadIdx.x; i < nq * a.vdim && nq <= kTile; i += kThreads)
+            out[(i / a.vdim) * a.out_stride + i % a.vdim] = __float2bfloat16_rn(0.0f);
+        return;
+    }
+    const int keys = pos0 + nq;
+    const int tiles = (keys + kTile - 1) / kTile;
+
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < NS; ++i) {
+            mbar_init(smem_u32(&bars->k_full[i]), 1);
+            mbar_init(smem_u32(&bars->k_free[i]), 1);
+            mbar_init(smem_u32(&bars->v_full[i]), 1);
+            mbar_init(smem_u32(&bars->v_free[i]), 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(smem_u32(&bars->s_full[i]), 1);
+            mbar_init(smem_u32(&bars->p_full[i]), 128);
+            mbar_init(smem_u32(&bars->p_free[i]), 1);
+        }
+        mbar_init(smem_u32(&bars->o_full), 1);
+        bars->abort = 0;
+    }
+    if (warp == 0) tmem_alloc(smem_u32(&bars->tmem), 512);
+    // Q rows into the swizzled operand layout, zeros beyond the portion
+    for (int i = threadIdx.x; i < kTile * CK * 8; i += kThreads) {
+        const int r = i / (CK * 8), c = i % (CK * 8);
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r < nq)
+            v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + ((t0 + r) * a.heads + h) * a.k_pad + c * 8);
+        *reinterpret_cast<uint4*>(q_s + (c >> 3) * kColTile + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+    }
+    fence_async_shared();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = bars->tmem;
+    volatile int* abort = &bars->abort;
+
+    if (warp == 8) {  // ---- K and V copies
+        const int gran = a.block_size < kTile ? a.block_size : kTile;  // rows per copy
+        const int32_t* table = a.tables + static_cast<int64_t>(row) * a.table_stride;
+        const SpkPageLayout kl{a.kv_heads, a.block_size, a.k_pad, 1}, vl{a.kv_heads, a.block_size, a.v_pad, 1};
+        int issued = 0;
+        for (int t = 0; t < tiles; ++t) {
+            const int stage = t % NS;
+            const uint32_t parity = ((t / NS) - 1) & 1;
+            const int valid = keys - t * kTile < kTile ? keys - t * kTile : kTile;
+            const int n = (valid + gran - 1) / gran;
+            auto copy = [&](const void* pool, const SpkPageLayout& l, int cols, uint8_t* dst, uint64_t* full) {
+                const uint32_t bar = smem_u32(full);
+                if (lane == 0) mbar_expect(bar, static_cast<uint32_t>(n * cols * gran * 128));
+                __syncwarp();
+                for (int i = lane; i < n * cols; i += 32) {
+                    const int p = i % n, c = i / n;
+                    const int j = t * kTile + p * gran;
+                    int64_t block = table[j / a.block_size];
+                    if (block < 0 || block >= a.num_blocks) {
+                        spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
+                        block = 0;
+                    }
+                    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(pool) + spk_page_base(l, block, g) +
+                                               c * (a.block_size << 6) + ((j % a.block_size) << 6);
+                    bulk_load(smem_u32(dst) + c * kColTile + p * gran * 128, src, gran * 128, bar);
+                }
+            };
+            // waits are made warp-uniform: a vote also brings the lanes back together
+            if (t >= NS && !__all_sync(~0u, mbar_wait(smem_u32(&bars->k_free[stage]), parity, abort))) break;
+            copy(a.k_pool, kl, CK, k_s + stage * Sh::kK, &bars->k_full[stage]);
+            if (t >= NS && !__all_sync(~0u, mbar_wait(smem_u32(&bars->v_free[stage]), parity, abort))) {
+                mbar_wait(smem_u32(&bars->k_full[stage]), (t / NS) & 1);
+                break;
+            }
+            copy(a.v_pool, vl, CV, v_s + stage * Sh::kV, &bars->v_full[stage]);
+            issued = t + 1;
+        }
+        if (*abort != 0)  // copies in flight land before the CTA's shared memory is given up
+            for (int t = issued > NS ? issued - NS : 0; t < issued; ++t) {
+                mbar_wait(smem_u32(&bars->k_full[t % NS]), (t / NS) & 1);
+                mbar_wait(smem_u32(&bars->v_full[t % NS]), (t / NS) & 1);
+            }
+    } else if (warp == 9) {  // ---- MMA issue
+        if (lane == 0) {
+            constexpr uint32_t idesc_s = idesc_bf16(kTile, kTile, false, false);
+            constexpr uint32_t idesc_o = idesc_bf16(kTile, CV * 64, false, true);
+            auto scores = [&](int t) {
+                const int stage = t % NS;
+                if (!mbar_wait(smem_u32(&bars->k_full[stage]), (t / NS) & 1, abort)) return false;
+                tc_fence_after();
+                const uint32_t qa = smem_u32(q_s), kb = smem_u32(k_s + stage * Sh::kK);
+#pragma unroll
+                for (int s = 0; s < CK * 4; ++s) {
+                    const uint32_t off = (s >> 2) * kColTile + (s & 3) * 32;
+                    mma_ss(tmem + kTmemS + (t & 1) * 128, desc_sw128(qa + off, 16, 1024), desc_sw128(kb + off, 16, 1024), idesc_s, s > 0);
+                }
+                mma_commit(smem_u32(&bars->k_free[stage]));
+                mma_commit(smem_u32(&bars->s_full[t & 1]));
+                return true;
+            };
+            bool ok = scores(0) && (tiles < 2 || scores(1));
+            for (int t = 0; ok && t < tiles; ++t) {
+                const int stage = t % NS, buf = t & 1;
+                ok = mbar_wait(smem_u32(&bars->v_full[stage]), (t / NS) & 1, abort) &&
+                     mbar_wait(smem_u32(&bars->p_full[buf]), (t >> 1) & 1, abort);
+                if (!ok) break;
+                tc_fence_after();
+                const uint32_t vb = smem_u32(v_s + stage * Sh::kV);
+                const int valid = keys - t * kTile < kTile ? keys - t * kTile : kTile;
+                const int steps = (valid + 15) >> 4;
+                for (int s = 0; s < steps; ++s) {
+                    const uint64_t vd = desc_sw128(vb + s * 2048, kColTile, 1024);
+                    mma_ts(tmem + kTmemO, tmem + kTmemS + buf * 128 + s * 8, vd, idesc_o, t > 0 || s > 0);
+                    mma_ts(tmem + kTmemO, tmem + kTmemLo + buf * 64 + s * 8, vd, idesc_o, true);
+                }
+                mma_commit(smem_u32(&bars->v_free[stage]));
+                mma_commit(smem_u32(&bars->p_free[buf]));
+                if (t + 2 < tiles)
+                    ok = mbar_wait(smem_u32(&bars->p_free[buf]), (t >> 1) & 1, abort) && scores(t + 2);
+            }
+            mma_commit(smem_u32(&bars->o_full));
+            mbar_wait(smem_u32(&bars->o_full), 0);  // nothing of this CTA is in the tensor pipe any more
+        }
+    } else {  // ---- scores to weights: warps 0-3 the even tiles, 4-7 the odd ones
+        const int wg = warp >> 2;
+        const int r = (warp & 3) * 32 + lane;
+        const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
+        const float c1 = -a.scale * kLog2e, c0 = -a.head_bias[h] * kLog2e;
+        bool ok = true;
+        for (int t = wg; t < tiles; t += 2) {
+            const int stage = t % NS;
+            ok = __all_sync(~0u, mbar_wait(smem_u32(&bars->s_full[wg]), (t >> 1) & 1, abort));
+            if (!ok) break;
+            tc_fence_after();
+            const int last = pos0 + r - t * kTile;  // last visible column of this row
+            const bool full = t * kTile + kTile - 1 <= pos0;
+            uint32_t buf[2][32];
+            const uint32_t sa = tmem + lanes + kTmemS + wg * 128, la = tmem + lanes + kTmemLo + wg * 64;
+            tmem_ld32(sa, buf[0]);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                uint32_t(&s)[32] = buf[c & 1];
+                tmem_wait_ld(s);
+                if (c < 3) tmem_ld32(sa + (c + 1) * 32, buf[(c + 1) & 1]);
+                uint32_t hi[16], lo[16];
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    float p0, p1;
+                    sigmoid2(fmaf(__uint_as_float(s[2 * i]), c1, c0), fmaf(__uint_as_float(s[2 * i + 1]), c1, c0), p0, p1);
+                    if (!full) {
+                        p0 = c * 32 + 2 * i <= last ? p0 : 0.0f;
+                        p1 = c * 32 + 2 * i + 1 <= last ? p1 : 0.0f;
+                    }
+                    split_bf16(p0, p1, hi[i], lo[i]);
+                }
+                // the hi half overlays score columns that have been read (16 c + 15 < 32 (c + 1))
+                tmem_st16(sa + c * 16, hi);
+                tmem_st16(la + c * 16, lo);
+            }
+            tmem_wait_st();
+            const int valid = keys - t * kTile;
+            if (valid < kTile && (valid & 15) != 0) {  // the last tile: clear the V rows its last MMA step reads beyond the end
+                ok = __all_sync(~0u, mbar_wait(smem_u32(&bars->v_full[stage]), (t / NS) & 1, abort));
+                if (!ok) break;
+                const int end = (valid + 15) & ~15;
+                for (int i = r; i < (end - valid) * CV * 8; i += 128) {
+                    const int c = i / ((end - valid) * 8), rest = i % ((end - valid) * 8);
+                    *reinterpret_cast<uint4*>(v_s + stage * Sh::kV + c * kColTile + (valid + (rest >> 3)) * 128 + ((rest & 7) << 4)) =
+                        make_uint4(0u, 0u, 0u, 0u);
+                }
+                fence_async_shared();
+            }
+            tc_fence_before();
+            mbar_arrive(smem_u32(&bars->p_full[wg]));
+        }
+        ok = __all_sync(~0u, ok && mbar_wait(smem_u32(&bars->o_full), 0, abort) && *abort == 0);
+        tc_fence_after();
+        const bool vec = a.vdim % 8 == 0 && a.out_stride % 8 == 0 && reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
+#pragma unroll
+        for (int c = 0; c < CV; ++c) {
+            const int col = (c * 2 + wg) * 32;
+            uint32_t o[32];
+            tmem_ld32(tmem + lanes + kTmemO + col, o);
+            tmem_wait_ld(o);
+            __nv_bfloat16* dst = out + r * a.out_stride + col;
+            if (r < nq && vec) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (col + 8 * i >= a.vdim) break;
+                    uint4 v;
+                    uint32_t* w = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+                        w[k] = ok ? pack_bf16(__uint_as_float(o[8 * i + 2 * k]) * a.out_scale, __uint_as_float(o[8 * i + 2 * k + 1]) * a.out_scale) : 0u;
+                    *reinterpret_cast<uint4*>(dst + 8 * i) = v;
+                }
+            } else if (r < nq) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i)
+                    if (col + i < a.vdim) dst[i] = __float2bfloat16_rn(ok ? __uint_as_float(o[i]) * a.out_scale : 0.0f);
+            }
+            __syncwarp();
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (threadIdx.x == 0 && *abort != 0) spk_flag(a.status, SPK_STATUS_DEVICE_WAIT_EXPIRED);
+    if (warp == 0) tmem_dealloc(tmem, 512);
+}
+
+template <int CK, int CV>
+int launch(const spk_sigmoid_attn_args& a, cudaStream_t s) {
+    constexpr int bytes = Shape<CK, CV>::kBytes;
+    static_assert(sizeof(Bars) <= 256 && bytes <= 227 * 1024, "shared memory");
+    const cudaError_t e = cudaFuncSetAttribute(sigmoid_prefill_kernel<CK, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return spk_set_cuda_error(e);
+    sigmoid_prefill_kernel<CK, CV><<<dim3(a.heads, a.n_tiles), kThreads, bytes, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+}  // namespace
+
+int spk_sigmoid_prefill_launch(const spk_sigmoid_attn_args& a, cudaStream_t s) {
+    if (a.n_tiles > 65535) return SPK_ERR_TOO_LARGE;
+    const int ck = a.k_pad / 64, cv = a.v_pad / 64;
+    if (ck == 1 && cv == 1) return launch<1, 1>(a, s);
+    if (ck == 1 && cv == 2) return launch<1, 2>(a, s);
+    if (ck == 2 && cv == 1) return launch<2, 1>(a, s);
+    return launch<2, 2>(a, s);
+}

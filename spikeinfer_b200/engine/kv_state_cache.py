@@ -31,13 +31,13 @@ class LayerCacheSpec:
 class PagedKVPool:
     """One K or V pool ``[num_blocks, kv_heads, block_size, pad]`` in the model dtype.
 
-    16-bit pools of up to 128 channels and pages of a multiple of eight rows are *tiled*: ``pad`` is the next multiple of 64
+    16-bit pools of up to 128 channels and pages of a multiple of sixteen rows are *tiled*: ``pad`` is the next multiple of 64
     and a page is stored in the 128-byte-swizzled order the tensor core reads shared memory in, so that a page copied as it
     is becomes part of an operand tile.  Other pools are plain rows.  Channels beyond ``dim`` stay zero."""
 
     def __init__(self, num_blocks: int, kv_heads: int, block_size: int, dim: int, dtype: torch.dtype, device) -> None:
         self.dim, self.block_size = dim, block_size
-        self.tiled = dtype == torch.bfloat16 and dim <= 128 and block_size % 8 == 0
+        self.tiled = dtype == torch.bfloat16 and dim <= 128 and block_size % 16 == 0
         self.pad = -(-dim // 64) * 64 if self.tiled else dim
         self.data = torch.zeros((num_blocks, kv_heads, block_size, self.pad), dtype=dtype, device=device)
 

@@ -110,31 +110,43 @@ def qk_prepare(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_pool, v_pool
 def sigmoid_attention(q: torch.Tensor, k_pool, v_pool, tables: torch.Tensor, head_bias: torch.Tensor, out: torch.Tensor, *,
                       heads: int, kv_heads: int, dim: int, vdim: int, scale: float, out_scale: float = 1.0,
                       plan=None, seq_lens: torch.Tensor | None = None, active: torch.Tensor | None = None,
-                      status: torch.Tensor | None = None) -> torch.Tensor:
+                      status: torch.Tensor | None = None, partial_sums: bool = False) -> torch.Tensor | None:
     """``out[t, h * vdim :] = out_scale * sum_j sigmoid(scale * q.k_j + head_bias[h]) v_j`` over the keys up to token t's own
     position, read through ``tables``.  ``out`` is a column range of a row-major matrix in the model dtype.  ``plan`` (a
-    ``PrefillPlan``): prefill form; None: decode form over ``seq_lens`` / ``active``."""
+    ``PrefillPlan``): prefill form; None: decode form over ``seq_lens`` / ``active``.
+
+    ``partial_sums`` (decode form): where the sizes allow it, leave ``out`` alone and return fp32 partial sums
+    ``[n, splits, heads * vdim]`` of key ranges, for :func:`gated_norm` to add up; otherwise ``out`` is written and None
+    returned."""
     _lib.require_cuda(q, "sigmoid_attention query")
     _f32(head_bias, "head_bias", heads)
     n = q.shape[0]
     if out.shape != (n, heads * vdim) or out.stride(1) != 1 or out.dtype != q.dtype:
         raise ValueError("out must be [n, heads * vdim] in the dtype of q with unit column stride")
-    tiles = None if plan is None else plan.tiles(int(_lib.load().spk_sigmoid_attn_tile_tokens()))
+    lib = _lib.load()
+    form = (_lib.dtype_code(q.dtype), k_pool.pad, v_pool.pad, int(k_pool.tiled), int(v_pool.tiled), k_pool.block_size)
+    tiles = None if plan is None else plan.tiles(int(lib.spk_sigmoid_attn_tile_tokens(*form)))
+    partials, splits = None, 0
+    if partial_sums and plan is None:
+        splits = int(lib.spk_sigmoid_attn_splits(*form, n, heads, kv_heads, tables.shape[1] * k_pool.block_size))
+        if splits:
+            partials = torch.empty((n, splits, heads * vdim), dtype=torch.float32, device=q.device)
     a = _lib.SigmoidAttnArgs(
         q=q.data_ptr(), k_pool=k_pool.data.data_ptr(), v_pool=v_pool.data.data_ptr(), tables=tables.data_ptr(),
         seq_lens=_ptr(seq_lens), active=_ptr(active), tiles=_ptr(tiles), head_bias=head_bias.data_ptr(), out=out.data_ptr(),
         out_stride=out.stride(0), table_stride=tables.stride(0), table_rows=tables.shape[0], max_blocks=tables.shape[1], n=n,
-        num_blocks=k_pool.data.shape[0], n_tiles=0 if tiles is None else tiles.shape[0], heads=heads, kv_heads=kv_heads, dim=dim,
-        vdim=vdim, k_pad=k_pool.pad, v_pad=v_pool.pad, k_tiled=int(k_pool.tiled), v_tiled=int(v_pool.tiled),
-        block_size=k_pool.block_size, dtype=_lib.dtype_code(q.dtype), scale=scale, out_scale=out_scale, status=_ptr(status))
+        num_blocks=k_pool.data.shape[0], partials=_ptr(partials), n_tiles=0 if tiles is None else tiles.shape[0], splits=splits,
+        heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, k_pad=k_pool.pad, v_pad=v_pool.pad, k_tiled=int(k_pool.tiled),
+        v_tiled=int(v_pool.tiled), block_size=k_pool.block_size, dtype=form[0], scale=scale, out_scale=out_scale,
+        status=_ptr(status))
     _call("spk_sigmoid_attn", a, q.device)
-    return out
+    return partials
 
 
 def decay_powers(decay, device) -> torch.Tensor:
-    """fp32 ``[heads, chunk + 1]``: the powers of every head's decay, evaluated in double precision."""
+    """fp32 ``[heads, powers]``: the powers 0, 1, 2 ... of every head's decay, evaluated in double precision."""
     d = torch.tensor(list(decay), dtype=torch.float64)
-    n = torch.arange(int(_lib.load().spk_decay_chunk_tokens()) + 1, dtype=torch.float64)
+    n = torch.arange(int(_lib.load().spk_decay_powers()), dtype=torch.float64)
     return (d[:, None] ** n[None, :]).to(torch.float32).to(device).contiguous()
 
 
@@ -161,7 +173,7 @@ def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: to
     if plan is None:
         _call("spk_decay_attn_step", a, q.device)
         return out
-    chunks, seqs = plan.chunks(int(lib.spk_decay_chunk_tokens()))
+    chunks, seqs = plan.chunks(int(lib.spk_decay_chunk_tokens(a.dtype, dim, vdim, n, heads)))
     need = int(lib.spk_decay_attn_workspace_bytes(chunks.shape[0], heads, dim, vdim))
     ws = torch.empty(need, dtype=torch.uint8, device=q.device)
     a.chunks, a.seqs, a.n_chunks, a.n_seqs = chunks.data_ptr(), seqs.data_ptr(), chunks.shape[0], seqs.shape[0]
@@ -171,16 +183,21 @@ def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: to
 
 
 def gated_norm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, out_offset: int, *, eps: float,
-               scale: float = 1.0, active: torch.Tensor | None = None) -> torch.Tensor:
-    """``out[:, out_offset:] = scale * rmsnorm(x) * weight * sigmoid(gate)`` over the whole width of ``x`` (fp32)."""
+               scale: float = 1.0, partials: torch.Tensor | None = None, left_scale: float = 1.0,
+               seq_lens: torch.Tensor | None = None, active: torch.Tensor | None = None) -> torch.Tensor:
+    """``out[:, out_offset:] = scale * rmsnorm(x) * weight * sigmoid(gate)`` over the whole width of ``x`` (fp32); with
+    ``partials`` of :func:`sigmoid_attention` also ``out[:, :left_width] = left_scale * (their sum)``."""
     _lib.require_cuda(x, "gated_norm input")
     n, width = x.shape
     _f32(x, "x")
     _f32(weight, "weight", width)
+    _f32(partials, "partials")
     if gate.shape != (n, width) or gate.stride(1) != 1 or gate.dtype != out.dtype or out.stride(1) != 1 or out.shape[1] < out_offset + width:
         raise ValueError("gate and out must be row-major in the model dtype and wide enough")
     a = _lib.GatedNormArgs(x=x.data_ptr(), w=weight.data_ptr(), gate=gate.data_ptr(), gate_stride=gate.stride(0), out=out.data_ptr(),
-                           out_stride=out.stride(0), active=_ptr(active), n=n, width=width, out_offset=out_offset,
-                           dtype=_lib.dtype_code(out.dtype), eps=eps, scale=scale)
+                           out_stride=out.stride(0), partials=_ptr(partials), seq_lens=_ptr(seq_lens), active=_ptr(active), n=n,
+                           width=width, out_offset=out_offset, splits=0 if partials is None else partials.shape[1],
+                           left_width=0 if partials is None else partials.shape[2], dtype=_lib.dtype_code(out.dtype), eps=eps,
+                           scale=scale, left_scale=left_scale)
     _call("spk_gated_norm", a, x.device)
     return out

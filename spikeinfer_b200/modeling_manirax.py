@@ -192,14 +192,17 @@ class ManiraxModel:
                        positions=positions, status=meta.status, **heads)
         common = dict(scale=lf.scale, out_scale=L.cfg.left_scale, status=meta.status, **heads)
         left = both[:, : L.left_width]
+        partials = None
         if meta.num_prefills:
             plan, active = meta.prefill_plan(), None
             sigmoid_attention(q, cache.k, cache.v, meta.row_tables, L.head_bias, left, plan=plan, **common)
         else:
             plan, active = None, meta.row_active
-            sigmoid_attention(q, cache.k, cache.v, meta.block_tables, L.head_bias, left, seq_lens=meta.seq_lens, active=active, **common)
+            partials = sigmoid_attention(q, cache.k, cache.v, meta.block_tables, L.head_bias, left, seq_lens=meta.seq_lens,
+                                         active=active, partial_sums=True, **common)
         o = decay_attention(rq, rk, rv, cache.states["decay"], L.decay, plan=plan, active=active, status=meta.status)
-        gated_norm(o, L.right_norm, rg, both, L.left_width, eps=eps, scale=L.cfg.right_scale, active=active)
+        gated_norm(o, L.right_norm, rg, both, L.left_width, eps=eps, scale=L.cfg.right_scale, partials=partials,
+                   left_scale=L.cfg.left_scale, seq_lens=meta.seq_lens, active=active)
         return self._matmul_f32(both, L.w_out)
 
     @torch.no_grad()
