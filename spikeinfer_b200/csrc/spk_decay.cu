@@ -40,44 +40,50 @@ decay_step_kernel(const spk_decay_attn_args a) {
     float* k = q + dim;
     float* v = k + dim;
     float* red = v + vdim;
-    const T* qr = static_cast<const T*>(a.q) + row * a.ld + static_cast<int64_t>(h) * dim;
-    const T* kr = static_cast<const T*>(a.k) + row * a.ld + static_cast<int64_t>(h) * dim;
-    const T* vr = static_cast<const T*>(a.v) + row * a.ld + static_cast<int64_t>(h) * vdim;
-    for (int d = threadIdx.x; d < dim; d += kThreads) {
-        q[d] = act(spk_to_float<T>(qr[d]), a.silu);
-        k[d] = act(spk_to_float<T>(kr[d]), a.silu);
-    }
-    for (int e = threadIdx.x; e < vdim; e += kThreads) v[e] = act(spk_to_float<T>(vr[e]), a.silu);
-    __syncthreads();
-    const float decay = a.decay_pow[h * kPow + 1];
     float* S = a.state + row * a.state_stride + static_cast<int64_t>(h) * dim * vdim;
     const int cols = vdim / W;
     const int slices = cols < kThreads ? kThreads / cols : 1;
     const int slice = threadIdx.x / cols;
+    constexpr int U = 8;  // state rows in flight per thread
+    float s[U][W];
+    auto load = [&](int d0, int c) {
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int d = d0 + u * slices;
+            if (d < dim) {
+                if (W == 4) {
+                    const float4 f = __ldcs(reinterpret_cast<const float4*>(S + static_cast<int64_t>(d) * vdim + c * W));
+                    s[u][0] = f.x; s[u][1 % W] = f.y; s[u][2 % W] = f.z; s[u][3 % W] = f.w;
+                } else {
+                    s[u][0] = S[static_cast<int64_t>(d) * vdim + c];
+                }
+            }
+        }
+    };
+    // the first rows are on their way before the projections are looked at
+    const bool mine = slice < slices;
+    const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
+    if (mine && first < cols) load(slice, first);
+    const T* qr = static_cast<const T*>(a.q) + row * a.ld + static_cast<int64_t>(h) * dim;
+    const T* kr = static_cast<const T*>(a.k) + row * a.ld + static_cast<int64_t>(h) * dim;
+    const T* vr = static_cast<const T*>(a.v) + row * a.ld + static_cast<int64_t>(h) * vdim;
+    for (int i = threadIdx.x; i < 2 * dim + vdim; i += kThreads) {
+        const T* src = i < dim ? qr + i : i < 2 * dim ? kr + (i - dim) : vr + (i - 2 * dim);
+        sm[i] = act(spk_to_float<T>(*src), a.silu);
+    }
+    __syncthreads();
+    const float decay = a.decay_pow[h * kPow + 1];
     for (int c0 = 0; c0 < cols; c0 += kThreads) {
-        const int c = c0 + (slices > 1 ? threadIdx.x % cols : threadIdx.x);
-        if (slice >= slices || c >= cols) continue;
+        const int c = c0 + first;
+        if (!mine || c >= cols) continue;
         float acc[W];
 #pragma unroll
         for (int i = 0; i < W; ++i) acc[i] = 0.0f;
         float vv[W];
 #pragma unroll
         for (int i = 0; i < W; ++i) vv[i] = v[c * W + i];
-        constexpr int U = 4;  // state rows in flight per thread
         for (int d0 = slice; d0 < dim; d0 += U * slices) {
-            float s[U][W];
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                const int d = d0 + u * slices;
-                if (d < dim) {
-                    if (W == 4) {
-                        const float4 f = *reinterpret_cast<const float4*>(S + static_cast<int64_t>(d) * vdim + c * W);
-                        s[u][0] = f.x; s[u][1 % W] = f.y; s[u][2 % W] = f.z; s[u][3 % W] = f.w;
-                    } else {
-                        s[u][0] = S[static_cast<int64_t>(d) * vdim + c];
-                    }
-                }
-            }
+            if (c0 > 0 || d0 > slice) load(d0, c);
 #pragma unroll
             for (int u = 0; u < U; ++u) {
                 const int d = d0 + u * slices;
@@ -89,8 +95,8 @@ decay_step_kernel(const spk_decay_attn_args a) {
                         acc[i] = fmaf(qd, s[u][i], acc[i]);
                     }
                     if (W == 4)
-                        *reinterpret_cast<float4*>(S + static_cast<int64_t>(d) * vdim + c * W) =
-                            make_float4(s[u][0], s[u][1 % W], s[u][2 % W], s[u][3 % W]);
+                        __stcs(reinterpret_cast<float4*>(S + static_cast<int64_t>(d) * vdim + c * W),
+                               make_float4(s[u][0], s[u][1 % W], s[u][2 % W], s[u][3 % W]));
                     else
                         S[static_cast<int64_t>(d) * vdim + c] = s[u][0];
                 }

@@ -21,47 +21,59 @@ constexpr int C = kDecayChunk;
 // x * sigmoid(x): 1 / (1 + 2^(-x log2 e))
 __device__ __forceinline__ float silu_fast(float x) { return x * rcp(1.0f + ex2(-1.4426950408889634f * x)); }
 
-__device__ __forceinline__ void load8(const __nv_bfloat16* p, int left, bool vec, float (&f)[8]) {
-    if (vec && left >= 8) {
-        const uint4 u = *reinterpret_cast<const uint4*>(p);
-        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+// Rows of one head of a chunk on their way into a shared-memory tile [64][W + 8]; rows and channels beyond the data are zero.
+// Asynchronous where the rows are 16-byte aligned.  A thread later transforms the very items it copied, so it needs no
+// barrier before that, only its own copies to have landed.
+template <int W>
+__device__ __forceinline__ void fetch(__nv_bfloat16* dst, const __nv_bfloat16* src, int64_t ld, int len, int width, bool vec) {
+    constexpr int ST = W + 8;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            f[2 * i] = __uint_as_float(w[i] << 16);
-            f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    for (int it = 0; it < C * (W / 8) / kThreads; ++it) {
+        const int i = threadIdx.x + it * kThreads;
+        const int r = i / (W / 8), c = (i % (W / 8)) * 8;
+        if (vec) {
+            const bool live = r < len && c < width;
+            cp_async16(smem_u32(dst + r * ST + c), live ? src + r * ld + c : src, live);
+        } else {
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+                dst[r * ST + c + k] = r < len && c + k < width ? src[r * ld + c + k] : __float2bfloat16_rn(0.0f);
         }
-    } else {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = i < left ? __bfloat162float(p[i]) : 0.0f;
     }
 }
 
-// Rows of one head of a chunk: activation, then to shared memory as bf16 (plain != NULL) and, times the row's decay
-// weight pw[top - row], as a bf16 pair (hi, lo != NULL).  Rows and channels beyond the data are zero.
-template <int W>
-__device__ __forceinline__ void stage(const __nv_bfloat16* src, int64_t ld, int len, int width, int silu, bool vec,
-                                      __nv_bfloat16* plain, __nv_bfloat16* hi, __nv_bfloat16* lo, const float* pw, int top) {
+// Activation of a fetched tile, in place (PLAIN) and, times the row's decay weight pw[top - row], as a bf16 pair (hi != NULL).
+template <int W, bool PLAIN>
+__device__ __forceinline__ void activate(__nv_bfloat16* tile, int len, int silu, __nv_bfloat16* hi, __nv_bfloat16* lo, const float* pw, int top) {
     constexpr int ST = W + 8;
-    for (int i = threadIdx.x; i < C * (W / 8); i += kThreads) {
+#pragma unroll
+    for (int it = 0; it < C * (W / 8) / kThreads; ++it) {
+        const int i = threadIdx.x + it * kThreads;
         const int r = i / (W / 8), c = (i % (W / 8)) * 8;
+        const uint4 u = *reinterpret_cast<const uint4*>(tile + r * ST + c);
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
         float f[8];
-        load8(src + r * ld + c, r < len ? width - c : 0, vec, f);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            f[2 * k] = __uint_as_float(w[k] << 16);
+            f[2 * k + 1] = __uint_as_float(w[k] & 0xffff0000u);
+        }
         if (silu) {
 #pragma unroll
             for (int k = 0; k < 8; ++k) f[k] = silu_fast(f[k]);
+            if (PLAIN)
+                *reinterpret_cast<uint4*>(tile + r * ST + c) =
+                    make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
         }
-        if (plain != nullptr)
-            *reinterpret_cast<uint4*>(plain + r * ST + c) =
-                make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
         if (hi != nullptr) {
-            const float w = r < len ? pw[top - r] : 0.0f;
-            uint4 a, b;
-            split_bf16(f[0] * w, f[1] * w, a.x, b.x);
-            split_bf16(f[2] * w, f[3] * w, a.y, b.y);
-            split_bf16(f[4] * w, f[5] * w, a.z, b.z);
-            split_bf16(f[6] * w, f[7] * w, a.w, b.w);
-            *reinterpret_cast<uint4*>(hi + r * ST + c) = a;
-            *reinterpret_cast<uint4*>(lo + r * ST + c) = b;
+            const float d = r < len ? pw[top - r] : 0.0f;
+            uint4 x, y;
+            split_bf16(f[0] * d, f[1] * d, x.x, y.x);
+            split_bf16(f[2] * d, f[3] * d, x.y, y.y);
+            split_bf16(f[4] * d, f[5] * d, x.z, y.z);
+            split_bf16(f[6] * d, f[7] * d, x.w, y.w);
+            *reinterpret_cast<uint4*>(hi + r * ST + c) = x;
+            *reinterpret_cast<uint4*>(lo + r * ST + c) = y;
         }
     }
 }
@@ -108,20 +120,30 @@ decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
     extern __shared__ __align__(16) __nv_bfloat16 sm[];
     __nv_bfloat16* hi = sm;
     __nv_bfloat16* lo = hi + C * SK;
-    __nv_bfloat16* v = lo + C * SK;
+    __nv_bfloat16* kb = lo + C * SK;      // two stages each of k and v
+    __nv_bfloat16* vb = kb + 2 * C * SK;
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const SpkChunk ci = spk_chunk(a, blockIdx.x);
     const float* pw = a.decay_pow + static_cast<int64_t>(h) * (kDecayMaxSpan + 1);
     const __nv_bfloat16* ks = static_cast<const __nv_bfloat16*>(a.k) + ci.start * a.ld + static_cast<int64_t>(h) * a.dim;
     const __nv_bfloat16* vs = static_cast<const __nv_bfloat16*>(a.v) + ci.start * a.ld + static_cast<int64_t>(h) * a.vdim;
     float acc[T::NT][4] = {};
-    for (int c0 = 0; c0 < ci.len; c0 += C) {
+    auto fetch_chunk = [&](int c0, int buf) {
         const int len = min(C, ci.len - c0);
+        fetch<T::D>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::V>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
+        cp_async_commit();
+    };
+    fetch_chunk(0, 0);
+    for (int c0 = 0, buf = 0; c0 < ci.len; c0 += C, buf ^= 1) {
+        const int len = min(C, ci.len - c0);
+        cp_async_wait_all();
+        __syncthreads();  // the previous chunk's products have read their operands
+        activate<T::D, false>(kb + buf * C * SK, len, a.silu, hi, lo, pw, ci.len - 1 - c0);
+        activate<T::V, true>(vb + buf * C * SV, len, a.silu, nullptr, nullptr, pw, 0);
+        if (c0 + C < ci.len) fetch_chunk(c0 + C, buf ^ 1);
         __syncthreads();
-        stage<T::D>(ks + c0 * a.ld, a.ld, len, a.dim, a.silu, vec_k, nullptr, hi, lo, pw, ci.len - 1 - c0);
-        stage<T::V>(vs + c0 * a.ld, a.ld, len, a.vdim, a.silu, vec_v, v, nullptr, nullptr, pw, 0);
-        __syncthreads();
-        add_outer<CD, CV>(acc, hi, lo, v, warp, lane);
+        add_outer<CD, CV>(acc, hi, lo, vb + buf * C * SV, warp, lane);
     }
     float* U = a.workspace + (static_cast<int64_t>(blockIdx.x) * a.heads + h) * a.dim * a.vdim;
     const int gid = lane >> 2, tig = lane & 3;
@@ -135,17 +157,17 @@ decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
 }
 
 template <int CD, int CV>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, CD * CV == 1 ? 2 : 1)
 decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool vec_v) {
     using T = StateTile<CD, CV>;
     constexpr int SK = T::D + 8, SV = T::V + 8;
     extern __shared__ __align__(16) __nv_bfloat16 sm[];
-    __nv_bfloat16* q = sm;
-    __nv_bfloat16* k = q + C * SK;
-    __nv_bfloat16* hi = k + C * SK;
+    __nv_bfloat16* qb = sm;               // two stages each of q, k and v
+    __nv_bfloat16* kb = qb + 2 * C * SK;
+    __nv_bfloat16* vb = kb + 2 * C * SK;
+    __nv_bfloat16* hi = vb + 2 * C * SV;  // decayed keys
     __nv_bfloat16* lo = hi + C * SK;
-    __nv_bfloat16* v = lo + C * SK;
-    __nv_bfloat16* sh = v + C * SV;   // state, hi and lo
+    __nv_bfloat16* sh = lo + C * SK;      // state, hi and lo
     __nv_bfloat16* sl = sh + T::D * SV;
     float* pw = reinterpret_cast<float*>(sl + T::D * SV);  // powers 0 .. 64 of this head's decay
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
@@ -167,13 +189,24 @@ decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
     const int i0 = (warp & 3) * 16;                 // this warp's 16 tokens
     constexpr int OC = T::V / 2, ON = OC / 8;       // and its half of the output columns
     const int e0 = (warp >> 2) * OC;
-    for (int c0 = 0; c0 < ci.len; c0 += C) {
+    auto fetch_chunk = [&](int c0, int buf) {
+        const int len = min(C, ci.len - c0);
+        fetch<T::D>(qb + buf * C * SK, qs + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::D>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::V>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
+        cp_async_commit();
+    };
+    fetch_chunk(0, 0);
+    for (int c0 = 0, buf = 0; c0 < ci.len; c0 += C, buf ^= 1) {
         const int len = min(C, ci.len - c0);
         const bool more = c0 + C < ci.len;
+        __nv_bfloat16 *q = qb + buf * C * SK, *k = kb + buf * C * SK, *v = vb + buf * C * SV;
+        cp_async_wait_all();
         __syncthreads();  // the previous chunk's reads are done (and pw is there)
-        stage<T::D>(qs + c0 * a.ld, a.ld, len, a.dim, a.silu, vec_k, q, nullptr, nullptr, pw, 0);
-        stage<T::D>(ks + c0 * a.ld, a.ld, len, a.dim, a.silu, vec_k, k, more ? hi : nullptr, lo, pw, len - 1);
-        stage<T::V>(vs + c0 * a.ld, a.ld, len, a.vdim, a.silu, vec_v, v, nullptr, nullptr, pw, 0);
+        activate<T::D, true>(q, len, a.silu, nullptr, nullptr, pw, 0);
+        activate<T::D, true>(k, len, a.silu, more ? hi : nullptr, lo, pw, len - 1);
+        activate<T::V, true>(v, len, a.silu, nullptr, nullptr, pw, 0);
+        if (more) fetch_chunk(c0 + C, buf ^ 1);
 #pragma unroll
         for (int n = 0; n < T::NT; ++n)
 #pragma unroll
@@ -286,13 +319,13 @@ int with_smem(F fn, size_t bytes, cudaStream_t s, const spk_decay_attn_args& a) 
 
 template <int CD, int CV>
 int sums(const spk_decay_attn_args& a, cudaStream_t s) {
-    constexpr size_t bytes = 2 * C * (2 * (CD * 64 + 8) + CV * 64 + 8);
+    constexpr size_t bytes = 2 * C * (4 * (CD * 64 + 8) + 2 * (CV * 64 + 8));
     return with_smem(decay_span_sum_kernel<CD, CV>, bytes, s, a);
 }
 
 template <int CD, int CV>
 int outputs(const spk_decay_attn_args& a, cudaStream_t s) {
-    constexpr size_t bytes = 2 * C * (4 * (CD * 64 + 8) + CV * 64 + 8) + 4 * CD * 64 * (CV * 64 + 8) + 4 * (C + 8);
+    constexpr size_t bytes = 2 * C * (6 * (CD * 64 + 8) + 2 * (CV * 64 + 8)) + 4 * CD * 64 * (CV * 64 + 8) + 4 * (C + 8);
     static_assert(bytes <= 227 * 1024, "shared memory");
     return with_smem(decay_span_out_kernel<CD, CV>, bytes, s, a);
 }
