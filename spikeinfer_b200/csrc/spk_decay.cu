@@ -299,6 +299,75 @@ gated_norm_kernel(const spk_gated_norm_args a) {
     }
 }
 
+// The same with four columns per access: at most 4 * kThreads * V columns, every operand aligned to four elements.
+template <typename T, int V>
+__global__ void __launch_bounds__(kThreads)
+gated_norm_vec_kernel(const spk_gated_norm_args a) {
+    __shared__ float part[32];
+    const int64_t t = blockIdx.x;
+    T* out = static_cast<T*>(a.out) + t * a.out_stride;
+    const bool live = a.active == nullptr || a.active[t] == 1;
+    const float* x = a.x + t * a.width;
+    const T* g = static_cast<const T*>(a.gate) + t * a.gate_stride;
+    float4 xv[V], gv[V], wv[V];
+    float ss[1] = {0.0f};
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (threadIdx.x + i * blockDim.x);
+        xv[i] = spk_load4<float, true>(x + c, a.width - c);
+        gv[i] = spk_load4<T, true>(g + c, a.width - c);
+        wv[i] = spk_load4<float, true>(a.w + c, a.width - c);
+    }
+    if (a.partials != nullptr) {
+        const int len = live ? a.seq_lens[t] : 0;
+        const int per = spk_split_keys(len, a.splits);
+        const int valid = (len + per - 1) / per;
+        const float* p = a.partials + t * a.splits * a.left_width;
+        for (int c = 4 * threadIdx.x; c < a.left_width; c += 4 * blockDim.x) {
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int k = 0; k < valid; ++k) {
+                const float4 y = spk_load4<float, true>(p + static_cast<int64_t>(k) * a.left_width + c, 4);
+                s.x += y.x; s.y += y.y; s.z += y.z; s.w += y.w;
+            }
+            const float m = a.left_scale;
+            spk_store4<T, true>(out + c, make_float4(s.x * m, s.y * m, s.z * m, s.w * m), 4);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss[0] += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+    spk_block_sum<1>(ss, part);
+    const float inv = a.scale / sqrtf(ss[0] / static_cast<float>(a.width) + a.eps);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (threadIdx.x + i * blockDim.x);
+        const float4 y = make_float4(xv[i].x * inv * wv[i].x * spk_sigmoid(gv[i].x), xv[i].y * inv * wv[i].y * spk_sigmoid(gv[i].y),
+                                     xv[i].z * inv * wv[i].z * spk_sigmoid(gv[i].z), xv[i].w * inv * wv[i].w * spk_sigmoid(gv[i].w));
+        spk_store4<T, true>(out + a.out_offset + c, live ? y : make_float4(0.f, 0.f, 0.f, 0.f), a.width - c);
+    }
+}
+
+template <typename T>
+int launch_gated(const spk_gated_norm_args& a, cudaStream_t s) {
+    const unsigned grid = static_cast<unsigned>(a.n);
+    auto aligned = [](const void* p, size_t bytes) { return reinterpret_cast<uintptr_t>(p) % bytes == 0; };
+    const bool vec = a.width % 4 == 0 && a.width <= 4 * kThreads * 4 && a.out_offset % 4 == 0 && a.out_stride % 4 == 0 && a.gate_stride % 4 == 0 &&
+                     aligned(a.x, 16) && aligned(a.w, 16) && aligned(a.gate, 4 * sizeof(T)) && aligned(a.out, 4 * sizeof(T)) &&
+                     (a.partials == nullptr || (a.left_width % 4 == 0 && aligned(a.partials, 16)));
+    if (!vec) {
+        gated_norm_kernel<T><<<grid, kThreads, 0, s>>>(a);
+    } else {
+        const int groups = a.width / 4;
+        const int threads = groups <= 128 && a.partials == nullptr ? 128 : kThreads;
+        const int v = (groups + threads - 1) / threads;
+        if (v <= 1) gated_norm_vec_kernel<T, 1><<<grid, threads, 0, s>>>(a);
+        else if (v <= 2) gated_norm_vec_kernel<T, 2><<<grid, threads, 0, s>>>(a);
+        else gated_norm_vec_kernel<T, 4><<<grid, threads, 0, s>>>(a);
+    }
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
 int check_decay(const spk_decay_attn_args* a) {
     if (a == nullptr) return SPK_ERR_NULL_POINTER;
     if (a->n < 0 || a->heads < 1 || a->dim < 1 || a->vdim < 1 || a->state_rows < 1 || a->heads > 65535) return SPK_ERR_BAD_SHAPE;
@@ -412,8 +481,5 @@ extern "C" int spk_gated_norm(const spk_gated_norm_args* a, void* stream) {
                                    a->left_width > a->out_offset))
         return SPK_ERR_BAD_SHAPE;
     cudaStream_t s = spk_stream(stream);
-    if (a->dtype == SPK_F32) gated_norm_kernel<float><<<static_cast<unsigned>(a->n), kThreads, 0, s>>>(*a);
-    else gated_norm_kernel<__nv_bfloat16><<<static_cast<unsigned>(a->n), kThreads, 0, s>>>(*a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return a->dtype == SPK_F32 ? launch_gated<float>(*a, s) : launch_gated<__nv_bfloat16>(*a, s);
 }

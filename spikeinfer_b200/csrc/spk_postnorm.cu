@@ -3,7 +3,7 @@
 //  * residual_norm_kernel: x' = layernorm(alpha * x + delta) * w (mean removed, no bias), or x' = embedding row; then
 //    what the next sublayer reads: x' itself, x' mixed per channel with the previous token's x' (token shift), or a second
 //    layer norm of x' (the model's last).  One launch per sublayer boundary.
-//  * poly_norm_kernel: a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square.
+//  * poly_norm_kernel, poly_norm_packed_kernel: a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's root mean square.
 //
 // The previous token's row is recomputed by the CTA that needs it when it lies in the same launch (it depends on nothing
 // but its own x and delta), and read from the sequence's state when the token is the first of its portion.  The
@@ -195,6 +195,78 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ coef, float 
     }
 }
 
+// bf16 rows in 16-byte groups that stay packed in registers between the two passes: G groups per thread.
+template <int G>
+__global__ void __launch_bounds__(512)
+poly_norm_packed_kernel(const __nv_bfloat16* __restrict__ z, const float* __restrict__ coef, float eps, __nv_bfloat16* __restrict__ out, int width) {
+    __shared__ float part[3 * 32];
+    const uint4* zr = reinterpret_cast<const uint4*>(z + static_cast<int64_t>(blockIdx.x) * width);
+    uint4* o = reinterpret_cast<uint4*>(out + static_cast<int64_t>(blockIdx.x) * width);
+    const int groups = width / 8;
+    uint4 raw[G];
+#pragma unroll
+    for (int v = 0; v < G; ++v) {
+        const int i = threadIdx.x + v * blockDim.x;
+        raw[v] = i < groups ? zr[i] : make_uint4(0u, 0u, 0u, 0u);
+    }
+    float s[3] = {0.0f, 0.0f, 0.0f};
+    auto moments = [&](float x) {
+        const float q = x * x;
+        s[0] += q;
+        s[1] = fmaf(q, q, s[1]);
+        s[2] = fmaf(q * q, q, s[2]);
+    };
+#pragma unroll
+    for (int v = 0; v < G; ++v) {
+        const uint32_t w[4] = {raw[v].x, raw[v].y, raw[v].z, raw[v].w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            moments(__uint_as_float(w[k] << 16));
+            moments(__uint_as_float(w[k] & 0xffff0000u));
+        }
+    }
+    spk_block_sum<3>(s, part);
+    const float n = static_cast<float>(width);
+    const float k1 = coef[0] / sqrtf(s[0] / n + eps), k2 = coef[1] / sqrtf(s[1] / n + eps);
+    const float k3 = coef[2] / sqrtf(s[2] / n + eps), k0 = coef[3];
+    auto f = [&](float x) { return fmaf(x, fmaf(x, fmaf(x, k3, k2), k1), k0); };
+#pragma unroll
+    for (int v = 0; v < G; ++v) {
+        const int i = threadIdx.x + v * blockDim.x;
+        uint32_t w[4] = {raw[v].x, raw[v].y, raw[v].z, raw[v].w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const __nv_bfloat162 b = __floats2bfloat162_rn(f(__uint_as_float(w[k] << 16)), f(__uint_as_float(w[k] & 0xffff0000u)));
+            w[k] = *reinterpret_cast<const uint32_t*>(&b);
+        }
+        if (i < groups) o[i] = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+}
+
+int launch_poly_packed(const void* z, const float* coef, float eps, void* out, int64_t rows, int64_t width, cudaStream_t s) {
+    const int groups = static_cast<int>(width / 8);
+    int threads = groups <= 512 ? 128 : groups <= 2048 ? 256 : 512;
+    if (rows < 2 * 148) threads = groups <= 128 ? 128 : groups <= 256 ? 256 : 512;  // few rows: spread a row wider
+    const int g = (groups + threads - 1) / threads;
+    const unsigned grid = static_cast<unsigned>(rows);
+    const __nv_bfloat16* zi = static_cast<const __nv_bfloat16*>(z);
+    __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+    const int w = static_cast<int>(width);
+#define SPK_PP(G_) poly_norm_packed_kernel<G_><<<grid, threads, 0, s>>>(zi, coef, eps, o, w)
+    switch (g) {
+        case 1: SPK_PP(1); break;
+        case 2: SPK_PP(2); break;
+        case 3: SPK_PP(3); break;
+        case 4: SPK_PP(4); break;
+        case 5: SPK_PP(5); break;
+        case 6: SPK_PP(6); break;
+        default: SPK_PP(8); break;
+    }
+#undef SPK_PP
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
 // Threads per row and four-element groups per thread for a row of `width` elements; 0 when too wide.
 int row_shape(int64_t width, int* v) {
     const int64_t groups = (width + 3) / 4;
@@ -296,6 +368,8 @@ extern "C" int spk_poly_norm(const void* z, const float* coef, float eps, void* 
     if (z == nullptr || coef == nullptr || out == nullptr) return SPK_ERR_NULL_POINTER;
     cudaStream_t s = spk_stream(stream);
     if (dtype == SPK_F32) return launch_poly<float>(z, coef, eps, out, rows, width, s);
+    if (dtype == SPK_BF16 && width % 8 == 0 && width <= 8 * 512 * 8 && reinterpret_cast<uintptr_t>(z) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0)
+        return launch_poly_packed(z, coef, eps, out, rows, width, s);
     if (dtype == SPK_BF16) return launch_poly<__nv_bfloat16>(z, coef, eps, out, rows, width, s);
     return SPK_ERR_BAD_DTYPE;
 }
