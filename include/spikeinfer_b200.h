@@ -521,7 +521,7 @@ typedef struct spk_sigmoid_attn_args {
     int32_t dtype;
     float scale;
     float out_scale;
-    float _pad;
+    int32_t overlap;            /* partial form only: see below */
     uint32_t* status;
 } spk_sigmoid_attn_args;
 int spk_sigmoid_attn_tile_tokens(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size);
@@ -557,9 +557,13 @@ typedef struct spk_decay_attn_args {
     int32_t heads, dim, vdim;
     int32_t silu;
     int32_t dtype;
-    int32_t _pad;
+    int32_t overlap;            /* _step only: see below */
     uint32_t* status;
 } spk_decay_attn_args;
+/* Launch overlap in a decode layer: spk_qk_prepare, then spk_decay_attn_step with overlap, then spk_sigmoid_attn (partial form)
+ * with overlap, back to back on one stream.  The caller vouches that the projections, tables and lengths were complete before
+ * spk_qk_prepare began.  The step kernel may then be placed while qk_prepare still runs, and lets the attention start only when
+ * qk_prepare is complete; the attention runs beside the step and both are complete when the launch after them begins. */
 int spk_decay_powers(void);
 /* Tokens per chunk of the prefill form for a call of n tokens: chunks may not be longer. */
 int spk_decay_chunk_tokens(int dtype, int dim, int vdim, int64_t n, int heads);

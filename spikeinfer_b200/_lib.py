@@ -116,14 +116,14 @@ class SigmoidAttnArgs(Structure):
 
     _fields_ = _fields("p q k_pool v_pool tables seq_lens active tiles head_bias out; l out_stride table_stride table_rows "
                        "max_blocks n num_blocks; p partials; i n_tiles splits heads kv_heads dim vdim k_pad v_pad k_tiled v_tiled block_size dtype; "
-                       "f scale out_scale _pad; p status")
+                       "f scale out_scale; i overlap; p status")
 
 
 class DecayAttnArgs(Structure):
     """Mirror of ``spk_decay_attn_args``."""
 
     _fields_ = _fields("p q k v; l ld; p state; l state_stride state_rows; p decay_pow out active chunks seqs workspace; "
-                       "l workspace_bytes n; i n_chunks n_seqs heads dim vdim silu dtype _pad; p status")
+                       "l workspace_bytes n; i n_chunks n_seqs heads dim vdim silu dtype overlap; p status")
 
 
 class GatedNormArgs(Structure):

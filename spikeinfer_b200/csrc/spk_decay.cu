@@ -33,6 +33,8 @@ decay_step_kernel(const spk_decay_attn_args a) {
     const int dim = a.dim, vdim = a.vdim;
     float* out = a.out + (row * a.heads + h) * vdim;
     if (a.active != nullptr && a.active[row] != 1) {
+        spk_grid_wait();
+        spk_grid_release();
         for (int e = threadIdx.x; e < vdim; e += kThreads) out[e] = 0.0f;
         return;
     }
@@ -64,6 +66,9 @@ decay_step_kernel(const spk_decay_attn_args a) {
     const bool mine = slice < slices;
     const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
     if (mine && first < cols) load(slice, first);
+    // what was launched before is complete from here on: the launch placed behind this one may rely on that
+    spk_grid_wait();
+    spk_grid_release();
     const T* qr = static_cast<const T*>(a.q) + row * a.ld + static_cast<int64_t>(h) * dim;
     const T* kr = static_cast<const T*>(a.k) + row * a.ld + static_cast<int64_t>(h) * dim;
     const T* vr = static_cast<const T*>(a.v) + row * a.ld + static_cast<int64_t>(h) * vdim;
@@ -397,10 +402,7 @@ int launch_step(const spk_decay_attn_args& a, cudaStream_t s) {
     const dim3 grid(a.heads, static_cast<unsigned>(a.n));
     const void* fn = vec ? reinterpret_cast<const void*>(decay_step_kernel<T, 4>) : reinterpret_cast<const void*>(decay_step_kernel<T, 1>);
     if (const int rc = smem_attr(fn, bytes)) return rc;
-    if (vec) decay_step_kernel<T, 4><<<grid, kThreads, bytes, s>>>(a);
-    else decay_step_kernel<T, 1><<<grid, kThreads, bytes, s>>>(a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return spk_launch(vec ? decay_step_kernel<T, 4> : decay_step_kernel<T, 1>, grid, kThreads, bytes, s, a, a.overlap != 0);
 }
 
 int launch_scan(const spk_decay_attn_args& a, cudaStream_t s) {

@@ -108,3 +108,26 @@ __host__ __device__ __forceinline__ int spk_split_keys(int len, int splits) {
     const int per = (len + splits - 1) / splits;
     return per <= 64 ? 64 : (per + 63) & ~63;
 }
+
+// Programmatic dependent launch: wait for the launches before this one, and let the launch after this one be placed.  Both
+// do nothing in a kernel that was launched plainly.
+__device__ __forceinline__ void spk_grid_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void spk_grid_release() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+
+template <typename Args>
+static inline int spk_launch(void (*fn)(Args), dim3 grid, int threads, size_t bytes, cudaStream_t s, const Args& args, bool overlap) {
+    cudaLaunchConfig_t cfg = {};
+    cudaLaunchAttribute attr = {};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(threads);
+    cfg.dynamicSmemBytes = bytes;
+    cfg.stream = s;
+    cfg.attrs = &attr;
+    cfg.numAttrs = overlap ? 1 : 0;
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, fn, args);
+    if (e != cudaSuccess) return spk_set_cuda_error(e);
+    spk_count_launch();
+    return SPK_OK;
+}

@@ -20,6 +20,7 @@ template <typename T>
 __global__ void __launch_bounds__(kThreads)
 qk_prepare_kernel(const spk_qk_prepare_args a) {
     extern __shared__ float sm[];
+    spk_grid_release();  // a launch that does not need this one's results may be placed beside it
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int slots = a.heads + 2 * a.kv_heads;
     const int64_t item = static_cast<int64_t>(blockIdx.x) * kWarps + warp;
@@ -81,6 +82,100 @@ qk_prepare_kernel(const spk_qk_prepare_args a) {
     } else {
         for (int c = lane; c < width; c += 32) page[spk_page_channel(lay, r, c)] = spk_from_float<T>(x[c] * inv);
     }
+}
+
+// The same for bf16 heads of DIM = 64 or 128 channels (q, k and v alike) in tiled pools, eight channels (16 bytes) per lane: a
+// rotated pair's channels sit in two lanes of the head.  rot_dims is a multiple of 16.
+template <int DIM>
+__global__ void __launch_bounds__(kThreads)
+qk_prepare_vec_kernel(const spk_qk_prepare_args a) {
+    spk_grid_release();
+    constexpr int LK = DIM / 8;  // lanes per head: 8 or 16, so a warp holds whole heads
+    const int lanes_t = (a.heads + 2 * a.kv_heads) * LK;
+    const int64_t item = static_cast<int64_t>(blockIdx.x) * kThreads + threadIdx.x;
+    const int64_t t = item / lanes_t;
+    const bool in = t < a.n;
+    const int l = static_cast<int>(item % lanes_t);
+    const int qk_lanes = (a.heads + a.kv_heads) * LK;
+    const bool is_v = l >= qk_lanes;
+    const int s = (is_v ? l - qk_lanes : l) / LK;  // head slot (q heads, then k heads) or v head
+    const int sub = l % LK;
+    const bool is_q = !is_v && s < a.heads;
+    const __nv_bfloat16* src = is_v ? static_cast<const __nv_bfloat16*>(a.v) + t * a.ld + s * DIM + sub * 8
+                             : is_q ? static_cast<const __nv_bfloat16*>(a.q) + t * a.ld + s * DIM + sub * 8
+                                    : static_cast<const __nv_bfloat16*>(a.k) + t * a.ld + (s - a.heads) * DIM + sub * 8;
+    const uint4 u = in ? *reinterpret_cast<const uint4*>(src) : make_uint4(0u, 0u, 0u, 0u);
+    float x[8];
+    {
+        const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            x[2 * k] = __uint_as_float(w[k] << 16);
+            x[2 * k + 1] = __uint_as_float(w[k] & 0xffff0000u);
+        }
+    }
+    const int half = a.rot_table != nullptr ? a.rot_dims / 2 : 0;
+    const int hl = half / 8;  // lanes of each half of the rotated channels
+    const bool low = sub < hl, turn = !is_v && sub < 2 * hl;
+    float y[8];
+    const int partner = (threadIdx.x & 31) + (turn ? (low ? hl : -hl) : 0);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) y[k] = __shfl_sync(~0u, x[k], partner);
+    if (turn && in) {
+        int64_t pos = a.positions[t];
+        if (pos < 0 || pos >= a.rot_positions) {
+            spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+            pos = 0;
+        }
+        const float4* cs = reinterpret_cast<const float4*>(reinterpret_cast<const float2*>(a.rot_table) + pos * half + (low ? sub : sub - hl) * 8);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float4 f = cs[k];  // (cos, sin) of two pairs
+            const float s0 = low ? -f.y : f.y, s1 = low ? -f.w : f.w;
+            x[2 * k] = x[2 * k] * f.x + y[2 * k] * s0;
+            x[2 * k + 1] = x[2 * k + 1] * f.z + y[2 * k + 1] * s1;
+        }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) ss = fmaf(x[k], x[k], ss);
+#pragma unroll
+    for (int o = LK / 2; o >= 1; o >>= 1) ss += __shfl_xor_sync(~0u, ss, o);
+    if (!in) return;
+    const float inv = a.unit_norm ? 1.0f / sqrtf(ss / static_cast<float>(DIM) + a.eps) : 1.0f;
+    uint4 r = u;
+    if (!is_v) {
+        uint32_t w[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const __nv_bfloat162 b = __floats2bfloat162_rn(x[2 * k] * inv, x[2 * k + 1] * inv);
+            w[k] = *reinterpret_cast<const uint32_t*>(&b);
+        }
+        r = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+    if (is_q) {
+        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.q_out) + (t * a.heads + s) * DIM + sub * 8) = r;
+        return;
+    }
+    const int64_t slot = a.slot_mapping[t];
+    const int64_t block = slot / a.block_size;
+    if (slot < 0 || block >= a.num_blocks) {
+        spk_flag(a.status, SPK_STATUS_BAD_SLOT);
+        return;
+    }
+    const SpkPageLayout lay{a.kv_heads, a.block_size, DIM, 1};
+    __nv_bfloat16* page = static_cast<__nv_bfloat16*>(is_v ? a.v_pool : a.k_pool) + spk_page_base(lay, block, is_v ? s : s - a.heads);
+    *reinterpret_cast<uint4*>(page + spk_page_channel(lay, static_cast<int>(slot % a.block_size), sub * 8)) = r;
+}
+
+template <int DIM>
+int launch_prepare_vec(const spk_qk_prepare_args& a, cudaStream_t s) {
+    const int64_t items = a.n * (a.heads + 2 * static_cast<int64_t>(a.kv_heads)) * (DIM / 8);
+    const int64_t grid = (items + kThreads - 1) / kThreads;
+    if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
+    qk_prepare_vec_kernel<DIM><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
 }
 
 // ---- attention, 32-bit -----------------------------------------------------------------------------------------
@@ -209,6 +304,11 @@ extern "C" int spk_qk_prepare(const spk_qk_prepare_args* a, void* stream) {
     if (a->q == nullptr || a->k == nullptr || a->v == nullptr || a->q_out == nullptr || a->k_pool == nullptr || a->v_pool == nullptr ||
         a->slot_mapping == nullptr)
         return SPK_ERR_NULL_POINTER;
+    auto at16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    if (a->dtype == SPK_BF16 && a->k_tiled && a->v_tiled && a->dim == a->vdim && (a->dim == 64 || a->dim == 128) && a->k_pad == a->dim &&
+        a->v_pad == a->vdim && a->ld % 8 == 0 && (a->rot_table == nullptr || (a->rot_dims % 16 == 0 && at16(a->rot_table))) && at16(a->q) &&
+        at16(a->k) && at16(a->v) && at16(a->q_out) && at16(a->k_pool) && at16(a->v_pool))
+        return a->dim == 64 ? launch_prepare_vec<64>(*a, spk_stream(stream)) : launch_prepare_vec<128>(*a, spk_stream(stream));
     const int64_t items = a->n * (a->heads + 2 * static_cast<int64_t>(a->kv_heads));
     const int64_t grid = (items + kWarps - 1) / kWarps;
     const size_t bytes = sizeof(float) * kWarps * a->dim;

@@ -45,11 +45,15 @@ sigmoid_decode_kernel(const spk_sigmoid_attn_args a) {
     const int len = (a.active == nullptr || a.active[row] == 1) ? a.seq_lens[row] : 0;
     if (len < 0 || len > a.max_blocks * a.block_size) {
         if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+        spk_grid_wait();
         return;
     }
     const int per = spk_split_keys(len, a.splits);
     const int lo = blockIdx.x * per, hi = min(lo + per, len);
-    if (lo >= len) return;
+    if (lo >= len) {
+        spk_grid_wait();
+        return;
+    }
     const int steps_cta = (hi - lo + kStep - 1) / kStep;
     const int steps = steps_cta > warp ? (steps_cta - warp + kWarps - 1) / kWarps : 0;
 
@@ -191,6 +195,8 @@ sigmoid_decode_kernel(const spk_sigmoid_attn_args a) {
         for (int w = 0; w < kWarps; ++w) sum += red[(w * 16 + r) * RW + e];
         part[i] = sum;
     }
+    // launched to overlap: the launch before this one is complete when this one is
+    spk_grid_wait();
 }
 
 template <int CK, int CV>
@@ -200,9 +206,7 @@ int launch(const spk_sigmoid_attn_args& a, cudaStream_t s) {
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     const int rep = a.heads / a.kv_heads;
     const dim3 grid(a.splits, a.kv_heads * ((rep + 15) / 16), static_cast<unsigned>(a.n));
-    sigmoid_decode_kernel<CK, CV><<<grid, kThreads, bytes, s>>>(a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return spk_launch(sigmoid_decode_kernel<CK, CV>, grid, kThreads, bytes, s, a, a.overlap != 0);
 }
 
 }  // namespace

@@ -110,14 +110,14 @@ def qk_prepare(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_pool, v_pool
 def sigmoid_attention(q: torch.Tensor, k_pool, v_pool, tables: torch.Tensor, head_bias: torch.Tensor, out: torch.Tensor, *,
                       heads: int, kv_heads: int, dim: int, vdim: int, scale: float, out_scale: float = 1.0,
                       plan=None, seq_lens: torch.Tensor | None = None, active: torch.Tensor | None = None,
-                      status: torch.Tensor | None = None, partial_sums: bool = False) -> torch.Tensor | None:
+                      status: torch.Tensor | None = None, partial_sums: bool = False, overlap_previous: bool = False) -> torch.Tensor | None:
     """``out[t, h * vdim :] = out_scale * sum_j sigmoid(scale * q.k_j + head_bias[h]) v_j`` over the keys up to token t's own
     position, read through ``tables``.  ``out`` is a column range of a row-major matrix in the model dtype.  ``plan`` (a
     ``PrefillPlan``): prefill form; None: decode form over ``seq_lens`` / ``active``.
 
     ``partial_sums`` (decode form): where the sizes allow it, leave ``out`` alone and return fp32 partial sums
     ``[n, splits, heads * vdim]`` of key ranges, for :func:`gated_norm` to add up; otherwise ``out`` is written and None
-    returned."""
+    returned.  ``overlap_previous``: this call directly follows :func:`decay_attention` and may run beside it."""
     _lib.require_cuda(q, "sigmoid_attention query")
     _f32(head_bias, "head_bias", heads)
     n = q.shape[0]
@@ -138,7 +138,7 @@ def sigmoid_attention(q: torch.Tensor, k_pool, v_pool, tables: torch.Tensor, hea
         num_blocks=k_pool.data.shape[0], partials=_ptr(partials), n_tiles=0 if tiles is None else tiles.shape[0], splits=splits,
         heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, k_pad=k_pool.pad, v_pad=v_pool.pad, k_tiled=int(k_pool.tiled),
         v_tiled=int(v_pool.tiled), block_size=k_pool.block_size, dtype=form[0], scale=scale, out_scale=out_scale,
-        status=_ptr(status))
+        overlap=int(overlap_previous and partials is not None), status=_ptr(status))
     _call("spk_sigmoid_attn", a, q.device)
     return partials
 
@@ -152,10 +152,12 @@ def decay_powers(decay, device) -> torch.Tensor:
 
 def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, powers: torch.Tensor, *,
                     plan=None, active: torch.Tensor | None = None, silu: bool = True,
-                    status: torch.Tensor | None = None) -> torch.Tensor:
+                    status: torch.Tensor | None = None, overlap_previous: bool = False) -> torch.Tensor:
     """``S <- decay S + k v^T, o = S^T q`` per head, silu on q, k and v first.  ``q``, ``k``, ``v`` are column ranges of one
     projection output; ``state`` fp32 ``[rows, heads, dim, vdim]`` is updated in place; ``powers`` from :func:`decay_powers`.
-    Returns fp32 ``[n, heads * vdim]``.  ``plan``: prefill form, None: decode form gated by ``active``."""
+    Returns fp32 ``[n, heads * vdim]``.  ``plan``: prefill form, None: decode form gated by ``active``.
+    ``overlap_previous`` (decode form): this call directly follows :func:`qk_prepare` of the same step, everything it reads was
+    complete before that began, and it may be placed while that still runs."""
     _lib.require_cuda(q, "decay_attention query")
     n = q.shape[0]
     rows, heads, dim, vdim = state.shape
@@ -169,7 +171,7 @@ def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: to
     a = _lib.DecayAttnArgs(
         q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), ld=ld, state=state.data_ptr(), state_stride=state.stride(0), state_rows=rows,
         decay_pow=powers.data_ptr(), out=out.data_ptr(), active=_ptr(active), n=n, heads=heads, dim=dim, vdim=vdim,
-        silu=int(silu), dtype=_lib.dtype_code(q.dtype), status=_ptr(status))
+        silu=int(silu), dtype=_lib.dtype_code(q.dtype), overlap=int(overlap_previous and plan is None), status=_ptr(status))
     if plan is None:
         _call("spk_decay_attn_step", a, q.device)
         return out

@@ -192,17 +192,19 @@ class ManiraxModel:
                        positions=positions, status=meta.status, **heads)
         common = dict(scale=lf.scale, out_scale=L.cfg.left_scale, status=meta.status, **heads)
         left = both[:, : L.left_width]
-        partials = None
         if meta.num_prefills:
-            plan, active = meta.prefill_plan(), None
+            plan = meta.prefill_plan()
+            o = decay_attention(rq, rk, rv, cache.states["decay"], L.decay, plan=plan, status=meta.status)
             sigmoid_attention(q, cache.k, cache.v, meta.row_tables, L.head_bias, left, plan=plan, **common)
+            partials = None
         else:
-            plan, active = None, meta.row_active
+            # three launches in a row: the recurrence is placed while K/V are being written, the attention runs beside it
+            o = decay_attention(rq, rk, rv, cache.states["decay"], L.decay, active=meta.row_active,
+                                overlap_previous=meta.tables_settled, status=meta.status)
             partials = sigmoid_attention(q, cache.k, cache.v, meta.block_tables, L.head_bias, left, seq_lens=meta.seq_lens,
-                                         active=active, partial_sums=True, **common)
-        o = decay_attention(rq, rk, rv, cache.states["decay"], L.decay, plan=plan, active=active, status=meta.status)
+                                         active=meta.row_active, partial_sums=True, overlap_previous=meta.tables_settled, **common)
         gated_norm(o, L.right_norm, rg, both, L.left_width, eps=eps, scale=L.cfg.right_scale, partials=partials,
-                   left_scale=L.cfg.left_scale, seq_lens=meta.seq_lens, active=active)
+                   left_scale=L.cfg.left_scale, seq_lens=meta.seq_lens, active=meta.row_active)
         return self._matmul_f32(both, L.w_out)
 
     @torch.no_grad()

@@ -33,6 +33,11 @@ CONFIGS = {
         layer(heads=24, kv_heads=1, dim=64, vdim=128, scale=0.1, rot=(32, 1e5, 2.0), r_heads=2, r_dim=128, r_vdim=64, decay=(0.7, 0.998), ff=256),
         layer(heads=12, kv_heads=1, dim=128, vdim=64, scale=0.06, rot=(128, 1e4, 8.0), r_heads=4, r_dim=64, r_vdim=128, decay=(0.3, 0.9, 0.99, 0.9995), ff=192),
     ], vocab=512, width=256, alpha=2.5),
+    # one head size throughout, a second wide layer whose keys and values are 128 channels
+    "even": config([
+        layer(heads=6, kv_heads=2, dim=64, vdim=64, scale=0.11, rot=(48, 2e4, 2.5), r_heads=3, r_dim=64, r_vdim=64, decay=(0.5, 0.93, 0.998), ff=136),
+        layer(heads=3, kv_heads=1, dim=128, vdim=128, scale=0.07, rot=(128, 1e6, 1.5), r_heads=2, r_dim=128, r_vdim=128, decay=(0.85, 0.9999), ff=104),
+    ], vocab=264, width=136, alpha=2.0),
     # more channels per head than the tensor-core forms take
     "large_heads": config([layer(heads=2, kv_heads=1, dim=160, vdim=144, rot=(96, 1e4, 3.0), r_heads=1, r_dim=136, r_vdim=130, decay=(0.95,))]),
 }

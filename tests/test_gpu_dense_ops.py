@@ -130,7 +130,9 @@ def test_poly_norm(dev, dtype, width):
 # ---- rotation, unit norm, pages ------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,rot,block_size", [
-    (4, 2, 32, 48, (16, 1e4, 4.0), 16), (3, 3, 21, 10, None, 4), (8, 1, 64, 128, (64, 500.0, 1.0), 32), (2, 1, 160, 16, (96, 1e5, 2.0), 8)])
+    (4, 2, 32, 48, (16, 1e4, 4.0), 16), (3, 3, 21, 10, None, 4), (8, 1, 64, 128, (64, 500.0, 1.0), 32), (2, 1, 160, 16, (96, 1e5, 2.0), 8),
+    (6, 2, 64, 64, (32, 1e4, 3.0), 16), (3, 1, 64, 64, (64, 700.0, 1.0), 32), (5, 5, 128, 128, (128, 1e5, 8.0), 16),
+    (4, 2, 128, 128, (48, 1e3, 2.0), 16), (2, 1, 64, 64, None, 16), (2, 1, 64, 64, (24, 1e3, 2.0), 16)])
 def test_qk_prepare(dev, dtype, heads, kv_heads, dim, vdim, rot, block_size):
     n, blocks = 9, 8
     g = gen(dim)

@@ -91,7 +91,7 @@ def test_token_by_token_equals_the_prompt(dev, name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name,cuts", [("mixed", [2] * 35), ("odd", [2, 3, 1, 1, 17, 2, 44]), ("wide", [1, 63, 2, 1, 1, 62, 2, 18]),
-                                       ("mixed", [64, 2, 64, 20]), ("large_heads", [16, 2, 31, 21]), ("wide", [130, 2, 18])])
+                                       ("mixed", [64, 2, 64, 20]), ("large_heads", [16, 2, 31, 21]), ("even", [100, 2, 1, 65, 12]), ("wide", [130, 2, 18])])
 def test_portions_of_several_sizes(dev, name, cuts, dtype):
     n = sum(cuts)
     tokens = prompt(name, n, 2)
@@ -118,7 +118,7 @@ def test_other_page_sizes(dev, dtype, block_size):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "wide"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "even"])
 def test_unequal_requests_together_and_alone(dev, name, dtype):
     """Portions of unequal requests in one call, decode steps of changing subsets, a row held between portions of its prompt
     while the others decode: each request as if it were alone."""
