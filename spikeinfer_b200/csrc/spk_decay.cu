@@ -185,10 +185,20 @@ decay_scan_kernel(const spk_decay_attn_args a) {
     float* slot = a.state + sq.z * a.state_stride + i;
     float S = sq.w > 0 ? *slot : 0.0f;
     float* w = a.workspace + sq.x * per_chunk + i;
-    for (int c = 0; c < sq.y; ++c, w += per_chunk) {
-        const float own = *w;
-        *w = S;
-        S = fmaf(pw[a.chunks[4 * (sq.x + c) + 1]], S, own);
+    constexpr int U = 8;  // chunks in flight: only S is a chain, the loads are not
+    for (int c0 = 0; c0 < sq.y; c0 += U) {
+        float own[U], p[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const bool in = c0 + u < sq.y;
+            own[u] = in ? w[(c0 + u) * per_chunk] : 0.0f;
+            p[u] = in ? pw[a.chunks[4 * (sq.x + c0 + u) + 1]] : 1.0f;
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            if (c0 + u < sq.y) w[(c0 + u) * per_chunk] = S;
+            S = fmaf(p[u], S, own[u]);
+        }
     }
     *slot = S;
 }

@@ -113,7 +113,7 @@ __device__ __forceinline__ void add_outer(float (&acc)[StateTile<CD, CV>::NT][4]
 }
 
 template <int CD, int CV>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 2)
 decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool vec_v) {
     using T = StateTile<CD, CV>;
     constexpr int SK = T::D + 8, SV = T::V + 8;
