@@ -443,8 +443,18 @@ extern "C" int spk_decay_powers(void) { return kPow; }
 
 extern "C" int spk_decay_chunk_tokens(int dtype, int dim, int vdim, int64_t n, int heads) {
     if (!spk_decay_tensor_form(dtype, dim, vdim) || n < 1 || heads < 1) return kChunk;
-    int span = kDecayMaxSpan;  // as long as two CTAs per SM remain
-    while (span > kChunk && n * heads < static_cast<int64_t>(span) * 2 * 148) span /= 2;
+    // the span whose waves of CTAs take least: a chunk is one unit, a CTA's set-up and its state's traffic one more
+    const int64_t slots = 148 * (dim <= 64 && vdim <= 64 ? 2 : 1);
+    int span = kChunk;
+    int64_t best = INT64_MAX;
+    for (int s = kChunk; s <= kDecayMaxSpan; s *= 2) {
+        const int64_t ctas = (n + s - 1) / s * heads;
+        const int64_t cost = (ctas + slots - 1) / slots * (s / kChunk + 1);
+        if (cost <= best) {
+            best = cost;
+            span = s;
+        }
+    }
     return span;
 }
 

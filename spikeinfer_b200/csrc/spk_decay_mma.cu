@@ -1,6 +1,6 @@
 // Prefill form of the decayed linear attention with bf16 projections on the tensor cores (heads of up to 128 channels).
 //
-// A stored state every `span` tokens (64 .. 512, chosen by the host so that the call fills the GPU) keeps the traffic of the
+// A stored state every `span` tokens (64 .. 512, chosen by the host for the call's size) keeps the traffic of the
 // states small; inside a span a CTA walks 64-token chunks with the running state in its registers:
 //  * decay_span_sum_kernel:  U = sum_j decay^(L-1-j) k_j v_j^T of a span of L tokens;
 //  * (the scan of spk_decay.cu turns the U of every span into the state the span starts from);

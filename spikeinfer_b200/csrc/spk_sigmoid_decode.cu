@@ -150,7 +150,7 @@ sigmoid_decode_kernel(const spk_sigmoid_attn_args a) {
             const int j0 = key0 + tig * 2;
             auto weigh = [&](float x, float y, float bias, int j, uint32_t& h, uint32_t& l) {
                 float p0, p1;
-                sigmoid2(fmaf(x, c1, bias), fmaf(y, c1, bias), p0, p1);
+                sigmoid2(f2_fma(f2_pack(x, y), f2_pack(c1, c1), f2_pack(bias, bias)), p0, p1);
                 split_bf16(j < hi ? p0 : 0.0f, j + 1 < hi ? p1 : 0.0f, h, l);
             };
             weigh(s0[0], s0[1], b0, j0, ph[0], pl[0]);

@@ -1,9 +1,10 @@
 // Prefill attention with sigmoid key weights on the fifth-generation tensor cores (tcgen05), bf16, head sizes up to 128.
 //
-// CTA = (128 query tokens of one portion, query head).  Ten warps:
+// CTA = (128 query tokens of one portion, query head).  Eleven warps:
 //  * warp 8 copies K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
 //    handful of plain bulk copies (cp.async.bulk), no tensor map, whatever pages the block table names;
-//  * warp 9 (one thread) issues the MMAs: S = Q K^T into one of two TMEM buffers, O += P V with P read from TMEM;
+//  * warp 9 (one thread) issues S = Q K^T into one of two TMEM buffers, warp 10 (one thread) O += P V with P read from TMEM,
+//    so that neither kind of MMA waits behind the other's operands;
 //  * warps 0-3 and 4-7 turn the even and the odd tiles' scores into weights (one thread per query row).
 // A weight is sigmoid(score) of its own key: no running maximum, no rescaling of O, no denominator.  Weights are computed in
 // 32 bits and enter the product as a bf16 pair (hi + lo: 16 significant bits), so O is a 32-bit sum of them to 2^-17.
@@ -19,7 +20,7 @@ using namespace spk_tc;
 constexpr int kTile = 128;            // query rows, and keys per step
 constexpr int kColTile = kTile * 128; // bytes of a 64-channel column tile
 constexpr int kSigmoidThreads = 256;
-constexpr int kThreads = kSigmoidThreads + 64;
+constexpr int kThreads = kSigmoidThreads + 96;
 constexpr uint32_t kTmemS = 0, kTmemLo = 256, kTmemO = 384;  // S/P-hi buffers 2 x 128, P-lo 2 x 64, O up to 128
 constexpr float kLog2e = 1.4426950408889634f;
 
@@ -31,7 +32,7 @@ struct Shape {
 };
 
 struct Bars {
-    uint64_t k_full[4], k_free[4], v_full[4], v_free[4], s_full[2], p_full[2], p_free[2], o_full;
+    uint64_t k_full[4], k_free[4], v_full[4], v_free[4], s_full[2], p_full[2], p_free[2], o_full, q_full, s_done;
     int abort;
     uint32_t tmem;
 };
@@ -79,17 +80,11 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
             mbar_init(smem_u32(&bars->p_free[i]), 1);
         }
         mbar_init(smem_u32(&bars->o_full), 1);
+        mbar_init(smem_u32(&bars->s_done), 1);
+        mbar_init(smem_u32(&bars->q_full), kSigmoidThreads);
         bars->abort = 0;
     }
     if (warp == 0) tmem_alloc(smem_u32(&bars->tmem), 512);
-    // Q rows into the swizzled operand layout, zeros beyond the portion
-    for (int i = threadIdx.x; i < kTile * CK * 8; i += kThreads) {
-        const int r = i / (CK * 8), c = i % (CK * 8);
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (r < nq)
-            v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + ((t0 + r) * a.heads + h) * a.k_pad + c * 8);
-        *reinterpret_cast<uint4*>(q_s + (c >> 3) * kColTile + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
-    }
     fence_async_shared();
     tc_fence_before();
     __syncthreads();
@@ -139,52 +134,67 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                 mbar_wait(smem_u32(&bars->k_full[t % NS]), (t / NS) & 1);
                 mbar_wait(smem_u32(&bars->v_full[t % NS]), (t / NS) & 1);
             }
-    } else if (warp == 9) {  // ---- MMA issue
+    } else if (warp == 9) {  // ---- scores
         if (lane == 0) {
-            constexpr uint32_t idesc_s = idesc_bf16(kTile, kTile, false, false);
-            constexpr uint32_t idesc_o = idesc_bf16(kTile, CV * 64, false, true);
-            auto scores = [&](int t) {
+            constexpr uint32_t idesc = idesc_bf16(kTile, kTile, false, false);
+            bool ok = mbar_wait(smem_u32(&bars->q_full), 0, abort);
+            for (int t = 0; ok && t < tiles; ++t) {
                 const int stage = t % NS;
-                if (!mbar_wait(smem_u32(&bars->k_full[stage]), (t / NS) & 1, abort)) return false;
+                // the buffer's previous weights (tile t - 2) have been multiplied
+                ok = (t < 2 || mbar_wait(smem_u32(&bars->p_free[t & 1]), ((t >> 1) - 1) & 1, abort)) &&
+                     mbar_wait(smem_u32(&bars->k_full[stage]), (t / NS) & 1, abort);
+                if (!ok) break;
                 tc_fence_after();
                 const uint32_t qa = smem_u32(q_s), kb = smem_u32(k_s + stage * Sh::kK);
 #pragma unroll
                 for (int s = 0; s < CK * 4; ++s) {
                     const uint32_t off = (s >> 2) * kColTile + (s & 3) * 32;
-                    mma_ss(tmem + kTmemS + (t & 1) * 128, desc_sw128(qa + off, 16, 1024), desc_sw128(kb + off, 16, 1024), idesc_s, s > 0);
+                    mma_ss(tmem + kTmemS + (t & 1) * 128, desc_sw128(qa + off, 16, 1024), desc_sw128(kb + off, 16, 1024), idesc, s > 0);
                 }
                 mma_commit(smem_u32(&bars->k_free[stage]));
                 mma_commit(smem_u32(&bars->s_full[t & 1]));
-                return true;
-            };
-            bool ok = scores(0) && (tiles < 2 || scores(1));
-            for (int t = 0; ok && t < tiles; ++t) {
+            }
+            mma_commit(smem_u32(&bars->s_done));
+            mbar_wait(smem_u32(&bars->s_done), 0);  // nothing this thread issued is in the tensor pipe any more
+        }
+    } else if (warp == 10) {  // ---- weighted sums
+        if (lane == 0) {
+            constexpr uint32_t idesc = idesc_bf16(kTile, CV * 64, false, true);
+            for (int t = 0; t < tiles; ++t) {
                 const int stage = t % NS, buf = t & 1;
-                ok = mbar_wait(smem_u32(&bars->v_full[stage]), (t / NS) & 1, abort) &&
-                     mbar_wait(smem_u32(&bars->p_full[buf]), (t >> 1) & 1, abort);
-                if (!ok) break;
+                if (!mbar_wait(smem_u32(&bars->v_full[stage]), (t / NS) & 1, abort) ||
+                    !mbar_wait(smem_u32(&bars->p_full[buf]), (t >> 1) & 1, abort))
+                    break;
                 tc_fence_after();
                 const uint32_t vb = smem_u32(v_s + stage * Sh::kV);
                 const int valid = keys - t * kTile < kTile ? keys - t * kTile : kTile;
                 const int steps = (valid + 15) >> 4;
                 for (int s = 0; s < steps; ++s) {
                     const uint64_t vd = desc_sw128(vb + s * 2048, kColTile, 1024);
-                    mma_ts(tmem + kTmemO, tmem + kTmemS + buf * 128 + s * 8, vd, idesc_o, t > 0 || s > 0);
-                    mma_ts(tmem + kTmemO, tmem + kTmemLo + buf * 64 + s * 8, vd, idesc_o, true);
+                    mma_ts(tmem + kTmemO, tmem + kTmemS + buf * 128 + s * 8, vd, idesc, t > 0 || s > 0);
+                    mma_ts(tmem + kTmemO, tmem + kTmemLo + buf * 64 + s * 8, vd, idesc, true);
                 }
-                mma_commit(smem_u32(&bars->v_free[stage]));
                 mma_commit(smem_u32(&bars->p_free[buf]));
-                if (t + 2 < tiles)
-                    ok = mbar_wait(smem_u32(&bars->p_free[buf]), (t >> 1) & 1, abort) && scores(t + 2);
+                mma_commit(smem_u32(&bars->v_free[stage]));
             }
             mma_commit(smem_u32(&bars->o_full));
-            mbar_wait(smem_u32(&bars->o_full), 0);  // nothing of this CTA is in the tensor pipe any more
+            mbar_wait(smem_u32(&bars->o_full), 0);
         }
     } else {  // ---- scores to weights: warps 0-3 the even tiles, 4-7 the odd ones
+        // Q rows into the swizzled operand layout, zeros beyond the portion
+        for (int i = threadIdx.x; i < kTile * CK * 8; i += kSigmoidThreads) {
+            const int r = i / (CK * 8), c = i % (CK * 8);
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (r < nq)
+                v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + ((t0 + r) * a.heads + h) * a.k_pad + c * 8);
+            *reinterpret_cast<uint4*>(q_s + (c >> 3) * kColTile + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+        }
+        fence_async_shared();
+        mbar_arrive(smem_u32(&bars->q_full));
         const int wg = warp >> 2;
         const int r = (warp & 3) * 32 + lane;
         const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
-        const float c1 = -a.scale * kLog2e, c0 = -a.head_bias[h] * kLog2e;
+        const uint64_t c1 = f2_pack(-a.scale * kLog2e, -a.scale * kLog2e), c0 = f2_pack(-a.head_bias[h] * kLog2e, -a.head_bias[h] * kLog2e);
         bool ok = true;
         for (int t = wg; t < tiles; t += 2) {
             const int stage = t % NS;
@@ -192,29 +202,39 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
             if (!ok) break;
             tc_fence_after();
             const int last = pos0 + r - t * kTile;  // last visible column of this row
-            const bool full = t * kTile + kTile - 1 <= pos0;
-            uint32_t buf[2][32];
             const uint32_t sa = tmem + lanes + kTmemS + wg * 128, la = tmem + lanes + kTmemLo + wg * 64;
-            tmem_ld32(sa, buf[0]);
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                uint32_t(&s)[32] = buf[c & 1];
-                tmem_wait_ld(s);
-                if (c < 3) tmem_ld32(sa + (c + 1) * 32, buf[(c + 1) & 1]);
+            // 32 score columns to weights; the hi half overlays score columns that have been read (16 c + 15 < 32 (c + 1))
+            auto weigh = [&](uint32_t (&sc)[32], int c) {
                 uint32_t hi[16], lo[16];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
                     float p0, p1;
-                    sigmoid2(fmaf(__uint_as_float(s[2 * i]), c1, c0), fmaf(__uint_as_float(s[2 * i + 1]), c1, c0), p0, p1);
-                    if (!full) {
-                        p0 = c * 32 + 2 * i <= last ? p0 : 0.0f;
-                        p1 = c * 32 + 2 * i + 1 <= last ? p1 : 0.0f;
-                    }
+                    sigmoid2(f2_fma(f2_pack(__uint_as_float(sc[2 * i]), __uint_as_float(sc[2 * i + 1])), c1, c0), p0, p1);
                     split_bf16(p0, p1, hi[i], lo[i]);
                 }
-                // the hi half overlays score columns that have been read (16 c + 15 < 32 (c + 1))
+                const int seen = last - c * 32;
+                if (!__all_sync(~0u, seen >= 31)) {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        const uint32_t m = (2 * i <= seen ? 0xffffu : 0u) | (2 * i + 1 <= seen ? 0xffff0000u : 0u);
+                        hi[i] &= m;
+                        lo[i] &= m;
+                    }
+                }
                 tmem_st16(sa + c * 16, hi);
                 tmem_st16(la + c * 16, lo);
+            };
+            // two chunks per turn, the next one's scores on their way meanwhile; rolled: the body has to fit the instruction cache
+            uint32_t even[32], odd[32];
+            tmem_ld32(sa, even);
+#pragma unroll 1
+            for (int c = 0; c < 4; c += 2) {
+                tmem_wait_ld(even);
+                tmem_ld32(sa + (c + 1) * 32, odd);
+                weigh(even, c);
+                tmem_wait_ld(odd);
+                if (c == 0) tmem_ld32(sa + 64, even);
+                weigh(odd, c + 1);
             }
             tmem_wait_st();
             const int valid = keys - t * kTile;

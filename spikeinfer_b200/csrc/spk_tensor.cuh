@@ -126,10 +126,36 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&v);
 }
+// Two 32-bit lanes in one instruction.
+__device__ __forceinline__ uint64_t f2_pack(float x, float y) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+    return r;
+}
+__device__ __forceinline__ void f2_unpack(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ uint64_t f2_fma(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t f2_add(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 // A pair of 32-bit values as two bf16 pairs whose sum carries 16 significant bits.
 __device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(x, y);
-    lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+    const uint64_t rest = f2_fma(f2_pack(__uint_as_float(hi << 16), __uint_as_float(hi & 0xffff0000u)), f2_pack(-1.0f, -1.0f), f2_pack(x, y));
+    float a, b;
+    f2_unpack(rest, a, b);
+    lo = pack_bf16(a, b);
 }
 
 __device__ __forceinline__ float ex2(float x) {
@@ -144,11 +170,12 @@ __device__ __forceinline__ float rcp(float x) {
 }
 // Two sigmoids, 1 / (1 + 2^u) each, with one reciprocal: r = 1 / (ab), 1/a = r b, 1/b = r a.  The exponents are capped
 // so that the product stays finite (a weight below 2^-60 counts as 2^-60).
-__device__ __forceinline__ void sigmoid2(float u0, float u1, float& p0, float& p1) {
-    const float a = 1.0f + ex2(fminf(u0, 60.0f)), b = 1.0f + ex2(fminf(u1, 60.0f));
+__device__ __forceinline__ void sigmoid2(uint64_t u, float& p0, float& p1) {
+    float u0, u1, a, b;
+    f2_unpack(u, u0, u1);
+    f2_unpack(f2_add(f2_pack(ex2(fminf(u0, 60.0f)), ex2(fminf(u1, 60.0f))), f2_pack(1.0f, 1.0f)), a, b);
     const float r = rcp(a * b);
-    p0 = r * b;
-    p1 = r * a;
+    f2_unpack(f2_mul(f2_pack(b, a), f2_pack(r, r)), p0, p1);
 }
 
 }  // namespace spk_tc
