@@ -1,11 +1,12 @@
 // Prefill attention with sigmoid key weights on the fifth-generation tensor cores (tcgen05), bf16, head sizes up to 128.
 //
-// CTA = (128 query tokens of one portion, query head).  Eleven warps:
-//  * warp 8 copies K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
+// CTA = (128 query tokens of one portion, query head).  Nineteen warps:
+//  * warp 16 copies K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
 //    handful of plain bulk copies (cp.async.bulk), no tensor map, whatever pages the block table names;
-//  * warp 9 (one thread) issues S = Q K^T into one of two TMEM buffers, warp 10 (one thread) O += P V with P read from TMEM,
+//  * warp 17 (one thread) issues S = Q K^T into one of two TMEM buffers, warp 18 (one thread) O += P V with P read from TMEM,
 //    so that neither kind of MMA waits behind the other's operands;
-//  * warps 0-3 and 4-7 turn the even and the odd tiles' scores into weights (one thread per query row).
+//  * warps 0-15 turn scores into weights: warpgroups 0 and 2 the two column halves of the even tiles, 1 and 3 those of the odd
+//    ones, one thread per query row and half.  The work is latency-bound, hence many warps of few registers.
 // A weight is sigmoid(score) of its own key: no running maximum, no rescaling of O, no denominator.  Weights are computed in
 // 32 bits and enter the product as a bf16 pair (hi + lo: 16 significant bits), so O is a 32-bit sum of them to 2^-17.
 // Visible keys are those up to the query's own position; the last tile's rows of V beyond the portion's end are cleared in
@@ -19,7 +20,7 @@ using namespace spk_tc;
 
 constexpr int kTile = 128;            // query rows, and keys per step
 constexpr int kColTile = kTile * 128; // bytes of a 64-channel column tile
-constexpr int kSigmoidThreads = 256;
+constexpr int kSigmoidThreads = 512;
 constexpr int kThreads = kSigmoidThreads + 96;
 constexpr uint32_t kTmemS = 0, kTmemLo = 256, kTmemO = 384;  // S/P-hi buffers 2 x 128, P-lo 2 x 64, O up to 128
 constexpr float kLog2e = 1.4426950408889634f;
@@ -76,7 +77,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
         }
         for (int i = 0; i < 2; ++i) {
             mbar_init(smem_u32(&bars->s_full[i]), 1);
-            mbar_init(smem_u32(&bars->p_full[i]), 128);
+            mbar_init(smem_u32(&bars->p_full[i]), 256);
             mbar_init(smem_u32(&bars->p_free[i]), 1);
         }
         mbar_init(smem_u32(&bars->o_full), 1);
@@ -92,7 +93,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
     const uint32_t tmem = bars->tmem;
     volatile int* abort = &bars->abort;
 
-    if (warp == 8) {  // ---- K and V copies
+    if (warp == 16) {  // ---- K and V copies
         const int gran = a.block_size < kTile ? a.block_size : kTile;  // rows per copy
         const int32_t* table = a.tables + static_cast<int64_t>(row) * a.table_stride;
         const SpkPageLayout kl{a.kv_heads, a.block_size, a.k_pad, 1}, vl{a.kv_heads, a.block_size, a.v_pad, 1};
@@ -134,7 +135,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                 mbar_wait(smem_u32(&bars->k_full[t % NS]), (t / NS) & 1);
                 mbar_wait(smem_u32(&bars->v_full[t % NS]), (t / NS) & 1);
             }
-    } else if (warp == 9) {  // ---- scores
+    } else if (warp == 17) {  // ---- scores
         if (lane == 0) {
             constexpr uint32_t idesc = idesc_bf16(kTile, kTile, false, false);
             bool ok = mbar_wait(smem_u32(&bars->q_full), 0, abort);
@@ -157,7 +158,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
             mma_commit(smem_u32(&bars->s_done));
             mbar_wait(smem_u32(&bars->s_done), 0);  // nothing this thread issued is in the tensor pipe any more
         }
-    } else if (warp == 10) {  // ---- weighted sums
+    } else if (warp == 18) {  // ---- weighted sums
         if (lane == 0) {
             constexpr uint32_t idesc = idesc_bf16(kTile, CV * 64, false, true);
             for (int t = 0; t < tiles; ++t) {
@@ -171,7 +172,8 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                 const int steps = (valid + 15) >> 4;
                 for (int s = 0; s < steps; ++s) {
                     const uint64_t vd = desc_sw128(vb + s * 2048, kColTile, 1024);
-                    mma_ts(tmem + kTmemO, tmem + kTmemS + buf * 128 + s * 8, vd, idesc, t > 0 || s > 0);
+                    // a half's weights lie in its own half of the score buffer
+                    mma_ts(tmem + kTmemO, tmem + kTmemS + buf * 128 + (s >> 2) * 64 + (s & 3) * 8, vd, idesc, t > 0 || s > 0);
                     mma_ts(tmem + kTmemO, tmem + kTmemLo + buf * 64 + s * 8, vd, idesc, true);
                 }
                 mma_commit(smem_u32(&bars->p_free[buf]));
@@ -180,7 +182,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
             mma_commit(smem_u32(&bars->o_full));
             mbar_wait(smem_u32(&bars->o_full), 0);
         }
-    } else {  // ---- scores to weights: warps 0-3 the even tiles, 4-7 the odd ones
+    } else {  // ---- scores to weights
         // Q rows into the swizzled operand layout, zeros beyond the portion
         for (int i = threadIdx.x; i < kTile * CK * 8; i += kSigmoidThreads) {
             const int r = i / (CK * 8), c = i % (CK * 8);
@@ -191,7 +193,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
         }
         fence_async_shared();
         mbar_arrive(smem_u32(&bars->q_full));
-        const int wg = warp >> 2;
+        const int wg = (warp >> 2) & 1, half = warp >> 3;  // tile parity, column half
         const int r = (warp & 3) * 32 + lane;
         const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
         const uint64_t c1 = f2_pack(-a.scale * kLog2e, -a.scale * kLog2e), c0 = f2_pack(-a.head_bias[h] * kLog2e, -a.head_bias[h] * kLog2e);
@@ -202,9 +204,13 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
             if (!ok) break;
             tc_fence_after();
             const int last = pos0 + r - t * kTile;  // last visible column of this row
-            const uint32_t sa = tmem + lanes + kTmemS + wg * 128, la = tmem + lanes + kTmemLo + wg * 64;
-            // 32 score columns to weights; the hi half overlays score columns that have been read (16 c + 15 < 32 (c + 1))
-            auto weigh = [&](uint32_t (&sc)[32], int c) {
+            const uint32_t sa = tmem + lanes + kTmemS + wg * 128 + half * 64, la = tmem + lanes + kTmemLo + wg * 64 + half * 32;
+            // 32 score columns at a time; the hi parts overlay columns of this half that have been read (16 c + 15 < 32 (c + 1))
+#pragma unroll 1
+            for (int c = 0; c < 2; ++c) {
+                uint32_t sc[32];
+                tmem_ld32(sa + c * 32, sc);
+                tmem_wait_ld(sc);
                 uint32_t hi[16], lo[16];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
@@ -212,7 +218,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                     sigmoid2(f2_fma(f2_pack(__uint_as_float(sc[2 * i]), __uint_as_float(sc[2 * i + 1])), c1, c0), p0, p1);
                     split_bf16(p0, p1, hi[i], lo[i]);
                 }
-                const int seen = last - c * 32;
+                const int seen = last - half * 64 - c * 32;
                 if (!__all_sync(~0u, seen >= 31)) {
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
@@ -223,18 +229,6 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                 }
                 tmem_st16(sa + c * 16, hi);
                 tmem_st16(la + c * 16, lo);
-            };
-            // two chunks per turn, the next one's scores on their way meanwhile; rolled: the body has to fit the instruction cache
-            uint32_t even[32], odd[32];
-            tmem_ld32(sa, even);
-#pragma unroll 1
-            for (int c = 0; c < 4; c += 2) {
-                tmem_wait_ld(even);
-                tmem_ld32(sa + (c + 1) * 32, odd);
-                weigh(even, c);
-                tmem_wait_ld(odd);
-                if (c == 0) tmem_ld32(sa + 64, even);
-                weigh(odd, c + 1);
             }
             tmem_wait_st();
             const int valid = keys - t * kTile;
@@ -242,7 +236,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
                 ok = __all_sync(~0u, mbar_wait(smem_u32(&bars->v_full[stage]), (t / NS) & 1, abort));
                 if (!ok) break;
                 const int end = (valid + 15) & ~15;
-                for (int i = r; i < (end - valid) * CV * 8; i += 128) {
+                for (int i = half * 128 + r; i < (end - valid) * CV * 8; i += 256) {
                     const int c = i / ((end - valid) * 8), rest = i % ((end - valid) * 8);
                     *reinterpret_cast<uint4*>(v_s + stage * Sh::kV + c * kColTile + (valid + (rest >> 3)) * 128 + ((rest & 7) << 4)) =
                         make_uint4(0u, 0u, 0u, 0u);
@@ -255,9 +249,7 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
         ok = __all_sync(~0u, ok && mbar_wait(smem_u32(&bars->o_full), 0, abort) && *abort == 0);
         tc_fence_after();
         const bool vec = a.vdim % 8 == 0 && a.out_stride % 8 == 0 && reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
-#pragma unroll
-        for (int c = 0; c < CV; ++c) {
-            const int col = (c * 2 + wg) * 32;
+        if (const int col = (warp >> 2) * 32; col < CV * 64) {  // a warpgroup writes 32 columns of the output
             uint32_t o[32];
             tmem_ld32(tmem + lanes + kTmemO + col, o);
             tmem_wait_ld(o);
