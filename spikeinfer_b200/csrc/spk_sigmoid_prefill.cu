@@ -1,8 +1,9 @@
 // Prefill attention with sigmoid key weights on the fifth-generation tensor cores (tcgen05), bf16, head sizes up to 128.
 //
-// CTA = (128 query tokens of one portion, query head).  Nineteen warps:
-//  * warp 16 copies K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
-//    handful of plain bulk copies (cp.async.bulk), no tensor map, whatever pages the block table names;
+// CTA = (128 query tokens of one portion, query head).  Twenty warps:
+//  * warps 16 and 19 copy K and V: a page of the pool is stored as the swizzled operand tile it becomes, so a 128-key tile is a
+//    handful of plain bulk copies (cp.async.bulk), no tensor map, whatever pages the block table names; one copy per lane, the
+//    next tile's block-table entries are read ahead;
 //  * warp 17 (one thread) issues S = Q K^T into one of two TMEM buffers, warp 18 (one thread) O += P V with P read from TMEM,
 //    so that neither kind of MMA waits behind the other's operands;
 //  * warps 0-15 turn scores into weights: warpgroups 0 and 2 the two column halves of the even tiles, 1 and 3 those of the odd
@@ -21,7 +22,7 @@ using namespace spk_tc;
 constexpr int kTile = 128;            // query rows, and keys per step
 constexpr int kColTile = kTile * 128; // bytes of a 64-channel column tile
 constexpr int kSigmoidThreads = 512;
-constexpr int kThreads = kSigmoidThreads + 96;
+constexpr int kThreads = kSigmoidThreads + 128;
 constexpr uint32_t kTmemS = 0, kTmemLo = 256, kTmemO = 384;  // S/P-hi buffers 2 x 128, P-lo 2 x 64, O up to 128
 constexpr float kLog2e = 1.4426950408889634f;
 
@@ -93,48 +94,50 @@ sigmoid_prefill_kernel(const spk_sigmoid_attn_args a) {
     const uint32_t tmem = bars->tmem;
     volatile int* abort = &bars->abort;
 
-    if (warp == 16) {  // ---- K and V copies
+    if (warp == 16 || warp == 19) {  // ---- K or V copies
+        const bool is_k = warp == 16;
+        const int cols = is_k ? CK : CV;
         const int gran = a.block_size < kTile ? a.block_size : kTile;  // rows per copy
+        const int per = kTile / gran;                                  // copies per column tile, at most 8
+        const int p = lane % per, c = lane / per;                      // this lane's copy
+        const int bs_log2 = 31 - __clz(a.block_size);
         const int32_t* table = a.tables + static_cast<int64_t>(row) * a.table_stride;
-        const SpkPageLayout kl{a.kv_heads, a.block_size, a.k_pad, 1}, vl{a.kv_heads, a.block_size, a.v_pad, 1};
+        const SpkPageLayout lay{a.kv_heads, a.block_size, is_k ? a.k_pad : a.v_pad, 1};
+        const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(is_k ? a.k_pool : a.v_pool);
+        uint8_t* stages = is_k ? k_s : v_s;
+        const int stage_bytes = is_k ? Sh::kK : Sh::kV;
+        uint64_t* full = is_k ? bars->k_full : bars->v_full;
+        uint64_t* free = is_k ? bars->k_free : bars->v_free;
+        auto entry = [&](int t) {
+            const int j = t * kTile + p * gran;
+            return t < tiles && j < keys ? table[j >> bs_log2] : 0;
+        };
+        int next = entry(0);
         int issued = 0;
         for (int t = 0; t < tiles; ++t) {
+            int64_t block = next;
+            next = entry(t + 1);
             const int stage = t % NS;
-            const uint32_t parity = ((t / NS) - 1) & 1;
             const int valid = keys - t * kTile < kTile ? keys - t * kTile : kTile;
             const int n = (valid + gran - 1) / gran;
-            auto copy = [&](const void* pool, const SpkPageLayout& l, int cols, uint8_t* dst, uint64_t* full) {
-                const uint32_t bar = smem_u32(full);
-                if (lane == 0) mbar_expect(bar, static_cast<uint32_t>(n * cols * gran * 128));
-                __syncwarp();
-                for (int i = lane; i < n * cols; i += 32) {
-                    const int p = i % n, c = i / n;
-                    const int j = t * kTile + p * gran;
-                    int64_t block = table[j / a.block_size];
-                    if (block < 0 || block >= a.num_blocks) {
-                        spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
-                        block = 0;
-                    }
-                    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(pool) + spk_page_base(l, block, g) +
-                                               c * (a.block_size << 6) + ((j % a.block_size) << 6);
-                    bulk_load(smem_u32(dst) + c * kColTile + p * gran * 128, src, gran * 128, bar);
-                }
-            };
             // waits are made warp-uniform: a vote also brings the lanes back together
-            if (t >= NS && !__all_sync(~0u, mbar_wait(smem_u32(&bars->k_free[stage]), parity, abort))) break;
-            copy(a.k_pool, kl, CK, k_s + stage * Sh::kK, &bars->k_full[stage]);
-            if (t >= NS && !__all_sync(~0u, mbar_wait(smem_u32(&bars->v_free[stage]), parity, abort))) {
-                mbar_wait(smem_u32(&bars->k_full[stage]), (t / NS) & 1);
-                break;
+            if (t >= NS && !__all_sync(~0u, mbar_wait(smem_u32(free + stage), ((t / NS) - 1) & 1, abort))) break;
+            const uint32_t bar = smem_u32(full + stage);
+            if (lane == 0) mbar_expect(bar, static_cast<uint32_t>(n * cols * gran * 128));
+            __syncwarp();
+            if (p < n && c < cols) {
+                if (block < 0 || block >= a.num_blocks) {
+                    spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
+                    block = 0;
+                }
+                const int j = t * kTile + p * gran;
+                const __nv_bfloat16* src = pool + spk_page_base(lay, block, g) + (c << (bs_log2 + 6)) + ((j & (a.block_size - 1)) << 6);
+                bulk_load(smem_u32(stages + stage * stage_bytes) + c * kColTile + p * gran * 128, src, gran * 128, bar);
             }
-            copy(a.v_pool, vl, CV, v_s + stage * Sh::kV, &bars->v_full[stage]);
             issued = t + 1;
         }
         if (*abort != 0)  // copies in flight land before the CTA's shared memory is given up
-            for (int t = issued > NS ? issued - NS : 0; t < issued; ++t) {
-                mbar_wait(smem_u32(&bars->k_full[t % NS]), (t / NS) & 1);
-                mbar_wait(smem_u32(&bars->v_full[t % NS]), (t / NS) & 1);
-            }
+            for (int t = issued > NS ? issued - NS : 0; t < issued; ++t) mbar_wait(smem_u32(full + t % NS), (t / NS) & 1);
     } else if (warp == 17) {  // ---- scores
         if (lane == 0) {
             constexpr uint32_t idesc = idesc_bf16(kTile, kTile, false, false);
