@@ -15,7 +15,6 @@ namespace {
 
 using namespace spk_tc;
 
-constexpr int kThreads = 256;
 constexpr int C = kDecayChunk;
 
 // x * sigmoid(x): 1 / (1 + 2^(-x log2 e))
@@ -24,12 +23,12 @@ __device__ __forceinline__ float silu_fast(float x) { return x * rcp(1.0f + ex2(
 // Rows of one head of a chunk on their way into a shared-memory tile [64][W + 8]; rows and channels beyond the data are zero.
 // Asynchronous where the rows are 16-byte aligned.  A thread later transforms the very items it copied, so it needs no
 // barrier before that, only its own copies to have landed.
-template <int W>
+template <int W, int NTH>
 __device__ __forceinline__ void fetch(__nv_bfloat16* dst, const __nv_bfloat16* src, int64_t ld, int len, int width, bool vec) {
     constexpr int ST = W + 8;
 #pragma unroll
-    for (int it = 0; it < C * (W / 8) / kThreads; ++it) {
-        const int i = threadIdx.x + it * kThreads;
+    for (int it = 0; it < C * (W / 8) / NTH; ++it) {
+        const int i = threadIdx.x + it * NTH;
         const int r = i / (W / 8), c = (i % (W / 8)) * 8;
         if (vec) {
             const bool live = r < len && c < width;
@@ -43,12 +42,12 @@ __device__ __forceinline__ void fetch(__nv_bfloat16* dst, const __nv_bfloat16* s
 }
 
 // Activation of a fetched tile, in place (PLAIN) and, times the row's decay weight pw[top - row], as a bf16 pair (hi != NULL).
-template <int W, bool PLAIN>
+template <int W, int NTH, bool PLAIN>
 __device__ __forceinline__ void activate(__nv_bfloat16* tile, int len, int silu, __nv_bfloat16* hi, __nv_bfloat16* lo, const float* pw, int top) {
     constexpr int ST = W + 8;
 #pragma unroll
-    for (int it = 0; it < C * (W / 8) / kThreads; ++it) {
-        const int i = threadIdx.x + it * kThreads;
+    for (int it = 0; it < C * (W / 8) / NTH; ++it) {
+        const int i = threadIdx.x + it * NTH;
         const int r = i / (W / 8), c = (i % (W / 8)) * 8;
         const uint4 u = *reinterpret_cast<const uint4*>(tile + r * ST + c);
         const uint32_t w[4] = {u.x, u.y, u.z, u.w};
@@ -78,20 +77,21 @@ __device__ __forceinline__ void activate(__nv_bfloat16* tile, int len, int silu,
     }
 }
 
-// This warp's part of the [D][V] state: 16 rows by COLS columns.
-template <int CD, int CV>
+// A warp's part of the [D][V] state when NW warps share it: 16 rows by COLS columns.
+template <int CD, int CV, int NW>
 struct StateTile {
-    static constexpr int D = CD * 64, V = CV * 64;
-    static constexpr int COLS = CD == 2 ? V : V / 2, NT = COLS / 8;
-    __device__ static int row0(int warp) { return (CD == 2 ? warp : warp & 3) * 16; }
-    __device__ static int col0(int warp) { return CD == 2 ? 0 : (warp >> 2) * COLS; }
+    static constexpr int D = CD * 64, V = CV * 64, THREADS = 32 * NW;
+    static constexpr int GROUPS = D / 16, COLS = V * GROUPS / NW, NT = COLS / 8;
+    static_assert(NT % 2 == 0, "pairs of column tiles");
+    __device__ static int row0(int warp) { return (warp % GROUPS) * 16; }
+    __device__ static int col0(int warp) { return (warp / GROUPS) * COLS; }
 };
 
 // acc += K^T V over the chunk's 64 tokens (K as the pair hi + lo)
-template <int CD, int CV>
-__device__ __forceinline__ void add_outer(float (&acc)[StateTile<CD, CV>::NT][4], const __nv_bfloat16* hi, const __nv_bfloat16* lo,
+template <int CD, int CV, int NW>
+__device__ __forceinline__ void add_outer(float (&acc)[StateTile<CD, CV, NW>::NT][4], const __nv_bfloat16* hi, const __nv_bfloat16* lo,
                                           const __nv_bfloat16* v, int warp, int lane) {
-    using T = StateTile<CD, CV>;
+    using T = StateTile<CD, CV, NW>;
     constexpr int SK = T::D + 8, SV = T::V + 8;
     const int m = lane >> 3, mr = lane & 7;
 #pragma unroll
@@ -112,10 +112,10 @@ __device__ __forceinline__ void add_outer(float (&acc)[StateTile<CD, CV>::NT][4]
     }
 }
 
-template <int CD, int CV>
-__global__ void __launch_bounds__(kThreads, 2)
+template <int CD, int CV, int NW>
+__global__ void __launch_bounds__(32 * NW, 2)
 decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool vec_v) {
-    using T = StateTile<CD, CV>;
+    using T = StateTile<CD, CV, NW>;
     constexpr int SK = T::D + 8, SV = T::V + 8;
     extern __shared__ __align__(16) __nv_bfloat16 sm[];
     __nv_bfloat16* hi = sm;
@@ -130,8 +130,8 @@ decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
     float acc[T::NT][4] = {};
     auto fetch_chunk = [&](int c0, int buf) {
         const int len = min(C, ci.len - c0);
-        fetch<T::D>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
-        fetch<T::V>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
+        fetch<T::D, T::THREADS>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::V, T::THREADS>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
         cp_async_commit();
     };
     fetch_chunk(0, 0);
@@ -139,11 +139,11 @@ decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
         const int len = min(C, ci.len - c0);
         cp_async_wait_all();
         __syncthreads();  // the previous chunk's products have read their operands
-        activate<T::D, false>(kb + buf * C * SK, len, a.silu, hi, lo, pw, ci.len - 1 - c0);
-        activate<T::V, true>(vb + buf * C * SV, len, a.silu, nullptr, nullptr, pw, 0);
+        activate<T::D, T::THREADS, false>(kb + buf * C * SK, len, a.silu, hi, lo, pw, ci.len - 1 - c0);
+        activate<T::V, T::THREADS, true>(vb + buf * C * SV, len, a.silu, nullptr, nullptr, pw, 0);
         if (c0 + C < ci.len) fetch_chunk(c0 + C, buf ^ 1);
         __syncthreads();
-        add_outer<CD, CV>(acc, hi, lo, vb + buf * C * SV, warp, lane);
+        add_outer<CD, CV, NW>(acc, hi, lo, vb + buf * C * SV, warp, lane);
     }
     float* U = a.workspace + (static_cast<int64_t>(blockIdx.x) * a.heads + h) * a.dim * a.vdim;
     const int gid = lane >> 2, tig = lane & 3;
@@ -156,10 +156,10 @@ decay_span_sum_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
         }
 }
 
-template <int CD, int CV>
-__global__ void __launch_bounds__(kThreads, CD * CV == 1 ? 2 : 1)
+template <int CD, int CV, int NW>
+__global__ void __launch_bounds__(32 * NW, CD * CV == 1 ? 2 : 1)
 decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool vec_v) {
-    using T = StateTile<CD, CV>;
+    using T = StateTile<CD, CV, NW>;
     constexpr int SK = T::D + 8, SV = T::V + 8;
     extern __shared__ __align__(16) __nv_bfloat16 sm[];
     __nv_bfloat16* qb = sm;               // two stages each of q, k and v
@@ -173,7 +173,7 @@ decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int m = lane >> 3, mr = lane & 7;
     const SpkChunk ci = spk_chunk(a, blockIdx.x);
-    for (int i = threadIdx.x; i <= C; i += kThreads) pw[i] = a.decay_pow[static_cast<int64_t>(h) * (kDecayMaxSpan + 1) + i];
+    for (int i = threadIdx.x; i <= C; i += T::THREADS) pw[i] = a.decay_pow[static_cast<int64_t>(h) * (kDecayMaxSpan + 1) + i];
     const __nv_bfloat16* qs = static_cast<const __nv_bfloat16*>(a.q) + ci.start * a.ld + static_cast<int64_t>(h) * a.dim;
     const __nv_bfloat16* ks = static_cast<const __nv_bfloat16*>(a.k) + ci.start * a.ld + static_cast<int64_t>(h) * a.dim;
     const __nv_bfloat16* vs = static_cast<const __nv_bfloat16*>(a.v) + ci.start * a.ld + static_cast<int64_t>(h) * a.vdim;
@@ -187,13 +187,13 @@ decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
             S[n][i] = d < a.dim && e < a.vdim ? S0[static_cast<int64_t>(d) * a.vdim + e] : 0.0f;
         }
     const int i0 = (warp & 3) * 16;                 // this warp's 16 tokens
-    constexpr int OC = T::V / 2, ON = OC / 8;       // and its half of the output columns
+    constexpr int OC = T::V / (NW / 4), ON = OC / 8;  // and its share of the output columns
     const int e0 = (warp >> 2) * OC;
     auto fetch_chunk = [&](int c0, int buf) {
         const int len = min(C, ci.len - c0);
-        fetch<T::D>(qb + buf * C * SK, qs + c0 * a.ld, a.ld, len, a.dim, vec_k);
-        fetch<T::D>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
-        fetch<T::V>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
+        fetch<T::D, T::THREADS>(qb + buf * C * SK, qs + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::D, T::THREADS>(kb + buf * C * SK, ks + c0 * a.ld, a.ld, len, a.dim, vec_k);
+        fetch<T::V, T::THREADS>(vb + buf * C * SV, vs + c0 * a.ld, a.ld, len, a.vdim, vec_v);
         cp_async_commit();
     };
     fetch_chunk(0, 0);
@@ -203,9 +203,9 @@ decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
         __nv_bfloat16 *q = qb + buf * C * SK, *k = kb + buf * C * SK, *v = vb + buf * C * SV;
         cp_async_wait_all();
         __syncthreads();  // the previous chunk's reads are done (and pw is there)
-        activate<T::D, true>(q, len, a.silu, nullptr, nullptr, pw, 0);
-        activate<T::D, true>(k, len, a.silu, more ? hi : nullptr, lo, pw, len - 1);
-        activate<T::V, true>(v, len, a.silu, nullptr, nullptr, pw, 0);
+        activate<T::D, T::THREADS, true>(q, len, a.silu, nullptr, nullptr, pw, 0);
+        activate<T::D, T::THREADS, true>(k, len, a.silu, more ? hi : nullptr, lo, pw, len - 1);
+        activate<T::V, T::THREADS, true>(v, len, a.silu, nullptr, nullptr, pw, 0);
         if (more) fetch_chunk(c0 + C, buf ^ 1);
 #pragma unroll
         for (int n = 0; n < T::NT; ++n)
@@ -301,18 +301,18 @@ decay_span_out_kernel(const spk_decay_attn_args a, const bool vec_k, const bool 
             for (int n = 0; n < T::NT; ++n)
 #pragma unroll
                 for (int i = 0; i < 4; ++i) S[n][i] *= w;
-            add_outer<CD, CV>(S, hi, lo, v, warp, lane);
+            add_outer<CD, CV, NW>(S, hi, lo, v, warp, lane);
         }
     }
 }
 
 template <typename F>
-int with_smem(F fn, size_t bytes, cudaStream_t s, const spk_decay_attn_args& a) {
+int with_smem(F fn, int threads, size_t bytes, cudaStream_t s, const spk_decay_attn_args& a) {
     const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     auto aligned = [&](const void* p, int width) { return reinterpret_cast<uintptr_t>(p) % 16 == 0 && a.ld % 8 == 0 && width % 8 == 0; };
     const bool vk = aligned(a.k, a.dim) && (a.q == nullptr || aligned(a.q, a.dim)), vv = aligned(a.v, a.vdim);
-    fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, vk, vv);
+    fn<<<dim3(a.n_chunks, a.heads), threads, bytes, s>>>(a, vk, vv);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -320,14 +320,15 @@ int with_smem(F fn, size_t bytes, cudaStream_t s, const spk_decay_attn_args& a) 
 template <int CD, int CV>
 int sums(const spk_decay_attn_args& a, cudaStream_t s) {
     constexpr size_t bytes = 2 * C * (4 * (CD * 64 + 8) + 2 * (CV * 64 + 8));
-    return with_smem(decay_span_sum_kernel<CD, CV>, bytes, s, a);
+    return with_smem(decay_span_sum_kernel<CD, CV, 8>, 256, bytes, s, a);
 }
 
 template <int CD, int CV>
 int outputs(const spk_decay_attn_args& a, cudaStream_t s) {
     constexpr size_t bytes = 2 * C * (6 * (CD * 64 + 8) + 2 * (CV * 64 + 8)) + 4 * CD * 64 * (CV * 64 + 8) + 4 * (C + 8);
     static_assert(bytes <= 227 * 1024, "shared memory");
-    return with_smem(decay_span_out_kernel<CD, CV>, bytes, s, a);
+    constexpr int NW = CD * CV == 4 ? 16 : 8;  // one CTA of sixteen warps per SM, or two of eight
+    return with_smem(decay_span_out_kernel<CD, CV, NW>, 32 * NW, bytes, s, a);
 }
 
 }  // namespace

@@ -3,10 +3,9 @@
 
 #include "spk_common.cuh"
 
-// Both pools tiled, 16-bit, at most 128 channels, pages of a multiple of 16 rows.
+// Both pools tiled, 16-bit, at most 128 channels, pages of 16 rows or a larger power of two.
 static inline bool spk_attn_tensor_form(int dtype, int k_pad, int v_pad, int k_tiled, int v_tiled, int block_size) {
-    return dtype == SPK_BF16 && k_tiled && v_tiled && k_pad <= 128 && v_pad <= 128 && block_size % 16 == 0 &&
-           (block_size <= 128 ? 128 % block_size == 0 : block_size % 128 == 0);
+    return dtype == SPK_BF16 && k_tiled && v_tiled && k_pad <= 128 && v_pad <= 128 && block_size >= 16 && (block_size & (block_size - 1)) == 0;
 }
 
 int spk_sigmoid_prefill_launch(const spk_sigmoid_attn_args& a, cudaStream_t s);
