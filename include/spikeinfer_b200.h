@@ -596,6 +596,236 @@ typedef struct spk_gated_norm_args {
 } spk_gated_norm_args;
 int spk_gated_norm(const spk_gated_norm_args* args, void* stream);
 
+/* ---------------------------------------------------------------------------
+ * Pre-norm decoder operators: residual stream in 32 bits with parallel branches, experts chosen by a token table, attention over
+ * a shared latent, gated delta rule with per-channel decay.  Same conventions as above.
+ * ------------------------------------------------------------------------- */
+
+/* One layer boundary of a decoder whose branches read the same x.  y = embed_scale * embed[ids[t]] when ids != NULL, else
+ * y = x + delta + pair_scale * sum_j pairs[pair_slots[t, j]] (delta or pairs may be NULL; a negative slot counts as zero).
+ * x_out <- y (may alias x); out1 <- y / rms(y) * w1; out2 <- y / rms(y) * w2 (w1, w2 may be NULL).
+ * out2_slots NULL: out2 is [n, width].  Otherwise row t goes to rows out2_slots[t, 0 .. out2_top) (negative: nowhere) of a
+ * matrix of out2_rows rows, plain, or with out2_tiled as the operand tiles of spk_experts (below). */
+typedef struct spk_rms_residual_args {
+    const float* x;
+    float* x_out;
+    const void* delta;          /* [n, width] in delta_dtype */
+    const void* embed;          /* [vocab, width] in dtype   */
+    const int64_t* ids;
+    int64_t vocab;
+    const float* pairs;         /* [pair_rows, width] */
+    const int32_t* pair_slots;  /* [n, pair_top] */
+    const float* w1;
+    void* out1;
+    const float* w2;
+    void* out2;
+    const int32_t* out2_slots;
+    int64_t pair_rows;
+    int64_t out2_rows;
+    int64_t n;
+    int64_t width;
+    int32_t pair_top, out2_top, out2_tiled;
+    int32_t dtype;
+    int32_t delta_dtype;
+    float embed_scale;
+    float pair_scale;
+    float eps;
+    uint32_t* status;
+} spk_rms_residual_args;
+int spk_rms_residual(const spk_rms_residual_args* args, void* stream);
+
+/* out[t, c] = gelu(z[t, c]), the tanh form; out has row stride out_stride, z is contiguous [n, width]. */
+int spk_gelu_tanh(const void* z, void* out, int64_t out_stride, int64_t n, int64_t width, int dtype, void* stream);
+
+/* Routing by token id for all expert layers of a step at once.  layers (device, 8 int64 each): address of the int32 table
+ * [vocab, top], top, experts, first column of the layer in slots' per-token total, first entry in segs, three reserved.
+ * slots [sum of top * n] (layer l's [n, top] at n * its first column) <- row of every (token, choice) pair in the layer's sorted
+ * matrix, -1 for tokens that take no part; segs [2 * sum of experts] (layer l at its first entry) <- per expert (first row, rows);
+ * first rows are multiples of eight. */
+typedef struct spk_expert_route_args {
+    const int64_t* layers;
+    const int64_t* ids;
+    const int32_t* active;      /* [n] or NULL */
+    int32_t* slots;
+    int32_t* segs;
+    int64_t n;
+    int64_t vocab;
+    int32_t n_layers;
+    int32_t max_experts;
+    uint32_t* status;
+} spk_expert_route_args;
+int spk_expert_route(const spk_expert_route_args* args, void* stream);
+/* Rows a sorted matrix needs for n tokens: segments padded to eight rows, and what a tile may touch beyond the last. */
+int64_t spk_expert_rows(int64_t n, int top, int experts);
+
+/* One product of every expert with its rows of a sorted matrix.
+ * gated != 0: out[r, f] = silu(x[r] . gate_e[f]) * (x[r] . up_e[f]), in dtype;  otherwise out[r, f] = x[r] . w_e[f], 32-bit.
+ * SPK_F32: x [rows, k], weights [experts][out_features (gate), out_features (up)][k], out [rows, out_features].
+ * SPK_BF16: operand tiles.  A matrix of R rows and K columns is stored as ceil(K / 64) column tiles of R x 128 bytes, the
+ * 16-byte group g of row r at group g ^ (r & 7); columns beyond K are zero.  x and the gated output are such matrices of `rows` rows;
+ * weights are [experts][blocks][ceil(k / 64)] pairs of such 128-row tiles: gate and up rows of 128 features (gated), or 256
+ * consecutive features. */
+typedef struct spk_experts_args {
+    const void* x;
+    const void* w;
+    void* out;
+    const int32_t* segs;        /* [experts][2] */
+    int64_t rows;
+    int64_t pairs;              /* upper bound of the rows in use (tokens * top) */
+    int32_t experts, k, out_features;
+    int32_t gated;
+    int32_t dtype;
+    int32_t _pad;
+    uint32_t* status;
+} spk_experts_args;
+int spk_experts(const spk_experts_args* args, void* stream);
+
+/* Cache row of the latent attention: `rank` latent channels, then (from channel rank_pad) rot_dim rotated ones.  A pool is
+ * [num_blocks][1][block_size][rank_pad + rot_pad]; tiled as above, or plain with rank_pad == rank, rot_pad == rot_dim.
+ *
+ * Per token: cq_out [n, q_rank] <- cq / rms(cq) * w_q; the pool row of slot_mapping[t] <- kv[0 .. rank) / rms * w_kv, and
+ * kv[rank .. rank + rot_dim) rotated by the table at positions[t].  kv NULL: only cq. */
+typedef struct spk_latent_prepare_args {
+    const void* cq;             /* row t at cq + t * ld */
+    const void* kv;             /* row t at kv + t * ld */
+    int64_t ld;
+    const float* w_q;
+    const float* w_kv;
+    void* cq_out;
+    void* pool;
+    const float* rot_table;     /* float2 [rot_positions, rot_dim / 2] */
+    const int64_t* positions;
+    const int64_t* slot_mapping;
+    int64_t rot_positions;
+    int64_t n;
+    int64_t num_blocks;
+    int32_t q_rank, rank, rot_dim, rank_pad, rot_pad, tiled;
+    int32_t block_size;
+    int32_t dtype;
+    float eps;
+    float _pad;
+    uint32_t* status;
+} spk_latent_prepare_args;
+int spk_latent_prepare(const spk_latent_prepare_args* args, void* stream);
+
+/* Queries that read the cache rows as they are: out[t, h, 0 .. rank) = W_uk[h]^T q[t, h, 0 .. dim), out[t, h, rank_pad ..) = the
+ * rotated q[t, h, dim ..); padding zero.  w_uk [heads * dim, rank]. */
+typedef struct spk_latent_query_args {
+    const void* q;              /* [n, heads, dim + rot_dim] */
+    const void* w_uk;
+    void* out;                  /* [n, heads, rank_pad + rot_pad] */
+    const float* rot_table;
+    const int64_t* positions;
+    int64_t rot_positions;
+    int64_t n;
+    int32_t heads, dim, rank, rot_dim, rank_pad, rot_pad;
+    int32_t dtype;
+    int32_t _pad;
+    uint32_t* status;
+} spk_latent_query_args;
+int spk_latent_query(const spk_latent_query_args* args, void* stream);
+
+/* Softmax attention of such queries over the cache rows: per token, head and key range the sum of exp(score - max) * latent
+ * (partials [n][splits][heads][rank]) and (max, sum of exp(score - max)) (stats [n][splits][heads][2]); scores are scaled.
+ * Prefill form: token t belongs to row token_rows[t] and sees positions[t] + 1 keys.  Decode form (token_rows NULL): row t,
+ * seq_lens[t] keys, inactive rows none.  A token's keys are cut into ranges of spk_split_keys(keys, splits) (csrc/spk_dense.cuh);
+ * ranges without keys are left as they are. */
+typedef struct spk_latent_attn_args {
+    const void* q;
+    const void* pool;
+    const int32_t* tables;
+    const int32_t* seq_lens;
+    const int32_t* active;
+    const int32_t* token_rows;
+    const int64_t* positions;
+    float* partials;
+    float* stats;
+    int64_t table_stride;
+    int64_t table_rows;
+    int64_t max_blocks;
+    int64_t n;
+    int64_t num_blocks;
+    int32_t splits;
+    int32_t heads, rank, rot_dim, rank_pad, rot_pad, tiled;
+    int32_t block_size;
+    int32_t dtype;
+    float scale;
+    uint32_t* status;
+} spk_latent_attn_args;
+int spk_latent_attn(const spk_latent_attn_args* args, void* stream);
+/* Key ranges a call of n tokens with at most max_keys keys should be cut into (1 or more). */
+int spk_latent_attn_splits(int dtype, int rank, int rot_dim, int rank_pad, int rot_pad, int tiled, int block_size, int64_t n, int heads,
+                           int64_t max_keys);
+
+/* out[t, h * vdim + e] = sigmoid(gate[t, h * vdim + e]) * (W_uv[h] . o)[e], o = the ranges' sums over (their denominators +
+ * exp(sink[h])).  w_uv [heads * vdim, rank]. */
+typedef struct spk_latent_out_args {
+    const float* partials;
+    const float* stats;
+    const float* sink;
+    const void* w_uv;
+    const void* gate;           /* row t at gate + t * gate_stride */
+    void* out;                  /* row t at out + t * out_stride */
+    const int32_t* seq_lens;    /* decode form */
+    const int32_t* active;
+    const int64_t* positions;   /* prefill form (seq_lens NULL): positions[t] + 1 keys */
+    int64_t gate_stride;
+    int64_t out_stride;
+    int64_t n;
+    int32_t splits, heads, vdim, rank;
+    int32_t dtype;
+    int32_t _pad;
+    uint32_t* status;
+} spk_latent_out_args;
+int spk_latent_out(const spk_latent_out_args* args, void* stream);
+
+/* Gated delta rule with one decay per head and key channel:
+ *   q, k, v <- silu(causal convolution of the projections, `taps` taps per channel);  q, k <- unit vectors per head, q * dim^-1/2;
+ *   S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  g = exp(-exp(a_log) softplus(a + dt_bias)), beta = sigmoid(b);
+ *   out = o / rms(o) * w_norm * sigmoid(gate).
+ * Head h reads q and k of head h / (heads / kv_heads).  state: 32-bit [state_rows][heads][dim][vdim].  conv_state: 32-bit
+ * [state_rows][taps][kv_heads * dim * 2 + heads * vdim], a ring: the projections of position p (q, k, v channels) in slot p % taps.
+ * a [n, heads * dim] and gate [n, heads * vdim] are column ranges with row stride ld2. */
+typedef struct spk_delta_args {
+    const void* q;
+    const void* k;
+    const void* v;
+    const void* b;
+    const void* a;
+    const void* gate;
+    int64_t ld;                 /* q, k, v, b */
+    int64_t ld2;                /* a, gate */
+    const float* conv_q;        /* [channels][taps], the last tap is the current token's */
+    const float* conv_k;
+    const float* conv_v;
+    const float* a_log;
+    const float* dt_bias;
+    const float* w_norm;
+    float* state;
+    float* conv_state;
+    int64_t state_rows;
+    const int64_t* positions;
+    const int32_t* active;      /* decode form */
+    void* out;                  /* row t, head h at out + t * out_stride + h * vdim */
+    int64_t out_stride;
+    const int32_t* chunks;      /* prefill form: int32 [n_chunks][4] = (first token, tokens, portion, index in the portion) */
+    const int32_t* portions;    /* int32 [n_portions][4] = (first token, tokens, row, tokens before) */
+    void* workspace;
+    int64_t workspace_bytes;
+    int64_t n;
+    int32_t n_chunks, n_portions;
+    int32_t heads, kv_heads, dim, vdim, taps;
+    int32_t dtype;
+    float eps;
+    float _pad;
+    uint32_t* status;
+} spk_delta_args;
+int spk_delta_step(const spk_delta_args* args, void* stream);
+/* Tokens per chunk of the prefill form, and its workspace. */
+int spk_delta_chunk_tokens(int dtype, int dim, int vdim);
+int64_t spk_delta_workspace_bytes(int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim);
+int spk_delta_prefill(const spk_delta_args* args, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

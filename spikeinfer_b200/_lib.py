@@ -133,6 +133,60 @@ class GatedNormArgs(Structure):
                        "left_width dtype; f eps scale left_scale")
 
 
+class RmsResidualArgs(Structure):
+    """Mirror of ``spk_rms_residual_args``."""
+
+    _fields_ = _fields("p x x_out delta embed ids; l vocab; p pairs pair_slots w1 out1 w2 out2 out2_slots; l pair_rows out2_rows n width; "
+                       "i pair_top out2_top out2_tiled dtype delta_dtype; f embed_scale pair_scale eps; p status")
+
+
+class ExpertRouteArgs(Structure):
+    """Mirror of ``spk_expert_route_args``."""
+
+    _fields_ = _fields("p layers ids active slots segs; l n vocab; i n_layers max_experts; p status")
+
+
+class ExpertsArgs(Structure):
+    """Mirror of ``spk_experts_args``."""
+
+    _fields_ = _fields("p x w out segs; l rows pairs; i experts k out_features gated dtype _pad; p status")
+
+
+class LatentPrepareArgs(Structure):
+    """Mirror of ``spk_latent_prepare_args``."""
+
+    _fields_ = _fields("p cq kv; l ld; p w_q w_kv cq_out pool rot_table positions slot_mapping; l rot_positions n num_blocks; "
+                       "i q_rank rank rot_dim rank_pad rot_pad tiled block_size dtype; f eps _pad; p status")
+
+
+class LatentQueryArgs(Structure):
+    """Mirror of ``spk_latent_query_args``."""
+
+    _fields_ = _fields("p q w_uk out rot_table positions; l rot_positions n; i heads dim rank rot_dim rank_pad rot_pad dtype _pad; p status")
+
+
+class LatentAttnArgs(Structure):
+    """Mirror of ``spk_latent_attn_args``."""
+
+    _fields_ = _fields("p q pool tables seq_lens active token_rows positions partials stats; l table_stride table_rows max_blocks n num_blocks; "
+                       "i splits heads rank rot_dim rank_pad rot_pad tiled block_size dtype; f scale; p status")
+
+
+class LatentOutArgs(Structure):
+    """Mirror of ``spk_latent_out_args``."""
+
+    _fields_ = _fields("p partials stats sink w_uv gate out seq_lens active positions; l gate_stride out_stride n; "
+                       "i splits heads vdim rank dtype _pad; p status")
+
+
+class DeltaArgs(Structure):
+    """Mirror of ``spk_delta_args``."""
+
+    _fields_ = _fields("p q k v b a gate; l ld ld2; p conv_q conv_k conv_v a_log dt_bias w_norm state conv_state; l state_rows; "
+                       "p positions active out; l out_stride; p chunks portions workspace; l workspace_bytes n; "
+                       "i n_chunks n_portions heads kv_heads dim vdim taps dtype; f eps _pad; p status")
+
+
 # name -> (restype, argtypes); every symbol include/spikeinfer_b200.h declares
 I64P = POINTER(c_int64)
 SIGNATURES = {
@@ -204,6 +258,20 @@ SIGNATURES = {
     "spk_decay_attn_step": (c_int, [POINTER(DecayAttnArgs), c_void_p]),
     "spk_decay_attn_chunks": (c_int, [POINTER(DecayAttnArgs), c_void_p]),
     "spk_gated_norm": (c_int, [POINTER(GatedNormArgs), c_void_p]),
+    "spk_rms_residual": (c_int, [POINTER(RmsResidualArgs), c_void_p]),
+    "spk_gelu_tanh": (c_int, [c_void_p, c_void_p, c_int64, c_int64, c_int64, c_int, c_void_p]),
+    "spk_expert_route": (c_int, [POINTER(ExpertRouteArgs), c_void_p]),
+    "spk_expert_rows": (c_int64, [c_int64, c_int, c_int]),
+    "spk_experts": (c_int, [POINTER(ExpertsArgs), c_void_p]),
+    "spk_latent_prepare": (c_int, [POINTER(LatentPrepareArgs), c_void_p]),
+    "spk_latent_query": (c_int, [POINTER(LatentQueryArgs), c_void_p]),
+    "spk_latent_attn_splits": (c_int, [c_int] * 7 + [c_int64, c_int, c_int64]),
+    "spk_latent_attn": (c_int, [POINTER(LatentAttnArgs), c_void_p]),
+    "spk_latent_out": (c_int, [POINTER(LatentOutArgs), c_void_p]),
+    "spk_delta_step": (c_int, [POINTER(DeltaArgs), c_void_p]),
+    "spk_delta_chunk_tokens": (c_int, [c_int] * 3),
+    "spk_delta_workspace_bytes": (c_int64, [c_int64] + [c_int] * 5),
+    "spk_delta_prefill": (c_int, [POINTER(DeltaArgs), c_void_p]),
     "spk_meta_release": (c_int, [c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
 }

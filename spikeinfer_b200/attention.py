@@ -99,9 +99,21 @@ class PrefillPlan:
         self.device = device
         self._tiles: dict[int, torch.Tensor] = {}
         self._chunks: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
+        self._portions: torch.Tensor | None = None
 
     def _table(self, entries: list[tuple[int, int, int, int]]) -> torch.Tensor:
         return torch.tensor(entries, dtype=torch.int32).to(self.device)
+
+    def portions(self) -> torch.Tensor:
+        """int32 ``[portions, 4]``: (first token, tokens, row, tokens before this portion)."""
+        if self._portions is None:
+            self._portions = self._table([(s, n, row, ctx) for s, n, ctx, row in zip(self.starts, self.lens, self.contexts, self.rows)])
+        return self._portions
+
+    @property
+    def most_keys(self) -> int:
+        """Keys the last token of the longest sequence sees."""
+        return max(c + n for c, n in zip(self.contexts, self.lens))
 
     def tiles(self, tokens: int) -> torch.Tensor:
         """int32 ``[n, 4]``: (first token, tokens, row, position of the first token), longest context first."""

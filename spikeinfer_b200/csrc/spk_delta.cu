@@ -1,0 +1,498 @@
+// Gated delta rule with one decay per head and key channel, and everything around it that enters the recurrence.
+//
+//   q, k, v <- silu(short causal convolution);  q, k <- unit vectors, q * dim^-1/2
+//   S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  out = o / rms(o) * w * sigmoid(gate)
+//
+//  * delta_step_kernel: one token per row (decode).  A CTA owns a (head, row): it convolves, normalises, decays, updates and reads the
+//    state and writes the gated output; the state is read and written once.
+//  * prefill: delta_prepare_kernel (convolutions, unit vectors, decays, step sizes), delta_scan_kernel (the recurrence, columns of the
+//    state in registers, tokens one after the other) and delta_out_kernel (norm and gate).
+// The convolution's past lives in a ring of `taps` slots per row: a step writes its own slot and reads the others, so heads that
+// share a key need no order among themselves.
+#include "spk_delta.cuh"
+#include "spk_tensor.cuh"
+
+namespace {
+
+using namespace spk_tc;
+
+constexpr int kThreads = 256;
+constexpr int kKeep = 16;  // state rows a thread of the step kernel keeps in registers
+
+// ---- decode ------------------------------------------------------------------------------------------------------------
+template <int W>
+__device__ __forceinline__ void load_state(float (&s)[W], const float* p) {
+    if (W == 4) {
+        const float4 f = __ldcs(reinterpret_cast<const float4*>(p));
+        s[0] = f.x; s[1 % W] = f.y; s[2 % W] = f.z; s[3 % W] = f.w;
+    } else {
+        s[0] = *p;
+    }
+}
+
+// CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  KEEP: a thread's
+// share of the state stays in registers between the two products; otherwise it is read twice.
+template <typename T, int W, bool KEEP>
+__global__ void __launch_bounds__(kThreads)
+delta_step_kernel(const spk_delta_args a) {
+    extern __shared__ float sm[];
+    __shared__ float part[3 * 32];
+    const int h = blockIdx.x;
+    const int64_t row = blockIdx.y;
+    const int dim = a.dim, vdim = a.vdim, rep = a.heads / a.kv_heads, g = h / rep;
+    T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(h) * vdim;
+    if (a.active != nullptr && a.active[row] != 1) {
+        for (int e = threadIdx.x; e < vdim; e += kThreads) out[e] = spk_from_float<T>(0.0f);
+        return;
+    }
+    float* q = sm;                 // [dim]
+    float* k = q + dim;            // [dim]
+    float* dec = k + dim;          // [dim]
+    float* v = dec + dim;          // [vdim]; the outputs afterwards
+    float* red = v + vdim;         // [slices][vdim]
+    float* S = a.state + (row * a.heads + h) * static_cast<int64_t>(dim) * vdim;
+    const int cols = vdim / W;
+    const int slices = cols < kThreads ? kThreads / cols : 1;
+    const int slice = slices > 1 ? threadIdx.x / cols : 0;
+    const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
+    const bool mine = slice < slices;
+    float s[KEEP ? kKeep : 1][W];
+    if (KEEP && mine) {  // on its way before the projections are looked at
+#pragma unroll
+        for (int u = 0; u < kKeep; ++u) {
+            const int d = slice + u * slices;
+            if (d < dim) load_state<W>(s[u], S + static_cast<int64_t>(d) * vdim + first * W);
+        }
+    }
+    const SpkDeltaShape sh = spk_delta_shape(a);
+    const int64_t pos = a.positions[row];
+    float* ring = a.conv_state + row * a.taps * sh.channels;
+    const int now_slot = static_cast<int>(pos % a.taps);
+    auto channel = [&](const void* src, int64_t c, int at, const float* w, bool keep) {  // one channel's convolution; `at`: its place in the ring
+        const float x = spk_to_float<T>(static_cast<const T*>(src)[row * a.ld + c]);
+        if (keep) ring[now_slot * sh.channels + at] = x;
+        return spk_conv_silu(w + c * a.taps, a.taps, x, [&](int back) {
+            const int64_t p = pos - back;
+            return p >= 0 ? ring[(p % a.taps) * sh.channels + at] : 0.0f;
+        });
+    };
+    const bool leader = h % rep == 0;
+    const float rate = expf(a.a_log[h]);
+    float sums[3] = {0.0f, 0.0f, 0.0f};
+    for (int c = threadIdx.x; c < dim; c += kThreads) {
+        const float x = channel(a.q, g * dim + c, g * dim + c, a.conv_q, leader);
+        const float y = channel(a.k, g * dim + c, sh.qk + g * dim + c, a.conv_k, leader);
+        q[c] = x;
+        k[c] = y;
+        sums[0] = fmaf(x, x, sums[0]);
+        sums[1] = fmaf(y, y, sums[1]);
+        const int64_t i = static_cast<int64_t>(h) * dim + c;
+        dec[c] = expf(spk_log_decay(spk_to_float<T>(static_cast<const T*>(a.a)[row * a.ld2 + i]) + a.dt_bias[i], rate));
+    }
+    for (int c = threadIdx.x; c < vdim; c += kThreads)
+        v[c] = channel(a.v, static_cast<int64_t>(h) * vdim + c, 2 * sh.qk + h * vdim + c, a.conv_v, true);
+    spk_block_sum<3>(sums, part);  // its barriers also publish q, k, v and the decays
+    const float qi = 1.0f / (sqrtf(sums[0] + 1e-6f) * sqrtf(static_cast<float>(dim))), ki = 1.0f / sqrtf(sums[1] + 1e-6f);
+    const float beta = spk_sigmoid(spk_to_float<T>(static_cast<const T*>(a.b)[row * a.ld + h]));
+    float square[1] = {0.0f};
+    for (int c0 = 0; c0 < cols; c0 += kThreads) {
+        const int c = c0 + first;
+        const bool in = mine && c < cols;
+        float acc[W] = {};
+        if (in) {
+            if (KEEP) {
+#pragma unroll
+                for (int u = 0; u < kKeep; ++u) {
+                    const int d = slice + u * slices;
+                    if (d < dim) {
+                        const float gd = dec[d], kd = k[d] * ki;
+#pragma unroll
+                        for (int i = 0; i < W; ++i) {
+                            s[u][i] *= gd;
+                            acc[i] = fmaf(kd, s[u][i], acc[i]);
+                        }
+                    }
+                }
+            } else {
+                for (int d = slice; d < dim; d += slices) {
+                    float x[W];
+                    load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
+                    const float w = dec[d] * (k[d] * ki);
+#pragma unroll
+                    for (int i = 0; i < W; ++i) acc[i] = fmaf(w, x[i], acc[i]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < W; ++i) red[slice * vdim + c * W + i] = acc[i];
+        }
+        __syncthreads();
+        float u_[W] = {};
+        if (in) {
+#pragma unroll
+            for (int i = 0; i < W; ++i) {
+                float sk = 0.0f;
+                for (int z = 0; z < slices; ++z) sk += red[z * vdim + c * W + i];
+                u_[i] = beta * (v[c * W + i] - sk);
+                acc[i] = 0.0f;
+            }
+        }
+        __syncthreads();  // the first product's parts have been read
+        if (in) {
+            auto update = [&](float (&x)[W], int d) {
+                const float kd = k[d] * ki, qd = q[d] * qi;
+#pragma unroll
+                for (int i = 0; i < W; ++i) {
+                    x[i] = fmaf(kd, u_[i], x[i]);
+                    acc[i] = fmaf(qd, x[i], acc[i]);
+                }
+                float* dst = S + static_cast<int64_t>(d) * vdim + c * W;
+                if (W == 4) __stcs(reinterpret_cast<float4*>(dst), make_float4(x[0], x[1 % W], x[2 % W], x[3 % W]));
+                else *dst = x[0];
+            };
+            if (KEEP) {
+#pragma unroll
+                for (int u = 0; u < kKeep; ++u) {
+                    const int d = slice + u * slices;
+                    if (d < dim) update(s[u], d);
+                }
+            } else {
+                for (int d = slice; d < dim; d += slices) {
+                    float x[W];
+                    load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
+#pragma unroll
+                    for (int i = 0; i < W; ++i) x[i] *= dec[d];
+                    update(x, d);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < W; ++i) red[slice * vdim + c * W + i] = acc[i];
+        }
+        __syncthreads();
+        if (in && slice == 0) {
+#pragma unroll
+            for (int i = 0; i < W; ++i) {
+                float o = 0.0f;
+                for (int z = 0; z < slices; ++z) o += red[z * vdim + c * W + i];
+                v[c * W + i] = o;
+                square[0] = fmaf(o, o, square[0]);
+            }
+        }
+    }
+    spk_block_sum<1>(square, part);
+    const float inv = 1.0f / sqrtf(square[0] / static_cast<float>(vdim) + a.eps);
+    const T* gate = static_cast<const T*>(a.gate) + row * a.ld2 + static_cast<int64_t>(h) * vdim;
+    for (int e = threadIdx.x; e < vdim; e += kThreads)
+        out[e] = spk_from_float<T>(v[e] * inv * a.w_norm[e] * spk_sigmoid(spk_to_float<T>(gate[e])));
+}
+
+// ---- prefill -----------------------------------------------------------------------------------------------------------
+constexpr int kChunk = 16;
+
+// What the recurrence reads, 32-bit: q [n][kv_heads][dim], k the same, v [n][heads][vdim], decays [n][heads][dim], beta [n][heads],
+// outputs [n][heads][vdim].
+struct Work {
+    float *q, *k, *v, *g, *beta, *o;
+};
+__host__ __device__ inline int64_t work_floats(int64_t n, int heads, int kv_heads, int dim, int vdim) {
+    return n * (2 * static_cast<int64_t>(kv_heads) * dim + static_cast<int64_t>(heads) * (dim + 2 * vdim) + ((heads + 3) & ~3));
+}
+__device__ __forceinline__ Work carve(const spk_delta_args& a) {
+    Work w;
+    const int64_t qk = a.n * a.kv_heads * a.dim, vv = a.n * a.heads * a.vdim;
+    w.q = static_cast<float*>(a.workspace);
+    w.k = w.q + qk;
+    w.g = w.k + qk;
+    w.v = w.g + a.n * a.heads * a.dim;
+    w.o = w.v + vv;
+    w.beta = w.o + vv;
+    return w;
+}
+
+// CTA = chunk of up to 16 tokens; a warp per (token, part): the key heads' q, their k, the heads' v, the heads' decays.
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+delta_prepare_kernel(const spk_delta_args a) {
+    const int4 ch = reinterpret_cast<const int4*>(a.chunks)[blockIdx.x];    // first token, tokens, portion, index
+    const int4 po = reinterpret_cast<const int4*>(a.portions)[ch.z];        // first token, tokens, row, tokens before
+    if (po.z < 0 || po.z >= a.state_rows) {
+        if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SLOT);
+        return;
+    }
+    const Work w = carve(a);
+    const SpkDeltaShape sh = spk_delta_shape(a);
+    const int lane = threadIdx.x & 31, parts = 2 * a.kv_heads + 2 * a.heads;
+    const float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
+    for (int item = threadIdx.x >> 5; item < ch.y * parts; item += kThreads / 32) {
+        const int64_t t = ch.x + item / parts;
+        int part = item % parts;
+        auto conv = [&](const void* src, int64_t c, int at, const float* taps) {
+            const T* p = static_cast<const T*>(src) + t * a.ld + c;
+            return spk_conv_silu(taps + c * a.taps, a.taps, spk_to_float<T>(*p), [&](int back) {
+                if (t - back >= po.x) return spk_to_float<T>(p[-back * a.ld]);
+                const int64_t pos = po.w + (t - po.x) - back;
+                return pos >= 0 ? ring[(pos % a.taps) * sh.channels + at] : 0.0f;
+            });
+        };
+        if (part < 2 * a.kv_heads) {
+            const bool is_q = part < a.kv_heads;
+            const int g = is_q ? part : part - a.kv_heads;
+            float* dst = (is_q ? w.q : w.k) + (t * a.kv_heads + g) * a.dim;
+            float ss = 0.0f;
+            for (int c = lane; c < a.dim; c += 32) {
+                const float x = conv(is_q ? a.q : a.k, g * a.dim + c, (is_q ? 0 : sh.qk) + g * a.dim + c, is_q ? a.conv_q : a.conv_k);
+                dst[c] = x;
+                ss = fmaf(x, x, ss);
+            }
+            float inv = 1.0f / sqrtf(spk_warp_sum(ss) + 1e-6f);
+            if (is_q) inv /= sqrtf(static_cast<float>(a.dim));
+            for (int c = lane; c < a.dim; c += 32) dst[c] *= inv;
+        } else if (part < 2 * a.kv_heads + a.heads) {
+            const int h = part - 2 * a.kv_heads;
+            for (int c = lane; c < a.vdim; c += 32)
+                w.v[(t * a.heads + h) * a.vdim + c] = conv(a.v, static_cast<int64_t>(h) * a.vdim + c, 2 * sh.qk + h * a.vdim + c, a.conv_v);
+        } else {
+            const int h = part - 2 * a.kv_heads - a.heads;
+            const float rate = expf(a.a_log[h]);
+            for (int c = lane; c < a.dim; c += 32) {
+                const int64_t i = static_cast<int64_t>(h) * a.dim + c;
+                w.g[t * a.heads * a.dim + i] = expf(spk_log_decay(spk_to_float<T>(static_cast<const T*>(a.a)[t * a.ld2 + i]) + a.dt_bias[i], rate));
+            }
+            if (lane == 0) w.beta[t * a.heads + h] = spk_sigmoid(spk_to_float<T>(static_cast<const T*>(a.b)[t * a.ld + h]));
+        }
+    }
+}
+
+// The recurrence, token by token.  CTA = (32 columns of a head's state, head, portion); four lanes share a column, each with every fourth
+// group of four key channels in registers: NR groups, dim <= 16 NR.  Both products are taken of the state before the step:
+//   S^T(g k) and S^T(g q) + (q . k) u, so one exchange per token serves them, and the update is off the chain.
+constexpr int kScanCols = 32;
+
+template <typename T, int NR>
+__global__ void __launch_bounds__(4 * kScanCols)
+delta_scan_kernel(const spk_delta_args a) {
+    constexpr int D = 16 * NR, kScanTokens = NR > 8 ? 4 : 8;  // tokens staged at a time
+    __shared__ __align__(16) float gs[2][kScanTokens][D], ks[2][kScanTokens][D], gk[2][kScanTokens][D], gq[2][kScanTokens][D];
+    __shared__ float qk[2][kScanTokens], bs[2][kScanTokens], vs[2][kScanTokens][kScanCols];
+    const int4 po = reinterpret_cast<const int4*>(a.portions)[blockIdx.z];
+    if (po.z < 0 || po.z >= a.state_rows) {
+        if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SLOT);
+        return;
+    }
+    const Work w = carve(a);
+    const SpkDeltaShape sh = spk_delta_shape(a);
+    const int h = blockIdx.y, rep = a.heads / a.kv_heads, g = h / rep;
+    const int col = threadIdx.x >> 2, part = threadIdx.x & 3, e = blockIdx.x * kScanCols + col;
+    const bool in = e < a.vdim;
+    float* S = a.state + (static_cast<int64_t>(po.z) * a.heads + h) * a.dim * a.vdim + e;
+    uint64_t s[NR][2];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        float f[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int d = 16 * i + 4 * part + j;
+            f[j] = po.w > 0 && in && d < a.dim ? S[static_cast<int64_t>(d) * a.vdim] : 0.0f;
+        }
+        s[i][0] = f2_pack(f[0], f[1]);
+        s[i][1] = f2_pack(f[2], f[3]);
+    }
+    auto stage = [&](int buf, int j0) {  // tokens j0 .. of the portion, a warp per token
+        const int lane = threadIdx.x & 31;
+        for (int j = threadIdx.x >> 5; j < kScanTokens && j0 + j < po.y; j += 4 * kScanCols / 32) {
+            const int64_t t = po.x + j0 + j;
+            const float *qr = w.q + (t * a.kv_heads + g) * a.dim, *kr = w.k + (t * a.kv_heads + g) * a.dim, *gr = w.g + (t * a.heads + h) * a.dim;
+            float dot = 0.0f;
+            for (int d = lane; d < D; d += 32) {
+                const bool live = d < a.dim;
+                const float x = live ? qr[d] : 0.0f, y = live ? kr[d] : 0.0f, z = live ? gr[d] : 0.0f;
+                gs[buf][j][d] = z;
+                ks[buf][j][d] = y;
+                gk[buf][j][d] = z * y;
+                gq[buf][j][d] = z * x;
+                dot = fmaf(x, y, dot);
+            }
+            dot = spk_warp_sum(dot);
+            if (lane == 0) {
+                qk[buf][j] = dot;
+                bs[buf][j] = w.beta[t * a.heads + h];
+            }
+            const int c = blockIdx.x * kScanCols + lane;
+            vs[buf][j][lane] = c < a.vdim ? w.v[(t * a.heads + h) * a.vdim + c] : 0.0f;
+        }
+    };
+    stage(0, 0);
+    __syncthreads();
+    for (int j0 = 0, buf = 0; j0 < po.y; j0 += kScanTokens, buf ^= 1) {
+        if (j0 + kScanTokens < po.y) stage(buf ^ 1, j0 + kScanTokens);
+        const int n = min(kScanTokens, po.y - j0);
+        for (int j = 0; j < n; ++j) {
+            uint64_t ak[2] = {0, 0}, aq[2] = {0, 0};
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(&gk[buf][j][16 * i + 4 * part]);
+                const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(&gq[buf][j][16 * i + 4 * part]);
+                ak[0] = f2_fma(s[i][0], x.x, ak[0]);
+                ak[1] = f2_fma(s[i][1], x.y, ak[1]);
+                aq[0] = f2_fma(s[i][0], y.x, aq[0]);
+                aq[1] = f2_fma(s[i][1], y.y, aq[1]);
+            }
+            float k0, k1, q0, q1;
+            f2_unpack(f2_add(ak[0], ak[1]), k0, k1);
+            f2_unpack(f2_add(aq[0], aq[1]), q0, q1);
+            float sk = k0 + k1, sq = q0 + q1;
+            sk += __shfl_xor_sync(~0u, sk, 1);
+            sq += __shfl_xor_sync(~0u, sq, 1);
+            sk += __shfl_xor_sync(~0u, sk, 2);
+            sq += __shfl_xor_sync(~0u, sq, 2);
+            const float u = bs[buf][j] * (vs[buf][j][col] - sk);
+            const uint64_t uu = f2_pack(u, u);
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const ulonglong2 z = *reinterpret_cast<const ulonglong2*>(&gs[buf][j][16 * i + 4 * part]);
+                const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(&ks[buf][j][16 * i + 4 * part]);
+                s[i][0] = f2_fma(s[i][0], z.x, f2_mul(y.x, uu));
+                s[i][1] = f2_fma(s[i][1], z.y, f2_mul(y.y, uu));
+            }
+            if (part == 0 && in) w.o[((static_cast<int64_t>(po.x) + j0 + j) * a.heads + h) * a.vdim + e] = fmaf(qk[buf][j], u, sq);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        float f[4];
+        f2_unpack(s[i][0], f[0], f[1]);
+        f2_unpack(s[i][1], f[2], f[3]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int d = 16 * i + 4 * part + j;
+            if (in && d < a.dim) S[static_cast<int64_t>(d) * a.vdim] = f[j];
+        }
+    }
+    // the convolution's last inputs, for the next portion or the first decode step
+    float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
+    const int keep = min(a.taps, po.y);
+    auto commit = [&](const void* src, int64_t c, int at) {
+        for (int b = 0; b < keep; ++b) {
+            const int64_t t = po.x + po.y - 1 - b, pos = static_cast<int64_t>(po.w) + po.y - 1 - b;
+            ring[(pos % a.taps) * sh.channels + at] = spk_to_float<T>(static_cast<const T*>(src)[t * a.ld + c]);
+        }
+    };
+    if (part == 0 && in) commit(a.v, static_cast<int64_t>(h) * a.vdim + e, 2 * sh.qk + h * a.vdim + e);
+    if (blockIdx.x == 0 && h % rep == 0)
+        for (int c = threadIdx.x; c < a.dim; c += 4 * kScanCols) {
+            commit(a.q, g * a.dim + c, g * a.dim + c);
+            commit(a.k, g * a.dim + c, sh.qk + g * a.dim + c);
+        }
+}
+
+// A warp per (token, head): norm over the head's outputs, weight, gate.
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+delta_out_kernel(const spk_delta_args a) {
+    const int64_t item = static_cast<int64_t>(blockIdx.x) * (kThreads / 32) + (threadIdx.x >> 5);
+    if (item >= a.n * a.heads) return;
+    const int lane = threadIdx.x & 31;
+    const int64_t t = item / a.heads;
+    const int h = static_cast<int>(item % a.heads);
+    const float* o = carve(a).o + item * a.vdim;
+    float ss = 0.0f;
+    for (int e = lane; e < a.vdim; e += 32) ss = fmaf(o[e], o[e], ss);
+    const float inv = 1.0f / sqrtf(spk_warp_sum(ss) / static_cast<float>(a.vdim) + a.eps);
+    const T* gate = static_cast<const T*>(a.gate) + t * a.ld2 + static_cast<int64_t>(h) * a.vdim;
+    T* out = static_cast<T*>(a.out) + t * a.out_stride + static_cast<int64_t>(h) * a.vdim;
+    for (int e = lane; e < a.vdim; e += 32) out[e] = spk_from_float<T>(o[e] * inv * a.w_norm[e] * spk_sigmoid(spk_to_float<T>(gate[e])));
+}
+
+int check(const spk_delta_args* a) {
+    if (a == nullptr) return SPK_ERR_NULL_POINTER;
+    if (a->n < 0 || a->heads < 1 || a->heads > 65535 || a->kv_heads < 1 || a->heads % a->kv_heads != 0 || a->dim < 1 || a->vdim < 1 || a->taps < 1 ||
+        a->state_rows < 1)
+        return SPK_ERR_BAD_SHAPE;
+    if (a->dtype != SPK_F32 && a->dtype != SPK_BF16) return SPK_ERR_BAD_DTYPE;
+    if (a->n == 0) return SPK_OK;
+    if (a->q == nullptr || a->k == nullptr || a->v == nullptr || a->b == nullptr || a->a == nullptr || a->gate == nullptr || a->conv_q == nullptr ||
+        a->conv_k == nullptr || a->conv_v == nullptr || a->a_log == nullptr || a->dt_bias == nullptr || a->w_norm == nullptr || a->state == nullptr ||
+        a->conv_state == nullptr || a->out == nullptr)
+        return SPK_ERR_NULL_POINTER;
+    return SPK_OK;
+}
+
+template <typename T, int W, bool KEEP>
+int launch_step_form(const spk_delta_args& a, size_t bytes, cudaStream_t s) {
+    if (bytes > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+        if (e != cudaSuccess) return spk_set_cuda_error(e);
+    }
+    delta_step_kernel<T, W, KEEP><<<dim3(a.heads, static_cast<unsigned>(a.n)), kThreads, bytes, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+template <typename T>
+int launch_step(const spk_delta_args& a, cudaStream_t s) {
+    const bool vec = a.vdim % 4 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0;
+    const int cols = vec ? a.vdim / 4 : a.vdim;
+    const int slices = cols < kThreads ? kThreads / cols : 1;
+    const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim);
+    if (bytes > 200 * 1024) return SPK_ERR_TOO_LARGE;
+    const bool keep = cols <= kThreads && a.dim <= kKeep * slices;
+    if (vec) return keep ? launch_step_form<T, 4, true>(a, bytes, s) : launch_step_form<T, 4, false>(a, bytes, s);
+    return keep ? launch_step_form<T, 1, true>(a, bytes, s) : launch_step_form<T, 1, false>(a, bytes, s);
+}
+
+template <typename T>
+int launch_prefill(const spk_delta_args& a, cudaStream_t s) {
+    if (a.dim > 256) return SPK_ERR_UNSUPPORTED;
+    delta_prepare_kernel<T><<<a.n_chunks, kThreads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    const dim3 grid((a.vdim + kScanCols - 1) / kScanCols, a.heads, a.n_portions);
+    const int threads = 4 * kScanCols;
+    if (a.dim <= 32) delta_scan_kernel<T, 2><<<grid, threads, 0, s>>>(a);
+    else if (a.dim <= 64) delta_scan_kernel<T, 4><<<grid, threads, 0, s>>>(a);
+    else if (a.dim <= 128) delta_scan_kernel<T, 8><<<grid, threads, 0, s>>>(a);
+    else delta_scan_kernel<T, 16><<<grid, threads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    const int64_t out_grid = (a.n * a.heads + kThreads / 32 - 1) / (kThreads / 32);
+    if (out_grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
+    delta_out_kernel<T><<<static_cast<unsigned>(out_grid), kThreads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+}  // namespace
+
+extern "C" int spk_delta_step(const spk_delta_args* a, void* stream) {
+    SpkRange nvtx_range("spk_delta_step");
+    const int rc = check(a);
+    if (rc != SPK_OK || a->n == 0) return rc;
+    if (a->positions == nullptr) return SPK_ERR_NULL_POINTER;
+    if (a->n > 65535) return SPK_ERR_TOO_LARGE;
+    if (a->n > a->state_rows) return SPK_ERR_BAD_SHAPE;
+    cudaStream_t s = spk_stream(stream);
+    return a->dtype == SPK_F32 ? launch_step<float>(*a, s) : launch_step<__nv_bfloat16>(*a, s);
+}
+
+extern "C" int spk_delta_chunk_tokens(int dtype, int dim, int vdim) {
+    (void)dtype;
+    (void)dim;
+    (void)vdim;
+    return kChunk;
+}
+
+extern "C" int64_t spk_delta_workspace_bytes(int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim) {
+    if (n < 1 || n_chunks < 1 || heads < 1 || kv_heads < 1 || dim < 1 || vdim < 1) return 0;
+    return static_cast<int64_t>(sizeof(float)) * work_floats(n, heads, kv_heads, dim, vdim);
+}
+
+extern "C" int spk_delta_prefill(const spk_delta_args* a, void* stream) {
+    SpkRange nvtx_range("spk_delta_prefill");
+    const int rc = check(a);
+    if (rc != SPK_OK || a->n == 0) return rc;
+    if (a->n_chunks < 1 || a->n_portions < 1 || a->n_portions > 65535) return SPK_ERR_BAD_SHAPE;
+    if (a->chunks == nullptr || a->portions == nullptr) return SPK_ERR_NULL_POINTER;
+    if (reinterpret_cast<uintptr_t>(a->chunks) % 16 != 0 || reinterpret_cast<uintptr_t>(a->portions) % 16 != 0) return SPK_ERR_BAD_STRIDE;
+    if (a->workspace == nullptr || a->workspace_bytes < spk_delta_workspace_bytes(a->n, a->n_chunks, a->heads, a->kv_heads, a->dim, a->vdim))
+        return SPK_ERR_WORKSPACE_TOO_SMALL;
+    cudaStream_t s = spk_stream(stream);
+    return a->dtype == SPK_F32 ? launch_prefill<float>(*a, s) : launch_prefill<__nv_bfloat16>(*a, s);
+}

@@ -131,3 +131,19 @@ static inline int spk_launch(void (*fn)(Args), dim3 grid, int threads, size_t by
     spk_count_launch();
     return SPK_OK;
 }
+
+// A row held by a CTA: V groups of four consecutive elements per thread, group v of thread i at element 4 (i + v * threads).
+template <int V>
+struct SpkRow {
+    float4 g[V];
+};
+
+// Threads per row and four-element groups per thread for a row of `width` elements; 0 when too wide.
+static inline int spk_row_shape(int64_t width, int* v) {
+    const int64_t groups = (width + 3) / 4;
+    const int threads = groups <= 128 ? (groups <= 32 ? 32 : groups <= 64 ? 64 : 128) : groups <= 256 ? 128 : groups <= 2048 ? 256 : 1024;
+    const int64_t need = (groups + threads - 1) / threads;
+    if (need > 8) return 0;
+    *v = need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : 8;
+    return threads;
+}

@@ -38,18 +38,13 @@ struct ResidualNormParams {
     uint32_t* status;
 };
 
-template <int V>
-struct Row {
-    float4 g[V];
-};
-
 __device__ __forceinline__ float4 f4_axpy(float a, float4 x, float4 y) {
     return make_float4(fmaf(a, x.x, y.x), fmaf(a, x.y, y.y), fmaf(a, x.z, y.z), fmaf(a, x.w, y.w));
 }
 
 // Layer norm of the row in registers (two passes over them: mean, then squared deviations).
 template <int V, bool VEC>
-__device__ __forceinline__ void layer_norm_row(Row<V>& y, const float* __restrict__ w, int width, float eps, float* part) {
+__device__ __forceinline__ void layer_norm_row(SpkRow<V>& y, const float* __restrict__ w, int width, float eps, float* part) {
     float s[1] = {0.0f};
 #pragma unroll
     for (int v = 0; v < V; ++v) s[0] += (y.g[v].x + y.g[v].y) + (y.g[v].z + y.g[v].w);
@@ -78,7 +73,7 @@ __device__ __forceinline__ void layer_norm_row(Row<V>& y, const float* __restric
 }
 
 template <typename T, typename TD, int V, bool VEC>
-__device__ __forceinline__ void new_row(const ResidualNormParams& p, int64_t t, int64_t commit_row, Row<V>& y, float* part) {
+__device__ __forceinline__ void new_row(const ResidualNormParams& p, int64_t t, int64_t commit_row, SpkRow<V>& y, float* part) {
     if (p.ids != nullptr) {
         const int64_t id = p.ids[t];
         const bool ok = id >= 0 && id < p.vocab;
@@ -109,7 +104,7 @@ residual_norm_kernel(const ResidualNormParams p, T* __restrict__ out) {
     __shared__ float part[32];
     const int64_t t0 = static_cast<int64_t>(blockIdx.x) * p.per_cta;
     const int64_t t1 = t0 + p.per_cta < p.n ? t0 + p.per_cta : p.n;
-    Row<V> before, y;
+    SpkRow<V> before, y;
     for (int64_t t = t0; t < t1; ++t) {
         // decode: token t is row t's only token; prefill: the portion's tables say
         const int32_t edge = p.token_edges != nullptr ? p.token_edges[t] : 3;
@@ -168,7 +163,7 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ coef, float 
     __shared__ float part[3 * 32];
     const T* zr = z + static_cast<int64_t>(blockIdx.x) * width;
     T* o = out + static_cast<int64_t>(blockIdx.x) * width;
-    Row<V> y;
+    SpkRow<V> y;
     float s[3] = {0.0f, 0.0f, 0.0f};
 #pragma unroll
     for (int v = 0; v < V; ++v) {
@@ -267,20 +262,10 @@ int launch_poly_packed(const void* z, const float* coef, float eps, void* out, i
     return SPK_OK;
 }
 
-// Threads per row and four-element groups per thread for a row of `width` elements; 0 when too wide.
-int row_shape(int64_t width, int* v) {
-    const int64_t groups = (width + 3) / 4;
-    const int threads = groups <= 128 ? (groups <= 32 ? 32 : groups <= 64 ? 64 : 128) : groups <= 256 ? 128 : groups <= 2048 ? 256 : 1024;
-    const int64_t need = (groups + threads - 1) / threads;
-    if (need > 8) return 0;
-    *v = need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : 8;
-    return threads;
-}
-
 template <typename T, typename TD>
 int launch_residual(const ResidualNormParams& p, void* out, cudaStream_t s) {
     int v = 1;
-    const int threads = row_shape(p.width, &v);
+    const int threads = spk_row_shape(p.width, &v);
     if (threads == 0) return SPK_ERR_TOO_LARGE;
     const unsigned grid = static_cast<unsigned>((p.n + p.per_cta - 1) / p.per_cta);
     const bool vec = p.width % 4 == 0;
@@ -302,7 +287,7 @@ int launch_residual(const ResidualNormParams& p, void* out, cudaStream_t s) {
 template <typename T>
 int launch_poly(const void* z, const float* coef, float eps, void* out, int64_t rows, int64_t width, cudaStream_t s) {
     int v = 1;
-    const int threads = row_shape(width, &v);
+    const int threads = spk_row_shape(width, &v);
     if (threads == 0) return SPK_ERR_TOO_LARGE;
     const unsigned grid = static_cast<unsigned>(rows);
     const bool vec = width % 4 == 0;

@@ -1,7 +1,7 @@
 """Cache of a decoder that mixes paged attention with recurrent layers.
 
 Per layer any of: a pair of dense K/V page pools (:class:`PagedKVPool`, addressed by the same block tables and slots as
-the spike pools), and named per-row states in 32 bits (one slot per batch row; a request keeps its row, and with it its
+the spike pools), a pool of shared-latent rows (:class:`PagedLatentPool`; a layer may read an earlier layer's), and named per-row states in 32 bits (one slot per batch row; a request keeps its row, and with it its
 slot, from its first token to its release).  A slot is never cleared when it is handed on: a portion that starts at position
 0 does not read it.
 """
@@ -22,10 +22,21 @@ class KVSpec:
 
 
 @dataclass(frozen=True)
+class LatentSpec:
+    """One layer's shared-latent cache: ``rank`` latent and ``rot_dim`` rotated channels per token, read by all heads."""
+
+    rank: int
+    rot_dim: int
+
+
+@dataclass(frozen=True)
 class LayerCacheSpec:
     kv: KVSpec | None = None
     states: tuple[tuple[str, tuple[int, ...]], ...] = ()
     """(name, shape) of every per-row state."""
+    latent: LatentSpec | None = None
+    latent_from: int | None = None
+    """The (earlier) layer whose latent pool this layer reads."""
 
 
 class PagedKVPool:
@@ -53,8 +64,33 @@ class PagedKVPool:
         return x[..., : self.dim].permute(0, 2, 1, 3).reshape(nb * bs, heads, self.dim)
 
 
+class PagedLatentPool(PagedKVPool):
+    """A pool of shared-latent cache rows: ``rank`` latent channels at 0, ``rot_dim`` rotated ones at ``rank_pad``; one pool head.
+    Tiled (see :class:`PagedKVPool`) in 16 bits, both parts padded to 64 channels; plain without padding otherwise."""
+
+    def __init__(self, num_blocks: int, block_size: int, rank: int, rot_dim: int, dtype: torch.dtype, device) -> None:
+        self.rank, self.rot_dim, self.block_size = rank, rot_dim, block_size
+        self.tiled = dtype == torch.bfloat16 and block_size % 16 == 0
+        self.rank_pad, self.rot_pad = (-(-x // 64) * 64 if self.tiled else x for x in (rank, rot_dim))
+        self.pad = self.dim = self.rank_pad + self.rot_pad
+        self.data = torch.zeros((num_blocks, 1, block_size, self.pad), dtype=dtype, device=device)
+
+    def rows(self) -> torch.Tensor:
+        """``[num_blocks * block_size, rank + rot_dim]`` in plain order (for checks)."""
+        x = super().rows()[:, 0]
+        return torch.cat((x[:, : self.rank], x[:, self.rank_pad: self.rank_pad + self.rot_dim]), dim=1)
+
+
 class LayerCache:
-    def __init__(self, spec: LayerCacheSpec, num_blocks: int, block_size: int, max_rows: int, dtype: torch.dtype, device) -> None:
+    def __init__(self, spec: LayerCacheSpec, num_blocks: int, block_size: int, max_rows: int, dtype: torch.dtype, device,
+                 earlier: list["LayerCache"] = ()) -> None:
+        self.latent = None
+        if spec.latent_from is not None:
+            if not 0 <= spec.latent_from < len(earlier) or earlier[spec.latent_from].latent is None:
+                raise ValueError(f"layer {spec.latent_from} holds no latent pool to share")
+            self.latent = earlier[spec.latent_from].latent
+        elif spec.latent is not None:
+            self.latent = PagedLatentPool(num_blocks, block_size, spec.latent.rank, spec.latent.rot_dim, dtype, device)
         self.k = self.v = None
         if spec.kv is not None:
             self.k = PagedKVPool(num_blocks, spec.kv.kv_heads, block_size, spec.kv.dim, dtype, device)
@@ -71,7 +107,9 @@ class PagedKVStateCache:
             raise ValueError(f"block_size must be a power of two, got {block_size}")
         self.num_blocks, self.block_size, self.max_rows = num_blocks, block_size, max_rows
         self.device = torch.device(device)
-        self.layers = [LayerCache(s, num_blocks, block_size, max_rows, dtype, self.device) for s in specs]
+        self.layers: list[LayerCache] = []
+        for s in specs:
+            self.layers.append(LayerCache(s, num_blocks, block_size, max_rows, dtype, self.device, self.layers))
 
     @property
     def pad_block(self) -> int:
@@ -83,8 +121,9 @@ class PagedKVStateCache:
 
     @property
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for layer in self.layers
-                   for t in (*(p.data for p in (layer.k, layer.v) if p is not None), *layer.states.values()))
+        tensors = {id(t): t for layer in self.layers
+                   for t in (*(p.data for p in (layer.k, layer.v, layer.latent) if p is not None), *layer.states.values())}
+        return sum(t.numel() * t.element_size() for t in tensors.values())  # a shared pool counts once
 
     def recurrent_tensors(self) -> tuple:
         """State that a replayed step would not rewrite by itself (snapshots save it)."""

@@ -1,4 +1,4 @@
-"""Operators of the dense (non-spiking) decoders (CUDA): post-norm residual boundary, polynomial norm activation, paged
+"""Operators of the dense (non-spiking) decoders (CUDA): post-norm and pre-norm residual boundaries, activations, paged
 attention with element-wise key weights, linear attention with a decaying state.
 
 Tensors are fp32 or bf16; 32-bit arithmetic throughout.  The decode forms (token t = batch row t) have fixed arguments and
@@ -202,4 +202,60 @@ def gated_norm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, out: t
                            left_width=0 if partials is None else partials.shape[2], dtype=_lib.dtype_code(out.dtype), eps=eps,
                            scale=scale, left_scale=left_scale)
     _call("spk_gated_norm", a, x.device)
+    return out
+
+
+def rms_residual(*, eps: float, x: torch.Tensor | None = None, delta: torch.Tensor | None = None, ids: torch.Tensor | None = None,
+                 embed: torch.Tensor | None = None, embed_scale: float = 1.0, x_out: torch.Tensor | None = None,
+                 pairs: torch.Tensor | None = None, pair_slots: torch.Tensor | None = None, pair_scale: float = 1.0,
+                 w1: torch.Tensor | None = None, out1: torch.Tensor | None = None, w2: torch.Tensor | None = None,
+                 out2: torch.Tensor | None = None, out2_slots: torch.Tensor | None = None, out2_tiled: bool = False,
+                 status: torch.Tensor | None = None) -> None:
+    """One layer boundary: ``y = x + delta + pair_scale * (rows pair_slots[t] of pairs)`` (or ``embed_scale * embed[ids]``), to
+    ``x_out`` (fp32, may be ``x``); ``out1 = rmsnorm(y) * w1`` and ``out2 = rmsnorm(y) * w2``.  ``out2_slots`` int32 ``[n, top]``:
+    ``out2`` is a sorted matrix of experts (:mod:`.experts`) and a row goes to all of its slots, as operand tiles with
+    ``out2_tiled``."""
+    some = x if x is not None else x_out if x_out is not None else out1
+    _lib.require_cuda(some, "rms_residual")
+    n, width = some.shape
+    for t, name in ((x, "x"), (x_out, "x_out")):
+        _f32(t, name, n * width)
+    for t, name in ((w1, "w1"), (w2, "w2")):
+        _f32(t, name, width)
+    _f32(pairs, "pairs")
+    if delta is not None and (delta.shape != (n, width) or not delta.is_contiguous()):
+        raise ValueError("delta must be contiguous [n, width]")
+    if ids is not None and (embed is None or not embed.is_contiguous() or embed.shape[1] != width or ids.numel() != n):
+        raise ValueError("embed must be a contiguous [vocab, width] table, ids one entry per row")
+    for o in (out1, out2 if out2_slots is None else None):
+        if o is not None and (o.shape != (n, width) or not o.is_contiguous()):
+            raise ValueError("out1 and out2 must be contiguous [n, width]")
+    outs = [t.dtype for t in (out1, out2, embed) if t is not None]
+    if len(set(outs)) > 1:
+        raise ValueError("outputs and embedding table must share one dtype")
+    for s in (pair_slots, out2_slots):
+        if s is not None and (s.dtype != torch.int32 or not s.is_contiguous() or s.shape[0] != n):
+            raise ValueError("slots must be contiguous int32 [n, top]")
+    a = _lib.RmsResidualArgs(
+        x=_ptr(x), x_out=_ptr(x_out), delta=_ptr(delta), embed=_ptr(embed), ids=_ptr(ids), vocab=0 if embed is None else embed.shape[0],
+        pairs=_ptr(pairs), pair_slots=_ptr(pair_slots), w1=_ptr(w1), out1=_ptr(out1), w2=_ptr(w2), out2=_ptr(out2),
+        out2_slots=_ptr(out2_slots), pair_rows=0 if pairs is None else pairs.shape[0],
+        out2_rows=0 if out2_slots is None else out2.numel() // out2.shape[-1] // (out2.shape[0] if out2_tiled else 1), n=n, width=width,
+        pair_top=0 if pair_slots is None else pair_slots.shape[1], out2_top=0 if out2_slots is None else out2_slots.shape[1],
+        out2_tiled=int(out2_tiled), dtype=_lib.dtype_code(outs[0] if outs else torch.float32),
+        delta_dtype=0 if delta is None else _lib.dtype_code(delta.dtype), embed_scale=embed_scale, pair_scale=pair_scale, eps=eps,
+        status=_ptr(status))
+    _call("spk_rms_residual", a, some.device)
+
+
+def gelu_tanh(z: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out = gelu(z)``, the tanh form; ``out`` may be a column range of a row-major matrix."""
+    _lib.require_cuda(z, "gelu_tanh input")
+    if not z.is_contiguous() or out.shape != z.shape or out.dtype != z.dtype or out.stride(1) != 1:
+        raise ValueError("z must be contiguous, out of the same shape and dtype with unit column stride")
+    lib = _lib.load()
+    with torch.cuda.device(z.device):
+        rc = lib.spk_gelu_tanh(z.data_ptr(), out.data_ptr(), out.stride(0), z.shape[0], z.shape[1], _lib.dtype_code(z.dtype),
+                               _lib.current_stream(z.device))
+    _lib.check(rc, "spk_gelu_tanh")
     return out

@@ -30,6 +30,8 @@ class ModelEntry:
 
 
 MODELS: dict[str, ModelEntry] = {
+    "Gotunex": ModelEntry("modeling_gotunex", "GotunexConfig", "GotunexModel", "PagedDecodeEngine", ("latent",),
+                          (torch.float32, torch.bfloat16)),
     "Manirax": ModelEntry("modeling_manirax", "ManiraxConfig", "ManiraxModel", "PagedDecodeEngine", ("dense",),
                           (torch.float32, torch.bfloat16)),
     "SpikingQwen": ModelEntry("modeling", "SpikingQwenConfig", "SpikingQwenModel", "SpikeDecodeEngine", ("spike",),
