@@ -1031,12 +1031,17 @@ def main() -> None:
     ap.add_argument("--repeats", type=int, default=5, help="timed regions per quantity (median, min and max are reported)")
     ap.add_argument("--no-serving", action="store_true", help="skip the closed-loop / open-loop serving measurements")
     ap.add_argument("--tokens", type=int, default=8192, help="tokens of --kernel-bench lif")
-    ap.add_argument("--workload", choices=["decode_0p5b", "tp7b", "manirax"], default="decode_0p5b",
+    ap.add_argument("--workload", choices=["decode_0p5b", "tp7b", "manirax", "gotunex"], default="decode_0p5b",
                     help="tp7b: the 7B-shape long-context tensor-parallel decode step (secondary line); manirax: prefill and "
-                         "decode of the Manirax design and its kernels, beside the spiking model of equal size")
+                         "decode of the Manirax design and its kernels, beside the spiking model of equal size; gotunex: the same of the "
+                         "Gotunex design, beside Manirax of equal size")
     ap.add_argument("--manirax-shapes", default="0.5b,7b4", help="--workload manirax: shapes to run, with commas between them")
     ap.add_argument("--manirax-kernels-only", action="store_true", help="--workload manirax: skip the throughput runs")
     ap.add_argument("--manirax-own-only", action="store_true", help="--workload manirax: skip the spiking kernels")
+    ap.add_argument("--gotunex-shapes", default="0.5b,7b4", help="--workload gotunex: shapes to run, with commas between them")
+    ap.add_argument("--gotunex-kernels-only", action="store_true", help="--workload gotunex: skip the throughput runs")
+    ap.add_argument("--gotunex-own-only", action="store_true", help="--workload gotunex: skip Manirax")
+    ap.add_argument("--gotunex-only", default="", help="--workload gotunex: only the kernels whose names start so, with commas between them")
     ap.add_argument("--tp-seqs", type=int, default=256, help="sequences per replica of --workload tp7b")
     ap.add_argument("--tp-size", type=int, default=0, help="tensor-parallel group size of --workload tp7b (default min(N, 4))")
     ap.add_argument("--tp-layers", type=int, default=0, help="layers of --workload tp7b (default 28)")
@@ -1050,6 +1055,10 @@ def main() -> None:
         import bench_manirax
 
         bench_manirax.run(args)
+    elif args.workload == "gotunex":
+        import bench_gotunex
+
+        bench_gotunex.run(args)
     elif args.kernel_bench:
         run_kernel_bench(args)
     elif args.impl == "reference":

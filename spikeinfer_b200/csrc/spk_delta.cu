@@ -66,6 +66,13 @@ delta_step_kernel(const spk_delta_args a) {
     }
     const SpkDeltaShape sh = spk_delta_shape(a);
     const int64_t pos = a.positions[row];
+    const bool fresh = pos == 0;  // whatever the slot holds, a sequence starts from zeros
+    if (KEEP && fresh) {
+#pragma unroll
+        for (int u = 0; u < (KEEP ? kKeep : 1); ++u)
+#pragma unroll
+            for (int i = 0; i < W; ++i) s[u][i] = 0.0f;
+    }
     float* ring = a.conv_state + row * a.taps * sh.channels;
     const int now_slot = static_cast<int>(pos % a.taps);
     auto channel = [&](const void* src, int64_t c, int at, const float* w, bool keep) {  // one channel's convolution; `at`: its place in the ring
@@ -119,7 +126,7 @@ delta_step_kernel(const spk_delta_args a) {
                     load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
                     const float w = dec[d] * (k[d] * ki);
 #pragma unroll
-                    for (int i = 0; i < W; ++i) acc[i] = fmaf(w, x[i], acc[i]);
+                    for (int i = 0; i < W; ++i) acc[i] = fresh ? 0.0f : fmaf(w, x[i], acc[i]);
                 }
             }
 #pragma unroll
@@ -160,7 +167,7 @@ delta_step_kernel(const spk_delta_args a) {
                     float x[W];
                     load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
 #pragma unroll
-                    for (int i = 0; i < W; ++i) x[i] *= dec[d];
+                    for (int i = 0; i < W; ++i) x[i] = fresh ? 0.0f : x[i] * dec[d];
                     update(x, d);
                 }
             }
