@@ -401,7 +401,7 @@ extern "C" int spk_latent_attn_splits(int dtype, int rank, int rot_dim, int rank
     (void)rank;
     (void)rot_dim;
     if (n < 1 || heads < 1 || max_keys < 1) return 1;
-    (void)spk_latent_tensor_form(dtype, rank_pad, rot_pad, tiled, block_size);
+    if (spk_latent_tensor_form(dtype, rank_pad, rot_pad, tiled, block_size)) return spk_latent_decode_splits(n, heads, max_keys);
     const int64_t ctas = n * ((heads + kHeadsPer - 1) / kHeadsPer);
     const int64_t want = (3 * 148 + ctas - 1) / ctas, most = (max_keys + 255) / 256;
     const int64_t splits = want < most ? want : most;
@@ -420,6 +420,11 @@ extern "C" int spk_latent_attn(const spk_latent_attn_args* a, void* stream) {
     if (a->token_rows != nullptr ? a->positions == nullptr : a->seq_lens == nullptr) return SPK_ERR_NULL_POINTER;
     if (a->token_rows == nullptr && a->n > a->table_rows) return SPK_ERR_BAD_SHAPE;
     cudaStream_t s = spk_stream(stream);
+    if (spk_latent_tensor_form(a->dtype, a->rank_pad, a->rot_pad, a->tiled, a->block_size)) {
+        // query rows and pages are read 16 bytes at a time
+        if (reinterpret_cast<uintptr_t>(a->q) % 16 != 0 || reinterpret_cast<uintptr_t>(a->pool) % 16 != 0) return SPK_ERR_BAD_STRIDE;
+        return spk_latent_decode_launch(*a, s);
+    }
     return a->dtype == SPK_F32 ? launch_simt<float>(*a, s) : launch_simt<__nv_bfloat16>(*a, s);
 }
 

@@ -10,8 +10,11 @@ __host__ __device__ __forceinline__ SpkPageLayout spk_latent_layout(int block_si
 
 // Tiled 16-bit pool of at most 512 latent and 64 rotated channels, pages of 16 rows or a larger power of two.
 static inline bool spk_latent_tensor_form(int dtype, int rank_pad, int rot_pad, int tiled, int block_size) {
-    return dtype == SPK_BF16 && tiled && rank_pad <= 512 && rot_pad <= 64 && block_size >= 16 && (block_size & (block_size - 1)) == 0;
+    return dtype == SPK_BF16 && tiled && rank_pad <= 512 && rot_pad == 64 && block_size >= 16 && (block_size & (block_size - 1)) == 0;
 }
+
+int spk_latent_decode_splits(int64_t n, int heads, int64_t max_keys);
+int spk_latent_decode_launch(const spk_latent_attn_args& a, cudaStream_t s);
 
 // Keys token t of a call sees: position + 1 in a prefill, the row's length in a decode step (0 for rows that sit out).
 template <typename Args>
