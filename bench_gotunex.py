@@ -190,10 +190,11 @@ def gotunex_kernels(shape: str, device, repeats: int, pk: dict, only=()) -> dict
         pos = torch.arange(n, device=device).repeat(seqs)
         rows = (torch.arange(seqs * n, device=device) // n).to(torch.int32)
         w_uk = rnd(H * D, K) * K ** -0.5
+        w_kv = latent.spelled_out_weights(w_uk, w_uv, H)
 
         def mk_pre():
             q, g, o = rnd(seqs * n, H * (D + R)), rnd(seqs * n, H * V), rnd(seqs * n, H * V)
-            return lambda: latent.latent_prefill(q, pool, tables, w_uk, w_uv, sink, g, o, rot_table=rot, positions=pos, token_rows=rows, plan=plan, heads=H, dim=D,
+            return lambda: latent.latent_prefill(q, pool, tables, w_uk, w_uv, w_kv, sink, g, o, rot_table=rot, positions=pos, token_rows=rows, plan=plan, heads=H, dim=D,
                                                  vdim=V, scale=0.07)
         nbytes = seqs * n * (H * (D + R + 2 * V) + K + R) * 2
         add(f"latent_attention prefill {seqs}x{n}", mk_pre, nbytes, seqs * n * (n + 1) // 2 * H * 2 * (D + R + V) + seqs * n * H * 2 * K * (D + V))

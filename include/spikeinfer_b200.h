@@ -779,6 +779,52 @@ typedef struct spk_latent_out_args {
 } spk_latent_out_args;
 int spk_latent_out(const spk_latent_out_args* args, void* stream);
 
+/* The same attention for long portions, keys and values spelled out per head (1 where these sizes have the form: bf16, tiled pool, heads of
+ * up to 128 channels and a rotated part of up to 64).
+ * spk_latent_gather: cache rows of whole sequences out of their pages.  rows int32 [n_rows][4] = (first destination row, rows (16 at
+ * most), batch row, first position); latents [n_ctx, rank_pad], rotated [n_ctx, 64].
+ * spk_latent_prefill: q [n, heads, dim + rot_dim] before its rotation; kv [n_ctx, heads * (dim_pad + vdim_pad)]: the heads' unrotated keys,
+ * then their values, padded to multiples of 64 channels with zeros; kr [n_ctx, 64] = rotated; tiles int32 [n_tiles][4] = (first token,
+ * tokens (128 at most), first context row of the sequence, position of the first token).  out as in spk_latent_out; scale > 0. */
+int spk_latent_prefill_form(int dtype, int dim, int rot_pad, int vdim, int tiled);
+typedef struct spk_latent_gather_args {
+    const void* pool;
+    const int32_t* tables;
+    const int32_t* rows;
+    void* latents;
+    void* rotated;
+    int64_t table_stride;
+    int64_t table_rows;
+    int64_t max_blocks;
+    int64_t num_blocks;
+    int64_t n_ctx;
+    int32_t n_rows, rank_pad, block_size, _pad;
+    uint32_t* status;
+} spk_latent_gather_args;
+int spk_latent_gather(const spk_latent_gather_args* args, void* stream);
+typedef struct spk_latent_prefill_args {
+    const void* q;
+    const void* kv;
+    const void* kr;
+    const int32_t* tiles;
+    const float* sink;
+    const void* gate;
+    void* out;
+    const float* rot_table;
+    int64_t rot_positions;
+    int64_t n;
+    int64_t n_ctx;
+    int64_t gate_stride;
+    int64_t out_stride;
+    int32_t n_tiles, heads, dim, rot_dim, vdim, dim_pad, vdim_pad;
+    int32_t vec_q, vec_out;     /* set by the call */
+    int32_t dtype;
+    float scale;
+    float _pad;
+    uint32_t* status;
+} spk_latent_prefill_args;
+int spk_latent_prefill(const spk_latent_prefill_args* args, void* stream);
+
 /* Gated delta rule with one decay per head and key channel:
  *   q, k, v <- silu(causal convolution of the projections, `taps` taps per channel);  q, k <- unit vectors per head, q * dim^-1/2;
  *   S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  g = exp(-exp(a_log) softplus(a + dt_bias)), beta = sigmoid(b);

@@ -179,6 +179,20 @@ class LatentOutArgs(Structure):
                        "i splits heads vdim rank dtype _pad; p status")
 
 
+class LatentGatherArgs(Structure):
+    """Mirror of ``spk_latent_gather_args``."""
+
+    _fields_ = _fields("p pool tables rows latents rotated; l table_stride table_rows max_blocks num_blocks n_ctx; i n_rows rank_pad block_size _pad; "
+                       "p status")
+
+
+class LatentPrefillArgs(Structure):
+    """Mirror of ``spk_latent_prefill_args``."""
+
+    _fields_ = _fields("p q kv kr tiles sink gate out rot_table; l rot_positions n n_ctx gate_stride out_stride; "
+                       "i n_tiles heads dim rot_dim vdim dim_pad vdim_pad vec_q vec_out dtype; f scale _pad; p status")
+
+
 class DeltaArgs(Structure):
     """Mirror of ``spk_delta_args``."""
 
@@ -268,6 +282,9 @@ SIGNATURES = {
     "spk_latent_attn_splits": (c_int, [c_int] * 7 + [c_int64, c_int, c_int64]),
     "spk_latent_attn": (c_int, [POINTER(LatentAttnArgs), c_void_p]),
     "spk_latent_out": (c_int, [POINTER(LatentOutArgs), c_void_p]),
+    "spk_latent_prefill_form": (c_int, [c_int] * 5),
+    "spk_latent_gather": (c_int, [POINTER(LatentGatherArgs), c_void_p]),
+    "spk_latent_prefill": (c_int, [POINTER(LatentPrefillArgs), c_void_p]),
     "spk_delta_step": (c_int, [POINTER(DeltaArgs), c_void_p]),
     "spk_delta_chunk_tokens": (c_int, [c_int] * 3),
     "spk_delta_workspace_bytes": (c_int64, [c_int64] + [c_int] * 5),

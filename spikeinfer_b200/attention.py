@@ -93,13 +93,15 @@ class PrefillPlan:
     tables, built on the host and copied once per batch; all layers share them."""
 
     def __init__(self, starts, lens, contexts, rows, device: torch.device) -> None:
-        self.starts, self.lens, self.contexts, self.rows = list(starts), list(lens), list(contexts), list(rows)
+        self.starts, self.lens, self.contexts_before, self.rows = list(starts), list(lens), list(contexts), list(rows)
         if len(self.rows) != len(self.lens):
             raise ValueError("every prefill portion needs its batch row")
         self.device = device
         self._tiles: dict[int, torch.Tensor] = {}
         self._chunks: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}
         self._portions: torch.Tensor | None = None
+        self._contexts: tuple[list[int], int, torch.Tensor] | None = None
+        self._context_tiles: dict[int, torch.Tensor] = {}
 
     def _table(self, entries: list[tuple[int, int, int, int]]) -> torch.Tensor:
         return torch.tensor(entries, dtype=torch.int32).to(self.device)
@@ -107,19 +109,41 @@ class PrefillPlan:
     def portions(self) -> torch.Tensor:
         """int32 ``[portions, 4]``: (first token, tokens, row, tokens before this portion)."""
         if self._portions is None:
-            self._portions = self._table([(s, n, row, ctx) for s, n, ctx, row in zip(self.starts, self.lens, self.contexts, self.rows)])
+            self._portions = self._table([(s, n, row, ctx) for s, n, ctx, row in zip(self.starts, self.lens, self.contexts_before, self.rows)])
         return self._portions
+
+    def contexts(self) -> tuple[list[int], int, torch.Tensor]:
+        """All portions' sequences laid out one after the other: first row of each, rows in all, and the work list that gathers them, int32
+        ``[n, 4]``: (first row, up to 16 rows, batch row, first position)."""
+        if self._contexts is None:
+            starts, at, rows = [], 0, []
+            for n, ctx, row in zip(self.lens, self.contexts_before, self.rows):
+                starts.append(at)
+                rows += [(at + lo, min(16, ctx + n - lo), row, lo) for lo in range(0, ctx + n, 16)]
+                at += ctx + n
+            self._contexts = (starts, at, self._table(rows))
+        return self._contexts
+
+    def context_tiles(self, tokens: int) -> torch.Tensor:
+        """int32 ``[n, 4]``: (first token, tokens, first row of the sequence in :meth:`contexts`, position of the first token), longest
+        context first."""
+        if tokens not in self._context_tiles:
+            out = [(s + lo, min(tokens, n - lo), at, ctx + lo)
+                   for s, n, ctx, at in zip(self.starts, self.lens, self.contexts_before, self.contexts()[0]) for lo in range(0, n, tokens)]
+            out.sort(key=lambda e: -e[3])
+            self._context_tiles[tokens] = self._table(out)
+        return self._context_tiles[tokens]
 
     @property
     def most_keys(self) -> int:
         """Keys the last token of the longest sequence sees."""
-        return max(c + n for c, n in zip(self.contexts, self.lens))
+        return max(c + n for c, n in zip(self.contexts_before, self.lens))
 
     def tiles(self, tokens: int) -> torch.Tensor:
         """int32 ``[n, 4]``: (first token, tokens, row, position of the first token), longest context first."""
         if tokens not in self._tiles:
             out = [(s + lo, min(tokens, n - lo), row, ctx + lo)
-                   for s, n, ctx, row in zip(self.starts, self.lens, self.contexts, self.rows) for lo in range(0, n, tokens)]
+                   for s, n, ctx, row in zip(self.starts, self.lens, self.contexts_before, self.rows) for lo in range(0, n, tokens)]
             out.sort(key=lambda e: -e[3])  # the tiles that see the most keys start first
             self._tiles[tokens] = self._table(out)
         return self._tiles[tokens]
@@ -129,7 +153,7 @@ class PrefillPlan:
         (first chunk, chunks, row, tokens before this portion)."""
         if tokens not in self._chunks:
             chunks, seqs = [], []
-            for i, (s, n, ctx, row) in enumerate(zip(self.starts, self.lens, self.contexts, self.rows)):
+            for i, (s, n, ctx, row) in enumerate(zip(self.starts, self.lens, self.contexts_before, self.rows)):
                 seqs.append((len(chunks), -(-n // tokens), row, ctx))
                 chunks += [(s + lo, min(tokens, n - lo), i, lo // tokens) for lo in range(0, n, tokens)]
             self._chunks[tokens] = (self._table(chunks), self._table(seqs))

@@ -137,6 +137,78 @@ latent_query_kernel(const spk_latent_query_args a) {
     rotate_query<T>(a, h, t0, rows);
 }
 
+// bf16 on the tensor cores: CTA = (head, 128 latent channels, 64 tokens), heads of up to 256 channels; warps 4 (tokens) x 2 (channels).
+constexpr int kMmaRows = 64, kMmaCols = 128;
+
+// `rows` x `width` elements into a padded tile, zeros beyond; asynchronous where rows are 16-byte aligned.
+__device__ __forceinline__ void fetch_tile(__nv_bfloat16* dst, int stride, const __nv_bfloat16* src, int64_t ld, int rows, int live_rows, int width, int live,
+                                           bool vec) {
+    const int groups = width / 8;
+    for (int i = threadIdx.x; i < rows * groups; i += blockDim.x) {
+        const int r = i / groups, c = (i % groups) * 8;
+        if (vec) {
+            const bool in = r < live_rows && c < live;
+            cp_async16(smem_u32(dst + r * stride + c), in ? src + r * ld + c : src, in);
+        } else {
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+                dst[r * stride + c + k] = r < live_rows && c + k < live ? src[r * ld + c + k] : __float2bfloat16_rn(0.0f);
+        }
+    }
+}
+
+__global__ void __launch_bounds__(kThreads)
+latent_query_mma_kernel(const spk_latent_query_args a, const int dp, const bool vec_q, const bool vec_w) {
+    extern __shared__ __align__(16) uint8_t raw[];
+    const int SQ = dp + 8;
+    constexpr int SW = kMmaCols + 8;
+    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(raw);  // [64][dp + 8]
+    __nv_bfloat16* ws = qs + kMmaRows * SQ;                      // [dp][128 + 8]
+    const int h = blockIdx.x, c0 = blockIdx.y * kMmaCols;
+    const int64_t t0 = static_cast<int64_t>(blockIdx.z) * kMmaRows;
+    const int rows = static_cast<int>(min(static_cast<int64_t>(kMmaRows), a.n - t0));
+    const int64_t ld = static_cast<int64_t>(a.heads) * (a.dim + a.rot_dim);
+    fetch_tile(ws, SW, static_cast<const __nv_bfloat16*>(a.w_uk) + static_cast<int64_t>(h) * a.dim * a.rank + c0, a.rank, dp, a.dim, kMmaCols,
+               a.rank - c0, vec_w);
+    fetch_tile(qs, SQ, static_cast<const __nv_bfloat16*>(a.q) + t0 * ld + static_cast<int64_t>(h) * (a.dim + a.rot_dim), ld, (rows + 15) & ~15, rows, dp,
+               a.dim, vec_q);
+    cp_async_commit();
+    if (blockIdx.y == 0) rotate_query<__nv_bfloat16>(a, h, t0, rows);
+    cp_async_wait_all();
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
+    const int i0 = (warp & 3) * 16, e0 = (warp >> 2) * 64;
+    if (i0 >= rows) return;
+    float acc[8][4] = {};
+    for (int d = 0; d < dp; d += 16) {
+        uint32_t x[4];
+        ldsm4(x, smem_u32(qs + (i0 + (lane & 15)) * SQ + d + (lane >> 4) * 8));
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+            uint32_t b[4];
+            ldsm4t(b, smem_u32(ws + (d + (m & 1) * 8 + mr) * SW + e0 + n * 8 + (m >> 1) * 8));
+            mma16816(acc[n], x, b[0], b[1]);
+            mma16816(acc[n + 1], x, b[2], b[3]);
+        }
+    }
+    const int W = a.rank_pad + a.rot_pad;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int r = i0 + gid + 8 * i;
+        if (r >= rows) continue;
+        __nv_bfloat16* o = static_cast<__nv_bfloat16*>(a.out) + ((t0 + r) * a.heads + h) * W;
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+            const int c = c0 + e0 + n * 8 + tig * 2;
+            if (c + 1 < a.rank && (W & 1) == 0) *reinterpret_cast<uint32_t*>(o + c) = pack_bf16(acc[n][2 * i], acc[n][2 * i + 1]);
+            else {
+                if (c < a.rank) o[c] = __float2bfloat16_rn(acc[n][2 * i]);
+                if (c + 1 < a.rank) o[c + 1] = __float2bfloat16_rn(acc[n][2 * i + 1]);
+            }
+        }
+    }
+}
+
 // ---- attention, 32-bit ---------------------------------------------------------------------------------------------------
 constexpr int kHeadsPer = kWarps;  // heads of a CTA, one warp each for the scores
 constexpr int kKeys = 32;
@@ -259,8 +331,7 @@ __device__ __forceinline__ void range_weights(const spk_latent_out_args& a, int 
     }
 }
 
-// CTA = (head, 16 tokens): any sizes.
-template <typename T>
+// 32-bit, CTA = (head, 16 tokens): any sizes.
 __global__ void __launch_bounds__(kThreads)
 latent_out_kernel(const spk_latent_out_args a) {
     extern __shared__ float sm[];
@@ -282,10 +353,10 @@ latent_out_kernel(const spk_latent_out_args a) {
     }
     __syncthreads();
     for (int e = threadIdx.x >> 5; e < a.vdim; e += kWarps) {
-        const T* w = static_cast<const T*>(a.w_uv) + (static_cast<int64_t>(h) * a.vdim + e) * a.rank;
+        const float* w = static_cast<const float*>(a.w_uv) + (static_cast<int64_t>(h) * a.vdim + e) * a.rank;
         float acc[kOutRows] = {};
         for (int c = lane; c < a.rank; c += 32) {
-            const float x = spk_to_float<T>(w[c]);
+            const float x = (w[c]);
 #pragma unroll
             for (int r = 0; r < kOutRows; ++r) acc[r] = fmaf(o[r * a.rank + c], x, acc[r]);
         }
@@ -297,9 +368,76 @@ latent_out_kernel(const spk_latent_out_args a) {
         }
         if (lane < rows) {
             const int64_t c = static_cast<int64_t>(h) * a.vdim + e;
-            const float g = spk_to_float<T>(static_cast<const T*>(a.gate)[(t0 + lane) * a.gate_stride + c]);
-            static_cast<T*>(a.out)[(t0 + lane) * a.out_stride + c] = spk_from_float<T>(mine * spk_sigmoid(g));
+            const float g = (static_cast<const float*>(a.gate)[(t0 + lane) * a.gate_stride + c]);
+            static_cast<float*>(a.out)[(t0 + lane) * a.out_stride + c] = (mine * spk_sigmoid(g));
         }
+    }
+}
+
+// bf16 on the tensor cores: CTA = (head, 16 tokens, 128 value channels), a warp per sixteen channels.  The ranges' sums are put together 64
+// latent channels at a time, right where the product reads them; the value matrix follows through a two-stage ring.
+template <bool VEC>
+__global__ void __launch_bounds__(kThreads)
+latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
+    constexpr int K = 64, S = K + 8;
+    extern __shared__ __align__(16) uint8_t raw[];
+    __nv_bfloat16* os = reinterpret_cast<__nv_bfloat16*>(raw);  // two stages of [16][72]
+    __nv_bfloat16* ws = os + 2 * kOutRows * S;                   // two stages of [128][72]
+    float* wts = reinterpret_cast<float*>(ws + 2 * kMmaCols * S);  // [16][splits]
+    const int h = blockIdx.x, e0 = blockIdx.z * kMmaCols;
+    const int64_t t0 = static_cast<int64_t>(blockIdx.y) * kOutRows;
+    const int rows = static_cast<int>(min(static_cast<int64_t>(kOutRows), a.n - t0));
+    const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w_uv) + (static_cast<int64_t>(h) * a.vdim + e0) * a.rank;
+    const int live = min(kMmaCols, a.vdim - e0);
+    fetch_tile(ws, S, w, a.rank, kMmaCols, live, K, a.rank, vec_w);
+    cp_async_commit();
+    range_weights(a, h, t0, rows, wts);
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
+    const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
+    const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank;
+    const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
+    float acc[2][4] = {};
+    for (int k0 = 0, buf = 0; k0 < a.rank; k0 += K, buf ^= 1) {
+        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < rows) {
+            for (int s = 0; s < a.splits; ++s) {
+                const float f = wts[r * a.splits + s];
+                if (f != 0.0f) {
+                    const float4 x = spk_load4<float, VEC>(part + s * step + k0 + c4, a.rank - k0 - c4);
+                    y = make_float4(fmaf(f, x.x, y.x), fmaf(f, x.y, y.y), fmaf(f, x.z, y.z), fmaf(f, x.w, y.w));
+                }
+            }
+        }
+        *reinterpret_cast<uint2*>(os + buf * kOutRows * S + r * S + c4) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
+        cp_async_wait_all();
+        __syncthreads();  // this stage is there, the previous one has been read
+        if (k0 + K < a.rank) fetch_tile(ws + (buf ^ 1) * kMmaCols * S, S, w + k0 + K, a.rank, kMmaCols, live, K, a.rank - k0 - K, vec_w);
+        cp_async_commit();
+        const __nv_bfloat16 *ob = os + buf * kOutRows * S, *wb = ws + buf * kMmaCols * S;
+#pragma unroll
+        for (int k = 0; k < K; k += 16) {
+            uint32_t x[4], b[4];
+            ldsm4(x, smem_u32(ob + (lane & 15) * S + k + (lane >> 4) * 8));
+            ldsm4(b, smem_u32(wb + (warp * 16 + (m >> 1) * 8 + mr) * S + k + (m & 1) * 8));
+            mma16816(acc[0], x, b[0], b[1]);
+            mma16816(acc[1], x, b[2], b[3]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int q = gid + 8 * i;
+        if (q >= rows) continue;
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int e = e0 + warp * 16 + n * 8 + tig * 2 + j;
+                if (e >= a.vdim) continue;
+                const int64_t c = static_cast<int64_t>(h) * a.vdim + e;
+                const float g = __bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(t0 + q) * a.gate_stride + c]);
+                static_cast<__nv_bfloat16*>(a.out)[(t0 + q) * a.out_stride + c] = __float2bfloat16_rn(acc[n][2 * i + j] * spk_sigmoid(g));
+            }
     }
 }
 
@@ -336,6 +474,33 @@ int launch_query(const spk_latent_query_args& a, cudaStream_t s) {
     return SPK_OK;
 }
 
+bool at16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
+
+int launch_query_mma(const spk_latent_query_args& a, cudaStream_t s) {
+    const int dp = (a.dim + 15) & ~15;
+    const int64_t tiles = (a.n + kMmaRows - 1) / kMmaRows;
+    if (tiles > 65535) return SPK_ERR_TOO_LARGE;
+    const size_t bytes = 2 * (static_cast<size_t>(kMmaRows) * (dp + 8) + static_cast<size_t>(dp) * (kMmaCols + 8));
+    if (const int rc = with_smem(reinterpret_cast<const void*>(latent_query_mma_kernel), bytes)) return rc;
+    const bool vq = at16(a.q) && (a.dim + a.rot_dim) % 8 == 0 && a.dim % 8 == 0, vw = at16(a.w_uk) && a.rank % 8 == 0;
+    latent_query_mma_kernel<<<dim3(a.heads, (a.rank + kMmaCols - 1) / kMmaCols, static_cast<unsigned>(tiles)), kThreads, bytes, s>>>(a, dp, vq, vw);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+int launch_out_mma(const spk_latent_out_args& a, cudaStream_t s) {
+    const int64_t tiles = (a.n + kOutRows - 1) / kOutRows;
+    if (tiles > 65535) return SPK_ERR_TOO_LARGE;
+    const size_t bytes = 2 * 2 * (kOutRows + kMmaCols) * 72 + sizeof(float) * kOutRows * a.splits;
+    const dim3 grid(a.heads, static_cast<unsigned>(tiles), (a.vdim + kMmaCols - 1) / kMmaCols);
+    const bool vec = a.rank % 4 == 0 && at16(a.partials), vw = at16(a.w_uv) && a.rank % 8 == 0;
+    auto* fn = vec ? latent_out_mma_kernel<true> : latent_out_mma_kernel<false>;
+    if (const int rc = with_smem(reinterpret_cast<const void*>(fn), bytes)) return rc;
+    fn<<<grid, kThreads, bytes, s>>>(a, vw);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
 template <typename T>
 int launch_simt(const spk_latent_attn_args& a, cudaStream_t s) {
     if (a.rank > kMaxChan * kThreads) return SPK_ERR_UNSUPPORTED;
@@ -348,13 +513,12 @@ int launch_simt(const spk_latent_attn_args& a, cudaStream_t s) {
     return SPK_OK;
 }
 
-template <typename T>
 int launch_out(const spk_latent_out_args& a, cudaStream_t s) {
     const int64_t tiles = (a.n + kOutRows - 1) / kOutRows;
     if (tiles > 65535) return SPK_ERR_TOO_LARGE;
     const size_t bytes = sizeof(float) * kOutRows * (a.splits + static_cast<size_t>(a.rank));
-    if (const int rc = with_smem(reinterpret_cast<const void*>(latent_out_kernel<T>), bytes)) return rc;
-    latent_out_kernel<T><<<dim3(a.heads, static_cast<unsigned>(tiles)), kThreads, bytes, s>>>(a);
+    if (const int rc = with_smem(reinterpret_cast<const void*>(latent_out_kernel), bytes)) return rc;
+    latent_out_kernel<<<dim3(a.heads, static_cast<unsigned>(tiles)), kThreads, bytes, s>>>(a);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -393,7 +557,8 @@ extern "C" int spk_latent_query(const spk_latent_query_args* a, void* stream) {
     if (a->n == 0) return SPK_OK;
     if (a->q == nullptr || a->w_uk == nullptr || a->out == nullptr || a->rot_table == nullptr || a->positions == nullptr) return SPK_ERR_NULL_POINTER;
     cudaStream_t s = spk_stream(stream);
-    return a->dtype == SPK_F32 ? launch_query<float>(*a, s) : launch_query<__nv_bfloat16>(*a, s);
+    if (a->dtype == SPK_BF16) return a->dim <= 256 ? launch_query_mma(*a, s) : launch_query<__nv_bfloat16>(*a, s);
+    return launch_query<float>(*a, s);
 }
 
 extern "C" int spk_latent_attn_splits(int dtype, int rank, int rot_dim, int rank_pad, int rot_pad, int tiled, int block_size, int64_t n, int heads,
@@ -438,5 +603,5 @@ extern "C" int spk_latent_out(const spk_latent_out_args* a, void* stream) {
         (a->seq_lens == nullptr && a->positions == nullptr))
         return SPK_ERR_NULL_POINTER;
     cudaStream_t s = spk_stream(stream);
-    return a->dtype == SPK_F32 ? launch_out<float>(*a, s) : launch_out<__nv_bfloat16>(*a, s);
+    return a->dtype == SPK_F32 ? launch_out(*a, s) : launch_out_mma(*a, s);
 }

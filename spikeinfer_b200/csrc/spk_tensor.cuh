@@ -102,6 +102,12 @@ __device__ __forceinline__ void tmem_ld32(uint32_t addr, uint32_t (&r)[32]) {
 __device__ __forceinline__ void tmem_wait_ld(uint32_t (&r)[32]) {
     asm volatile("tcgen05.wait::ld.sync.aligned;" : SPK_R8(r, 0), SPK_R8(r, 8), SPK_R8(r, 16), SPK_R8(r, 24) : : "memory");
 }
+// Sixteen columns, complete on return.
+__device__ __forceinline__ void tmem_ld16(uint32_t addr, uint32_t (&r)[16]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                 : SPK_W8(r, 0), SPK_W8(r, 8) : "r"(addr) : "memory");
+    asm volatile("tcgen05.wait::ld.sync.aligned;" : SPK_R8(r, 0), SPK_R8(r, 8) : : "memory");
+}
 __device__ __forceinline__ void tmem_st16(uint32_t addr, const uint32_t (&r)[16]) {
     asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
                  ::"r"(addr), SPK_I8(r, 0), SPK_I8(r, 8) : "memory");

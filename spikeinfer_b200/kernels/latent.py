@@ -6,6 +6,7 @@ key weights are 32-bit."""
 from __future__ import annotations
 
 import torch
+import torch.nn.functional as F
 
 from .. import _lib
 from .dense import _call, _f32, _ptr
@@ -80,4 +81,58 @@ def latent_attention(q: torch.Tensor, pool, tables: torch.Tensor, sink: torch.Te
         seq_lens=None if prefill else seq_lens.data_ptr(), active=_ptr(active), positions=_ptr(positions), gate_stride=gate.stride(0),
         out_stride=out.stride(0), n=n, splits=splits, heads=heads, vdim=vdim, rank=pool.rank, dtype=code, status=_ptr(status))
     _call("spk_latent_out", b, q.device)
+    return out
+
+
+PREFILL_TILE = 128          # query tokens per tile of the spelled-out form
+PREFILL_MIN_TOKENS = 64     # fewer tokens in a call are taken into the latent space one by one
+PREFILL_CONTEXT_RATIO = 32  # spelling keys and values out pays off up to this many cache rows per query token
+PREFILL_MAX_BYTES = 8 << 30
+
+
+def spelled_out_weights(w_uk: torch.Tensor, w_uv: torch.Tensor, heads: int) -> torch.Tensor:
+    """Key and value matrices of all heads stacked, every head padded to a multiple of 64 channels with zeros."""
+    def pad(w):
+        d = w.shape[0] // heads
+        return F.pad(w.view(heads, d, -1), (0, 0, 0, -d % 64)).flatten(0, 1)
+    return torch.cat((pad(w_uk), pad(w_uv))).contiguous()
+
+
+def latent_prefill(q: torch.Tensor, pool, tables: torch.Tensor, w_uk: torch.Tensor, w_uv: torch.Tensor, w_kv: torch.Tensor | None, sink: torch.Tensor,
+                   gate: torch.Tensor, out: torch.Tensor, *, rot_table: torch.Tensor, positions: torch.Tensor, token_rows: torch.Tensor, plan, heads: int,
+                   dim: int, vdim: int, scale: float, spelled_out: bool | None = None, status: torch.Tensor | None = None) -> torch.Tensor:
+    """Attention of the tokens of prefill portions (``plan``), ``q [n, heads * (dim + rot_dim)]`` as projected.  Long portions spell keys and
+    values out (``w_kv`` from :func:`spelled_out_weights`; ``spelled_out`` overrides the choice), others take the queries into the latent
+    space.  The rest as in :func:`latent_attention`."""
+    lib = _lib.load()
+    n = q.shape[0]
+    code = _lib.dtype_code(q.dtype)
+    possible = w_kv is not None and scale > 0 and bool(lib.spk_latent_prefill_form(code, dim, pool.rot_pad, vdim, int(pool.tiled)))
+    if spelled_out is None:
+        rows = sum(plan.contexts_before) + sum(plan.lens)
+        spelled_out = possible and n >= PREFILL_MIN_TOKENS and rows <= PREFILL_CONTEXT_RATIO * n and rows * w_kv.shape[0] * 2 <= PREFILL_MAX_BYTES
+    if not spelled_out:
+        ql = latent_query(q, w_uk, pool, rot_table, positions, heads=heads, dim=dim, status=status)
+        return latent_attention(ql, pool, tables, sink, w_uv, gate, out, vdim=vdim, scale=scale, token_rows=token_rows, positions=positions,
+                                most_keys=plan.most_keys, status=status)
+    if not possible:
+        raise ValueError("these sizes have no spelled-out form")
+    _f32(sink, "sink", heads)
+    if not q.is_contiguous() or q.shape[1] != heads * (dim + pool.rot_dim) or out.shape != (n, heads * vdim) or gate.shape != out.shape:
+        raise ValueError("q, gate and out do not fit the head sizes")
+    _, total, rows = plan.contexts()
+    latents = torch.empty((total, pool.rank_pad), dtype=q.dtype, device=q.device)
+    rotated = torch.empty((total, 64), dtype=q.dtype, device=q.device)
+    g = _lib.LatentGatherArgs(pool=pool.data.data_ptr(), tables=tables.data_ptr(), rows=rows.data_ptr(), latents=latents.data_ptr(), rotated=rotated.data_ptr(),
+                              table_stride=tables.stride(0), table_rows=tables.shape[0], max_blocks=tables.shape[1], num_blocks=pool.data.shape[0],
+                              n_ctx=total, n_rows=rows.shape[0], rank_pad=pool.rank_pad, block_size=pool.block_size, status=_ptr(status))
+    _call("spk_latent_gather", g, q.device)
+    kv = F.linear(latents[:, : pool.rank], w_kv)
+    tiles = plan.context_tiles(PREFILL_TILE)
+    a = _lib.LatentPrefillArgs(
+        q=q.data_ptr(), kv=kv.data_ptr(), kr=rotated.data_ptr(), tiles=tiles.data_ptr(), sink=sink.data_ptr(), gate=gate.data_ptr(), out=out.data_ptr(),
+        rot_table=rot_table.data_ptr(), rot_positions=rot_table.shape[0], n=n, n_ctx=total, gate_stride=gate.stride(0), out_stride=out.stride(0),
+        n_tiles=tiles.shape[0], heads=heads, dim=dim, rot_dim=pool.rot_dim, vdim=vdim, dim_pad=-(-dim // 64) * 64, vdim_pad=-(-vdim // 64) * 64,
+        dtype=code, scale=scale, status=_ptr(status))
+    _call("spk_latent_prefill", a, q.device)
     return out

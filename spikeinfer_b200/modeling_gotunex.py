@@ -27,7 +27,7 @@ from .engine.kv_state_cache import LatentSpec, LayerCacheSpec, PagedKVStateCache
 from .kernels.delta import delta_rule
 from .kernels.dense import gelu_tanh, rms_residual
 from .kernels.experts import ExpertRouter, ExpertWeights, experts_forward
-from .kernels.latent import latent_attention, latent_prepare, latent_query
+from .kernels.latent import latent_attention, latent_prefill, latent_prepare, latent_query, spelled_out_weights
 from .rotary import RotaryConfig
 
 
@@ -156,6 +156,7 @@ class _LatentAttention:
         self.w_uq = _expect("uq", get("mix.uq"), c.heads * (c.dim + c.rot_dim), c.q_rank)
         self.w_uk = _expect("uk", get("mix.uk"), c.heads * c.dim, c.kv_rank)
         self.w_uv = _expect("uv", get("mix.uv"), c.heads * c.vdim, c.kv_rank)
+        self.w_kv = spelled_out_weights(self.w_uk, self.w_uv, c.heads) if self.w_uk.dtype == torch.bfloat16 else None
         self.sink = _expect("sink", f32("mix.sink"), c.heads)
         self.out_width = c.heads * c.vdim
         self.w_o = _expect("o", get("mix.o"), width, self.out_width)
@@ -171,14 +172,14 @@ class _LatentAttention:
         own = {} if c.kv_from is not None else dict(kv=z[:, self.at["dkv"]], w_kv=self.kv_norm, pool=pool, rot_table=rot, positions=positions,
                                                     slot_mapping=meta.slot_mapping)
         cq = latent_prepare(z[:, self.at["dq"]], self.q_norm, eps=model.config.eps, status=meta.status, **own)
-        q = latent_query(model._matmul(cq, self.w_uq), self.w_uk, pool, rot, positions, heads=c.heads, dim=c.dim, status=meta.status)
+        q, gate = model._matmul(cq, self.w_uq), z[:, self.at["g"]]
+        common = dict(vdim=c.vdim, scale=c.scale, status=meta.status)
         if meta.num_prefills:
-            where = dict(token_rows=meta.token_rows, positions=positions, most_keys=meta.prefill_plan().most_keys)
-            tables = meta.row_tables
-        else:
-            where = dict(seq_lens=meta.seq_lens, active=meta.row_active)
-            tables = meta.block_tables
-        latent_attention(q, pool, tables, self.sink, self.w_uv, z[:, self.at["g"]], out, vdim=c.vdim, scale=c.scale, status=meta.status, **where)
+            latent_prefill(q, pool, meta.row_tables, self.w_uk, self.w_uv, self.w_kv, self.sink, gate, out, rot_table=rot, positions=positions,
+                           token_rows=meta.token_rows, plan=meta.prefill_plan(), heads=c.heads, dim=c.dim, **common)
+            return
+        ql = latent_query(q, self.w_uk, pool, rot, positions, heads=c.heads, dim=c.dim, status=meta.status)
+        latent_attention(ql, pool, meta.block_tables, self.sink, self.w_uv, gate, out, seq_lens=meta.seq_lens, active=meta.row_active, **common)
 
 
 class _ChannelDelta:

@@ -63,7 +63,8 @@ def test_registry_knows_the_design():
 def test_argument_structs_have_the_header_layout(tmp_path):
     names = {"spk_rms_residual_args": _lib.RmsResidualArgs, "spk_expert_route_args": _lib.ExpertRouteArgs, "spk_experts_args": _lib.ExpertsArgs,
              "spk_latent_prepare_args": _lib.LatentPrepareArgs, "spk_latent_query_args": _lib.LatentQueryArgs,
-             "spk_latent_attn_args": _lib.LatentAttnArgs, "spk_latent_out_args": _lib.LatentOutArgs, "spk_delta_args": _lib.DeltaArgs}
+             "spk_latent_attn_args": _lib.LatentAttnArgs, "spk_latent_out_args": _lib.LatentOutArgs, "spk_delta_args": _lib.DeltaArgs,
+             "spk_latent_gather_args": _lib.LatentGatherArgs, "spk_latent_prefill_args": _lib.LatentPrefillArgs}
     lines = [f'printf("{c}.{f} %zu\\n", offsetof({c}, {f}));' for c, s in names.items() for f, _ in s._fields_]
     lines += [f'printf("{c} %zu\\n", sizeof({c}));' for c in names]
     src = tmp_path / "layout.c"
@@ -138,6 +139,10 @@ def test_latent_pools_and_sharing():
 def test_portion_table():
     plan = PrefillPlan([0, 5, 7], [5, 2, 40], [0, 31, 8], [3, 0, 1], torch.device("cpu"))
     assert plan.portions().tolist() == [[0, 5, 3, 0], [5, 2, 0, 31], [7, 40, 1, 8]] and plan.most_keys == 48
+    starts, total, rows = plan.contexts()
+    assert (starts, total) == ([0, 5, 38], 86)
+    assert rows.tolist() == [[0, 5, 3, 0], [5, 16, 0, 0], [21, 16, 0, 16], [37, 1, 0, 32], [38, 16, 1, 0], [54, 16, 1, 16], [70, 16, 1, 32]]
+    assert sorted(plan.context_tiles(32).tolist()) == [[0, 5, 0, 0], [5, 2, 5, 31], [7, 32, 38, 8], [39, 8, 38, 40]]
 
 
 # ---- the plain implementation itself ---------------------------------------------------------------------------

@@ -288,6 +288,48 @@ def test_attention_decode_and_prefill(dev, status, heads, dim, rot_dim, vdim, ra
         assert rel(out[t], reference(i, q[t], gate[t], [p])[0]) < TOL[dtype] * (1 if dtype == F32 else 2), (i, p)
 
 
+@pytest.mark.parametrize("block_size", [16, 64])
+@pytest.mark.parametrize("heads,dim,rot_dim,vdim,rank", [s for s in SIZES if s[1] <= 128 and s[2] <= 64])
+def test_spelled_out_prefill(dev, status, heads, dim, rot_dim, vdim, rank, block_size):
+    """Portions of several sequences, some behind a cached context: the form with keys and values spelled out against the plain
+    implementation (a few positions of each) and against the other form (all)."""
+    g = gen(heads + dim)
+    rnd = lambda *s: torch.randn(*s, generator=g)
+    ctx, lens, dtype = [0, 37, 200, 0, 128], [70, 5, 300, 1, 129], BF
+    rot, scale = dict(dims=rot_dim, base=800.0), 0.4 / math.sqrt(dim + rot_dim)
+    table = RotaryConfig(rot_dim, 800.0).table(512, dev)
+    seqs = [(rnd(c + n, rank + rot_dim)).to(dtype).float() for c, n in zip(ctx, lens)]
+    seqs[2][450] *= 6                                    # late scores above everything before: the reference moves
+    seqs[2][451:460, :] *= 3
+    pool, tables = filled_pool(dev, dtype, seqs, rank, rot_dim, block_size, 5)
+    w_uk, w_uv = ((rnd(heads * d, rank) / math.sqrt(rank)).to(dtype) for d in (dim, vdim))
+    sink = rnd(heads) * 2
+    sink[0] = 6.0
+    n = sum(lens)
+    starts = [sum(lens[:i]) for i in range(5)]
+    q, gate = (rnd(n, heads * (dim + rot_dim)) * 3).to(dtype), rnd(n, heads * vdim).to(dtype)
+    pos = torch.cat([torch.arange(c, c + m) for c, m in zip(ctx, lens)]).to(dev)
+    rows = torch.cat([torch.full((m,), i, dtype=torch.int32) for i, m in enumerate(lens)]).to(dev)
+    plan = PrefillPlan(starts, lens, ctx, list(range(5)), dev)
+    dd = lambda t: t.to(dev)
+    w_kv = kl.spelled_out_weights(dd(w_uk), dd(w_uv), heads)
+    outs = []
+    for form in (True, False):
+        out = torch.full((n, heads * vdim + 8), float("nan"), dtype=dtype, device=dev)[:, : heads * vdim]
+        kl.latent_prefill(dd(q), pool, tables, dd(w_uk), dd(w_uv), w_kv, dd(sink), dd(gate), out, rot_table=table, positions=pos, token_rows=rows, plan=plan,
+                          heads=heads, dim=dim, vdim=vdim, scale=scale, spelled_out=form, status=status)
+        outs.append(out.cpu())
+    assert rel(outs[0], outs[1]) < 3e-2
+    f = lambda t: t.double()
+    for i, picks in enumerate([(0, 1, 15, 16, 63, 64, 69), (0, 4), (0, 55, 56, 183, 184, 249, 250, 251, 299), (0,), (0, 1, 127, 128)]):
+        t = [starts[i] + p for p in picks]
+        c = f(seqs[i])
+        want = attention_reference(f(q[t]).view(len(t), heads, -1), c[:, :rank], c[:, rank:], f(w_uk), f(w_uv), f(sink), f(gate[t]),
+                                   [ctx[i] + p for p in picks], rot, scale, heads, dim, vdim)
+        for k in range(len(t)):
+            assert rel(outs[0][t[k]], want[k]) < 2.4e-2, (i, picks[k])
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,rank", [(2, 56), (20, 256), (4, 512)])
 def test_one_key_stands_out(dev, status, heads, rank, dtype):
@@ -326,6 +368,19 @@ def test_one_key_stands_out(dev, status, heads, rank, dtype):
             assert (row.float().cpu() - loud).abs().max() < 0.1, j
         if j > 0:
             assert out[0].abs().max() < 0.1, j
+        if dtype == BF:  # a whole portion, keys and values spelled out
+            m = 320
+            lo = min(max(j - 100, 0), n - m)
+            plan = PrefillPlan([0], [m], [lo], [0], dev)
+            qs = dd(q[:1].flatten(1).to(dtype)).expand(m, -1).contiguous()
+            full = torch.empty(m, heads * vdim, dtype=dtype, device=dev)
+            kl.latent_prefill(qs, pool, tables, dd(w_uk.to(dtype)), dd(w_uv.to(dtype)), kl.spelled_out_weights(dd(w_uk.to(dtype)), dd(w_uv.to(dtype)), heads),
+                              sink, gate[:1].expand(m, -1).contiguous(), full, rot_table=table, positions=torch.arange(lo, lo + m, device=dev),
+                              token_rows=torch.zeros(m, dtype=torch.int32, device=dev), plan=plan, heads=heads, dim=dim, vdim=vdim, scale=0.5,
+                              spelled_out=True, status=status)
+            assert (full[j - lo:].float().cpu() - loud).abs().max() < 0.1, j
+            if j > lo:
+                assert full[: j - lo].abs().max() < 0.1, j
 
 
 def test_a_sink_takes_its_share(dev, status):
