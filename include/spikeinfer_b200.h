@@ -856,6 +856,7 @@ typedef struct spk_delta_args {
     int64_t out_stride;
     const int32_t* chunks;      /* prefill form: int32 [n_chunks][4] = (first token, tokens, portion, index in the portion) */
     const int32_t* portions;    /* int32 [n_portions][4] = (first token, tokens, row, tokens before) */
+    const int32_t* seqs;        /* int32 [n_portions][4] = (first chunk, chunks, row, tokens before) */
     void* workspace;
     int64_t workspace_bytes;
     int64_t n;
@@ -869,7 +870,7 @@ typedef struct spk_delta_args {
 int spk_delta_step(const spk_delta_args* args, void* stream);
 /* Tokens per chunk of the prefill form, and its workspace. */
 int spk_delta_chunk_tokens(int dtype, int dim, int vdim);
-int64_t spk_delta_workspace_bytes(int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim);
+int64_t spk_delta_workspace_bytes(int dtype, int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim);
 int spk_delta_prefill(const spk_delta_args* args, void* stream);
 
 #ifdef __cplusplus

@@ -197,7 +197,7 @@ class DeltaArgs(Structure):
     """Mirror of ``spk_delta_args``."""
 
     _fields_ = _fields("p q k v b a gate; l ld ld2; p conv_q conv_k conv_v a_log dt_bias w_norm state conv_state; l state_rows; "
-                       "p positions active out; l out_stride; p chunks portions workspace; l workspace_bytes n; "
+                       "p positions active out; l out_stride; p chunks portions seqs workspace; l workspace_bytes n; "
                        "i n_chunks n_portions heads kv_heads dim vdim taps dtype; f eps _pad; p status")
 
 
@@ -287,7 +287,7 @@ SIGNATURES = {
     "spk_latent_prefill": (c_int, [POINTER(LatentPrefillArgs), c_void_p]),
     "spk_delta_step": (c_int, [POINTER(DeltaArgs), c_void_p]),
     "spk_delta_chunk_tokens": (c_int, [c_int] * 3),
-    "spk_delta_workspace_bytes": (c_int64, [c_int64] + [c_int] * 5),
+    "spk_delta_workspace_bytes": (c_int64, [c_int, c_int64] + [c_int] * 5),
     "spk_delta_prefill": (c_int, [POINTER(DeltaArgs), c_void_p]),
     "spk_meta_release": (c_int, [c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),

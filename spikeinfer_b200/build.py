@@ -35,7 +35,7 @@ COMPONENTS = {
     "dense": ("spk_postnorm.cu", "spk_paged_attn.cu", "spk_sigmoid_prefill.cu", "spk_sigmoid_decode.cu", "spk_decay.cu",
               "spk_decay_mma.cu"),
     "latent": ("spk_prenorm.cu", "spk_experts.cu", "spk_experts_mma.cu", "spk_latent.cu", "spk_latent_decode.cu",
-               "spk_latent_prefill.cu", "spk_delta.cu"),
+               "spk_latent_prefill.cu", "spk_delta.cu", "spk_delta_mma.cu"),
 }
 
 

@@ -5,8 +5,9 @@
 //
 //  * delta_step_kernel: one token per row (decode).  A CTA owns a (head, row): it convolves, normalises, decays, updates and reads the
 //    state and writes the gated output; the state is read and written once.
-//  * prefill: delta_prepare_kernel (convolutions, unit vectors, decays, step sizes), delta_scan_kernel (the recurrence, columns of the
-//    state in registers, tokens one after the other) and delta_out_kernel (norm and gate).
+//  * prefill, any sizes, 32-bit: delta_prepare_kernel (convolutions, unit vectors, decays, step sizes), delta_scan_kernel (the
+//    recurrence, columns of the state in registers, tokens one after the other); bf16 heads of up to 128 channels take the chunked
+//    form of spk_delta_mma.cu instead.  delta_out_kernel (norm and gate) ends both.
 // The convolution's past lives in a ring of `taps` slots per row: a step writes its own slot and reads the others, so heads that
 // share a key need no order among themselves.
 #include "spk_delta.cuh"
@@ -17,7 +18,6 @@ namespace {
 using namespace spk_tc;
 
 constexpr int kThreads = 256;
-constexpr int kKeep = 16;  // state rows a thread of the step kernel keeps in registers
 
 // ---- decode ------------------------------------------------------------------------------------------------------------
 template <int W>
@@ -30,9 +30,9 @@ __device__ __forceinline__ void load_state(float (&s)[W], const float* p) {
     }
 }
 
-// CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  KEEP: a thread's
-// share of the state stays in registers between the two products; otherwise it is read twice.
-template <typename T, int W, bool KEEP>
+// CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  KEEP: rows of the
+// state that are a thread's share and stay in its registers between the two products; 0: any share, read twice.
+template <typename T, int W, int KEEP>
 __global__ void __launch_bounds__(kThreads)
 delta_step_kernel(const spk_delta_args a) {
     extern __shared__ float sm[];
@@ -56,10 +56,10 @@ delta_step_kernel(const spk_delta_args a) {
     const int slice = slices > 1 ? threadIdx.x / cols : 0;
     const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
     const bool mine = slice < slices;
-    float s[KEEP ? kKeep : 1][W];
+    float s[KEEP > 0 ? KEEP : 1][W];
     if (KEEP && mine) {  // on its way before the projections are looked at
 #pragma unroll
-        for (int u = 0; u < kKeep; ++u) {
+        for (int u = 0; u < KEEP; ++u) {
             const int d = slice + u * slices;
             if (d < dim) load_state<W>(s[u], S + static_cast<int64_t>(d) * vdim + first * W);
         }
@@ -69,35 +69,48 @@ delta_step_kernel(const spk_delta_args a) {
     const bool fresh = pos == 0;  // whatever the slot holds, a sequence starts from zeros
     if (KEEP && fresh) {
 #pragma unroll
-        for (int u = 0; u < (KEEP ? kKeep : 1); ++u)
+        for (int u = 0; u < KEEP; ++u)
 #pragma unroll
             for (int i = 0; i < W; ++i) s[u][i] = 0.0f;
     }
     float* ring = a.conv_state + row * a.taps * sh.channels;
-    const int now_slot = static_cast<int>(pos % a.taps);
-    auto channel = [&](const void* src, int64_t c, int at, const float* w, bool keep) {  // one channel's convolution; `at`: its place in the ring
-        const float x = spk_to_float<T>(static_cast<const T*>(src)[row * a.ld + c]);
-        if (keep) ring[now_slot * sh.channels + at] = x;
-        return spk_conv_silu(w + c * a.taps, a.taps, x, [&](int back) {
-            const int64_t p = pos - back;
-            return p >= 0 ? ring[(p % a.taps) * sh.channels + at] : 0.0f;
-        });
-    };
+    const int now_slot = static_cast<int>(static_cast<uint64_t>(pos) % static_cast<uint32_t>(a.taps));
+    const int past = pos < a.taps - 1 ? static_cast<int>(pos) : a.taps - 1;  // earlier tokens the convolution sees
     const bool leader = h % rep == 0;
-    const float rate = expf(a.a_log[h]);
     float sums[3] = {0.0f, 0.0f, 0.0f};
-    for (int c = threadIdx.x; c < dim; c += kThreads) {
-        const float x = channel(a.q, g * dim + c, g * dim + c, a.conv_q, leader);
-        const float y = channel(a.k, g * dim + c, sh.qk + g * dim + c, a.conv_k, leader);
-        q[c] = x;
-        k[c] = y;
-        sums[0] = fmaf(x, x, sums[0]);
-        sums[1] = fmaf(y, y, sums[1]);
-        const int64_t i = static_cast<int64_t>(h) * dim + c;
-        dec[c] = expf(spk_log_decay(spk_to_float<T>(static_cast<const T*>(a.a)[row * a.ld2 + i]) + a.dt_bias[i], rate));
+    // one channel of q, k, the decays or v per thread and turn
+    for (int i = threadIdx.x; i < 3 * dim + vdim; i += kThreads) {
+        if (i >= 2 * dim && i < 3 * dim) {
+            const int d = i - 2 * dim;
+            const int64_t c = static_cast<int64_t>(h) * dim + d;
+            dec[d] = expf(spk_log_decay(spk_to_float<T>(static_cast<const T*>(a.a)[row * a.ld2 + c]) + a.dt_bias[c], expf(a.a_log[h])));
+            continue;
+        }
+        const int part_of = i < dim ? 0 : i < 2 * dim ? 1 : 2;
+        const int local = part_of == 0 ? i : part_of == 1 ? i - dim : i - 3 * dim;
+        const int c = part_of == 2 ? h * vdim + local : g * dim + local;  // channel of its projection
+        const int at = c + part_of * sh.qk;                                // and its place in the ring
+        const void* src = part_of == 0 ? a.q : part_of == 1 ? a.k : a.v;
+        const float* w = (part_of == 0 ? a.conv_q : part_of == 1 ? a.conv_k : a.conv_v) + static_cast<int64_t>(c) * a.taps;
+        const float x = spk_to_float<T>(static_cast<const T*>(src)[row * a.ld + c]);
+        float y = x * w[a.taps - 1];
+#pragma unroll 4
+        for (int back = 1; back <= past; ++back) {
+            const int slot = now_slot >= back ? now_slot - back : now_slot - back + a.taps;
+            y = fmaf(ring[slot * sh.channels + at], w[a.taps - 1 - back], y);
+        }
+        y = spk_silu(y);
+        if (leader || part_of == 2) ring[now_slot * sh.channels + at] = x;
+        if (part_of == 0) {
+            q[local] = y;
+            sums[0] = fmaf(y, y, sums[0]);
+        } else if (part_of == 1) {
+            k[local] = y;
+            sums[1] = fmaf(y, y, sums[1]);
+        } else {
+            v[local] = y;
+        }
     }
-    for (int c = threadIdx.x; c < vdim; c += kThreads)
-        v[c] = channel(a.v, static_cast<int64_t>(h) * vdim + c, 2 * sh.qk + h * vdim + c, a.conv_v, true);
     spk_block_sum<3>(sums, part);  // its barriers also publish q, k, v and the decays
     const float qi = 1.0f / (sqrtf(sums[0] + 1e-6f) * sqrtf(static_cast<float>(dim))), ki = 1.0f / sqrtf(sums[1] + 1e-6f);
     const float beta = spk_sigmoid(spk_to_float<T>(static_cast<const T*>(a.b)[row * a.ld + h]));
@@ -109,7 +122,7 @@ delta_step_kernel(const spk_delta_args a) {
         if (in) {
             if (KEEP) {
 #pragma unroll
-                for (int u = 0; u < kKeep; ++u) {
+                for (int u = 0; u < KEEP; ++u) {
                     const int d = slice + u * slices;
                     if (d < dim) {
                         const float gd = dec[d], kd = k[d] * ki;
@@ -158,7 +171,7 @@ delta_step_kernel(const spk_delta_args a) {
             };
             if (KEEP) {
 #pragma unroll
-                for (int u = 0; u < kKeep; ++u) {
+                for (int u = 0; u < KEEP; ++u) {
                     const int d = slice + u * slices;
                     if (d < dim) update(s[u], d);
                 }
@@ -193,7 +206,6 @@ delta_step_kernel(const spk_delta_args a) {
 }
 
 // ---- prefill -----------------------------------------------------------------------------------------------------------
-constexpr int kChunk = 16;
 
 // What the recurrence reads, 32-bit: q [n][kv_heads][dim], k the same, v [n][heads][vdim], decays [n][heads][dim], beta [n][heads],
 // outputs [n][heads][vdim].
@@ -203,7 +215,7 @@ struct Work {
 __host__ __device__ inline int64_t work_floats(int64_t n, int heads, int kv_heads, int dim, int vdim) {
     return n * (2 * static_cast<int64_t>(kv_heads) * dim + static_cast<int64_t>(heads) * (dim + 2 * vdim) + ((heads + 3) & ~3));
 }
-__device__ __forceinline__ Work carve(const spk_delta_args& a) {
+__host__ __device__ inline Work carve(const spk_delta_args& a) {
     Work w;
     const int64_t qk = a.n * a.kv_heads * a.dim, vv = a.n * a.heads * a.vdim;
     w.q = static_cast<float*>(a.workspace);
@@ -376,32 +388,24 @@ delta_scan_kernel(const spk_delta_args a) {
         }
     }
     // the convolution's last inputs, for the next portion or the first decode step
-    float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
-    const int keep = min(a.taps, po.y);
-    auto commit = [&](const void* src, int64_t c, int at) {
-        for (int b = 0; b < keep; ++b) {
-            const int64_t t = po.x + po.y - 1 - b, pos = static_cast<int64_t>(po.w) + po.y - 1 - b;
-            ring[(pos % a.taps) * sh.channels + at] = spk_to_float<T>(static_cast<const T*>(src)[t * a.ld + c]);
-        }
-    };
-    if (part == 0 && in) commit(a.v, static_cast<int64_t>(h) * a.vdim + e, 2 * sh.qk + h * a.vdim + e);
+    if (part == 0 && in) spk_commit_conv<T>(a, po, sh, a.v, static_cast<int64_t>(h) * a.vdim + e, 2 * sh.qk + h * a.vdim + e);
     if (blockIdx.x == 0 && h % rep == 0)
         for (int c = threadIdx.x; c < a.dim; c += 4 * kScanCols) {
-            commit(a.q, g * a.dim + c, g * a.dim + c);
-            commit(a.k, g * a.dim + c, sh.qk + g * a.dim + c);
+            spk_commit_conv<T>(a, po, sh, a.q, g * a.dim + c, g * a.dim + c);
+            spk_commit_conv<T>(a, po, sh, a.k, g * a.dim + c, sh.qk + g * a.dim + c);
         }
 }
 
 // A warp per (token, head): norm over the head's outputs, weight, gate.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
-delta_out_kernel(const spk_delta_args a) {
+delta_out_kernel(const spk_delta_args a, const float* __restrict__ outputs) {
     const int64_t item = static_cast<int64_t>(blockIdx.x) * (kThreads / 32) + (threadIdx.x >> 5);
     if (item >= a.n * a.heads) return;
     const int lane = threadIdx.x & 31;
     const int64_t t = item / a.heads;
     const int h = static_cast<int>(item % a.heads);
-    const float* o = carve(a).o + item * a.vdim;
+    const float* o = outputs + item * a.vdim;
     float ss = 0.0f;
     for (int e = lane; e < a.vdim; e += 32) ss = fmaf(o[e], o[e], ss);
     const float inv = 1.0f / sqrtf(spk_warp_sum(ss) / static_cast<float>(a.vdim) + a.eps);
@@ -424,7 +428,7 @@ int check(const spk_delta_args* a) {
     return SPK_OK;
 }
 
-template <typename T, int W, bool KEEP>
+template <typename T, int W, int KEEP>
 int launch_step_form(const spk_delta_args& a, size_t bytes, cudaStream_t s) {
     if (bytes > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
@@ -442,9 +446,20 @@ int launch_step(const spk_delta_args& a, cudaStream_t s) {
     const int slices = cols < kThreads ? kThreads / cols : 1;
     const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim);
     if (bytes > 200 * 1024) return SPK_ERR_TOO_LARGE;
-    const bool keep = cols <= kThreads && a.dim <= kKeep * slices;
-    if (vec) return keep ? launch_step_form<T, 4, true>(a, bytes, s) : launch_step_form<T, 4, false>(a, bytes, s);
-    return keep ? launch_step_form<T, 1, true>(a, bytes, s) : launch_step_form<T, 1, false>(a, bytes, s);
+    const int share = cols <= kThreads ? (a.dim + slices - 1) / slices : 1 << 30;  // state rows per thread
+    if (!vec) return share <= 16 ? launch_step_form<T, 1, 16>(a, bytes, s) : launch_step_form<T, 1, 0>(a, bytes, s);
+    if (share <= 4) return launch_step_form<T, 4, 4>(a, bytes, s);
+    if (share <= 8) return launch_step_form<T, 4, 8>(a, bytes, s);
+    return share <= 16 ? launch_step_form<T, 4, 16>(a, bytes, s) : launch_step_form<T, 4, 0>(a, bytes, s);
+}
+
+template <typename T>
+int launch_out(const spk_delta_args& a, const float* outputs, cudaStream_t s) {
+    const int64_t grid = (a.n * a.heads + kThreads / 32 - 1) / (kThreads / 32);
+    if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
+    delta_out_kernel<T><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
 }
 
 template <typename T>
@@ -459,11 +474,7 @@ int launch_prefill(const spk_delta_args& a, cudaStream_t s) {
     else if (a.dim <= 128) delta_scan_kernel<T, 8><<<grid, threads, 0, s>>>(a);
     else delta_scan_kernel<T, 16><<<grid, threads, 0, s>>>(a);
     SPK_CHECK_LAUNCH();
-    const int64_t out_grid = (a.n * a.heads + kThreads / 32 - 1) / (kThreads / 32);
-    if (out_grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
-    delta_out_kernel<T><<<static_cast<unsigned>(out_grid), kThreads, 0, s>>>(a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return launch_out<T>(a, carve(a).o, s);
 }
 
 }  // namespace
@@ -483,11 +494,12 @@ extern "C" int spk_delta_chunk_tokens(int dtype, int dim, int vdim) {
     (void)dtype;
     (void)dim;
     (void)vdim;
-    return kChunk;
+    return kDeltaChunk;
 }
 
-extern "C" int64_t spk_delta_workspace_bytes(int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim) {
+extern "C" int64_t spk_delta_workspace_bytes(int dtype, int64_t n, int n_chunks, int heads, int kv_heads, int dim, int vdim) {
     if (n < 1 || n_chunks < 1 || heads < 1 || kv_heads < 1 || dim < 1 || vdim < 1) return 0;
+    if (spk_delta_tensor_form(dtype, dim, vdim)) return spk_delta_mma_bytes(n_chunks, heads, dim, vdim) + static_cast<int64_t>(sizeof(float)) * n * heads * vdim;
     return static_cast<int64_t>(sizeof(float)) * work_floats(n, heads, kv_heads, dim, vdim);
 }
 
@@ -496,10 +508,17 @@ extern "C" int spk_delta_prefill(const spk_delta_args* a, void* stream) {
     const int rc = check(a);
     if (rc != SPK_OK || a->n == 0) return rc;
     if (a->n_chunks < 1 || a->n_portions < 1 || a->n_portions > 65535) return SPK_ERR_BAD_SHAPE;
-    if (a->chunks == nullptr || a->portions == nullptr) return SPK_ERR_NULL_POINTER;
-    if (reinterpret_cast<uintptr_t>(a->chunks) % 16 != 0 || reinterpret_cast<uintptr_t>(a->portions) % 16 != 0) return SPK_ERR_BAD_STRIDE;
-    if (a->workspace == nullptr || a->workspace_bytes < spk_delta_workspace_bytes(a->n, a->n_chunks, a->heads, a->kv_heads, a->dim, a->vdim))
+    if (a->chunks == nullptr || a->portions == nullptr || a->seqs == nullptr) return SPK_ERR_NULL_POINTER;
+    if (reinterpret_cast<uintptr_t>(a->chunks) % 16 != 0 || reinterpret_cast<uintptr_t>(a->portions) % 16 != 0 ||
+        reinterpret_cast<uintptr_t>(a->seqs) % 16 != 0 || reinterpret_cast<uintptr_t>(a->workspace) % 16 != 0)
+        return SPK_ERR_BAD_STRIDE;
+    if (a->workspace == nullptr || a->workspace_bytes < spk_delta_workspace_bytes(a->dtype, a->n, a->n_chunks, a->heads, a->kv_heads, a->dim, a->vdim))
         return SPK_ERR_WORKSPACE_TOO_SMALL;
     cudaStream_t s = spk_stream(stream);
+    if (spk_delta_tensor_form(a->dtype, a->dim, a->vdim)) {
+        float* outputs = reinterpret_cast<float*>(static_cast<uint8_t*>(a->workspace) + spk_delta_mma_bytes(a->n_chunks, a->heads, a->dim, a->vdim));
+        if (const int e = spk_delta_mma_launch(*a, outputs, s)) return e;
+        return launch_out<__nv_bfloat16>(*a, outputs, s);
+    }
     return a->dtype == SPK_F32 ? launch_prefill<float>(*a, s) : launch_prefill<__nv_bfloat16>(*a, s);
 }

@@ -21,3 +21,21 @@ __device__ __forceinline__ float spk_conv_silu(const float* taps_of_channel, int
     for (int s = 1; s < taps; ++s) y = fmaf(before(s), taps_of_channel[taps - 1 - s], y);
     return spk_silu(y);
 }
+
+// One channel's last inputs of a portion into the row's ring.
+template <typename T>
+__device__ __forceinline__ void spk_commit_conv(const spk_delta_args& a, const int4& po, const SpkDeltaShape& sh, const void* src, int64_t c, int at) {
+    float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
+    const int keep = min(a.taps, po.y);
+    for (int b = 0; b < keep; ++b) {
+        const int64_t t = po.x + po.y - 1 - b;
+        ring[((po.w + po.y - 1 - b) % a.taps) * sh.channels + at] = spk_to_float<T>(static_cast<const T*>(src)[t * a.ld + c]);
+    }
+}
+
+constexpr int kDeltaChunk = 16;  // tokens per chunk of the prefill forms
+
+// 16-bit projections and heads of at most 128 channels run on the tensor cores.
+static inline bool spk_delta_tensor_form(int dtype, int dim, int vdim) { return dtype == SPK_BF16 && dim <= 128 && vdim <= 128; }
+int64_t spk_delta_mma_bytes(int n_chunks, int heads, int dim, int vdim);
+int spk_delta_mma_launch(const spk_delta_args& a, float* outputs, cudaStream_t s);

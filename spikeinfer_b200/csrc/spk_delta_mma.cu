@@ -1,0 +1,504 @@
+// Prefill form of the gated delta rule on the tensor cores: bf16 projections, heads of up to 128 key and 128 value channels.
+//
+// Over a chunk of 16 tokens, with G_t the product of the decays up to token t and the state S at the chunk's start,
+//   A[t, s] = k_t . (k_s * G_t / G_s)  (s < t),   B[t, s] = q_t . (k_s * G_t / G_s)  (s <= t),
+//   (1 + beta A) W = beta (k * G),   (1 + beta A) U0 = beta v        (forward substitution, one column per thread)
+//   u = U0 - W S,   o = (q * G) S + B u,   S <- G_16 S + (k * G_16 / G)^T u.
+// Ratios of G are running products of decays, never quotients: any decay is exact, a vanishing one included.
+//  * delta_chunk_kernel, all chunks at once: convolutions, unit vectors, decays, A, B, and the operands W, q G, k G_16 / G, B, U0 of
+//    the recurrence, laid out as the shared-memory image they become.
+//  * delta_chain_kernel, chunk after chunk: a warp owns sixteen value columns; S^T lives in its registers as the accumulators of the
+//    update, which are, as they are, the A operand of the next chunk's products (and u^T that of the update).  One bulk copy brings a
+//    chunk's operands.
+// 32-bit quantities enter a product as bf16 pairs (hi + lo, three MMAs), sums are 32-bit.
+#include "spk_delta.cuh"
+#include "spk_tensor.cuh"
+
+namespace {
+
+using namespace spk_tc;
+
+constexpr int C = kDeltaChunk;
+constexpr int kThreads = 256;
+
+// A chunk's operands in bytes from the image's start; SD elements per row of W, Q and K.
+template <int DP>
+struct Image {
+    static constexpr int SD = DP + 8, SB = 24, SU = C + 2;
+    static constexpr int kRows = C * SD * 2;                                              // bytes of one of the six matrices
+    static constexpr int kWh = 0, kWl = kRows, kQh = 2 * kRows, kQl = 3 * kRows, kKh = 4 * kRows, kKl = 5 * kRows;
+    static constexpr int kBh = 6 * kRows, kBl = kBh + C * SB * 2, kE = kBl + C * SB * 2;  // B, then G_16
+    static constexpr int kU = kE + DP * 4;                                                // U0^T [vdim padded to 16][SU], 32-bit
+};
+
+// Lanes L = 0 .. 31 end up with the sum over the warp of v[L].
+__device__ __forceinline__ float transpose_sum(float (&v)[32]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int o = 16; o >= 1; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+            v[i] = keep + __shfl_xor_sync(~0u, send, o);
+        }
+    }
+    return v[0];
+}
+
+// Channel c of a projection over the chunk's tokens through its convolution and silu into dst[t * stride]; zero beyond the chunk.
+template <int TAPS>
+__device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4& po, int64_t t0, int len, const void* src, int64_t c, const float* ring,
+                                             int channels, int at, const float* w, float* dst, int stride) {
+    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(src) + t0 * a.ld + c;
+    const int taps = TAPS > 0 ? TAPS : a.taps;
+    const int before = static_cast<int>(t0 - po.x);  // tokens of the portion ahead of the chunk
+    auto raw = [&](int j) {  // projection of token t0 + j, j < 0 reaching back into the portion, then into the ring
+        if (j >= 0 || before + j >= 0) return __bfloat162float(p[j * a.ld]);
+        const int pos = po.w + before + j;
+        return pos >= 0 ? ring[(pos % taps) * channels + at] : 0.0f;
+    };
+    if (TAPS > 0) {
+        float f[TAPS > 0 ? TAPS : 1], win[TAPS > 0 ? TAPS : 1], x[C];
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) f[i] = w[c * TAPS + i];
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i) win[i + 1] = raw(i - (TAPS - 1));
+#pragma unroll
+        for (int t = 0; t < C; ++t) x[t] = t < len ? __bfloat162float(p[t * a.ld]) : 0.0f;
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+#pragma unroll
+            for (int i = 0; i < TAPS - 1; ++i) win[i] = win[i + 1];
+            win[TAPS - 1] = x[t];
+            float y = 0.0f;
+#pragma unroll
+            for (int i = 0; i < TAPS; ++i) y = fmaf(win[i], f[i], y);
+            dst[t * stride] = t < len ? y * rcp(1.0f + ex2(-1.4426950408889634f * y)) : 0.0f;
+        }
+    } else {
+        for (int t = 0; t < C; ++t) {
+            float y = 0.0f;
+            if (t < len)
+                for (int i = 0; i < taps; ++i) y = fmaf(raw(t - (taps - 1 - i)), w[c * taps + i], y);
+            dst[t * stride] = t < len ? y * rcp(1.0f + ex2(-1.4426950408889634f * y)) : 0.0f;
+        }
+    }
+}
+
+// CTA = (chunk, head).
+template <int DP, int TAPS>
+__global__ void __launch_bounds__(kThreads)
+delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp) {
+    using I = Image<DP>;
+    constexpr int PL = DP / 32;  // channels per lane
+    extern __shared__ __align__(16) float sm[];
+    float* q = sm;               // [C][DP]
+    float* k = q + C * DP;
+    float* g = k + C * DP;       // decays
+    float* G = g + C * DP;       // their products from the chunk's start
+    float* v = G + C * DP;       // [C][vp]
+    __shared__ __align__(16) float A[C][C], B[C][C];
+    __shared__ float qi[C], ki[C], beta[C];
+    const int h = blockIdx.y, grp = h / (a.heads / a.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int4 ch = reinterpret_cast<const int4*>(a.chunks)[blockIdx.x];  // first token, tokens, portion, index
+    const int4 po = reinterpret_cast<const int4*>(a.portions)[ch.z];      // first token, tokens, row, tokens before
+    if (po.z < 0 || po.z >= a.state_rows) {
+        if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SLOT);
+        return;
+    }
+    const int64_t t0 = ch.x;
+    const int len = ch.y, dim = a.dim, vdim = a.vdim;
+    const SpkDeltaShape sh = spk_delta_shape(a);
+    const float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
+    // work items in an order that gives every warp one kind: k channels, q channels, v columns, decays
+    for (int i = threadIdx.x; i < 3 * DP + vp; i += kThreads) {
+        if (i < 2 * DP) {
+            const bool is_k = i < DP;
+            const int d = is_k ? i : i - DP;
+            float* dst = (is_k ? k : q) + d;
+            if (d < dim) {
+                conv_channel<TAPS>(a, po, t0, len, is_k ? a.k : a.q, static_cast<int64_t>(grp) * dim + d, ring, sh.channels, (is_k ? sh.qk : 0) + grp * dim + d,
+                                   is_k ? a.conv_k : a.conv_q, dst, DP);
+            } else {
+#pragma unroll
+                for (int t = 0; t < C; ++t) dst[t * DP] = 0.0f;
+            }
+        } else if (i < 3 * DP) {
+            const int d = i - 2 * DP;
+            float run = 1.0f, x[C];
+            const int64_t c = static_cast<int64_t>(h) * dim + d;
+#pragma unroll
+            for (int t = 0; t < C; ++t) x[t] = d < dim && t < len ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.a)[(t0 + t) * a.ld2 + c]) : 0.0f;
+            const float bias = d < dim ? a.dt_bias[c] : 0.0f, rate = expf(a.a_log[h]);
+#pragma unroll
+            for (int t = 0; t < C; ++t) {
+                const float dec = d < dim && t < len ? expf(spk_log_decay(x[t] + bias, rate)) : 1.0f;
+                run *= dec;
+                g[t * DP + d] = dec;
+                G[t * DP + d] = run;
+            }
+        } else {
+            const int e = i - 3 * DP;
+            if (e < vdim) {
+                conv_channel<TAPS>(a, po, t0, len, a.v, static_cast<int64_t>(h) * vdim + e, ring, sh.channels, 2 * sh.qk + h * vdim + e, a.conv_v, v + e, vp);
+            } else {
+#pragma unroll
+                for (int t = 0; t < C; ++t) v[t * vp + e] = 0.0f;
+            }
+        }
+    }
+    if (threadIdx.x < C)
+        beta[threadIdx.x] = static_cast<int>(threadIdx.x) < len ? spk_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(a.b)[(t0 + threadIdx.x) * a.ld + h])) : 0.0f;
+    __syncthreads();
+    // norms: two tokens per warp
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int t = 2 * warp + i;
+        float x = 0.0f, y = 0.0f;
+#pragma unroll
+        for (int j = 0; j < PL; ++j) {
+            const float a1 = q[t * DP + lane + 32 * j], b1 = k[t * DP + lane + 32 * j];
+            x = fmaf(a1, a1, x);
+            y = fmaf(b1, b1, y);
+        }
+        x = spk_warp_sum(x);
+        y = spk_warp_sum(y);
+        if (lane == 0) {
+            qi[t] = 1.0f / (sqrtf(x + 1e-6f) * sqrtf(static_cast<float>(dim)));
+            ki[t] = 1.0f / sqrtf(y + 1e-6f);
+        }
+    }
+    // A and B: warp w walks from tokens w and 15 - w to the chunk's end, fifteen steps in all, and sums 32 products over its lanes
+    {
+        const int s0 = warp, s1 = C - 1 - warp;
+        float x[PL], part[32];
+        auto load = [&](float (&r)[PL], const float* m, int t) {
+            if (PL == 4) {
+                const float4 f = *reinterpret_cast<const float4*>(m + t * DP + 4 * lane);
+                r[0] = f.x; r[1] = f.y; r[2 % PL] = f.z; r[3 % PL] = f.w;
+            } else {
+                const float2 f = *reinterpret_cast<const float2*>(m + t * DP + 2 * lane);
+                r[0] = f.x; r[1] = f.y;
+            }
+        };
+        auto dot = [&](const float (&p)[PL], const float (&r)[PL]) {
+            float s = p[0] * r[0];
+#pragma unroll
+            for (int j = 1; j < PL; ++j) s = fmaf(p[j], r[j], s);
+            return s;
+        };
+        float y[PL], z[PL];
+        load(x, k, s1);
+        load(y, q, s1);
+        part[31] = dot(x, y);
+        load(x, k, s0);
+        load(y, q, s0);
+        part[30] = dot(x, y);
+        const int first = C - 1 - s0;  // steps that start from s0
+#pragma unroll
+        for (int i = 0; i < C - 1; ++i) {
+            if (i == first) load(x, k, s1);
+            const int t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
+            load(y, g, t);
+#pragma unroll
+            for (int j = 0; j < PL; ++j) x[j] *= y[j];
+            load(y, k, t);
+            load(z, q, t);
+            part[i] = dot(x, y);
+            part[C - 1 + i] = dot(x, z);
+        }
+        const float total = transpose_sum(part);
+        __syncthreads();  // the norms are there
+        const int i = lane < C - 1 ? lane : lane < 2 * (C - 1) ? lane - (C - 1) : lane;
+        if (lane < 2 * (C - 1)) {
+            const int s = i < first ? s0 : s1, t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
+            if (lane < C - 1) A[t][s] = total * ki[t] * ki[s];
+            else B[t][s] = total * qi[t] * ki[s];
+        } else {
+            const int s = lane == 30 ? s0 : s1;
+            B[s][s] = total * qi[s] * ki[s];
+        }
+    }
+    __syncthreads();
+    uint8_t* image = static_cast<uint8_t*>(a.workspace) + (static_cast<int64_t>(blockIdx.x) * a.heads + h) * image_bytes;
+    if (threadIdx.x < C * C / 2) {
+        const int t = threadIdx.x >> 3, s = (threadIdx.x & 7) * 2;
+        uint32_t hi, lo;
+        split_bf16(s <= t ? B[t][s] : 0.0f, s + 1 <= t ? B[t][s + 1] : 0.0f, hi, lo);
+        *reinterpret_cast<uint32_t*>(image + I::kBh + (t * I::SB + s) * 2) = hi;
+        *reinterpret_cast<uint32_t*>(image + I::kBl + (t * I::SB + s) * 2) = lo;
+    }
+    // one column per thread: forward substitution, then the operands
+    for (int i = threadIdx.x; i < DP + vp; i += kThreads) {
+        const bool is_w = i < DP;  // uniform over a warp
+        const int e = i - DP;
+        float w[C];
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            float x = is_w ? k[t * DP + i] * ki[t] * G[t * DP + i] : v[t * vp + e];
+#pragma unroll
+            for (int s4 = 0; s4 < t; s4 += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(&A[t][s4]);
+                x = fmaf(-f.x, w[s4], x);
+                if (s4 + 1 < t) x = fmaf(-f.y, w[s4 + 1], x);
+                if (s4 + 2 < t) x = fmaf(-f.z, w[s4 + 2], x);
+                if (s4 + 3 < t) x = fmaf(-f.w, w[s4 + 3], x);
+            }
+            w[t] = beta[t] * x;
+        }
+        if (!is_w) {
+            float* u = reinterpret_cast<float*>(image + I::kU) + e * I::SU;
+#pragma unroll
+            for (int t = 0; t < C; t += 2) *reinterpret_cast<float2*>(u + t) = make_float2(w[t], w[t + 1]);
+            continue;
+        }
+        // lanes trade tokens in pairs, so that a store carries two channels
+        const bool odd = lane & 1;
+        auto put = [&](int t, float x0, float x1, int hi_at, int lo_at) {  // this column's values at tokens t and t + 1
+            const float got = __shfl_xor_sync(~0u, odd ? x0 : x1, 1);
+            uint32_t hi, lo;
+            split_bf16(odd ? got : x0, odd ? x1 : got, hi, lo);
+            const int at = ((t + (odd ? 1 : 0)) * I::SD + (i & ~1)) * 2;
+            *reinterpret_cast<uint32_t*>(image + hi_at + at) = hi;
+            *reinterpret_cast<uint32_t*>(image + lo_at + at) = lo;
+        };
+        float rest = 1.0f;  // product of the decays behind the token
+#pragma unroll
+        for (int t = C - 2; t >= 0; t -= 2) {
+            const float y1 = k[(t + 1) * DP + i] * ki[t + 1] * rest;
+            rest *= g[(t + 1) * DP + i];
+            const float y0 = k[t * DP + i] * ki[t] * rest;
+            rest *= g[t * DP + i];
+            put(t, y0, y1, I::kKh, I::kKl);
+            put(t, w[t], w[t + 1], I::kWh, I::kWl);
+            put(t, q[t * DP + i] * qi[t] * G[t * DP + i], q[(t + 1) * DP + i] * qi[t + 1] * G[(t + 1) * DP + i], I::kQh, I::kQl);
+        }
+        reinterpret_cast<float*>(image + I::kE)[i] = G[(C - 1) * DP + i];
+    }
+}
+
+// CTA = (NW * 16 value columns of a head, head, portion); warp NW copies.
+template <int DP, int NW>
+struct Chain {
+    static constexpr int kHead = Image<DP>::kU, kU = NW * 16 * Image<DP>::SU * 4;
+    static constexpr int kStage = (kHead + kU + 127) & ~127;
+    static constexpr int NS = 3;
+    static constexpr int kBytes = NS * kStage + 128 + 2 * NS * 8;
+};
+
+template <int DP, int NW>
+__global__ void __launch_bounds__(32 * NW + 32)
+delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp, float* __restrict__ outputs) {
+    using I = Image<DP>;
+    using K = Chain<DP, NW>;
+    constexpr int NS = K::NS;
+    extern __shared__ uint8_t raw[];
+    uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 127) & ~uintptr_t(127));
+    uint64_t* full = reinterpret_cast<uint64_t*>(base + NS * K::kStage);
+    uint64_t* empty = full + NS;
+    __shared__ int abort_flag;
+    volatile int* abort = &abort_flag;
+    const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int4 po = reinterpret_cast<const int4*>(a.portions)[blockIdx.z];  // first token, tokens, row, tokens before
+    const int4 sq = reinterpret_cast<const int4*>(a.seqs)[blockIdx.z];      // first chunk, chunks, row, tokens before
+    if (po.z < 0 || po.z >= a.state_rows) return;                            // flagged by the chunks
+    const int v0 = blockIdx.x * NW * 16;
+    const int columns = min(NW * 16, vp - v0);
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < NS; ++i) {
+            mbar_init(smem_u32(full + i), 1);
+            mbar_init(smem_u32(empty + i), NW);
+        }
+        abort_flag = 0;
+    }
+    fence_async_shared();
+    __syncthreads();
+    if (warp == NW) {
+        if (lane == 0) {
+            int issued = 0;
+            for (int c = 0; c < sq.y; ++c) {
+                const int st = c % NS;
+                if (c >= NS && !mbar_wait(smem_u32(empty + st), ((c / NS) - 1) & 1, abort)) break;
+                const uint8_t* src = static_cast<const uint8_t*>(a.workspace) + (static_cast<int64_t>(sq.x + c) * a.heads + h) * image_bytes;
+                const uint32_t bar = smem_u32(full + st), dst = smem_u32(base + st * K::kStage);
+                const uint32_t ub = static_cast<uint32_t>(columns) * I::SU * 4;
+                mbar_expect(bar, K::kHead + ub);
+                bulk_load(dst, src, K::kHead, bar);
+                bulk_load(dst + K::kHead, src + I::kU + v0 * I::SU * 4, ub, bar);
+                issued = c + 1;
+            }
+            if (*abort != 0) {  // copies in flight land before the CTA's shared memory is given up
+                for (int c = issued > NS ? issued - NS : 0; c < issued; ++c) mbar_wait(smem_u32(full + c % NS), (c / NS) & 1);
+                spk_flag(a.status, SPK_STATUS_DEVICE_WAIT_EXPIRED);
+            }
+        }
+    } else {
+        const int gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
+        constexpr int NT = DP / 8;
+        const int dim = a.dim, vdim = a.vdim, v1 = v0 + warp * 16 + gid;
+        const bool live = warp * 16 < columns;  // a warp without columns only keeps the ring going
+        float* state = a.state + (static_cast<int64_t>(po.z) * a.heads + h) * dim * vdim;
+        float S[NT][4];
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = n * 8 + tig * 2 + (i & 1), e = v1 + (i >> 1) * 8;
+                S[n][i] = live && po.w > 0 && d < dim && e < vdim ? state[static_cast<int64_t>(d) * vdim + e] : 0.0f;
+            }
+        for (int c = 0; c < sq.y; ++c) {
+            const int st = c % NS;
+            if (!__all_sync(~0u, mbar_wait(smem_u32(full + st), (c / NS) & 1, abort))) break;
+            const uint8_t* im = base + st * K::kStage;
+            const uint32_t at = smem_u32(im);
+            if (live) {
+                // u^T and o^T: columns (tokens) 0-7 and 8-15, main and cross terms apart
+                float u[2][4] = {}, uc[2][4] = {}, o[2][4] = {}, oc[2][4] = {};
+                const uint32_t row = ((m >> 1) * 8 + mr) * I::SD * 2 + (m & 1) * 16;
+#pragma unroll
+                for (int j = 0; j < DP / 16; ++j) {
+                    uint32_t sh[4], sl[4], bh[4], bl[4];
+                    split_bf16(S[2 * j][0], S[2 * j][1], sh[0], sl[0]);
+                    split_bf16(S[2 * j][2], S[2 * j][3], sh[1], sl[1]);
+                    split_bf16(S[2 * j + 1][0], S[2 * j + 1][1], sh[2], sl[2]);
+                    split_bf16(S[2 * j + 1][2], S[2 * j + 1][3], sh[3], sl[3]);
+                    ldsm4(bh, at + I::kWh + row + j * 32);
+                    ldsm4(bl, at + I::kWl + row + j * 32);
+                    mma16816(u[0], sh, bh[0], bh[1]);
+                    mma16816(u[1], sh, bh[2], bh[3]);
+                    mma16816(uc[0], sh, bl[0], bl[1]);
+                    mma16816(uc[1], sh, bl[2], bl[3]);
+                    mma16816(uc[0], sl, bh[0], bh[1]);
+                    mma16816(uc[1], sl, bh[2], bh[3]);
+                    ldsm4(bh, at + I::kQh + row + j * 32);
+                    ldsm4(bl, at + I::kQl + row + j * 32);
+                    mma16816(o[0], sh, bh[0], bh[1]);
+                    mma16816(o[1], sh, bh[2], bh[3]);
+                    mma16816(oc[0], sh, bl[0], bl[1]);
+                    mma16816(oc[1], sh, bl[2], bl[3]);
+                    mma16816(oc[0], sl, bh[0], bh[1]);
+                    mma16816(oc[1], sl, bh[2], bh[3]);
+                }
+                const float* U = reinterpret_cast<const float*>(im + K::kHead) + (warp * 16 + gid) * I::SU + tig * 2;
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        const float2 f = *reinterpret_cast<const float2*>(U + i * 8 * I::SU + n * 8);
+                        u[n][2 * i] = f.x - (u[n][2 * i] + uc[n][2 * i]);
+                        u[n][2 * i + 1] = f.y - (u[n][2 * i + 1] + uc[n][2 * i + 1]);
+                    }
+                uint32_t uh[4], ul[4];
+                split_bf16(u[0][0], u[0][1], uh[0], ul[0]);
+                split_bf16(u[0][2], u[0][3], uh[1], ul[1]);
+                split_bf16(u[1][0], u[1][1], uh[2], ul[2]);
+                split_bf16(u[1][2], u[1][3], uh[3], ul[3]);
+                // S^T <- G_16 S^T + u^T K
+                const float* E = reinterpret_cast<const float*>(im + I::kE) + tig * 2;
+                const uint32_t krow = ((m & 1) * 8 + mr) * I::SD * 2 + (m >> 1) * 16;
+#pragma unroll
+                for (int n = 0; n < NT; n += 2) {
+                    uint32_t bh[4], bl[4];
+                    ldsm4t(bh, at + I::kKh + krow + n * 16);
+                    ldsm4t(bl, at + I::kKl + krow + n * 16);
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const float2 f = *reinterpret_cast<const float2*>(E + (n + x) * 8);
+                        S[n + x][0] *= f.x;
+                        S[n + x][1] *= f.y;
+                        S[n + x][2] *= f.x;
+                        S[n + x][3] *= f.y;
+                        mma16816(S[n + x], uh, bh[2 * x], bh[2 * x + 1]);
+                        mma16816(S[n + x], uh, bl[2 * x], bl[2 * x + 1]);
+                        mma16816(S[n + x], ul, bh[2 * x], bh[2 * x + 1]);
+                    }
+                }
+                {
+                    uint32_t bh[4], bl[4];
+                    const uint32_t brow = ((m >> 1) * 8 + mr) * I::SB * 2 + (m & 1) * 16;
+                    ldsm4(bh, at + I::kBh + brow);
+                    ldsm4(bl, at + I::kBl + brow);
+                    mma16816(o[0], uh, bh[0], bh[1]);
+                    mma16816(o[1], uh, bh[2], bh[3]);
+                    mma16816(oc[0], uh, bl[0], bl[1]);
+                    mma16816(oc[1], uh, bl[2], bl[3]);
+                    mma16816(oc[0], ul, bh[0], bh[1]);
+                    mma16816(oc[1], ul, bh[2], bh[3]);
+                }
+                const int left = po.y - c * C;
+                float* dst = outputs + ((static_cast<int64_t>(po.x) + c * C) * a.heads + h) * vdim;
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int t = n * 8 + tig * 2 + (i & 1), e = v1 + (i >> 1) * 8;
+                        if (t < left && e < vdim) dst[static_cast<int64_t>(t) * a.heads * vdim + e] = o[n][i] + oc[n][i];
+                    }
+            }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(empty + st));
+        }
+        if (live) {
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int d = n * 8 + tig * 2 + (i & 1), e = v1 + (i >> 1) * 8;
+                    if (d < dim && e < vdim) state[static_cast<int64_t>(d) * vdim + e] = S[n][i];
+                }
+        }
+        // the convolution's last inputs, for the next portion or the first decode step
+        const SpkDeltaShape shp = spk_delta_shape(a);
+        const int rep = a.heads / a.kv_heads, grp = h / rep;
+        for (int i = threadIdx.x; i < columns; i += 32 * NW)
+            if (v0 + i < vdim) spk_commit_conv<__nv_bfloat16>(a, po, shp, a.v, static_cast<int64_t>(h) * vdim + v0 + i, 2 * shp.qk + h * vdim + v0 + i);
+        if (blockIdx.x == 0 && h % rep == 0)
+            for (int d = threadIdx.x; d < dim; d += 32 * NW) {
+                spk_commit_conv<__nv_bfloat16>(a, po, shp, a.q, static_cast<int64_t>(grp) * dim + d, grp * dim + d);
+                spk_commit_conv<__nv_bfloat16>(a, po, shp, a.k, static_cast<int64_t>(grp) * dim + d, shp.qk + grp * dim + d);
+            }
+    }
+    __syncthreads();
+}
+
+int padded_v(int vdim) { return (vdim + 15) & ~15; }
+int64_t image_size(int dim, int vdim) {
+    const int64_t u = static_cast<int64_t>(padded_v(vdim)) * Image<64>::SU * 4;
+    return (dim <= 64 ? Image<64>::kU : Image<128>::kU) + u;
+}
+
+template <int DP, int NW>
+int launch_chain(const spk_delta_args& a, int64_t image, int vp, float* outputs, cudaStream_t s) {
+    constexpr int bytes = Chain<DP, NW>::kBytes;
+    const cudaError_t e = cudaFuncSetAttribute(delta_chain_kernel<DP, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return spk_set_cuda_error(e);
+    delta_chain_kernel<DP, NW><<<dim3((vp + NW * 16 - 1) / (NW * 16), a.heads, a.n_portions), 32 * NW + 32, bytes, s>>>(a, image, vp, outputs);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
+template <int DP>
+int launch(const spk_delta_args& a, float* outputs, cudaStream_t s) {
+    const int vp = padded_v(a.vdim);
+    const int64_t image = image_size(a.dim, a.vdim);
+    const size_t bytes = sizeof(float) * C * (4 * DP + static_cast<size_t>(vp));
+    auto* fn = a.taps == 4 ? delta_chunk_kernel<DP, 4> : delta_chunk_kernel<DP, 0>;
+    const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+    if (e != cudaSuccess) return spk_set_cuda_error(e);
+    fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, image, vp);
+    SPK_CHECK_LAUNCH();
+    // few chains: spread a head's columns over more CTAs
+    const int64_t chains = static_cast<int64_t>(a.heads) * a.n_portions;
+    if (chains * ((vp + 63) / 64) >= 148) return launch_chain<DP, 4>(a, image, vp, outputs, s);
+    if (chains * ((vp + 31) / 32) >= 148) return launch_chain<DP, 2>(a, image, vp, outputs, s);
+    return launch_chain<DP, 1>(a, image, vp, outputs, s);
+}
+
+}  // namespace
+
+int64_t spk_delta_mma_bytes(int n_chunks, int heads, int dim, int vdim) { return static_cast<int64_t>(n_chunks) * heads * image_size(dim, vdim); }
+
+int spk_delta_mma_launch(const spk_delta_args& a, float* outputs, cudaStream_t s) {
+    return a.dim <= 64 ? launch<64>(a, outputs, s) : launch<128>(a, outputs, s);
+}

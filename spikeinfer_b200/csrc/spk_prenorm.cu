@@ -5,8 +5,11 @@
 //    One launch per layer boundary.
 //  * gelu_kernel: the tanh form of gelu.
 #include "spk_experts.cuh"
+#include "spk_tensor.cuh"
 
 namespace {
+
+using namespace spk_tc;
 
 template <typename T, typename TD, int V, bool VEC>
 __global__ void __launch_bounds__(1024)
@@ -132,11 +135,29 @@ int launch_boundary(const spk_rms_residual_args& p, cudaStream_t s) {
     return SPK_OK;
 }
 
+// z / 2 (1 + tanh(y)) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+    return z / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));
+}
+__device__ __forceinline__ float gelu_tanh_fast(float z) {  // for 16-bit results
+    return z * rcp(1.0f + ex2(-2.302208198f * fmaf(0.044715f * z * z, z, z)));  // 2 sqrt(2 / pi) log2(e)
 }
 
 constexpr int kGeluThreads = 256;
+
+// bf16, eight elements per thread; everything aligned to them.
+__global__ void __launch_bounds__(kGeluThreads)
+gelu_vec_kernel(const __nv_bfloat16* __restrict__ z, __nv_bfloat16* __restrict__ out, int64_t out_stride, int width) {
+    const int c = 8 * (blockIdx.x * kGeluThreads + threadIdx.x);
+    if (c >= width) return;
+    const int64_t t = blockIdx.y;
+    const uint4 u = __ldcs(reinterpret_cast<const uint4*>(z + t * width + c));
+    uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+        w[k] = pack_bf16(gelu_tanh_fast(__uint_as_float(w[k] << 16)), gelu_tanh_fast(__uint_as_float(w[k] & 0xffff0000u)));
+    *reinterpret_cast<uint4*>(out + t * out_stride + c) = make_uint4(w[0], w[1], w[2], w[3]);
+}
 
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(kGeluThreads)
@@ -151,10 +172,16 @@ gelu_kernel(const T* __restrict__ z, T* __restrict__ out, int64_t out_stride, in
 
 template <typename T>
 int launch_gelu(const void* z, void* out, int64_t out_stride, int64_t n, int64_t width, cudaStream_t s) {
+    auto at = [](const void* p, size_t b) { return reinterpret_cast<uintptr_t>(p) % b == 0; };
+    if (sizeof(T) == 2 && width % 8 == 0 && out_stride % 8 == 0 && at(z, 16) && at(out, 16) && n <= 65535) {
+        const dim3 grid(static_cast<unsigned>((width / 8 + kGeluThreads - 1) / kGeluThreads), static_cast<unsigned>(n));
+        gelu_vec_kernel<<<grid, kGeluThreads, 0, s>>>(static_cast<const __nv_bfloat16*>(z), static_cast<__nv_bfloat16*>(out), out_stride, static_cast<int>(width));
+        SPK_CHECK_LAUNCH();
+        return SPK_OK;
+    }
     const int64_t per = (width + 3) / 4, groups = n * per, grid = (groups + kGeluThreads - 1) / kGeluThreads;
     if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
-    const bool vec = width % 4 == 0 && out_stride % 4 == 0 && reinterpret_cast<uintptr_t>(z) % (4 * sizeof(T)) == 0 &&
-                     reinterpret_cast<uintptr_t>(out) % (4 * sizeof(T)) == 0;
+    const bool vec = width % 4 == 0 && out_stride % 4 == 0 && at(z, 4 * sizeof(T)) && at(out, 4 * sizeof(T));
     const T* zi = static_cast<const T*>(z);
     T* o = static_cast<T*>(out);
     const unsigned g = static_cast<unsigned>(grid);

@@ -42,10 +42,11 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b: torch.Tenso
         _call("spk_delta_step", args, q.device)
         return out
     lib = _lib.load()
-    chunks, _ = plan.chunks(int(lib.spk_delta_chunk_tokens(args.dtype, dim, vdim)))
+    chunks, seqs = plan.chunks(int(lib.spk_delta_chunk_tokens(args.dtype, dim, vdim)))
     portions = plan.portions()
-    need = int(lib.spk_delta_workspace_bytes(n, chunks.shape[0], heads, kv_heads, dim, vdim))
+    need = int(lib.spk_delta_workspace_bytes(args.dtype, n, chunks.shape[0], heads, kv_heads, dim, vdim))
     ws = torch.empty(need, dtype=torch.uint8, device=q.device)
+    args.seqs = seqs.data_ptr()
     args.chunks, args.portions, args.n_chunks, args.n_portions = chunks.data_ptr(), portions.data_ptr(), chunks.shape[0], portions.shape[0]
     args.workspace, args.workspace_bytes = ws.data_ptr(), need
     _call("spk_delta_prefill", args, q.device)
