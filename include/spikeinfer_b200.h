@@ -681,7 +681,7 @@ typedef struct spk_experts_args {
 int spk_experts(const spk_experts_args* args, void* stream);
 
 /* Cache row of the latent attention: `rank` latent channels, then (from channel rank_pad) rot_dim rotated ones.  A pool is
- * [num_blocks][1][block_size][rank_pad + rot_pad]; tiled as above, or plain with rank_pad == rank, rot_pad == rot_dim.
+ * [num_blocks][block_size][rank_pad + rot_pad]; tiled (csrc/spk_latent.cuh), or plain with rank_pad == rank, rot_pad == rot_dim.
  *
  * Per token: cq_out [n, q_rank] <- cq / rms(cq) * w_q; the pool row of slot_mapping[t] <- kv[0 .. rank) / rms * w_kv, and
  * kv[rank .. rank + rot_dim) rotated by the table at positions[t].  kv NULL: only cq. */

@@ -32,9 +32,9 @@ __device__ __forceinline__ void load_state(float (&s)[W], const float* p) {
 
 // CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  KEEP: rows of the
 // state that are a thread's share and stay in its registers between the two products; 0: any share, read twice.
-template <typename T, int W, int KEEP>
-__global__ void __launch_bounds__(kThreads)
-delta_step_kernel(const spk_delta_args a) {
+template <typename T, int W, int KEEP, int NT>
+__global__ void __launch_bounds__(NT, NT == 128 ? 6 : 2)
+delta_step_kernel(const spk_delta_args a, const int prefetch) {
     extern __shared__ float sm[];
     __shared__ float part[3 * 32];
     const int h = blockIdx.x;
@@ -42,7 +42,7 @@ delta_step_kernel(const spk_delta_args a) {
     const int dim = a.dim, vdim = a.vdim, rep = a.heads / a.kv_heads, g = h / rep;
     T* out = static_cast<T*>(a.out) + row * a.out_stride + static_cast<int64_t>(h) * vdim;
     if (a.active != nullptr && a.active[row] != 1) {
-        for (int e = threadIdx.x; e < vdim; e += kThreads) out[e] = spk_from_float<T>(0.0f);
+        for (int e = threadIdx.x; e < vdim; e += NT) out[e] = spk_from_float<T>(0.0f);
         return;
     }
     float* q = sm;                 // [dim]
@@ -52,7 +52,7 @@ delta_step_kernel(const spk_delta_args a) {
     float* red = v + vdim;         // [slices][vdim]
     float* S = a.state + (row * a.heads + h) * static_cast<int64_t>(dim) * vdim;
     const int cols = vdim / W;
-    const int slices = cols < kThreads ? kThreads / cols : 1;
+    const int slices = cols < NT ? NT / cols : 1;
     const int slice = slices > 1 ? threadIdx.x / cols : 0;
     const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
     const bool mine = slice < slices;
@@ -63,6 +63,11 @@ delta_step_kernel(const spk_delta_args a) {
             const int d = slice + u * slices;
             if (d < dim) load_state<W>(s[u], S + static_cast<int64_t>(d) * vdim + first * W);
         }
+    }
+    if (threadIdx.x == 0 && prefetch > 0) {  // the state of the CTA that follows this one on its SM
+        const int64_t next = row * a.heads + h + prefetch, bytes = static_cast<int64_t>(dim) * vdim * 4;
+        if (next < a.n * a.heads)
+            asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(__cvta_generic_to_global(a.state + next * dim * vdim)), "r"(static_cast<uint32_t>(bytes)) : "memory");
     }
     const SpkDeltaShape sh = spk_delta_shape(a);
     const int64_t pos = a.positions[row];
@@ -79,7 +84,7 @@ delta_step_kernel(const spk_delta_args a) {
     const bool leader = h % rep == 0;
     float sums[3] = {0.0f, 0.0f, 0.0f};
     // one channel of q, k, the decays or v per thread and turn
-    for (int i = threadIdx.x; i < 3 * dim + vdim; i += kThreads) {
+    for (int i = threadIdx.x; i < 3 * dim + vdim; i += NT) {
         if (i >= 2 * dim && i < 3 * dim) {
             const int d = i - 2 * dim;
             const int64_t c = static_cast<int64_t>(h) * dim + d;
@@ -115,7 +120,7 @@ delta_step_kernel(const spk_delta_args a) {
     const float qi = 1.0f / (sqrtf(sums[0] + 1e-6f) * sqrtf(static_cast<float>(dim))), ki = 1.0f / sqrtf(sums[1] + 1e-6f);
     const float beta = spk_sigmoid(spk_to_float<T>(static_cast<const T*>(a.b)[row * a.ld + h]));
     float square[1] = {0.0f};
-    for (int c0 = 0; c0 < cols; c0 += kThreads) {
+    for (int c0 = 0; c0 < cols; c0 += NT) {
         const int c = c0 + first;
         const bool in = mine && c < cols;
         float acc[W] = {};
@@ -201,7 +206,7 @@ delta_step_kernel(const spk_delta_args a) {
     spk_block_sum<1>(square, part);
     const float inv = 1.0f / sqrtf(square[0] / static_cast<float>(vdim) + a.eps);
     const T* gate = static_cast<const T*>(a.gate) + row * a.ld2 + static_cast<int64_t>(h) * vdim;
-    for (int e = threadIdx.x; e < vdim; e += kThreads)
+    for (int e = threadIdx.x; e < vdim; e += NT)
         out[e] = spk_from_float<T>(v[e] * inv * a.w_norm[e] * spk_sigmoid(spk_to_float<T>(gate[e])));
 }
 
@@ -414,6 +419,29 @@ delta_out_kernel(const spk_delta_args a, const float* __restrict__ outputs) {
     for (int e = lane; e < a.vdim; e += 32) out[e] = spk_from_float<T>(o[e] * inv * a.w_norm[e] * spk_sigmoid(spk_to_float<T>(gate[e])));
 }
 
+// The same with four channels per lane: V / 4 lanes per head, everything aligned to four elements.
+template <typename T, int V>
+__global__ void __launch_bounds__(kThreads)
+delta_out_vec_kernel(const spk_delta_args a, const float* __restrict__ outputs) {
+    constexpr int L = V / 4;
+    const int64_t item = static_cast<int64_t>(blockIdx.x) * (kThreads / L) + threadIdx.x / L;
+    const bool in = item < a.n * a.heads;
+    const int c = 4 * (threadIdx.x % L);
+    const int64_t t = item / a.heads;
+    const int64_t at = (item % a.heads) * V + c;
+    const float4 o = in ? __ldcs(reinterpret_cast<const float4*>(outputs + item * V + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 g = spk_load4<T, true>(static_cast<const T*>(a.gate) + (in ? t * a.ld2 + at : 0), 4);
+    const float4 w = *reinterpret_cast<const float4*>(a.w_norm + c);
+    float ss = (o.x * o.x + o.y * o.y) + (o.z * o.z + o.w * o.w);
+#pragma unroll
+    for (int s = L / 2; s >= 1; s >>= 1) ss += __shfl_xor_sync(~0u, ss, s);
+    if (!in) return;
+    const float inv = 1.0f / sqrtf(ss / static_cast<float>(V) + a.eps);
+    spk_store4<T, true>(static_cast<T*>(a.out) + t * a.out_stride + at,
+                        make_float4(o.x * inv * w.x * spk_sigmoid(g.x), o.y * inv * w.y * spk_sigmoid(g.y), o.z * inv * w.z * spk_sigmoid(g.z),
+                                    o.w * inv * w.w * spk_sigmoid(g.w)), 4);
+}
+
 int check(const spk_delta_args* a) {
     if (a == nullptr) return SPK_ERR_NULL_POINTER;
     if (a->n < 0 || a->heads < 1 || a->heads > 65535 || a->kv_heads < 1 || a->heads % a->kv_heads != 0 || a->dim < 1 || a->vdim < 1 || a->taps < 1 ||
@@ -428,13 +456,19 @@ int check(const spk_delta_args* a) {
     return SPK_OK;
 }
 
-template <typename T, int W, int KEEP>
-int launch_step_form(const spk_delta_args& a, size_t bytes, cudaStream_t s) {
+template <typename T, int W, int KEEP, int NT>
+int launch_step_form(const spk_delta_args& a, cudaStream_t s) {
+    const int cols = a.vdim / W, slices = cols < NT ? NT / cols : 1;
+    const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim);
+    if (bytes > 200 * 1024) return SPK_ERR_TOO_LARGE;
     if (bytes > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+        const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, KEEP, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
         if (e != cudaSuccess) return spk_set_cuda_error(e);
     }
-    delta_step_kernel<T, W, KEEP><<<dim3(a.heads, static_cast<unsigned>(a.n)), kThreads, bytes, s>>>(a);
+    // large states: a CTA has the next one's on its way into L2 while it computes
+    const int64_t state = static_cast<int64_t>(a.dim) * a.vdim * 4;
+    const int prefetch = state >= 32 * 1024 && state % 16 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0 ? 2 * 148 : 0;
+    delta_step_kernel<T, W, KEEP, NT><<<dim3(a.heads, static_cast<unsigned>(a.n)), NT, bytes, s>>>(a, prefetch);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -443,18 +477,28 @@ template <typename T>
 int launch_step(const spk_delta_args& a, cudaStream_t s) {
     const bool vec = a.vdim % 4 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0;
     const int cols = vec ? a.vdim / 4 : a.vdim;
-    const int slices = cols < kThreads ? kThreads / cols : 1;
-    const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim);
-    if (bytes > 200 * 1024) return SPK_ERR_TOO_LARGE;
-    const int share = cols <= kThreads ? (a.dim + slices - 1) / slices : 1 << 30;  // state rows per thread
-    if (!vec) return share <= 16 ? launch_step_form<T, 1, 16>(a, bytes, s) : launch_step_form<T, 1, 0>(a, bytes, s);
-    if (share <= 4) return launch_step_form<T, 4, 4>(a, bytes, s);
-    if (share <= 8) return launch_step_form<T, 4, 8>(a, bytes, s);
-    return share <= 16 ? launch_step_form<T, 4, 16>(a, bytes, s) : launch_step_form<T, 4, 0>(a, bytes, s);
+    auto share = [&](int threads) {  // state rows per thread
+        const int slices = cols < threads ? threads / cols : 1;
+        return cols <= threads ? (a.dim + slices - 1) / slices : 1 << 30;
+    };
+    if (!vec) return share(256) <= 16 ? launch_step_form<T, 1, 16, 256>(a, s) : launch_step_form<T, 1, 0, 256>(a, s);
+    if (share(128) <= 8) return launch_step_form<T, 4, 8, 128>(a, s);
+    return share(256) <= 16 ? launch_step_form<T, 4, 16, 256>(a, s) : launch_step_form<T, 4, 0, 256>(a, s);
 }
 
 template <typename T>
 int launch_out(const spk_delta_args& a, const float* outputs, cudaStream_t s) {
+    auto at = [](const void* p, size_t b) { return reinterpret_cast<uintptr_t>(p) % b == 0; };
+    if ((a.vdim == 64 || a.vdim == 128) && a.ld2 % 4 == 0 && a.out_stride % 4 == 0 && at(a.gate, 4 * sizeof(T)) && at(a.out, 4 * sizeof(T)) &&
+        at(outputs, 16) && at(a.w_norm, 16)) {
+        const int per = kThreads / (a.vdim / 4);
+        const int64_t grid = (a.n * a.heads + per - 1) / per;
+        if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
+        if (a.vdim == 64) delta_out_vec_kernel<T, 64><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);
+        else delta_out_vec_kernel<T, 128><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);
+        SPK_CHECK_LAUNCH();
+        return SPK_OK;
+    }
     const int64_t grid = (a.n * a.heads + kThreads / 32 - 1) / (kThreads / 32);
     if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
     delta_out_kernel<T><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);

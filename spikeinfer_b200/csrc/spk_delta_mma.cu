@@ -88,7 +88,7 @@ __device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4
 
 // CTA = (chunk, head).
 template <int DP, int TAPS>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 3)
 delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp) {
     using I = Image<DP>;
     constexpr int PL = DP / 32;  // channels per lane
@@ -288,7 +288,7 @@ struct Chain {
 };
 
 template <int DP, int NW>
-__global__ void __launch_bounds__(32 * NW + 32)
+__global__ void __launch_bounds__(32 * NW + 32, 2)
 delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp, float* __restrict__ outputs) {
     using I = Image<DP>;
     using K = Chain<DP, NW>;

@@ -55,8 +55,8 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
         for (int i = lane; i < half; i += 32) {
             const float2 f = rot_factor(a.rot_table, a.rot_positions, half, pos, i, a.status);
             const float u = spk_to_float<T>(src[i]), v = spk_to_float<T>(src[i + half]);
-            page[spk_page_channel(lay, r, a.rank_pad + i)] = spk_from_float<T>(u * f.x - v * f.y);
-            page[spk_page_channel(lay, r, a.rank_pad + i + half)] = spk_from_float<T>(v * f.x + u * f.y);
+            page[spk_latent_channel(lay, r, a.rank_pad + i)] = spk_from_float<T>(u * f.x - v * f.y);
+            page[spk_latent_channel(lay, r, a.rank_pad + i + half)] = spk_from_float<T>(v * f.x + u * f.y);
         }
         return;
     }
@@ -75,12 +75,12 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
         if (part == 0) {
             spk_store4<T, VEC>(static_cast<T*>(a.cq_out) + t * width + c, y, width - c);
         } else if (VEC) {
-            spk_store4<T, VEC>(page + spk_page_channel(lay, r, c), y, width - c);
+            spk_store4<T, VEC>(page + spk_latent_channel(lay, r, c), y, width - c);
         } else {
             const float e[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-                if (c + k < width) page[spk_page_channel(lay, r, c + k)] = spk_from_float<T>(e[k]);
+                if (c + k < width) page[spk_latent_channel(lay, r, c + k)] = spk_from_float<T>(e[k]);
         }
     }
 }
@@ -168,12 +168,15 @@ latent_query_mma_kernel(const spk_latent_query_args a, const int dp, const bool 
     const int64_t t0 = static_cast<int64_t>(blockIdx.z) * kMmaRows;
     const int rows = static_cast<int>(min(static_cast<int64_t>(kMmaRows), a.n - t0));
     const int64_t ld = static_cast<int64_t>(a.heads) * (a.dim + a.rot_dim);
+    if (c0 >= a.rank) {  // the last CTA of a head and token block turns the rotated part
+        rotate_query<__nv_bfloat16>(a, h, t0, rows);
+        return;
+    }
     fetch_tile(ws, SW, static_cast<const __nv_bfloat16*>(a.w_uk) + static_cast<int64_t>(h) * a.dim * a.rank + c0, a.rank, dp, a.dim, kMmaCols,
                a.rank - c0, vec_w);
     fetch_tile(qs, SQ, static_cast<const __nv_bfloat16*>(a.q) + t0 * ld + static_cast<int64_t>(h) * (a.dim + a.rot_dim), ld, (rows + 15) & ~15, rows, dp,
                a.dim, vec_q);
     cp_async_commit();
-    if (blockIdx.y == 0) rotate_query<__nv_bfloat16>(a, h, t0, rows);
     cp_async_wait_all();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
@@ -253,7 +256,7 @@ latent_attn_simt_kernel(const spk_latent_attn_args a) {
                 const int64_t block = table[j / a.block_size];
                 if (block >= 0 && block < a.num_blocks)
                     v = spk_to_float<T>(static_cast<const T*>(a.pool)[spk_page_base(lay, block, 0) +
-                                        spk_page_channel(lay, static_cast<int>(j % a.block_size), c < a.rank ? c : a.rank_pad + c - a.rank)]);
+                                        spk_latent_channel(lay, static_cast<int>(j % a.block_size), c < a.rank ? c : a.rank_pad + c - a.rank)]);
                 else if (c == 0)
                     spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
             }
@@ -374,51 +377,69 @@ latent_out_kernel(const spk_latent_out_args a) {
     }
 }
 
-// bf16 on the tensor cores: CTA = (head, 16 tokens, 128 value channels), a warp per sixteen channels.  The ranges' sums are put together 64
-// latent channels at a time, right where the product reads them; the value matrix follows through a two-stage ring.
+// bf16 on the tensor cores: CTA = (head, 16 tokens, 128 value channels), a warp per sixteen channels.  The ranges' sums are put together
+// with all of a thread's loads in flight at once, while the first stages of the value matrix are on their way.
+constexpr int kOutStages = 4;
+
 template <bool VEC>
 __global__ void __launch_bounds__(kThreads)
 latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
     constexpr int K = 64, S = K + 8;
     extern __shared__ __align__(16) uint8_t raw[];
-    __nv_bfloat16* os = reinterpret_cast<__nv_bfloat16*>(raw);  // two stages of [16][72]
-    __nv_bfloat16* ws = os + 2 * kOutRows * S;                   // two stages of [128][72]
-    float* wts = reinterpret_cast<float*>(ws + 2 * kMmaCols * S);  // [16][splits]
+    const int chunks = (a.rank + K - 1) / K, SO = chunks * K + 8;
+    __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(raw);   // stages of [128][72]
+    __nv_bfloat16* os = ws + kOutStages * kMmaCols * S;           // [16][rank, padded + 8]
+    float* wts = reinterpret_cast<float*>(os + kOutRows * SO);   // [16][splits]
     const int h = blockIdx.x, e0 = blockIdx.z * kMmaCols;
     const int64_t t0 = static_cast<int64_t>(blockIdx.y) * kOutRows;
     const int rows = static_cast<int>(min(static_cast<int64_t>(kOutRows), a.n - t0));
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w_uv) + (static_cast<int64_t>(h) * a.vdim + e0) * a.rank;
-    const int live = min(kMmaCols, a.vdim - e0);
-    fetch_tile(ws, S, w, a.rank, kMmaCols, live, K, a.rank, vec_w);
-    cp_async_commit();
+    const int live = min(kMmaCols, a.vdim - e0), used = (live + 15) & ~15;
+    auto fetch = [&](int c) {
+        if (c < chunks) fetch_tile(ws + (c % kOutStages) * kMmaCols * S, S, w + c * K, a.rank, used, live, K, a.rank - c * K, vec_w);
+        cp_async_commit();
+    };
+    for (int c = 0; c < kOutStages - 1; ++c) fetch(c);
     range_weights(a, h, t0, rows, wts);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
-    const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
-    const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank;
-    const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
-    float acc[2][4] = {};
-    for (int k0 = 0, buf = 0; k0 < a.rank; k0 += K, buf ^= 1) {
-        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < rows) {
-            for (int s = 0; s < a.splits; ++s) {
-                const float f = wts[r * a.splits + s];
-                if (f != 0.0f) {
-                    const float4 x = spk_load4<float, VEC>(part + s * step + k0 + c4, a.rank - k0 - c4);
-                    y = make_float4(fmaf(f, x.x, y.x), fmaf(f, x.y, y.y), fmaf(f, x.z, y.z), fmaf(f, x.w, y.w));
+    {
+        const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
+        const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank + c4;
+        const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
+        constexpr int U = 8;
+        for (int g = 0; g < chunks; g += U) {
+            float4 y[U];
+#pragma unroll
+            for (int u = 0; u < U; ++u) y[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < rows) {
+                for (int s = 0; s < a.splits; ++s) {
+                    const float f = wts[r * a.splits + s];
+                    if (f == 0.0f) continue;
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        const float4 x = spk_load4<float, VEC>(part + s * step + (g + u) * K, a.rank - (g + u) * K - c4);
+                        y[u] = make_float4(fmaf(f, x.x, y[u].x), fmaf(f, x.y, y[u].y), fmaf(f, x.z, y[u].z), fmaf(f, x.w, y[u].w));
+                    }
                 }
             }
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+                if (g + u < chunks)
+                    *reinterpret_cast<uint2*>(os + r * SO + (g + u) * K + c4) = make_uint2(pack_bf16(y[u].x, y[u].y), pack_bf16(y[u].z, y[u].w));
         }
-        *reinterpret_cast<uint2*>(os + buf * kOutRows * S + r * S + c4) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
-        cp_async_wait_all();
-        __syncthreads();  // this stage is there, the previous one has been read
-        if (k0 + K < a.rank) fetch_tile(ws + (buf ^ 1) * kMmaCols * S, S, w + k0 + K, a.rank, kMmaCols, live, K, a.rank - k0 - K, vec_w);
-        cp_async_commit();
-        const __nv_bfloat16 *ob = os + buf * kOutRows * S, *wb = ws + buf * kMmaCols * S;
+    }
+    float acc[2][4] = {};
+    for (int c = 0; c < chunks; ++c) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(kOutStages - 2) : "memory");
+        __syncthreads();  // this stage is there, the one before has been read
+        fetch(c + kOutStages - 1);
+        if (warp * 16 >= used) continue;
+        const __nv_bfloat16 *ob = os + c * K, *wb = ws + (c % kOutStages) * kMmaCols * S;
 #pragma unroll
         for (int k = 0; k < K; k += 16) {
             uint32_t x[4], b[4];
-            ldsm4(x, smem_u32(ob + (lane & 15) * S + k + (lane >> 4) * 8));
+            ldsm4(x, smem_u32(ob + (lane & 15) * SO + k + (lane >> 4) * 8));
             ldsm4(b, smem_u32(wb + (warp * 16 + (m >> 1) * 8 + mr) * S + k + (m & 1) * 8));
             mma16816(acc[0], x, b[0], b[1]);
             mma16816(acc[1], x, b[2], b[3]);
@@ -483,7 +504,7 @@ int launch_query_mma(const spk_latent_query_args& a, cudaStream_t s) {
     const size_t bytes = 2 * (static_cast<size_t>(kMmaRows) * (dp + 8) + static_cast<size_t>(dp) * (kMmaCols + 8));
     if (const int rc = with_smem(reinterpret_cast<const void*>(latent_query_mma_kernel), bytes)) return rc;
     const bool vq = at16(a.q) && (a.dim + a.rot_dim) % 8 == 0 && a.dim % 8 == 0, vw = at16(a.w_uk) && a.rank % 8 == 0;
-    latent_query_mma_kernel<<<dim3(a.heads, (a.rank + kMmaCols - 1) / kMmaCols, static_cast<unsigned>(tiles)), kThreads, bytes, s>>>(a, dp, vq, vw);
+    latent_query_mma_kernel<<<dim3(a.heads, (a.rank + kMmaCols - 1) / kMmaCols + 1, static_cast<unsigned>(tiles)), kThreads, bytes, s>>>(a, dp, vq, vw);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -491,7 +512,7 @@ int launch_query_mma(const spk_latent_query_args& a, cudaStream_t s) {
 int launch_out_mma(const spk_latent_out_args& a, cudaStream_t s) {
     const int64_t tiles = (a.n + kOutRows - 1) / kOutRows;
     if (tiles > 65535) return SPK_ERR_TOO_LARGE;
-    const size_t bytes = 2 * 2 * (kOutRows + kMmaCols) * 72 + sizeof(float) * kOutRows * a.splits;
+    const size_t bytes = 2 * (static_cast<size_t>(kOutStages) * kMmaCols * 72 + kOutRows * (((a.rank + 63) / 64) * 64 + 8)) + sizeof(float) * kOutRows * a.splits;
     const dim3 grid(a.heads, static_cast<unsigned>(tiles), (a.vdim + kMmaCols - 1) / kMmaCols);
     const bool vec = a.rank % 4 == 0 && at16(a.partials), vw = at16(a.w_uv) && a.rank % 8 == 0;
     auto* fn = vec ? latent_out_mma_kernel<true> : latent_out_mma_kernel<false>;

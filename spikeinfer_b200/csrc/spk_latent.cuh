@@ -3,9 +3,16 @@
 
 #include "spk_dense.cuh"
 
-// A cache row: `rank` latent channels at 0, rot_dim rotated channels at rank_pad; one pool head.
+// A cache row: `rank` latent channels at 0, rot_dim rotated channels at rank_pad; one pool head.  Tiled pages hold eight rows after the other,
+// and of eight rows 64 channels after the other: 1 KB atoms of 8 x 128 bytes, the 16-byte group g of row r at group g ^ (r & 7).  So any run
+// of whole pages laid end to end is one operand of the tensor core, with all channels, whichever of rows and channels it sums over.
 __host__ __device__ __forceinline__ SpkPageLayout spk_latent_layout(int block_size, int rank_pad, int rot_pad, int tiled) {
     return SpkPageLayout{1, block_size, rank_pad + rot_pad, tiled};
+}
+
+__device__ __forceinline__ int spk_latent_channel(const SpkPageLayout& p, int r, int d) {
+    if (!p.tiled) return r * p.dim_pad + d;
+    return (r >> 3) * (p.dim_pad << 3) + ((d >> 6) << 9) + ((r & 7) << 6) + ((((d >> 3) & 7) ^ (r & 7)) << 3) + (d & 7);
 }
 
 // Tiled 16-bit pool of at most 512 latent and 64 rotated channels, pages of 16 rows or a larger power of two.

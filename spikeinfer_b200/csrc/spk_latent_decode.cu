@@ -3,8 +3,8 @@
 // All heads read the same cache rows, so a CTA takes 32 heads of a token at once over a range of its keys, and the cache rows are the M
 // operand of both products: S^T = K Q^T (64 keys x 32 heads) and O^T += V^T P^T (128 latent channels x 32 heads per MMA), V being the
 // latent part of the very tile K is.  No row of the accumulators is padding, a step reads the cache once and stays bound by that.
-//  * warp 4 copies: a page of the pool is stored as the swizzled operand tile it becomes, so a 64-key stage is a handful of plain bulk
-//    copies (cp.async.bulk) whatever pages the block table names;
+//  * warp 4 copies: pages laid end to end are an operand as they are (spk_latent.cuh), so a 64-key stage is one plain bulk copy
+//    (cp.async.bulk) per page, all channels at once, whatever pages the block table names;
 //  * warp 5 issues S^T into one of two TMEM buffers, warp 6 the weighted sums;
 //  * warps 0-3 turn scores into weights, sixteen keys each, in the fragment layout of tcgen05.ld.16x256b: two keys x eight heads per lane.
 // Weights are exp2(score - reference), 32-bit, and enter the product as a bf16 pair side by side (columns 0-31 the high, 32-63 the
@@ -18,7 +18,8 @@ namespace {
 using namespace spk_tc;
 
 constexpr int kKeys = 64;                  // keys per step
-constexpr int kColTile = kKeys * 128;      // bytes of a 64-channel column tile of a step
+constexpr int kAtom = 1024;                // bytes of eight rows x 64 channels
+constexpr int kPTile = kKeys * 128;        // a step's weights: 64 keys x (32 high | 32 low parts)
 constexpr int kHeads = 32;                 // heads of a CTA
 constexpr int kQTile = kHeads * 128;
 constexpr int kSoftThreads = 128;
@@ -30,9 +31,10 @@ constexpr float kSlack = 8.0f;             // a score may exceed the reference b
 template <int CL>
 struct Shape {
     static constexpr int CT = CL + 1, MB = (CL + 1) / 2;
-    static constexpr int kStage = CT * kColTile;
+    static constexpr int kGroup = CT * kAtom;  // eight rows
+    static constexpr int kStage = kKeys / 8 * kGroup;
     static constexpr int NS = CT > 6 ? 2 : CT > 4 ? 3 : 4;
-    static constexpr int kBytes = NS * kStage + CT * kQTile + 2 * kColTile + 1024 + 1536;
+    static constexpr int kBytes = NS * kStage + CT * kQTile + 2 * kPTile + 1024 + 1536;
     static constexpr int kColumns = MB > 2 ? 512 : 256;  // scores 2 x 32, then MB x 64 sums
 };
 constexpr uint32_t kTmemO = 2 * kHeads;
@@ -77,7 +79,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
     uint8_t* q_s = base + NS * Sh::kStage;
     uint8_t* p_s = q_s + CT * kQTile;
-    Bars* bars = reinterpret_cast<Bars*>(p_s + 2 * kColTile);
+    Bars* bars = reinterpret_cast<Bars*>(p_s + 2 * kPTile);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         for (int i = 0; i < NS; ++i) {
@@ -122,20 +124,16 @@ latent_decode_kernel(const spk_latent_attn_args a) {
             // waits are made warp-uniform: a vote also brings the lanes back together
             if (s >= NS && !__all_sync(~0u, mbar_wait(smem_u32(&bars->free[st]), ((s / NS) - 1) & 1, abort))) break;
             const uint32_t bar = smem_u32(&bars->full[st]);
-            if (lane == 0) mbar_expect(bar, static_cast<uint32_t>(n * CT * gran * 128));
+            if (lane == 0) mbar_expect(bar, static_cast<uint32_t>(n * gran * CT * 128));
             __syncwarp();
-            for (int i0 = 0; i0 < n * CT; i0 += 32) {
-                const int i = i0 + lane, p = i % n, c = i / n;
-                int64_t block = __shfl_sync(~0u, mine, p);
-                if (i < n * CT) {
-                    if (block < 0 || block >= a.num_blocks) {
-                        spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
-                        block = 0;
-                    }
-                    const __nv_bfloat16* src = pool + spk_page_base(lay, block, 0) + (static_cast<int64_t>(c) << (bs_log2 + 6)) +
-                                               (((j0 + p * gran) & (a.block_size - 1)) << 6);
-                    bulk_load(smem_u32(base + st * Sh::kStage) + c * kColTile + p * gran * 128, src, gran * 128, bar);
+            if (lane < n) {
+                int64_t block = mine;
+                if (block < 0 || block >= a.num_blocks) {
+                    spk_flag(a.status, SPK_STATUS_BAD_BLOCK);
+                    block = 0;
                 }
+                const __nv_bfloat16* src = pool + spk_page_base(lay, block, 0) + ((j0 + lane * gran) & (a.block_size - 1)) * (CT * 64);
+                bulk_load(smem_u32(base + st * Sh::kStage) + lane * gran * CT * 128, src, gran * CT * 128, bar);
             }
             issued = s + 1;
         }
@@ -155,7 +153,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
                 const uint32_t ka = smem_u32(base + st * Sh::kStage), qa = smem_u32(q_s);
 #pragma unroll
                 for (int k = 0; k < CT * 4; ++k)
-                    mma_ss(tmem + (s & 1) * kHeads, desc_sw128(ka + (k >> 2) * kColTile + (k & 3) * 32, 16, 1024),
+                    mma_ss(tmem + (s & 1) * kHeads, desc_sw128(ka + (k >> 2) * kAtom + (k & 3) * 32, 16, Sh::kGroup),
                            desc_sw128(qa + (k >> 2) * kQTile + (k & 3) * 32, 16, 1024), idesc, k > 0);
                 mma_commit(smem_u32(&bars->s_full[s & 1]));
             }
@@ -169,13 +167,13 @@ latent_decode_kernel(const spk_latent_attn_args a) {
                 const int st = s % NS;
                 if (!mbar_wait(smem_u32(&bars->p_full[s & 1]), (s >> 1) & 1, abort)) break;
                 tc_fence_after();
-                const uint32_t va = smem_u32(base + st * Sh::kStage), pa = smem_u32(p_s + (s & 1) * kColTile);
+                const uint32_t va = smem_u32(base + st * Sh::kStage), pa = smem_u32(p_s + (s & 1) * kPTile);
                 const int steps = (min(kKeys, hi - lo - s * kKeys) + 15) >> 4;
                 for (int k = 0; k < steps; ++k) {
                     const uint64_t pd = desc_sw128(pa + k * 2048, 16, 1024);
 #pragma unroll
                     for (int b = 0; b < MB; ++b)
-                        mma_ss(tmem + kTmemO + b * 2 * kHeads, desc_sw128(va + b * 2 * kColTile + k * 2048, kColTile, 1024), pd, idesc, s > 0 || k > 0);
+                        mma_ss(tmem + kTmemO + b * 2 * kHeads, desc_sw128(va + b * 2 * kAtom + k * 2 * Sh::kGroup, kAtom, Sh::kGroup), pd, idesc, s > 0 || k > 0);
                 }
                 mma_commit(smem_u32(&bars->free[st]));
                 mma_commit(smem_u32(&bars->p_free[s & 1]));
@@ -268,7 +266,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
                 }
             }
             if (s >= 2) __all_sync(~0u, mbar_wait(smem_u32(&bars->p_free[buf]), ((s >> 1) - 1) & 1, abort));
-            uint8_t* p = p_s + buf * kColTile;
+            uint8_t* p = p_s + buf * kPTile;
 #pragma unroll
             for (int g = 0; g < 4; ++g) {
 #pragma unroll
@@ -290,8 +288,8 @@ latent_decode_kernel(const spk_latent_attn_args a) {
                 __all_sync(~0u, mbar_wait(smem_u32(&bars->full[st]), (s / NS) & 1, abort));
                 const int end = (valid + 15) & ~15;
                 for (int i = threadIdx.x; i < (end - valid) * CL * 8; i += kSoftThreads) {
-                    const int c = i / ((end - valid) * 8), rest = i % ((end - valid) * 8);
-                    *reinterpret_cast<uint4*>(base + st * Sh::kStage + c * kColTile + (valid + (rest >> 3)) * 128 + ((rest & 7) << 4)) =
+                    const int c = i / ((end - valid) * 8), rest = i % ((end - valid) * 8), r = valid + (rest >> 3);
+                    *reinterpret_cast<uint4*>(base + st * Sh::kStage + (r >> 3) * Sh::kGroup + c * kAtom + (r & 7) * 128 + ((rest & 7) << 4)) =
                         make_uint4(0u, 0u, 0u, 0u);
                 }
             }

@@ -380,7 +380,7 @@ latent_gather_kernel(const spk_latent_gather_args a) {
             block = a.num_blocks - 1;
         }
         const uint4 v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.pool) + spk_page_base(lay, block, 0) +
-                                                         spk_page_channel(lay, p % a.block_size, g * 8));
+                                                         spk_latent_channel(lay, p % a.block_size, g * 8));
         __nv_bfloat16* dst = g < own ? static_cast<__nv_bfloat16*>(a.latents) + static_cast<int64_t>(e.x + r) * a.rank_pad + g * 8
                                      : static_cast<__nv_bfloat16*>(a.rotated) + static_cast<int64_t>(e.x + r) * 64 + (g - own) * 8;
         *reinterpret_cast<uint4*>(dst) = v;

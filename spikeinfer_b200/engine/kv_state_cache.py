@@ -66,7 +66,8 @@ class PagedKVPool:
 
 class PagedLatentPool(PagedKVPool):
     """A pool of shared-latent cache rows: ``rank`` latent channels at 0, ``rot_dim`` rotated ones at ``rank_pad``; one pool head.
-    Tiled (see :class:`PagedKVPool`) in 16 bits, both parts padded to 64 channels; plain without padding otherwise."""
+    In 16 bits pages are tiled and both parts padded to 64 channels: eight rows after the other, of eight rows 64 channels after
+    the other, swizzled as in :class:`PagedKVPool`, so that pages laid end to end are one operand.  Plain without padding otherwise."""
 
     def __init__(self, num_blocks: int, block_size: int, rank: int, rot_dim: int, dtype: torch.dtype, device) -> None:
         self.rank, self.rot_dim, self.block_size = rank, rot_dim, block_size
@@ -77,7 +78,13 @@ class PagedLatentPool(PagedKVPool):
 
     def rows(self) -> torch.Tensor:
         """``[num_blocks * block_size, rank + rot_dim]`` in plain order (for checks)."""
-        x = super().rows()[:, 0]
+        nb, _, bs, pad = self.data.shape
+        x = self.data.view(nb * bs, pad)
+        if self.tiled:
+            x = self.data.view(nb, bs // 8, pad // 64, 8, 8, 8)
+            r = torch.arange(8, device=x.device)
+            group = r[None, :] ^ r[:, None]  # stored place of group c in row r
+            x = x.gather(4, group.view(1, 1, 1, 8, 8, 1).expand(x.shape)).transpose(2, 3).reshape(nb * bs, pad)
         return torch.cat((x[:, : self.rank], x[:, self.rank_pad: self.rank_pad + self.rot_dim]), dim=1)
 
 

@@ -126,8 +126,8 @@ def test_latent_pools_and_sharing():
     assert pool.tiled and (pool.rank_pad, pool.rot_pad, pool.pad) == (64, 64, 128)
     plain = PagedLatentPool(3, 16, 56, 16, torch.float32, "cpu")
     assert not plain.tiled and plain.pad == 72 and plain.rows().shape == (48, 72)
-    pool.data.view(3, -1)[1, 64 * 16 + 5 * 64 + ((1 ^ 5) << 3) + 2] = 7.0     # page 1, row 5, rotated channel 10
-    assert pool.rows()[16 + 5, 56 + 10] == 7.0
+    pool.data.view(3, -1)[1, 8 * 128 + 512 + 5 * 64 + ((1 ^ 5) << 3) + 2] = 7.0     # page 1, row 13, rotated channel 10
+    assert pool.rows()[16 + 13, 56 + 10] == 7.0
     specs = [LayerCacheSpec(states=(("s", (2, 3)),)), LayerCacheSpec(latent=LatentSpec(8, 4)), LayerCacheSpec(latent_from=1)]
     cache = PagedKVStateCache(specs, 4, 16, 2, torch.float32, "cpu")
     assert cache.layers[2].latent is cache.layers[1].latent and cache.nbytes == 4 * (2 * 6 + 4 * 16 * 12)

@@ -260,11 +260,11 @@ def test_used_slots_and_pages_may_hold_anything(dev):
             if layer.latent is not None:
                 layer.latent.data.fill_(float("nan"))
                 if layer.latent.tiled:  # padding channels stay zero
-                    plain = layer.latent.data.view(*layer.latent.data.shape[:2], layer.latent.pad // 64, layer.latent.block_size, 8, 8)
-                    r = torch.arange(layer.latent.block_size, device=dev)
+                    atoms = layer.latent.data.view(-1, layer.latent.pad // 64, 8, 8, 8)
+                    r = torch.arange(8, device=dev)
                     for c in range(layer.latent.pad):
                         if layer.latent.rank <= c < layer.latent.rank_pad or c >= layer.latent.rank_pad + layer.latent.rot_dim:
-                            plain[:, :, c // 64, r, ((c // 8) % 8) ^ (r & 7), c % 8] = 0
+                            atoms[:, c // 64, r, ((c // 8) % 8) ^ r, c % 8] = 0
         tokens = prompt("mixed", 40, 3)
         want, _ = reference("mixed", tuple(tokens))
         row = eng.open_request()

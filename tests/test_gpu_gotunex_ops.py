@@ -185,10 +185,9 @@ def filled_pool(dev, dtype, seqs, rank, rot_dim, block_size, seed, blocks=None):
             at += 1
     x = plain.view(nb, 1, block_size, pool.pad)
     if pool.tiled:
-        r = torch.arange(block_size)
-        source = torch.arange(8)[None, :] ^ (r[:, None] & 7)
-        x = x.view(nb, 1, block_size, pool.pad // 64, 8, 8).permute(0, 1, 3, 2, 4, 5)
-        x = x.gather(4, source.view(1, 1, 1, block_size, 8, 1).expand(x.shape)).reshape(nb, 1, block_size, pool.pad)
+        r = torch.arange(8)
+        x = x.view(nb, block_size // 8, 8, pool.pad // 64, 8, 8).transpose(2, 3)
+        x = x.gather(4, (r[None, :] ^ r[:, None]).view(1, 1, 1, 8, 8, 1).expand(x.shape)).reshape(nb, 1, block_size, pool.pad)
     pool.data.copy_(x.to(dtype))
     return pool, tables.to(dev)
 
