@@ -4,7 +4,7 @@
 //   S <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  out = o / rms(o) * w * sigmoid(gate)
 //
 //  * delta_step_kernel: one token per row (decode).  A CTA owns a (head, row): it convolves, normalises, decays, updates and reads the
-//    state and writes the gated output; the state is read and written once.
+//    state and writes the gated output; the state crosses the memory bus once each way.
 //  * prefill, any sizes, 32-bit: delta_prepare_kernel (convolutions, unit vectors, decays, step sizes), delta_scan_kernel (the
 //    recurrence, columns of the state in registers, tokens one after the other); bf16 heads of up to 128 channels take the chunked
 //    form of spk_delta_mma.cu instead.  delta_out_kernel (norm and gate) ends both.
@@ -20,23 +20,15 @@ using namespace spk_tc;
 constexpr int kThreads = 256;
 
 // ---- decode ------------------------------------------------------------------------------------------------------------
-template <int W>
-__device__ __forceinline__ void load_state(float (&s)[W], const float* p) {
-    if (W == 4) {
-        const float4 f = __ldcs(reinterpret_cast<const float4*>(p));
-        s[0] = f.x; s[1 % W] = f.y; s[2 % W] = f.z; s[3 % W] = f.w;
-    } else {
-        s[0] = *p;
-    }
-}
-
-// CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  KEEP: rows of the
-// state that are a thread's share and stay in its registers between the two products; 0: any share, read twice.
-template <typename T, int W, int KEEP, int NT>
-__global__ void __launch_bounds__(NT, NT == 128 ? 6 : 2)
-delta_step_kernel(const spk_delta_args a, const int prefetch) {
-    extern __shared__ float sm[];
+// CTA (head, row).  W columns per thread (4: 16-byte accesses); threads = (column group, slice of the key channels).  STAGED: the state
+// comes into shared memory with one bulk copy while the convolutions run, is updated there and leaves with another; otherwise it is
+// read twice from where it is.
+template <typename T, int W, bool STAGED, int NT>
+__global__ void __launch_bounds__(NT)
+delta_step_kernel(const spk_delta_args a) {
+    extern __shared__ __align__(128) float sm[];
     __shared__ float part[3 * 32];
+    __shared__ uint64_t arrived;
     const int h = blockIdx.x;
     const int64_t row = blockIdx.y;
     const int dim = a.dim, vdim = a.vdim, rep = a.heads / a.kv_heads, g = h / rep;
@@ -45,154 +37,172 @@ delta_step_kernel(const spk_delta_args a, const int prefetch) {
         for (int e = threadIdx.x; e < vdim; e += NT) out[e] = spk_from_float<T>(0.0f);
         return;
     }
-    float* q = sm;                 // [dim]
-    float* k = q + dim;            // [dim]
-    float* dec = k + dim;          // [dim]
-    float* v = dec + dim;          // [vdim]; the outputs afterwards
-    float* red = v + vdim;         // [slices][vdim]
     float* S = a.state + (row * a.heads + h) * static_cast<int64_t>(dim) * vdim;
+    float* held = sm;                                                        // [dim][vdim] (STAGED)
+    float* q = sm + (STAGED ? static_cast<int64_t>(dim) * vdim : 0);         // [dim]
+    float* k = q + dim;                                                      // [dim]
+    float* dec = k + dim;                                                    // [dim]
+    float* v = dec + dim;                                                    // [vdim]; the outputs afterwards
+    float* red = v + vdim;                                                   // [slices][vdim]
+    const uint32_t state_bytes = static_cast<uint32_t>(dim) * vdim * 4;
+    if (STAGED && threadIdx.x == 0) {
+        mbar_init(smem_u32(&arrived), 1);
+        fence_async_shared();
+        mbar_expect(smem_u32(&arrived), state_bytes);
+        bulk_load(smem_u32(held), S, state_bytes, smem_u32(&arrived));
+    }
     const int cols = vdim / W;
     const int slices = cols < NT ? NT / cols : 1;
     const int slice = slices > 1 ? threadIdx.x / cols : 0;
     const int first = slices > 1 ? threadIdx.x % cols : threadIdx.x;
     const bool mine = slice < slices;
-    float s[KEEP > 0 ? KEEP : 1][W];
-    if (KEEP && mine) {  // on its way before the projections are looked at
-#pragma unroll
-        for (int u = 0; u < KEEP; ++u) {
-            const int d = slice + u * slices;
-            if (d < dim) load_state<W>(s[u], S + static_cast<int64_t>(d) * vdim + first * W);
-        }
-    }
-    if (threadIdx.x == 0 && prefetch > 0) {  // the state of the CTA that follows this one on its SM
-        const int64_t next = row * a.heads + h + prefetch, bytes = static_cast<int64_t>(dim) * vdim * 4;
-        if (next < a.n * a.heads)
-            asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(__cvta_generic_to_global(a.state + next * dim * vdim)), "r"(static_cast<uint32_t>(bytes)) : "memory");
-    }
     const SpkDeltaShape sh = spk_delta_shape(a);
     const int64_t pos = a.positions[row];
     const bool fresh = pos == 0;  // whatever the slot holds, a sequence starts from zeros
-    if (KEEP && fresh) {
-#pragma unroll
-        for (int u = 0; u < KEEP; ++u)
-#pragma unroll
-            for (int i = 0; i < W; ++i) s[u][i] = 0.0f;
-    }
     float* ring = a.conv_state + row * a.taps * sh.channels;
     const int now_slot = static_cast<int>(static_cast<uint64_t>(pos) % static_cast<uint32_t>(a.taps));
     const int past = pos < a.taps - 1 ? static_cast<int>(pos) : a.taps - 1;  // earlier tokens the convolution sees
     const bool leader = h % rep == 0;
+    const T* gate = static_cast<const T*>(a.gate) + row * a.ld2 + static_cast<int64_t>(h) * vdim;
     float sums[3] = {0.0f, 0.0f, 0.0f};
-    // one channel of q, k, the decays or v per thread and turn
-    for (int i = threadIdx.x; i < 3 * dim + vdim; i += NT) {
-        if (i >= 2 * dim && i < 3 * dim) {
-            const int d = i - 2 * dim;
-            const int64_t c = static_cast<int64_t>(h) * dim + d;
-            dec[d] = expf(spk_log_decay(spk_to_float<T>(static_cast<const T*>(a.a)[row * a.ld2 + c]) + a.dt_bias[c], expf(a.a_log[h])));
-            continue;
+    // one channel of q, k, the decays or v per thread and turn; two turns' loads are in flight together
+    struct Item {
+        float x, w0, back[3], w[3], bias;
+        int kind, local, at;  // 0 q, 1 k, 2 v, 3 decay, -1 none
+        const float* taps;
+    };
+    const int items = 3 * dim + vdim;
+    auto fetch = [&](int i) {
+        Item it;
+        it.kind = i >= items ? -1 : i < dim ? 0 : i < 2 * dim ? 1 : i < 3 * dim ? 3 : 2;
+        if (it.kind < 0) return it;
+        if (it.kind == 3) {
+            it.local = i - 2 * dim;
+            const int c = h * dim + it.local;
+            it.x = spk_to_float<T>(static_cast<const T*>(a.a)[row * a.ld2 + c]);
+            it.bias = a.dt_bias[c];
+            it.w0 = a.a_log[h];
+            return it;
         }
-        const int part_of = i < dim ? 0 : i < 2 * dim ? 1 : 2;
-        const int local = part_of == 0 ? i : part_of == 1 ? i - dim : i - 3 * dim;
-        const int c = part_of == 2 ? h * vdim + local : g * dim + local;  // channel of its projection
-        const int at = c + part_of * sh.qk;                                // and its place in the ring
-        const void* src = part_of == 0 ? a.q : part_of == 1 ? a.k : a.v;
-        const float* w = (part_of == 0 ? a.conv_q : part_of == 1 ? a.conv_k : a.conv_v) + static_cast<int64_t>(c) * a.taps;
-        const float x = spk_to_float<T>(static_cast<const T*>(src)[row * a.ld + c]);
-        float y = x * w[a.taps - 1];
-#pragma unroll 4
-        for (int back = 1; back <= past; ++back) {
-            const int slot = now_slot >= back ? now_slot - back : now_slot - back + a.taps;
-            y = fmaf(ring[slot * sh.channels + at], w[a.taps - 1 - back], y);
+        it.local = it.kind == 0 ? i : it.kind == 1 ? i - dim : i - 3 * dim;
+        const int c = it.kind == 2 ? h * vdim + it.local : g * dim + it.local;  // channel of its projection
+        it.at = c + it.kind * sh.qk;                                             // and its place in the ring
+        const void* src = it.kind == 0 ? a.q : it.kind == 1 ? a.k : a.v;
+        it.taps = (it.kind == 0 ? a.conv_q : it.kind == 1 ? a.conv_k : a.conv_v) + static_cast<int64_t>(c) * a.taps;
+        it.x = spk_to_float<T>(static_cast<const T*>(src)[row * a.ld + c]);
+        it.w0 = it.taps[a.taps - 1];
+#pragma unroll
+        for (int b = 1; b <= 3; ++b) {
+            const bool in = b <= past;
+            const int slot = now_slot >= b ? now_slot - b : now_slot - b + a.taps;
+            it.back[b - 1] = in ? ring[slot * sh.channels + it.at] : 0.0f;
+            it.w[b - 1] = in ? it.taps[a.taps - 1 - b] : 0.0f;
+        }
+        return it;
+    };
+    auto finish = [&](const Item& it) {
+        if (it.kind < 0) return;
+        if (it.kind == 3) {
+            dec[it.local] = expf(spk_log_decay(it.x + it.bias, expf(it.w0)));
+            return;
+        }
+        float y = it.x * it.w0;
+#pragma unroll
+        for (int b = 0; b < 3; ++b) y = fmaf(it.back[b], it.w[b], y);
+        for (int b = 4; b <= past; ++b) {
+            const int slot = now_slot >= b ? now_slot - b : now_slot - b + a.taps;
+            y = fmaf(ring[slot * sh.channels + it.at], it.taps[a.taps - 1 - b], y);
         }
         y = spk_silu(y);
-        if (leader || part_of == 2) ring[now_slot * sh.channels + at] = x;
-        if (part_of == 0) {
-            q[local] = y;
+        if (leader || it.kind == 2) ring[now_slot * sh.channels + it.at] = it.x;
+        if (it.kind == 0) {
+            q[it.local] = y;
             sums[0] = fmaf(y, y, sums[0]);
-        } else if (part_of == 1) {
-            k[local] = y;
+        } else if (it.kind == 1) {
+            k[it.local] = y;
             sums[1] = fmaf(y, y, sums[1]);
         } else {
-            v[local] = y;
+            v[it.local] = y;
         }
+    };
+    const float raw_beta = spk_to_float<T>(static_cast<const T*>(a.b)[row * a.ld + h]);
+    for (int i = threadIdx.x; i < items; i += 2 * NT) {
+        const Item x = fetch(i), y = fetch(i + NT);
+        finish(x);
+        finish(y);
     }
+    const float gate_mine = static_cast<int>(threadIdx.x) < vdim ? spk_to_float<T>(gate[threadIdx.x]) : 0.0f;
+    const float norm_mine = static_cast<int>(threadIdx.x) < vdim ? a.w_norm[threadIdx.x] : 0.0f;
     spk_block_sum<3>(sums, part);  // its barriers also publish q, k, v and the decays
     const float qi = 1.0f / (sqrtf(sums[0] + 1e-6f) * sqrtf(static_cast<float>(dim))), ki = 1.0f / sqrtf(sums[1] + 1e-6f);
-    const float beta = spk_sigmoid(spk_to_float<T>(static_cast<const T*>(a.b)[row * a.ld + h]));
+    const float beta = spk_sigmoid(raw_beta);
+    if (STAGED && !mbar_wait(smem_u32(&arrived), 0) && threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_DEVICE_WAIT_EXPIRED);
+    const float* from = STAGED ? held : S;
+    float* to = STAGED ? held : S;
+    auto load = [&](float (&x)[W], int d, int c) {
+        const float* p = from + static_cast<int64_t>(d) * vdim + c * W;
+        if (W == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(p);
+            x[0] = f.x; x[1 % W] = f.y; x[2 % W] = f.z; x[3 % W] = f.w;
+        } else {
+            x[0] = *p;
+        }
+#pragma unroll
+        for (int i = 0; i < W; ++i) x[i] = fresh ? 0.0f : x[i] * dec[d];
+    };
     float square[1] = {0.0f};
     for (int c0 = 0; c0 < cols; c0 += NT) {
         const int c = c0 + first;
         const bool in = mine && c < cols;
         float acc[W] = {};
         if (in) {
-            if (KEEP) {
+#pragma unroll 4
+            for (int d = slice; d < dim; d += slices) {
+                float x[W];
+                load(x, d, c);
+                const float kd = k[d] * ki;
 #pragma unroll
-                for (int u = 0; u < KEEP; ++u) {
-                    const int d = slice + u * slices;
-                    if (d < dim) {
-                        const float gd = dec[d], kd = k[d] * ki;
-#pragma unroll
-                        for (int i = 0; i < W; ++i) {
-                            s[u][i] *= gd;
-                            acc[i] = fmaf(kd, s[u][i], acc[i]);
-                        }
-                    }
-                }
-            } else {
-                for (int d = slice; d < dim; d += slices) {
-                    float x[W];
-                    load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
-                    const float w = dec[d] * (k[d] * ki);
-#pragma unroll
-                    for (int i = 0; i < W; ++i) acc[i] = fresh ? 0.0f : fmaf(w, x[i], acc[i]);
-                }
+                for (int i = 0; i < W; ++i) acc[i] = fmaf(kd, x[i], acc[i]);
             }
 #pragma unroll
             for (int i = 0; i < W; ++i) red[slice * vdim + c * W + i] = acc[i];
         }
         __syncthreads();
-        float u_[W] = {};
+        float u[W] = {};
         if (in) {
 #pragma unroll
             for (int i = 0; i < W; ++i) {
                 float sk = 0.0f;
                 for (int z = 0; z < slices; ++z) sk += red[z * vdim + c * W + i];
-                u_[i] = beta * (v[c * W + i] - sk);
+                u[i] = beta * (v[c * W + i] - sk);
                 acc[i] = 0.0f;
             }
         }
         __syncthreads();  // the first product's parts have been read
         if (in) {
-            auto update = [&](float (&x)[W], int d) {
+#pragma unroll 4
+            for (int d = slice; d < dim; d += slices) {
+                float x[W];
+                load(x, d, c);
                 const float kd = k[d] * ki, qd = q[d] * qi;
 #pragma unroll
                 for (int i = 0; i < W; ++i) {
-                    x[i] = fmaf(kd, u_[i], x[i]);
+                    x[i] = fmaf(kd, u[i], x[i]);
                     acc[i] = fmaf(qd, x[i], acc[i]);
                 }
-                float* dst = S + static_cast<int64_t>(d) * vdim + c * W;
-                if (W == 4) __stcs(reinterpret_cast<float4*>(dst), make_float4(x[0], x[1 % W], x[2 % W], x[3 % W]));
+                float* dst = to + static_cast<int64_t>(d) * vdim + c * W;
+                if (W == 4) *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1 % W], x[2 % W], x[3 % W]);
                 else *dst = x[0];
-            };
-            if (KEEP) {
-#pragma unroll
-                for (int u = 0; u < KEEP; ++u) {
-                    const int d = slice + u * slices;
-                    if (d < dim) update(s[u], d);
-                }
-            } else {
-                for (int d = slice; d < dim; d += slices) {
-                    float x[W];
-                    load_state<W>(x, S + static_cast<int64_t>(d) * vdim + c * W);
-#pragma unroll
-                    for (int i = 0; i < W; ++i) x[i] = fresh ? 0.0f : x[i] * dec[d];
-                    update(x, d);
-                }
             }
 #pragma unroll
             for (int i = 0; i < W; ++i) red[slice * vdim + c * W + i] = acc[i];
         }
+        if (STAGED) fence_async_shared();
         __syncthreads();
+        if (STAGED && c0 + NT >= cols && threadIdx.x == 0) {
+            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(__cvta_generic_to_global(S)), "r"(smem_u32(held)), "r"(state_bytes) : "memory");
+            asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+        }
         if (in && slice == 0) {
 #pragma unroll
             for (int i = 0; i < W; ++i) {
@@ -205,9 +215,11 @@ delta_step_kernel(const spk_delta_args a, const int prefetch) {
     }
     spk_block_sum<1>(square, part);
     const float inv = 1.0f / sqrtf(square[0] / static_cast<float>(vdim) + a.eps);
-    const T* gate = static_cast<const T*>(a.gate) + row * a.ld2 + static_cast<int64_t>(h) * vdim;
-    for (int e = threadIdx.x; e < vdim; e += NT)
-        out[e] = spk_from_float<T>(v[e] * inv * a.w_norm[e] * spk_sigmoid(spk_to_float<T>(gate[e])));
+    for (int e = threadIdx.x; e < vdim; e += NT) {
+        const bool own = e == static_cast<int>(threadIdx.x);
+        out[e] = spk_from_float<T>(v[e] * inv * (own ? norm_mine : a.w_norm[e]) * spk_sigmoid(own ? gate_mine : spk_to_float<T>(gate[e])));
+    }
+    if (STAGED && threadIdx.x == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");  // the copy has read shared memory
 }
 
 // ---- prefill -----------------------------------------------------------------------------------------------------------
@@ -456,19 +468,16 @@ int check(const spk_delta_args* a) {
     return SPK_OK;
 }
 
-template <typename T, int W, int KEEP, int NT>
+template <typename T, int W, bool STAGED, int NT>
 int launch_step_form(const spk_delta_args& a, cudaStream_t s) {
     const int cols = a.vdim / W, slices = cols < NT ? NT / cols : 1;
-    const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim);
+    const size_t bytes = sizeof(float) * (3 * static_cast<size_t>(a.dim) + a.vdim + static_cast<size_t>(slices) * a.vdim + (STAGED ? static_cast<size_t>(a.dim) * a.vdim : 0));
     if (bytes > 200 * 1024) return SPK_ERR_TOO_LARGE;
     if (bytes > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, KEEP, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+        const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, W, STAGED, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
         if (e != cudaSuccess) return spk_set_cuda_error(e);
     }
-    // large states: a CTA has the next one's on its way into L2 while it computes
-    const int64_t state = static_cast<int64_t>(a.dim) * a.vdim * 4;
-    const int prefetch = state >= 32 * 1024 && state % 16 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0 ? 2 * 148 : 0;
-    delta_step_kernel<T, W, KEEP, NT><<<dim3(a.heads, static_cast<unsigned>(a.n)), NT, bytes, s>>>(a, prefetch);
+    delta_step_kernel<T, W, STAGED, NT><<<dim3(a.heads, static_cast<unsigned>(a.n)), NT, bytes, s>>>(a);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -476,14 +485,10 @@ int launch_step_form(const spk_delta_args& a, cudaStream_t s) {
 template <typename T>
 int launch_step(const spk_delta_args& a, cudaStream_t s) {
     const bool vec = a.vdim % 4 == 0 && reinterpret_cast<uintptr_t>(a.state) % 16 == 0;
-    const int cols = vec ? a.vdim / 4 : a.vdim;
-    auto share = [&](int threads) {  // state rows per thread
-        const int slices = cols < threads ? threads / cols : 1;
-        return cols <= threads ? (a.dim + slices - 1) / slices : 1 << 30;
-    };
-    if (!vec) return share(256) <= 16 ? launch_step_form<T, 1, 16, 256>(a, s) : launch_step_form<T, 1, 0, 256>(a, s);
-    if (share(128) <= 8) return launch_step_form<T, 4, 8, 128>(a, s);
-    return share(256) <= 16 ? launch_step_form<T, 4, 16, 256>(a, s) : launch_step_form<T, 4, 0, 256>(a, s);
+    const int64_t state = static_cast<int64_t>(a.dim) * a.vdim * 4;
+    if (!vec) return launch_step_form<T, 1, false, 256>(a, s);
+    if (state <= 20 * 1024) return launch_step_form<T, 4, true, 128>(a, s);
+    return state <= 100 * 1024 ? launch_step_form<T, 4, true, 256>(a, s) : launch_step_form<T, 4, false, 256>(a, s);
 }
 
 template <typename T>

@@ -111,46 +111,42 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     const int len = ch.y, dim = a.dim, vdim = a.vdim;
     const SpkDeltaShape sh = spk_delta_shape(a);
     const float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
-    // work items in an order that gives every warp one kind: k channels, q channels, v columns, decays
-    for (int i = threadIdx.x; i < 3 * DP + vp; i += kThreads) {
-        if (i < 2 * DP) {
-            const bool is_k = i < DP;
-            const int d = is_k ? i : i - DP;
-            float* dst = (is_k ? k : q) + d;
-            if (d < dim) {
-                conv_channel<TAPS>(a, po, t0, len, is_k ? a.k : a.q, static_cast<int64_t>(grp) * dim + d, ring, sh.channels, (is_k ? sh.qk : 0) + grp * dim + d,
-                                   is_k ? a.conv_k : a.conv_q, dst, DP);
-            } else {
+    // decays, spread over all threads; then a channel of k, q or v per thread and turn
+    {
+        const float rate = expf(a.a_log[h]);
 #pragma unroll
-                for (int t = 0; t < C; ++t) dst[t * DP] = 0.0f;
-            }
-        } else if (i < 3 * DP) {
-            const int d = i - 2 * DP;
-            float run = 1.0f, x[C];
+        for (int i = threadIdx.x; i < C * DP; i += kThreads) {
+            const int t = i / DP, d = i % DP;
             const int64_t c = static_cast<int64_t>(h) * dim + d;
-#pragma unroll
-            for (int t = 0; t < C; ++t) x[t] = d < dim && t < len ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.a)[(t0 + t) * a.ld2 + c]) : 0.0f;
-            const float bias = d < dim ? a.dt_bias[c] : 0.0f, rate = expf(a.a_log[h]);
-#pragma unroll
-            for (int t = 0; t < C; ++t) {
-                const float dec = d < dim && t < len ? expf(spk_log_decay(x[t] + bias, rate)) : 1.0f;
-                run *= dec;
-                g[t * DP + d] = dec;
-                G[t * DP + d] = run;
-            }
+            const bool in = d < dim && t < len;
+            const float x = in ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.a)[(t0 + t) * a.ld2 + c]) + a.dt_bias[c] : 0.0f;
+            g[i] = in ? expf(spk_log_decay(x, rate)) : 1.0f;
+        }
+    }
+    for (int i = threadIdx.x; i < 2 * DP + vp; i += kThreads) {
+        const int kind = i < DP ? 0 : i < 2 * DP ? 1 : 2;  // k, q, v: uniform over a warp
+        const int c = i - kind * DP, width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : DP;
+        float* dst = (kind == 0 ? k : kind == 1 ? q : v) + c;
+        if (c < width) {
+            const int head = kind == 2 ? h : grp;
+            conv_channel<TAPS>(a, po, t0, len, kind == 0 ? a.k : kind == 1 ? a.q : a.v, static_cast<int64_t>(head) * width + c, ring, sh.channels,
+                               (kind == 0 ? sh.qk : kind == 1 ? 0 : 2 * sh.qk) + head * width + c, kind == 0 ? a.conv_k : kind == 1 ? a.conv_q : a.conv_v, dst, stride);
         } else {
-            const int e = i - 3 * DP;
-            if (e < vdim) {
-                conv_channel<TAPS>(a, po, t0, len, a.v, static_cast<int64_t>(h) * vdim + e, ring, sh.channels, 2 * sh.qk + h * vdim + e, a.conv_v, v + e, vp);
-            } else {
 #pragma unroll
-                for (int t = 0; t < C; ++t) v[t * vp + e] = 0.0f;
-            }
+            for (int t = 0; t < C; ++t) dst[t * stride] = 0.0f;
         }
     }
     if (threadIdx.x < C)
         beta[threadIdx.x] = static_cast<int>(threadIdx.x) < len ? spk_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(a.b)[(t0 + threadIdx.x) * a.ld + h])) : 0.0f;
     __syncthreads();
+    if (threadIdx.x < DP) {
+        float run = 1.0f;
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            run *= g[t * DP + threadIdx.x];
+            G[t * DP + threadIdx.x] = run;
+        }
+    }
     // norms: two tokens per warp
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -229,52 +225,64 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
         *reinterpret_cast<uint32_t*>(image + I::kBh + (t * I::SB + s) * 2) = hi;
         *reinterpret_cast<uint32_t*>(image + I::kBl + (t * I::SB + s) * 2) = lo;
     }
-    // one column per thread: forward substitution, then the operands
-    for (int i = threadIdx.x; i < DP + vp; i += kThreads) {
-        const bool is_w = i < DP;  // uniform over a warp
-        const int e = i - DP;
-        float w[C];
+    // one column of W, U0, q G or k G_16 / G per thread and turn
+    const int cols = DP + vp;
+    // lanes trade tokens in pairs, so that a store carries two channels
+    const bool odd = lane & 1;
+    auto put = [&](int t, int d, float x0, float x1, int hi_at, int lo_at) {  // column d's values at tokens t and t + 1
+        const float got = __shfl_xor_sync(~0u, odd ? x0 : x1, 1);
+        uint32_t hi, lo;
+        split_bf16(odd ? got : x0, odd ? x1 : got, hi, lo);
+        const int at = ((t + (odd ? 1 : 0)) * I::SD + (d & ~1)) * 2;
+        *reinterpret_cast<uint32_t*>(image + hi_at + at) = hi;
+        *reinterpret_cast<uint32_t*>(image + lo_at + at) = lo;
+    };
+    const int cols32 = (cols + 31) & ~31;
+    for (int i = threadIdx.x; i < cols32 + 2 * DP; i += kThreads) {
+        if (i < cols32) {  // forward substitution
+            const bool is_w = i < DP;  // uniform over a warp
+            const int e = i - DP;
+            if (!is_w && e >= vp) continue;
+            float w[C];
 #pragma unroll
-        for (int t = 0; t < C; ++t) {
-            float x = is_w ? k[t * DP + i] * ki[t] * G[t * DP + i] : v[t * vp + e];
+            for (int t = 0; t < C; ++t) {
+                float x = is_w ? k[t * DP + i] * ki[t] * G[t * DP + i] : v[t * vp + e];
 #pragma unroll
-            for (int s4 = 0; s4 < t; s4 += 4) {
-                const float4 f = *reinterpret_cast<const float4*>(&A[t][s4]);
-                x = fmaf(-f.x, w[s4], x);
-                if (s4 + 1 < t) x = fmaf(-f.y, w[s4 + 1], x);
-                if (s4 + 2 < t) x = fmaf(-f.z, w[s4 + 2], x);
-                if (s4 + 3 < t) x = fmaf(-f.w, w[s4 + 3], x);
+                for (int s4 = 0; s4 < t; s4 += 4) {
+                    const float4 f = *reinterpret_cast<const float4*>(&A[t][s4]);
+                    x = fmaf(-f.x, w[s4], x);
+                    if (s4 + 1 < t) x = fmaf(-f.y, w[s4 + 1], x);
+                    if (s4 + 2 < t) x = fmaf(-f.z, w[s4 + 2], x);
+                    if (s4 + 3 < t) x = fmaf(-f.w, w[s4 + 3], x);
+                }
+                w[t] = beta[t] * x;
             }
-            w[t] = beta[t] * x;
-        }
-        if (!is_w) {
-            float* u = reinterpret_cast<float*>(image + I::kU) + e * I::SU;
+            if (is_w) {
 #pragma unroll
-            for (int t = 0; t < C; t += 2) *reinterpret_cast<float2*>(u + t) = make_float2(w[t], w[t + 1]);
-            continue;
-        }
-        // lanes trade tokens in pairs, so that a store carries two channels
-        const bool odd = lane & 1;
-        auto put = [&](int t, float x0, float x1, int hi_at, int lo_at) {  // this column's values at tokens t and t + 1
-            const float got = __shfl_xor_sync(~0u, odd ? x0 : x1, 1);
-            uint32_t hi, lo;
-            split_bf16(odd ? got : x0, odd ? x1 : got, hi, lo);
-            const int at = ((t + (odd ? 1 : 0)) * I::SD + (i & ~1)) * 2;
-            *reinterpret_cast<uint32_t*>(image + hi_at + at) = hi;
-            *reinterpret_cast<uint32_t*>(image + lo_at + at) = lo;
-        };
-        float rest = 1.0f;  // product of the decays behind the token
+                for (int t = 0; t < C; t += 2) put(t, i, w[t], w[t + 1], I::kWh, I::kWl);
+            } else {
+                float* u = reinterpret_cast<float*>(image + I::kU) + e * I::SU;
 #pragma unroll
-        for (int t = C - 2; t >= 0; t -= 2) {
-            const float y1 = k[(t + 1) * DP + i] * ki[t + 1] * rest;
-            rest *= g[(t + 1) * DP + i];
-            const float y0 = k[t * DP + i] * ki[t] * rest;
-            rest *= g[t * DP + i];
-            put(t, y0, y1, I::kKh, I::kKl);
-            put(t, w[t], w[t + 1], I::kWh, I::kWl);
-            put(t, q[t * DP + i] * qi[t] * G[t * DP + i], q[(t + 1) * DP + i] * qi[t + 1] * G[(t + 1) * DP + i], I::kQh, I::kQl);
+                for (int t = 0; t < C; t += 2) *reinterpret_cast<float2*>(u + t) = make_float2(w[t], w[t + 1]);
+            }
+        } else if (i < cols32 + DP) {
+            const int d = i - cols32;
+#pragma unroll
+            for (int t = 0; t < C; t += 2)
+                put(t, d, q[t * DP + d] * qi[t] * G[t * DP + d], q[(t + 1) * DP + d] * qi[t + 1] * G[(t + 1) * DP + d], I::kQh, I::kQl);
+            reinterpret_cast<float*>(image + I::kE)[d] = G[(C - 1) * DP + d];
+        } else {
+            const int d = i - cols32 - DP;
+            float rest = 1.0f;  // product of the decays behind the token
+#pragma unroll
+            for (int t = C - 2; t >= 0; t -= 2) {
+                const float y1 = k[(t + 1) * DP + d] * ki[t + 1] * rest;
+                rest *= g[(t + 1) * DP + d];
+                const float y0 = k[t * DP + d] * ki[t] * rest;
+                rest *= g[t * DP + d];
+                put(t, d, y0, y1, I::kKh, I::kKl);
+            }
         }
-        reinterpret_cast<float*>(image + I::kE)[i] = G[(C - 1) * DP + i];
     }
 }
 
@@ -283,7 +291,7 @@ template <int DP, int NW>
 struct Chain {
     static constexpr int kHead = Image<DP>::kU, kU = NW * 16 * Image<DP>::SU * 4;
     static constexpr int kStage = (kHead + kU + 127) & ~127;
-    static constexpr int NS = 3;
+    static constexpr int NS = DP == 64 ? 6 : NW >= 4 ? 3 : 5;
     static constexpr int kBytes = NS * kStage + 128 + 2 * NS * 8;
 };
 

@@ -63,14 +63,23 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
     const int width = part == 0 ? a.q_rank : a.rank;
     const T* src = part == 0 ? static_cast<const T*>(a.cq) + t * a.ld : static_cast<const T*>(a.kv) + t * a.ld;
     const float* w = part == 0 ? a.w_q : a.w_kv;
+    constexpr int KEEP = VEC ? 12 : 1;  // groups of four a lane keeps between the two passes
+    float4 keep[KEEP];
     float ss = 0.0f;
-    for (int c = 4 * lane; c < width; c += 128) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        keep[i] = spk_load4<T, VEC>(src + c, width - c);
+    }
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) ss += (keep[i].x * keep[i].x + keep[i].y * keep[i].y) + (keep[i].z * keep[i].z + keep[i].w * keep[i].w);
+    for (int c = 4 * (lane + 32 * KEEP); c < width; c += 128) {
         const float4 x = spk_load4<T, VEC>(src + c, width - c);
         ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
     }
     const float inv = 1.0f / sqrtf(spk_warp_sum(ss) / static_cast<float>(width) + a.eps);
-    for (int c = 4 * lane; c < width; c += 128) {
-        const float4 x = spk_load4<T, VEC>(src + c, width - c), m = spk_load4<float, VEC>(w + c, width - c);
+    auto put = [&](int c, const float4& x) {
+        const float4 m = spk_load4<float, VEC>(w + c, width - c);
         const float4 y = make_float4(x.x * inv * m.x, x.y * inv * m.y, x.z * inv * m.z, x.w * inv * m.w);
         if (part == 0) {
             spk_store4<T, VEC>(static_cast<T*>(a.cq_out) + t * width + c, y, width - c);
@@ -82,7 +91,11 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
             for (int k = 0; k < 4; ++k)
                 if (c + k < width) page[spk_latent_channel(lay, r, c + k)] = spk_from_float<T>(e[k]);
         }
-    }
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (4 * (lane + 32 * i) < width) put(4 * (lane + 32 * i), keep[i]);
+    for (int c = 4 * (lane + 32 * KEEP); c < width; c += 128) put(c, spk_load4<T, VEC>(src + c, width - c));
 }
 
 // ---- queries ---------------------------------------------------------------------------------------------------------
@@ -310,28 +323,36 @@ latent_attn_simt_kernel(const spk_latent_attn_args a) {
 constexpr int kOutRows = 16;
 
 // Weight of every (token, key range) of a head: exp(max_s - M) / (sum of denominators and exp(sink), relative to M); 0 where a range has
-// no keys.  wts [kOutRows][splits]; a warp per two tokens.
+// no keys.  wts [kOutRows][splits]; half a warp per token, up to 64 ranges.
 __device__ __forceinline__ void range_weights(const spk_latent_out_args& a, int h, int64_t t0, int rows, float* wts) {
-    const int lane = threadIdx.x & 31;
-    for (int r = threadIdx.x >> 5; r < kOutRows; r += kWarps) {
-        const int64_t t = t0 + r;
-        const int64_t len = r < rows ? spk_visible_keys(a, t, a.seq_lens == nullptr) : 0;
-        const int per = spk_split_keys(static_cast<int>(len), a.splits);
-        const int valid = static_cast<int>((len + per - 1) / per);
-        const float sink = a.sink[h];
-        float m = sink;
-        for (int s = lane; s < valid; s += 32) m = fmaxf(m, a.stats[2 * ((t * a.splits + s) * a.heads + h)]);
+    static_assert(2 * kWarps == kOutRows, "half a warp per token");
+    const int r = threadIdx.x >> 4, l = threadIdx.x & 15;
+    const int64_t t = t0 + r;
+    const float sink = a.sink[h];
+    const int64_t len = r < rows ? spk_visible_keys(a, t, a.seq_lens == nullptr) : 0;
+    const int per = spk_split_keys(static_cast<int>(len), a.splits);
+    const int valid = static_cast<int>((len + per - 1) / per);
+    float2 st[4];
+    float m = sink, den = 0.0f;
 #pragma unroll
-        for (int o = 16; o >= 1; o >>= 1) m = fmaxf(m, __shfl_xor_sync(~0u, m, o));
-        float den = 0.0f;
-        for (int s = lane; s < valid; s += 32) {
-            const float2 st = *reinterpret_cast<const float2*>(a.stats + 2 * ((t * a.splits + s) * a.heads + h));
-            den = fmaf(st.y, expf(st.x - m), den);
-        }
-        den = spk_warp_sum(den) + expf(sink - m);
-        for (int s = lane; s < a.splits; s += 32)
-            wts[r * a.splits + s] = s < valid ? expf(a.stats[2 * ((t * a.splits + s) * a.heads + h)] - m) / den : 0.0f;
+    for (int i = 0; i < 4; ++i) {
+        const int s = l + 16 * i;
+        st[i] = s < valid ? *reinterpret_cast<const float2*>(a.stats + 2 * ((t * a.splits + s) * a.heads + h)) : make_float2(-INFINITY, 0.0f);
+        m = fmaxf(m, st[i].x);
     }
+#pragma unroll
+    for (int o = 8; o >= 1; o >>= 1) m = fmaxf(m, __shfl_xor_sync(~0u, m, o));
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        st[i].x = expf(st[i].x - m);
+        den = fmaf(st[i].y, st[i].x, den);
+    }
+#pragma unroll
+    for (int o = 8; o >= 1; o >>= 1) den += __shfl_xor_sync(~0u, den, o);
+    den += expf(sink - m);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+        if (l + 16 * i < a.splits) wts[r * a.splits + l + 16 * i] = st[i].x / den;
 }
 
 // 32-bit, CTA = (head, 16 tokens): any sizes.
@@ -597,7 +618,7 @@ extern "C" int spk_latent_attn_splits(int dtype, int rank, int rot_dim, int rank
 extern "C" int spk_latent_attn(const spk_latent_attn_args* a, void* stream) {
     SpkRange nvtx_range("spk_latent_attn");
     if (a == nullptr) return SPK_ERR_NULL_POINTER;
-    if (a->n < 0 || a->n > 0x7fffffffLL || a->heads < 1 || a->splits < 1 || a->splits > 65535 || a->num_blocks < 1 || a->max_blocks < 1 ||
+    if (a->n < 0 || a->n > 0x7fffffffLL || a->heads < 1 || a->splits < 1 || a->splits > 64 || a->num_blocks < 1 || a->max_blocks < 1 ||
         bad_row(a->rank, a->rot_dim, a->rank_pad, a->rot_pad, a->tiled, a->block_size))
         return SPK_ERR_BAD_SHAPE;
     if (bad_dtype(a->dtype)) return SPK_ERR_BAD_DTYPE;
@@ -617,7 +638,7 @@ extern "C" int spk_latent_attn(const spk_latent_attn_args* a, void* stream) {
 extern "C" int spk_latent_out(const spk_latent_out_args* a, void* stream) {
     SpkRange nvtx_range("spk_latent_out");
     if (a == nullptr) return SPK_ERR_NULL_POINTER;
-    if (a->n < 0 || a->heads < 1 || a->vdim < 1 || a->rank < 1 || a->splits < 1) return SPK_ERR_BAD_SHAPE;
+    if (a->n < 0 || a->heads < 1 || a->vdim < 1 || a->rank < 1 || a->splits < 1 || a->splits > 64) return SPK_ERR_BAD_SHAPE;
     if (bad_dtype(a->dtype)) return SPK_ERR_BAD_DTYPE;
     if (a->n == 0) return SPK_OK;
     if (a->partials == nullptr || a->stats == nullptr || a->sink == nullptr || a->w_uv == nullptr || a->gate == nullptr || a->out == nullptr ||

@@ -80,7 +80,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     uint8_t* q_s = base + NS * Sh::kStage;
     uint8_t* p_s = q_s + CT * kQTile;
     Bars* bars = reinterpret_cast<Bars*>(p_s + 2 * kPTile);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = __shfl_sync(~0u, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         for (int i = 0; i < NS; ++i) {
             mbar_init(smem_u32(&bars->full[i]), 1);
@@ -101,7 +101,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem = bars->tmem;
+    const uint32_t tmem = __shfl_sync(~0u, bars->tmem, 0);
     volatile int* abort = &bars->abort;
 
     if (warp == 4) {  // ---- cache rows
@@ -140,56 +140,62 @@ latent_decode_kernel(const spk_latent_attn_args a) {
         if (*abort != 0)  // copies in flight land before the CTA's shared memory is given up
             for (int s = issued > NS ? issued - NS : 0; s < issued; ++s) mbar_wait(smem_u32(&bars->full[s % NS]), (s / NS) & 1);
     } else if (warp == 5) {  // ---- scores
-        if (lane == 0) {
-            constexpr uint32_t idesc = idesc_bf16(kKeys, kHeads, false, false);
-            bool ok = mbar_wait(smem_u32(&bars->q_full), 0, abort);
-            for (int s = 0; ok && s < tiles; ++s) {
-                const int st = s % NS;
-                // the buffer's previous scores have been read when that step's weights are complete
-                ok = (s < 2 || mbar_wait(smem_u32(&bars->p_full[s & 1]), ((s >> 1) - 1) & 1, abort)) &&
-                     mbar_wait(smem_u32(&bars->full[st]), (s / NS) & 1, abort);
-                if (!ok) break;
-                tc_fence_after();
-                const uint32_t ka = smem_u32(base + st * Sh::kStage), qa = smem_u32(q_s);
+        constexpr uint32_t idesc = idesc_bf16(kKeys, kHeads, false, false);
+        const uint32_t who = elect_one();
+        // descriptors of one operand differ in the start address alone
+        const uint64_t kd0 = desc_sw128(smem_u32(base), 16, Sh::kGroup), qd = desc_sw128(smem_u32(q_s), 16, 1024);
+        bool ok = __all_sync(~0u, mbar_wait(smem_u32(&bars->q_full), 0, abort));
+        for (int s = 0; ok && s < tiles; ++s) {
+            const int st = s % NS;
+            // the buffer's previous scores have been read when that step's weights are complete
+            ok = __all_sync(~0u, (s < 2 || mbar_wait(smem_u32(&bars->p_full[s & 1]), ((s >> 1) - 1) & 1, abort)) &&
+                                     mbar_wait(smem_u32(&bars->full[st]), (s / NS) & 1, abort));
+            if (!ok) break;
+            tc_fence_after();
+            const uint64_t kd = kd0 + (st * Sh::kStage >> 4);
 #pragma unroll
-                for (int k = 0; k < CT * 4; ++k)
-                    mma_ss(tmem + (s & 1) * kHeads, desc_sw128(ka + (k >> 2) * kAtom + (k & 3) * 32, 16, Sh::kGroup),
-                           desc_sw128(qa + (k >> 2) * kQTile + (k & 3) * 32, 16, 1024), idesc, k > 0);
-                mma_commit(smem_u32(&bars->s_full[s & 1]));
-            }
-            mma_commit(smem_u32(&bars->s_done));
-            mbar_wait(smem_u32(&bars->s_done), 0);  // nothing this thread issued is in the tensor pipe any more
+            for (int k = 0; k < CT * 4; ++k)
+                mma_ss_by(who, tmem + (s & 1) * kHeads, kd + (((k >> 2) * kAtom + (k & 3) * 32) >> 4), qd + (((k >> 2) * kQTile + (k & 3) * 32) >> 4), idesc, k > 0);
+            if (who) mma_commit(smem_u32(&bars->s_full[s & 1]));
+            __syncwarp();
         }
+        if (who) mma_commit(smem_u32(&bars->s_done));
+        mbar_wait(smem_u32(&bars->s_done), 0);  // nothing this warp issued is in the tensor pipe any more
     } else if (warp == 6) {  // ---- weighted sums
-        if (lane == 0) {
-            constexpr uint32_t idesc = idesc_bf16(128, 2 * kHeads, true, true);
-            for (int s = 0; s < tiles; ++s) {
-                const int st = s % NS;
-                if (!mbar_wait(smem_u32(&bars->p_full[s & 1]), (s >> 1) & 1, abort)) break;
-                tc_fence_after();
-                const uint32_t va = smem_u32(base + st * Sh::kStage), pa = smem_u32(p_s + (s & 1) * kPTile);
-                const int steps = (min(kKeys, hi - lo - s * kKeys) + 15) >> 4;
-                for (int k = 0; k < steps; ++k) {
-                    const uint64_t pd = desc_sw128(pa + k * 2048, 16, 1024);
+        constexpr uint32_t idesc = idesc_bf16(128, 2 * kHeads, true, true);
+        const uint32_t who = elect_one();
+        const uint64_t vd0 = desc_sw128(smem_u32(base), kAtom, Sh::kGroup), pd0 = desc_sw128(smem_u32(p_s), 16, 1024);
+        for (int s = 0; s < tiles; ++s) {
+            const int st = s % NS;
+            if (!__all_sync(~0u, mbar_wait(smem_u32(&bars->p_full[s & 1]), (s >> 1) & 1, abort))) break;
+            tc_fence_after();
+            const uint64_t vd = vd0 + (st * Sh::kStage >> 4), pd = pd0 + ((s & 1) * kPTile >> 4);
+            const int steps = (min(kKeys, hi - lo - s * kKeys) + 15) >> 4;
 #pragma unroll
-                    for (int b = 0; b < MB; ++b)
-                        mma_ss(tmem + kTmemO + b * 2 * kHeads, desc_sw128(va + b * 2 * kAtom + k * 2 * Sh::kGroup, kAtom, Sh::kGroup), pd, idesc, s > 0 || k > 0);
-                }
+            for (int k = 0; k < kKeys / 16; ++k) {
+                if (k >= steps) break;
+#pragma unroll
+                for (int b = 0; b < MB; ++b)
+                    mma_ss_by(who, tmem + kTmemO + b * 2 * kHeads, vd + ((b * 2 * kAtom + k * 2 * Sh::kGroup) >> 4), pd + (k * 2048 >> 4), idesc, s > 0 || k > 0);
+            }
+            if (who) {
                 mma_commit(smem_u32(&bars->free[st]));
                 mma_commit(smem_u32(&bars->p_free[s & 1]));
             }
-            mma_commit(smem_u32(&bars->o_full));
-            mbar_wait(smem_u32(&bars->o_full), 0);
+            __syncwarp();
         }
+        if (who) mma_commit(smem_u32(&bars->o_full));
+        mbar_wait(smem_u32(&bars->o_full), 0);
     } else {  // ---- scores to weights
         // query rows into the operand layout, zeros beyond the heads
         const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + (t * a.heads + h0) * (CT * 64);
+#pragma unroll 6
         for (int i = threadIdx.x; i < kHeads * CT * 8; i += kSoftThreads) {
             const int r = i / (CT * 8), c = i % (CT * 8);
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (r < nh) v = *reinterpret_cast<const uint4*>(q + r * (CT * 64) + c * 8);
-            *reinterpret_cast<uint4*>(q_s + (c >> 3) * kQTile + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+            cp_async16(smem_u32(q_s) + (c >> 3) * kQTile + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (r < nh ? r * (CT * 64) + c * 8 : 0), r < nh);
         }
+        cp_async_commit();
+        cp_async_wait_all();
         fence_async_shared();
         mbar_arrive(smem_u32(&bars->q_full));
         const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
