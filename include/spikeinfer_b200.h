@@ -749,6 +749,8 @@ typedef struct spk_latent_attn_args {
     int32_t heads, rank, rot_dim, rank_pad, rot_pad, tiled;
     int32_t block_size;
     int32_t dtype;
+    int32_t overlap;            /* tensor form: may be placed while the launch ahead (spk_latent_query) still runs; the caller vouches that
+                                 * tables, lengths and rows of the portion's other tokens were complete before that began */
     float scale;
     uint32_t* status;
 } spk_latent_attn_args;
@@ -774,7 +776,7 @@ typedef struct spk_latent_out_args {
     int64_t n;
     int32_t splits, heads, vdim, rank;
     int32_t dtype;
-    int32_t _pad;
+    int32_t overlap;            /* bf16: directly follows spk_latent_attn and may be placed while that still runs */
     uint32_t* status;
 } spk_latent_out_args;
 int spk_latent_out(const spk_latent_out_args* args, void* stream);

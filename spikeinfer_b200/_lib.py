@@ -169,14 +169,14 @@ class LatentAttnArgs(Structure):
     """Mirror of ``spk_latent_attn_args``."""
 
     _fields_ = _fields("p q pool tables seq_lens active token_rows positions partials stats; l table_stride table_rows max_blocks n num_blocks; "
-                       "i splits heads rank rot_dim rank_pad rot_pad tiled block_size dtype; f scale; p status")
+                       "i splits heads rank rot_dim rank_pad rot_pad tiled block_size dtype overlap; f scale; p status")
 
 
 class LatentOutArgs(Structure):
     """Mirror of ``spk_latent_out_args``."""
 
     _fields_ = _fields("p partials stats sink w_uv gate out seq_lens active positions; l gate_stride out_stride n; "
-                       "i splits heads vdim rank dtype _pad; p status")
+                       "i splits heads vdim rank dtype overlap; p status")
 
 
 class LatentGatherArgs(Structure):

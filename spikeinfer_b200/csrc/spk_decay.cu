@@ -412,7 +412,7 @@ int launch_step(const spk_decay_attn_args& a, cudaStream_t s) {
     const dim3 grid(a.heads, static_cast<unsigned>(a.n));
     const void* fn = vec ? reinterpret_cast<const void*>(decay_step_kernel<T, 4>) : reinterpret_cast<const void*>(decay_step_kernel<T, 1>);
     if (const int rc = smem_attr(fn, bytes)) return rc;
-    return spk_launch(vec ? decay_step_kernel<T, 4> : decay_step_kernel<T, 1>, grid, kThreads, bytes, s, a, a.overlap != 0);
+    return spk_launch(vec ? decay_step_kernel<T, 4> : decay_step_kernel<T, 1>, grid, kThreads, bytes, s, a.overlap != 0, a);
 }
 
 int launch_scan(const spk_decay_attn_args& a, cudaStream_t s) {

@@ -136,7 +136,7 @@ delta_step_kernel(const spk_delta_args a) {
     spk_block_sum<3>(sums, part);  // its barriers also publish q, k, v and the decays
     const float qi = 1.0f / (sqrtf(sums[0] + 1e-6f) * sqrtf(static_cast<float>(dim))), ki = 1.0f / sqrtf(sums[1] + 1e-6f);
     const float beta = spk_sigmoid(raw_beta);
-    if (STAGED && !mbar_wait(smem_u32(&arrived), 0) && threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_DEVICE_WAIT_EXPIRED);
+    if (STAGED && !mbar_wait(smem_u32(&arrived), 0) && !mbar_wait(smem_u32(&arrived), 0) && threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_DEVICE_WAIT_EXPIRED);
     const float* from = STAGED ? held : S;
     float* to = STAGED ? held : S;
     auto load = [&](float (&x)[W], int d, int c) {
@@ -449,9 +449,8 @@ delta_out_vec_kernel(const spk_delta_args a, const float* __restrict__ outputs) 
     for (int s = L / 2; s >= 1; s >>= 1) ss += __shfl_xor_sync(~0u, ss, s);
     if (!in) return;
     const float inv = 1.0f / sqrtf(ss / static_cast<float>(V) + a.eps);
-    spk_store4<T, true>(static_cast<T*>(a.out) + t * a.out_stride + at,
-                        make_float4(o.x * inv * w.x * spk_sigmoid(g.x), o.y * inv * w.y * spk_sigmoid(g.y), o.z * inv * w.z * spk_sigmoid(g.z),
-                                    o.w * inv * w.w * spk_sigmoid(g.w)), 4);
+    auto gated = [&](float x, float m, float y) { return x * inv * m * (sizeof(T) == 2 ? sigmoid_fast(y) : spk_sigmoid(y)); };
+    spk_store4<T, true>(static_cast<T*>(a.out) + t * a.out_stride + at, make_float4(gated(o.x, w.x, g.x), gated(o.y, w.y, g.y), gated(o.z, w.z, g.z), gated(o.w, w.w, g.w)), 4);
 }
 
 int check(const spk_delta_args* a) {

@@ -111,18 +111,16 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     const int len = ch.y, dim = a.dim, vdim = a.vdim;
     const SpkDeltaShape sh = spk_delta_shape(a);
     const float* ring = a.conv_state + static_cast<int64_t>(po.z) * a.taps * sh.channels;
-    // decays, spread over all threads; then a channel of k, q or v per thread and turn
-    {
-        const float rate = expf(a.a_log[h]);
+    // the decays' raw values are on their way while the convolutions run, a channel of k, q or v per thread and turn
+    constexpr int RAW = C * DP / kThreads;
+    float raw_a[RAW];
 #pragma unroll
-        for (int i = threadIdx.x; i < C * DP; i += kThreads) {
-            const int t = i / DP, d = i % DP;
-            const int64_t c = static_cast<int64_t>(h) * dim + d;
-            const bool in = d < dim && t < len;
-            const float x = in ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.a)[(t0 + t) * a.ld2 + c]) + a.dt_bias[c] : 0.0f;
-            g[i] = in ? expf(spk_log_decay(x, rate)) : 1.0f;
-        }
+    for (int j = 0; j < RAW; ++j) {
+        const int i = threadIdx.x + j * kThreads, t = i / DP, d = i % DP;
+        raw_a[j] = d < dim && t < len ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.a)[(t0 + t) * a.ld2 + static_cast<int64_t>(h) * dim + d]) : 0.0f;
     }
+    const int my_d = threadIdx.x % DP;  // kThreads is a multiple of DP: one channel for all of a thread's values
+    const float bias = my_d < dim ? a.dt_bias[static_cast<int64_t>(h) * dim + my_d] : 0.0f, rate = expf(a.a_log[h]);
     for (int i = threadIdx.x; i < 2 * DP + vp; i += kThreads) {
         const int kind = i < DP ? 0 : i < 2 * DP ? 1 : 2;  // k, q, v: uniform over a warp
         const int c = i - kind * DP, width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : DP;
@@ -135,6 +133,11 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
 #pragma unroll
             for (int t = 0; t < C; ++t) dst[t * stride] = 0.0f;
         }
+    }
+#pragma unroll
+    for (int j = 0; j < RAW; ++j) {
+        const int i = threadIdx.x + j * kThreads;
+        g[i] = my_d < dim && i / DP < len ? expf(spk_log_decay(raw_a[j] + bias, rate)) : 1.0f;
     }
     if (threadIdx.x < C)
         beta[threadIdx.x] = static_cast<int>(threadIdx.x) < len ? spk_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(a.b)[(t0 + threadIdx.x) * a.ld + h])) : 0.0f;
@@ -291,7 +294,7 @@ template <int DP, int NW>
 struct Chain {
     static constexpr int kHead = Image<DP>::kU, kU = NW * 16 * Image<DP>::SU * 4;
     static constexpr int kStage = (kHead + kU + 127) & ~127;
-    static constexpr int NS = DP == 64 ? 6 : NW >= 4 ? 3 : 5;
+    static constexpr int NS = DP == 64 ? 4 : 3;
     static constexpr int kBytes = NS * kStage + 128 + 2 * NS * 8;
 };
 
@@ -496,11 +499,7 @@ int launch(const spk_delta_args& a, float* outputs, cudaStream_t s) {
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, image, vp);
     SPK_CHECK_LAUNCH();
-    // few chains: spread a head's columns over more CTAs
-    const int64_t chains = static_cast<int64_t>(a.heads) * a.n_portions;
-    if (chains * ((vp + 63) / 64) >= 148) return launch_chain<DP, 4>(a, image, vp, outputs, s);
-    if (chains * ((vp + 31) / 32) >= 148) return launch_chain<DP, 2>(a, image, vp, outputs, s);
-    return launch_chain<DP, 1>(a, image, vp, outputs, s);
+    return launch_chain<DP, 4>(a, image, vp, outputs, s);  // a warp per scheduler: the chain is bound by its MMAs
 }
 
 }  // namespace

@@ -114,8 +114,8 @@ __host__ __device__ __forceinline__ int spk_split_keys(int len, int splits) {
 __device__ __forceinline__ void spk_grid_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void spk_grid_release() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
-template <typename Args>
-static inline int spk_launch(void (*fn)(Args), dim3 grid, int threads, size_t bytes, cudaStream_t s, const Args& args, bool overlap) {
+template <typename... Params, typename... Args>
+static inline int spk_launch(void (*fn)(Params...), dim3 grid, int threads, size_t bytes, cudaStream_t s, bool overlap, const Args&... args) {
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute attr = {};
     attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -126,7 +126,7 @@ static inline int spk_launch(void (*fn)(Args), dim3 grid, int threads, size_t by
     cfg.stream = s;
     cfg.attrs = &attr;
     cfg.numAttrs = overlap ? 1 : 0;
-    const cudaError_t e = cudaLaunchKernelEx(&cfg, fn, args);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, fn, args...);
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     spk_count_launch();
     return SPK_OK;

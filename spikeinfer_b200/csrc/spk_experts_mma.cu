@@ -21,7 +21,7 @@ constexpr int kTileW = 128 * 128;  // bytes of a 128-row, 64-column weight tile
 template <int TN>
 struct Shape {
     static constexpr int kStage = 2 * kTileW + TN * 128;
-    static constexpr int NS = TN >= 256 ? 3 : TN >= 128 ? 4 : TN >= 64 ? 5 : 6;
+    static constexpr int NS = TN >= 256 ? 3 : TN >= 128 ? 4 : TN >= 64 ? 5 : 3;  // the narrow form leaves room for a second CTA
     static constexpr int kBytes = NS * kStage + 1024 + 256;
     static constexpr int kColumns = 2 * TN < 32 ? 32 : 2 * TN;
 };
@@ -33,7 +33,7 @@ struct Bars {
 };
 
 template <int TN, bool GATED>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, TN <= 32 ? 2 : 1)
 experts_kernel(const spk_experts_args a, const int blocks, const int ktiles) {
     using Sh = Shape<TN>;
     constexpr int NS = Sh::NS;

@@ -398,38 +398,41 @@ latent_out_kernel(const spk_latent_out_args a) {
     }
 }
 
-// bf16 on the tensor cores: CTA = (head, 16 tokens, 128 value channels), a warp per sixteen channels.  The ranges' sums are put together
-// with all of a thread's loads in flight at once, while the first stages of the value matrix are on their way.
-constexpr int kOutStages = 4;
+// bf16 on the tensor cores: CTA = (head, 16 tokens, 64 value channels); warps 4 (sixteen channels each) x 2 (halves of every 128 latent
+// channels).  The ranges' sums are put together with all of a thread's loads in flight at once; the value matrix comes through a ring whose
+// first stages are on their way before the launch ahead of this one is waited for.
+constexpr int kOutStages = 4, kOutCols = 64, kOutK = 128;
 
 template <bool VEC>
 __global__ void __launch_bounds__(kThreads)
 latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
-    constexpr int K = 64, S = K + 8;
+    constexpr int S = kOutK + 8;
     extern __shared__ __align__(16) uint8_t raw[];
-    const int chunks = (a.rank + K - 1) / K, SO = chunks * K + 8;
-    __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(raw);   // stages of [128][72]
-    __nv_bfloat16* os = ws + kOutStages * kMmaCols * S;           // [16][rank, padded + 8]
+    const int chunks = (a.rank + kOutK - 1) / kOutK, SO = chunks * kOutK + 8;
+    __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(raw);   // stages of [64][136]
+    __nv_bfloat16* os = ws + kOutStages * kOutCols * S;           // [16][rank, padded + 8]
     float* wts = reinterpret_cast<float*>(os + kOutRows * SO);   // [16][splits]
-    const int h = blockIdx.x, e0 = blockIdx.z * kMmaCols;
+    const int h = blockIdx.x, e0 = blockIdx.z * kOutCols;
     const int64_t t0 = static_cast<int64_t>(blockIdx.y) * kOutRows;
     const int rows = static_cast<int>(min(static_cast<int64_t>(kOutRows), a.n - t0));
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w_uv) + (static_cast<int64_t>(h) * a.vdim + e0) * a.rank;
-    const int live = min(kMmaCols, a.vdim - e0), used = (live + 15) & ~15;
+    const int live = min(kOutCols, a.vdim - e0), used = (live + 15) & ~15;
     auto fetch = [&](int c) {
-        if (c < chunks) fetch_tile(ws + (c % kOutStages) * kMmaCols * S, S, w + c * K, a.rank, used, live, K, a.rank - c * K, vec_w);
+        if (c < chunks) fetch_tile(ws + (c % kOutStages) * kOutCols * S, S, w + c * kOutK, a.rank, used, live, kOutK, a.rank - c * kOutK, vec_w);
         cp_async_commit();
     };
     for (int c = 0; c < kOutStages - 1; ++c) fetch(c);
+    spk_grid_wait();
     range_weights(a, h, t0, rows, wts);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
+    const int cw = (warp & 3) * 16, kw = (warp >> 2) * 64;
     {
+        constexpr int U = 8, K = 64;
         const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
         const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank + c4;
         const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
-        constexpr int U = 8;
-        for (int g = 0; g < chunks; g += U) {
+        for (int g = 0; g < 2 * chunks; g += U) {
             float4 y[U];
 #pragma unroll
             for (int u = 0; u < U; ++u) y[u] = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -446,7 +449,7 @@ latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
             }
 #pragma unroll
             for (int u = 0; u < U; ++u)
-                if (g + u < chunks)
+                if (g + u < 2 * chunks)
                     *reinterpret_cast<uint2*>(os + r * SO + (g + u) * K + c4) = make_uint2(pack_bf16(y[u].x, y[u].y), pack_bf16(y[u].z, y[u].w));
         }
     }
@@ -455,31 +458,39 @@ latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
         asm volatile("cp.async.wait_group %0;" ::"n"(kOutStages - 2) : "memory");
         __syncthreads();  // this stage is there, the one before has been read
         fetch(c + kOutStages - 1);
-        if (warp * 16 >= used) continue;
-        const __nv_bfloat16 *ob = os + c * K, *wb = ws + (c % kOutStages) * kMmaCols * S;
+        if (cw >= used) continue;
+        const __nv_bfloat16 *ob = os + c * kOutK + kw, *wb = ws + (c % kOutStages) * kOutCols * S + kw;
 #pragma unroll
-        for (int k = 0; k < K; k += 16) {
+        for (int k = 0; k < 64; k += 16) {
             uint32_t x[4], b[4];
             ldsm4(x, smem_u32(ob + (lane & 15) * SO + k + (lane >> 4) * 8));
-            ldsm4(b, smem_u32(wb + (warp * 16 + (m >> 1) * 8 + mr) * S + k + (m & 1) * 8));
+            ldsm4(b, smem_u32(wb + (cw + (m >> 1) * 8 + mr) * S + k + (m & 1) * 8));
             mma16816(acc[0], x, b[0], b[1]);
             mma16816(acc[1], x, b[2], b[3]);
         }
     }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        const int q = gid + 8 * i;
-        if (q >= rows) continue;
+    __syncthreads();
+    float* half = reinterpret_cast<float*>(ws);  // the second halves' sums [64 channels][17]
+    if (kw > 0 && cw < used) {
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int e = e0 + warp * 16 + n * 8 + tig * 2 + j;
-                if (e >= a.vdim) continue;
-                const int64_t c = static_cast<int64_t>(h) * a.vdim + e;
-                const float g = __bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(t0 + q) * a.gate_stride + c]);
-                static_cast<__nv_bfloat16*>(a.out)[(t0 + q) * a.out_stride + c] = __float2bfloat16_rn(acc[n][2 * i + j] * spk_sigmoid(g));
-            }
+            for (int i = 0; i < 4; ++i) half[(cw + n * 8 + tig * 2 + (i & 1)) * 17 + gid + 8 * (i >> 1)] = acc[n][i];
+    }
+    __syncthreads();
+    if (kw > 0 || cw >= used) return;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int q = gid + 8 * (i >> 1);
+        if (q >= rows) continue;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const int e = cw + n * 8 + tig * 2 + (i & 1);
+            if (e >= live) continue;
+            const int64_t c = static_cast<int64_t>(h) * a.vdim + e0 + e;
+            const float g = __bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(t0 + q) * a.gate_stride + c]);
+            static_cast<__nv_bfloat16*>(a.out)[(t0 + q) * a.out_stride + c] = __float2bfloat16_rn((acc[n][i] + half[e * 17 + q]) * sigmoid_fast(g));
+        }
     }
 }
 
@@ -533,14 +544,12 @@ int launch_query_mma(const spk_latent_query_args& a, cudaStream_t s) {
 int launch_out_mma(const spk_latent_out_args& a, cudaStream_t s) {
     const int64_t tiles = (a.n + kOutRows - 1) / kOutRows;
     if (tiles > 65535) return SPK_ERR_TOO_LARGE;
-    const size_t bytes = 2 * (static_cast<size_t>(kOutStages) * kMmaCols * 72 + kOutRows * (((a.rank + 63) / 64) * 64 + 8)) + sizeof(float) * kOutRows * a.splits;
-    const dim3 grid(a.heads, static_cast<unsigned>(tiles), (a.vdim + kMmaCols - 1) / kMmaCols);
+    const size_t bytes = 2 * (static_cast<size_t>(kOutStages) * kOutCols * (kOutK + 8) + kOutRows * ((a.rank + kOutK - 1) / kOutK * kOutK + 8)) + sizeof(float) * kOutRows * a.splits;
+    const dim3 grid(a.heads, static_cast<unsigned>(tiles), (a.vdim + kOutCols - 1) / kOutCols);
     const bool vec = a.rank % 4 == 0 && at16(a.partials), vw = at16(a.w_uv) && a.rank % 8 == 0;
     auto* fn = vec ? latent_out_mma_kernel<true> : latent_out_mma_kernel<false>;
     if (const int rc = with_smem(reinterpret_cast<const void*>(fn), bytes)) return rc;
-    fn<<<grid, kThreads, bytes, s>>>(a, vw);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return spk_launch(fn, grid, kThreads, bytes, s, a.overlap != 0, a, vw);
 }
 
 template <typename T>

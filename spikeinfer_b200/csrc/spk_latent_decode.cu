@@ -68,11 +68,15 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     // uniform over the CTA: nothing has been set up yet
     if (len < 0 || len > a.max_blocks * a.block_size || row < 0 || row >= a.table_rows) {
         if (threadIdx.x == 0) spk_flag(a.status, SPK_STATUS_BAD_SEQ_LEN);
+        spk_grid_wait();
         return;
     }
     const int per = spk_split_keys(static_cast<int>(len), a.splits);
     const int lo = blockIdx.z * per, hi = static_cast<int>(min(static_cast<int64_t>(lo) + per, len));
-    if (lo >= len) return;
+    if (lo >= len) {  // launched to overlap: the launch before this one is complete when this one is
+        spk_grid_wait();
+        return;
+    }
     const int tiles = (hi - lo + kKeys - 1) / kKeys;
 
     extern __shared__ uint8_t raw[];
@@ -103,6 +107,9 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     tc_fence_after();
     const uint32_t tmem = __shfl_sync(~0u, bars->tmem, 0);
     volatile int* abort = &bars->abort;
+    // the rows written and the queries made by the launches ahead are complete from here on; the launch behind may be placed
+    spk_grid_wait();
+    spk_grid_release();
 
     if (warp == 4) {  // ---- cache rows
         const int gran = a.block_size < kKeys ? a.block_size : kKeys;  // rows per copy
@@ -355,9 +362,7 @@ int launch(const spk_latent_attn_args& a, cudaStream_t s) {
     const cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     const dim3 grid(static_cast<unsigned>(a.n), (a.heads + kHeads - 1) / kHeads, a.splits);
-    latent_decode_kernel<CL><<<grid, kThreads, bytes, s>>>(a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return spk_launch(latent_decode_kernel<CL>, grid, kThreads, bytes, s, a.overlap != 0, a);
 }
 
 }  // namespace

@@ -334,15 +334,15 @@ latent_prefill_kernel(const spk_latent_prefill_args a, const __grid_constant__ C
                     uint32_t* w = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
                     for (int k = 0; k < 4; ++k)
-                        w[k] = pack_bf16(__uint_as_float(o[8 * i + 2 * k]) * inv * spk_sigmoid(__uint_as_float(gw[k] << 16)),
-                                         __uint_as_float(o[8 * i + 2 * k + 1]) * inv * spk_sigmoid(__uint_as_float(gw[k] & 0xffff0000u)));
+                        w[k] = pack_bf16(__uint_as_float(o[8 * i + 2 * k]) * inv * sigmoid_fast(__uint_as_float(gw[k] << 16)),
+                                         __uint_as_float(o[8 * i + 2 * k + 1]) * inv * sigmoid_fast(__uint_as_float(gw[k] & 0xffff0000u)));
                     *reinterpret_cast<uint4*>(out + e) = v;
                 }
             } else if (r < nq) {
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
                     const int e = c * 16 + i;
-                    if (e < a.vdim) out[e] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv * spk_sigmoid(__bfloat162float(gate[e])));
+                    if (e < a.vdim) out[e] = __float2bfloat16_rn(__uint_as_float(o[i]) * inv * sigmoid_fast(__bfloat162float(gate[e])));
                 }
             }
             __syncwarp();

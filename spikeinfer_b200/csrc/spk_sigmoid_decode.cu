@@ -206,7 +206,7 @@ int launch(const spk_sigmoid_attn_args& a, cudaStream_t s) {
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     const int rep = a.heads / a.kv_heads;
     const dim3 grid(a.splits, a.kv_heads * ((rep + 15) / 16), static_cast<unsigned>(a.n));
-    return spk_launch(sigmoid_decode_kernel<CK, CV>, grid, kThreads, bytes, s, a, a.overlap != 0);
+    return spk_launch(sigmoid_decode_kernel<CK, CV>, grid, kThreads, bytes, s, a.overlap != 0, a);
 }
 
 }  // namespace

@@ -187,6 +187,8 @@ __device__ __forceinline__ float rcp(float x) {
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// A sigmoid for 16-bit results.
+__device__ __forceinline__ float sigmoid_fast(float x) { return rcp(1.0f + ex2(-1.4426950408889634f * x)); }
 // Two sigmoids, 1 / (1 + 2^u) each, with one reciprocal: r = 1 / (ab), 1/a = r b, 1/b = r a.  The exponents are capped
 // so that the product stays finite (a weight below 2^-60 counts as 2^-60).
 __device__ __forceinline__ void sigmoid2(uint64_t u, float& p0, float& p1) {

@@ -53,11 +53,12 @@ def latent_query(q: torch.Tensor, w_uk: torch.Tensor, pool, rot_table: torch.Ten
 
 def latent_attention(q: torch.Tensor, pool, tables: torch.Tensor, sink: torch.Tensor, w_uv: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, *,
                      vdim: int, scale: float, seq_lens: torch.Tensor | None = None, active: torch.Tensor | None = None,
-                     token_rows: torch.Tensor | None = None, positions: torch.Tensor | None = None, most_keys: int | None = None,
+                     token_rows: torch.Tensor | None = None, positions: torch.Tensor | None = None, most_keys: int | None = None, overlap_previous: bool = False,
                      status: torch.Tensor | None = None) -> torch.Tensor:
     """``out[t, h vdim :] = sigmoid(gate) * W_uv[h] (softmax with sink over the visible cache rows)`` for queries of :func:`latent_query`.
     ``token_rows`` / ``positions``: tokens of prefill portions (token t sees ``positions[t] + 1`` keys of its row); without them the
-    decode form over ``seq_lens`` / ``active``."""
+    decode form over ``seq_lens`` / ``active``.  ``overlap_previous``: this call directly follows :func:`latent_query` and may be placed while
+    that still runs (tables and lengths were complete before it began)."""
     _lib.require_cuda(q, "latent_attention query")
     n, heads, _ = q.shape
     _f32(sink, "sink", heads)
@@ -74,12 +75,13 @@ def latent_attention(q: torch.Tensor, pool, tables: torch.Tensor, sink: torch.Te
         q=q.data_ptr(), pool=pool.data.data_ptr(), tables=tables.data_ptr(), seq_lens=_ptr(seq_lens), active=_ptr(active), token_rows=_ptr(token_rows),
         positions=_ptr(positions), partials=partials.data_ptr(), stats=stats.data_ptr(), table_stride=tables.stride(0), table_rows=tables.shape[0],
         max_blocks=tables.shape[1], n=n, num_blocks=pool.data.shape[0], splits=splits, heads=heads, rank=pool.rank, rot_dim=pool.rot_dim,
-        rank_pad=pool.rank_pad, rot_pad=pool.rot_pad, tiled=int(pool.tiled), block_size=pool.block_size, dtype=code, scale=scale, status=_ptr(status))
+        rank_pad=pool.rank_pad, rot_pad=pool.rot_pad, tiled=int(pool.tiled), block_size=pool.block_size, dtype=code, overlap=int(overlap_previous), scale=scale, status=_ptr(status))
     _call("spk_latent_attn", a, q.device)
     b = _lib.LatentOutArgs(
         partials=partials.data_ptr(), stats=stats.data_ptr(), sink=sink.data_ptr(), w_uv=w_uv.data_ptr(), gate=gate.data_ptr(), out=out.data_ptr(),
         seq_lens=None if prefill else seq_lens.data_ptr(), active=_ptr(active), positions=_ptr(positions), gate_stride=gate.stride(0),
-        out_stride=out.stride(0), n=n, splits=splits, heads=heads, vdim=vdim, rank=pool.rank, dtype=code, status=_ptr(status))
+        out_stride=out.stride(0), n=n, splits=splits, heads=heads, vdim=vdim, rank=pool.rank, dtype=code, overlap=1,
+        status=_ptr(status))
     _call("spk_latent_out", b, q.device)
     return out
 

@@ -179,7 +179,8 @@ class _LatentAttention:
                            token_rows=meta.token_rows, plan=meta.prefill_plan(), heads=c.heads, dim=c.dim, **common)
             return
         ql = latent_query(q, self.w_uk, pool, rot, positions, heads=c.heads, dim=c.dim, status=meta.status)
-        latent_attention(ql, pool, meta.block_tables, self.sink, self.w_uv, gate, out, seq_lens=meta.seq_lens, active=meta.row_active, **common)
+        latent_attention(ql, pool, meta.block_tables, self.sink, self.w_uv, gate, out, seq_lens=meta.seq_lens, active=meta.row_active,
+                         overlap_previous=meta.tables_settled, **common)
 
 
 class _ChannelDelta:
@@ -266,6 +267,9 @@ class GotunexModel:
             layer.route_index = i
         self.router = ExpertRouter([layer.experts for layer in routed], c.vocab) if routed else None
         self._rot: dict[RotaryConfig, torch.Tensor] = {}
+        # the feed-forward reads the same x as the mixer: steps of up to this many tokens run it on a stream of its own beside it
+        self.side_tokens = 1024
+        self._side = torch.cuda.Stream(device=self.device)
 
     def prepare(self, max_positions: int) -> None:
         """Engine hook: positions ``0 .. max_positions - 1`` may be fed (tabulates the rotary factors)."""
@@ -320,13 +324,21 @@ class GotunexModel:
             mixed = L.mixer.out_width
             both = torch.empty((n, L.w_out.shape[1]), dtype=self.dtype, device=self.device)
             added = {}
-            if L.up is not None:
-                gelu_tanh(self._matmul(hand["out2"], L.up), both[:, mixed:])
-            elif L.experts is not None:
-                route = routes[L.route_index]
-                added = dict(pairs=experts_forward(hand["out2"], L.experts, route, meta.status), pair_slots=route.slots, pair_scale=1.0 / L.experts.top)
+            main, beside = torch.cuda.current_stream(self.device), n <= self.side_tokens and L.norm2 is not None
+            if beside:
+                self._side.wait_stream(main)
+            with torch.cuda.stream(self._side if beside else main):
+                if L.up is not None:
+                    gelu_tanh(self._matmul(hand["out2"], L.up), both[:, mixed:])
+                elif L.experts is not None:
+                    route = routes[L.route_index]
+                    added = dict(pairs=experts_forward(hand["out2"], L.experts, route, meta.status), pair_slots=route.slots, pair_scale=1.0 / L.experts.top)
             L.mixer.forward(self, h, both[:, :mixed], positions, caches[i], meta)
+            if beside and L.up is not None:
+                main.wait_stream(self._side)
             delta = self._matmul_f32(both, L.w_out)
+            if beside and L.experts is not None:
+                main.wait_stream(self._side)
             hand = reads(i + 1)
             rms_residual(x=x, delta=delta, **added, **hand, **common)
             if residuals is not None:
