@@ -88,7 +88,7 @@ __device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4
 
 // CTA = (chunk, head).
 template <int DP, int TAPS>
-__global__ void __launch_bounds__(kThreads, 3)
+__global__ void __launch_bounds__(kThreads, 4)
 delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp) {
     using I = Image<DP>;
     constexpr int PL = DP / 32;  // channels per lane
@@ -171,23 +171,25 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     // A and B: warp w walks from tokens w and 15 - w to the chunk's end, fifteen steps in all, and sums 32 products over its lanes
     {
         const int s0 = warp, s1 = C - 1 - warp;
-        float x[PL], part[32];
-        auto load = [&](float (&r)[PL], const float* m, int t) {
+        constexpr int P2 = PL / 2;
+        uint64_t x[P2], y[P2], z[P2];
+        float part[32];
+        auto load = [&](uint64_t (&r)[P2], const float* m, int t) {
             if (PL == 4) {
-                const float4 f = *reinterpret_cast<const float4*>(m + t * DP + 4 * lane);
-                r[0] = f.x; r[1] = f.y; r[2 % PL] = f.z; r[3 % PL] = f.w;
+                const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(m + t * DP + 4 * lane);
+                r[0] = f.x;
+                r[P2 - 1] = f.y;
             } else {
-                const float2 f = *reinterpret_cast<const float2*>(m + t * DP + 2 * lane);
-                r[0] = f.x; r[1] = f.y;
+                r[0] = *reinterpret_cast<const uint64_t*>(m + t * DP + 2 * lane);
             }
         };
-        auto dot = [&](const float (&p)[PL], const float (&r)[PL]) {
-            float s = p[0] * r[0];
-#pragma unroll
-            for (int j = 1; j < PL; ++j) s = fmaf(p[j], r[j], s);
-            return s;
+        auto dot = [&](const uint64_t (&p)[P2], const uint64_t (&r)[P2]) {
+            uint64_t s = f2_mul(p[0], r[0]);
+            if (P2 == 2) s = f2_fma(p[P2 - 1], r[P2 - 1], s);
+            float a0, a1;
+            f2_unpack(s, a0, a1);
+            return a0 + a1;
         };
-        float y[PL], z[PL];
         load(x, k, s1);
         load(y, q, s1);
         part[31] = dot(x, y);
@@ -201,7 +203,7 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
             const int t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
             load(y, g, t);
 #pragma unroll
-            for (int j = 0; j < PL; ++j) x[j] *= y[j];
+            for (int j = 0; j < P2; ++j) x[j] = f2_mul(x[j], y[j]);
             load(y, k, t);
             load(z, q, t);
             part[i] = dot(x, y);
