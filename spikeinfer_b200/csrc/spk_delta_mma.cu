@@ -24,11 +24,11 @@ constexpr int kThreads = 256;
 // A chunk's operands in bytes from the image's start; SD elements per row of W, Q and K.
 template <int DP>
 struct Image {
-    static constexpr int SD = DP + 8, SB = 24, SU = C + 2;
+    static constexpr int SD = DP + 8, SB = 24, SU = 64 + 4;  // of U0, 64 columns at a time
     static constexpr int kRows = C * SD * 2;                                              // bytes of one of the six matrices
     static constexpr int kWh = 0, kWl = kRows, kQh = 2 * kRows, kQl = 3 * kRows, kKh = 4 * kRows, kKl = 5 * kRows;
     static constexpr int kBh = 6 * kRows, kBl = kBh + C * SB * 2, kE = kBl + C * SB * 2;  // B, then G_16
-    static constexpr int kU = kE + DP * 4;                                                // U0^T [vdim padded to 16][SU], 32-bit
+    static constexpr int kU = kE + DP * 4;                                                // U0 [vdim / 64][C][SU], 32-bit
 };
 
 // Lanes L = 0 .. 31 end up with the sum over the warp of v[L].
@@ -86,18 +86,75 @@ __device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4
     }
 }
 
+// A and B by running products of the decays: warp w of eight walks from tokens w and 15 - w to the chunk's end, fifteen steps in all, and
+// sums 32 products over its lanes.
+template <int DP>
+__device__ __noinline__ void pair_products(const float* q, const float* k, const float* g, const float* qi, const float* ki, float (*A)[C], float (*B)[C],
+                                           int warp, int lane) {
+    constexpr int SQ = DP + 8, P2 = DP / 64;  // channel pairs per lane
+    const int s0 = warp, s1 = C - 1 - warp;
+    uint64_t x[P2], y[P2], z[P2];
+    float part[32];
+    auto load = [&](uint64_t (&r)[P2], const float* m, int t) {
+        if (P2 == 2) {
+            const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(m + t * SQ + 4 * lane);
+            r[0] = f.x;
+            r[P2 - 1] = f.y;
+        } else {
+            r[0] = *reinterpret_cast<const uint64_t*>(m + t * SQ + 2 * lane);
+        }
+    };
+    auto dot = [&](const uint64_t (&p)[P2], const uint64_t (&r)[P2]) {
+        uint64_t s = f2_mul(p[0], r[0]);
+        if (P2 == 2) s = f2_fma(p[P2 - 1], r[P2 - 1], s);
+        float a0, a1;
+        f2_unpack(s, a0, a1);
+        return a0 + a1;
+    };
+    load(x, k, s1);
+    load(y, q, s1);
+    part[31] = dot(x, y);
+    load(x, k, s0);
+    load(y, q, s0);
+    part[30] = dot(x, y);
+    const int first = C - 1 - s0;  // steps that start from s0
+#pragma unroll
+    for (int i = 0; i < C - 1; ++i) {
+        if (i == first) load(x, k, s1);
+        const int t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
+        load(y, g, t);
+#pragma unroll
+        for (int j = 0; j < P2; ++j) x[j] = f2_mul(x[j], y[j]);
+        load(y, k, t);
+        load(z, q, t);
+        part[i] = dot(x, y);
+        part[C - 1 + i] = dot(x, z);
+    }
+    const float total = transpose_sum(part);
+    if (lane < 2 * (C - 1)) {
+        const int i = lane < C - 1 ? lane : lane - (C - 1);
+        const int s = i < first ? s0 : s1, t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
+        if (lane < C - 1) A[t][s] = total * ki[t] * ki[s];
+        else B[t][s] = total * qi[t] * ki[s];
+    } else {
+        const int s = lane == 30 ? s0 : s1;
+        B[s][s] = total * qi[s] * ki[s];
+    }
+}
+
 // CTA = (chunk, head).
 template <int DP, int TAPS>
 __global__ void __launch_bounds__(kThreads, 4)
 delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp) {
     using I = Image<DP>;
-    constexpr int PL = DP / 32;  // channels per lane
+    constexpr int SQ = DP + 8;   // row stride: MMA fragments read without bank conflicts
+    constexpr float kSmallest = 1e-30f;
     extern __shared__ __align__(16) float sm[];
-    float* q = sm;               // [C][DP]
-    float* k = q + C * DP;
-    float* g = k + C * DP;       // decays
-    float* G = g + C * DP;       // their products from the chunk's start
-    float* v = G + C * DP;       // [C][vp]
+    float* q = sm;               // [C][SQ]
+    float* k = q + C * SQ;
+    float* g = k + C * SQ;       // decays
+    float* G = g + C * SQ;       // their products from the chunk's start
+    float* v = G + C * SQ;       // [C][vp]
     __shared__ __align__(16) float A[C][C], B[C][C];
     __shared__ float qi[C], ki[C], beta[C];
     const int h = blockIdx.y, grp = h / (a.heads / a.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -123,7 +180,7 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     const float bias = my_d < dim ? a.dt_bias[static_cast<int64_t>(h) * dim + my_d] : 0.0f, rate = expf(a.a_log[h]);
     for (int i = threadIdx.x; i < 2 * DP + vp; i += kThreads) {
         const int kind = i < DP ? 0 : i < 2 * DP ? 1 : 2;  // k, q, v: uniform over a warp
-        const int c = i - kind * DP, width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : DP;
+        const int c = i - kind * DP, width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : SQ;
         float* dst = (kind == 0 ? k : kind == 1 ? q : v) + c;
         if (c < width) {
             const int head = kind == 2 ? h : grp;
@@ -136,18 +193,18 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     }
 #pragma unroll
     for (int j = 0; j < RAW; ++j) {
-        const int i = threadIdx.x + j * kThreads;
-        g[i] = my_d < dim && i / DP < len ? expf(spk_log_decay(raw_a[j] + bias, rate)) : 1.0f;
+        const int t = (threadIdx.x + j * kThreads) / DP;
+        g[t * SQ + my_d] = my_d < dim && t < len ? expf(spk_log_decay(raw_a[j] + bias, rate)) : 1.0f;
     }
     if (threadIdx.x < C)
         beta[threadIdx.x] = static_cast<int>(threadIdx.x) < len ? spk_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(a.b)[(t0 + threadIdx.x) * a.ld + h])) : 0.0f;
     __syncthreads();
+    float run = 1.0f;
     if (threadIdx.x < DP) {
-        float run = 1.0f;
 #pragma unroll
         for (int t = 0; t < C; ++t) {
-            run *= g[t * DP + threadIdx.x];
-            G[t * DP + threadIdx.x] = run;
+            run *= g[t * SQ + threadIdx.x];
+            G[t * SQ + threadIdx.x] = run;
         }
     }
     // norms: two tokens per warp
@@ -156,8 +213,8 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
         const int t = 2 * warp + i;
         float x = 0.0f, y = 0.0f;
 #pragma unroll
-        for (int j = 0; j < PL; ++j) {
-            const float a1 = q[t * DP + lane + 32 * j], b1 = k[t * DP + lane + 32 * j];
+        for (int j = 0; j < DP / 32; ++j) {
+            const float a1 = q[t * SQ + lane + 32 * j], b1 = k[t * SQ + lane + 32 * j];
             x = fmaf(a1, a1, x);
             y = fmaf(b1, b1, y);
         }
@@ -168,70 +225,8 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
             ki[t] = 1.0f / sqrtf(y + 1e-6f);
         }
     }
-    // A and B: warp w walks from tokens w and 15 - w to the chunk's end, fifteen steps in all, and sums 32 products over its lanes
-    {
-        const int s0 = warp, s1 = C - 1 - warp;
-        constexpr int P2 = PL / 2;
-        uint64_t x[P2], y[P2], z[P2];
-        float part[32];
-        auto load = [&](uint64_t (&r)[P2], const float* m, int t) {
-            if (PL == 4) {
-                const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(m + t * DP + 4 * lane);
-                r[0] = f.x;
-                r[P2 - 1] = f.y;
-            } else {
-                r[0] = *reinterpret_cast<const uint64_t*>(m + t * DP + 2 * lane);
-            }
-        };
-        auto dot = [&](const uint64_t (&p)[P2], const uint64_t (&r)[P2]) {
-            uint64_t s = f2_mul(p[0], r[0]);
-            if (P2 == 2) s = f2_fma(p[P2 - 1], r[P2 - 1], s);
-            float a0, a1;
-            f2_unpack(s, a0, a1);
-            return a0 + a1;
-        };
-        load(x, k, s1);
-        load(y, q, s1);
-        part[31] = dot(x, y);
-        load(x, k, s0);
-        load(y, q, s0);
-        part[30] = dot(x, y);
-        const int first = C - 1 - s0;  // steps that start from s0
-#pragma unroll
-        for (int i = 0; i < C - 1; ++i) {
-            if (i == first) load(x, k, s1);
-            const int t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
-            load(y, g, t);
-#pragma unroll
-            for (int j = 0; j < P2; ++j) x[j] = f2_mul(x[j], y[j]);
-            load(y, k, t);
-            load(z, q, t);
-            part[i] = dot(x, y);
-            part[C - 1 + i] = dot(x, z);
-        }
-        const float total = transpose_sum(part);
-        __syncthreads();  // the norms are there
-        const int i = lane < C - 1 ? lane : lane < 2 * (C - 1) ? lane - (C - 1) : lane;
-        if (lane < 2 * (C - 1)) {
-            const int s = i < first ? s0 : s1, t = i < first ? s0 + 1 + i : s1 + 1 + i - first;
-            if (lane < C - 1) A[t][s] = total * ki[t] * ki[s];
-            else B[t][s] = total * qi[t] * ki[s];
-        } else {
-            const int s = lane == 30 ? s0 : s1;
-            B[s][s] = total * qi[s] * ki[s];
-        }
-    }
-    __syncthreads();
+    const bool steep = __syncthreads_or(run < kSmallest);  // a channel all but forgets within the chunk
     uint8_t* image = static_cast<uint8_t*>(a.workspace) + (static_cast<int64_t>(blockIdx.x) * a.heads + h) * image_bytes;
-    if (threadIdx.x < C * C / 2) {
-        const int t = threadIdx.x >> 3, s = (threadIdx.x & 7) * 2;
-        uint32_t hi, lo;
-        split_bf16(s <= t ? B[t][s] : 0.0f, s + 1 <= t ? B[t][s + 1] : 0.0f, hi, lo);
-        *reinterpret_cast<uint32_t*>(image + I::kBh + (t * I::SB + s) * 2) = hi;
-        *reinterpret_cast<uint32_t*>(image + I::kBl + (t * I::SB + s) * 2) = lo;
-    }
-    // one column of W, U0, q G or k G_16 / G per thread and turn
-    const int cols = DP + vp;
     // lanes trade tokens in pairs, so that a store carries two channels
     const bool odd = lane & 1;
     auto put = [&](int t, int d, float x0, float x1, int hi_at, int lo_at) {  // column d's values at tokens t and t + 1
@@ -242,69 +237,116 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
         *reinterpret_cast<uint32_t*>(image + hi_at + at) = hi;
         *reinterpret_cast<uint32_t*>(image + lo_at + at) = lo;
     };
-    const int cols32 = (cols + 31) & ~31;
-    for (int i = threadIdx.x; i < cols32 + 2 * DP; i += kThreads) {
-        if (i < cols32) {  // forward substitution
-            const bool is_w = i < DP;  // uniform over a warp
-            const int e = i - DP;
-            if (!is_w && e >= vp) continue;
-            float w[C];
+    // A and B.  Steep chunks: products of running decays by all warps.  Otherwise A = (k G) (k / G)^T and B = (q G) (k / G)^T on the tensor
+    // cores, a warp each (nothing below 1e-30 is divided by), beside the other warps' operands.
+    if (steep) {
+        pair_products<DP>(q, k, g, qi, ki, A, B, warp, lane);
+    } else if (warp < 2) {
+        const float *left = warp == 0 ? k : q, *li = warp == 0 ? ki : qi;
+        const int gid = lane >> 2, tig = lane & 3;
+        float acc[2][4] = {}, cross[2][4] = {};
+#pragma unroll 2
+        for (int d0 = 0; d0 < DP; d0 += 16) {
+            uint32_t lh[4], ll[4], rh[4], rl[4];
 #pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float x = is_w ? k[t * DP + i] * ki[t] * G[t * DP + i] : v[t * vp + e];
-#pragma unroll
-                for (int s4 = 0; s4 < t; s4 += 4) {
-                    const float4 f = *reinterpret_cast<const float4*>(&A[t][s4]);
-                    x = fmaf(-f.x, w[s4], x);
-                    if (s4 + 1 < t) x = fmaf(-f.y, w[s4 + 1], x);
-                    if (s4 + 2 < t) x = fmaf(-f.z, w[s4 + 2], x);
-                    if (s4 + 3 < t) x = fmaf(-f.w, w[s4 + 3], x);
-                }
-                w[t] = beta[t] * x;
+            for (int i = 0; i < 4; ++i) {  // left rows gid (+ 8), channels + 8; right: tokens gid (+ 8) of k / G
+                const int at = (gid + 8 * (i & 1)) * SQ + d0 + 2 * tig + 8 * (i >> 1);
+                const float2 x = *reinterpret_cast<const float2*>(left + at), y = *reinterpret_cast<const float2*>(k + at), z = *reinterpret_cast<const float2*>(G + at);
+                split_bf16(x.x * z.x, x.y * z.y, lh[i], ll[i]);
+                split_bf16(__fdividef(y.x, z.x), __fdividef(y.y, z.y), rh[i], rl[i]);
             }
-            if (is_w) {
 #pragma unroll
-                for (int t = 0; t < C; t += 2) put(t, i, w[t], w[t + 1], I::kWh, I::kWl);
+            for (int n = 0; n < 2; ++n) {
+                mma16816(acc[n], lh, rh[n], rh[2 + n]);
+                mma16816(cross[n], lh, rl[n], rl[2 + n]);
+                mma16816(cross[n], ll, rh[n], rh[2 + n]);
+            }
+        }
+        float(*M)[C] = warp == 0 ? A : B;
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int t = gid + 8 * (i >> 1), s = n * 8 + tig * 2 + (i & 1);
+                M[t][s] = s <= t ? (acc[n][i] + cross[n][i]) * li[t] * ki[s] : 0.0f;
+            }
+    }
+    {  // a column of q G or k G_16 / G per thread and turn
+        const int skip = steep ? 0 : 64;
+        for (int i = static_cast<int>(threadIdx.x) - skip; i < 2 * DP; i += kThreads - skip) {
+            if (i < 0) break;  // uniform over a warp
+            if (i < DP) {
+#pragma unroll
+                for (int t = 0; t < C; t += 2)
+                    put(t, i, q[t * SQ + i] * qi[t] * G[t * SQ + i], q[(t + 1) * SQ + i] * qi[t + 1] * G[(t + 1) * SQ + i], I::kQh, I::kQl);
+                reinterpret_cast<float*>(image + I::kE)[i] = G[(C - 1) * SQ + i];
             } else {
-                float* u = reinterpret_cast<float*>(image + I::kU) + e * I::SU;
+                const int d = i - DP;
+                float rest = 1.0f;  // product of the decays behind the token
 #pragma unroll
-                for (int t = 0; t < C; t += 2) *reinterpret_cast<float2*>(u + t) = make_float2(w[t], w[t + 1]);
+                for (int t = C - 2; t >= 0; t -= 2) {
+                    const float y1 = k[(t + 1) * SQ + d] * ki[t + 1] * rest;
+                    rest *= g[(t + 1) * SQ + d];
+                    const float y0 = k[t * SQ + d] * ki[t] * rest;
+                    rest *= g[t * SQ + d];
+                    put(t, d, y0, y1, I::kKh, I::kKl);
+                }
             }
-        } else if (i < cols32 + DP) {
-            const int d = i - cols32;
+        }
+    }
+    __syncthreads();
+    if (threadIdx.x < C * C / 2) {
+        const int t = threadIdx.x >> 3, s = (threadIdx.x & 7) * 2;
+        uint32_t hi, lo;
+        split_bf16(s <= t ? B[t][s] : 0.0f, s + 1 <= t ? B[t][s + 1] : 0.0f, hi, lo);
+        *reinterpret_cast<uint32_t*>(image + I::kBh + (t * I::SB + s) * 2) = hi;
+        *reinterpret_cast<uint32_t*>(image + I::kBl + (t * I::SB + s) * 2) = lo;
+    }
+    // forward substitution, a column of W or U0 per thread and turn
+    for (int i = threadIdx.x; i < DP + vp; i += kThreads) {
+        const bool is_w = i < DP;  // uniform over a warp
+        const int e = i - DP;
+        float w[C];
 #pragma unroll
-            for (int t = 0; t < C; t += 2)
-                put(t, d, q[t * DP + d] * qi[t] * G[t * DP + d], q[(t + 1) * DP + d] * qi[t + 1] * G[(t + 1) * DP + d], I::kQh, I::kQl);
-            reinterpret_cast<float*>(image + I::kE)[d] = G[(C - 1) * DP + d];
+        for (int t = 0; t < C; ++t) {
+            float x = is_w ? k[t * SQ + i] * ki[t] * G[t * SQ + i] : v[t * vp + e];
+#pragma unroll
+            for (int s4 = 0; s4 < t; s4 += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(&A[t][s4]);
+                x = fmaf(-f.x, w[s4], x);
+                if (s4 + 1 < t) x = fmaf(-f.y, w[s4 + 1], x);
+                if (s4 + 2 < t) x = fmaf(-f.z, w[s4 + 2], x);
+                if (s4 + 3 < t) x = fmaf(-f.w, w[s4 + 3], x);
+            }
+            w[t] = beta[t] * x;
+        }
+        if (is_w) {
+#pragma unroll
+            for (int t = 0; t < C; t += 2) put(t, i, w[t], w[t + 1], I::kWh, I::kWl);
         } else {
-            const int d = i - cols32 - DP;
-            float rest = 1.0f;  // product of the decays behind the token
+            float* u = reinterpret_cast<float*>(image + I::kU) + (e >> 6) * C * I::SU + (e & 63);
 #pragma unroll
-            for (int t = C - 2; t >= 0; t -= 2) {
-                const float y1 = k[(t + 1) * DP + d] * ki[t + 1] * rest;
-                rest *= g[(t + 1) * DP + d];
-                const float y0 = k[t * DP + d] * ki[t] * rest;
-                rest *= g[t * DP + d];
-                put(t, d, y0, y1, I::kKh, I::kKl);
-            }
+            for (int t = 0; t < C; ++t) u[t * I::SU] = w[t];
         }
     }
 }
 
 // CTA = (NW * 16 value columns of a head, head, portion); warp NW copies.
-template <int DP, int NW>
+constexpr int NW = 4;  // a warp per scheduler: the chain is bound by its MMAs
+
+template <int DP>
 struct Chain {
-    static constexpr int kHead = Image<DP>::kU, kU = NW * 16 * Image<DP>::SU * 4;
+    static constexpr int kHead = Image<DP>::kU, kU = C * Image<DP>::SU * 4;
     static constexpr int kStage = (kHead + kU + 127) & ~127;
     static constexpr int NS = DP == 64 ? 4 : 3;
     static constexpr int kBytes = NS * kStage + 128 + 2 * NS * 8;
 };
 
-template <int DP, int NW>
+template <int DP>
 __global__ void __launch_bounds__(32 * NW + 32, 2)
-delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp, float* __restrict__ outputs) {
+delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, float* __restrict__ outputs) {
     using I = Image<DP>;
-    using K = Chain<DP, NW>;
+    using K = Chain<DP>;
     constexpr int NS = K::NS;
     extern __shared__ uint8_t raw[];
     uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 127) & ~uintptr_t(127));
@@ -317,7 +359,7 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     const int4 sq = reinterpret_cast<const int4*>(a.seqs)[blockIdx.z];      // first chunk, chunks, row, tokens before
     if (po.z < 0 || po.z >= a.state_rows) return;                            // flagged by the chunks
     const int v0 = blockIdx.x * NW * 16;
-    const int columns = min(NW * 16, vp - v0);
+    const int columns = min(NW * 16, a.vdim - v0);
     if (threadIdx.x == 0) {
         for (int i = 0; i < NS; ++i) {
             mbar_init(smem_u32(full + i), 1);
@@ -335,10 +377,9 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
                 if (c >= NS && !mbar_wait(smem_u32(empty + st), ((c / NS) - 1) & 1, abort)) break;
                 const uint8_t* src = static_cast<const uint8_t*>(a.workspace) + (static_cast<int64_t>(sq.x + c) * a.heads + h) * image_bytes;
                 const uint32_t bar = smem_u32(full + st), dst = smem_u32(base + st * K::kStage);
-                const uint32_t ub = static_cast<uint32_t>(columns) * I::SU * 4;
-                mbar_expect(bar, K::kHead + ub);
+                mbar_expect(bar, K::kHead + K::kU);
                 bulk_load(dst, src, K::kHead, bar);
-                bulk_load(dst + K::kHead, src + I::kU + v0 * I::SU * 4, ub, bar);
+                bulk_load(dst + K::kHead, src + I::kU + blockIdx.x * K::kU, K::kU, bar);
                 issued = c + 1;
             }
             if (*abort != 0) {  // copies in flight land before the CTA's shared memory is given up
@@ -393,15 +434,11 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
                     mma16816(oc[0], sl, bh[0], bh[1]);
                     mma16816(oc[1], sl, bh[2], bh[3]);
                 }
-                const float* U = reinterpret_cast<const float*>(im + K::kHead) + (warp * 16 + gid) * I::SU + tig * 2;
+                const float* U = reinterpret_cast<const float*>(im + K::kHead) + tig * 2 * I::SU + warp * 16 + gid;
 #pragma unroll
                 for (int n = 0; n < 2; ++n)
 #pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        const float2 f = *reinterpret_cast<const float2*>(U + i * 8 * I::SU + n * 8);
-                        u[n][2 * i] = f.x - (u[n][2 * i] + uc[n][2 * i]);
-                        u[n][2 * i + 1] = f.y - (u[n][2 * i + 1] + uc[n][2 * i + 1]);
-                    }
+                    for (int i = 0; i < 4; ++i) u[n][i] = U[(n * 8 + (i & 1)) * I::SU + (i >> 1) * 8] - (u[n][i] + uc[n][i]);
                 uint32_t uh[4], ul[4];
                 split_bf16(u[0][0], u[0][1], uh[0], ul[0]);
                 split_bf16(u[0][2], u[0][3], uh[1], ul[1]);
@@ -475,18 +512,18 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     __syncthreads();
 }
 
-int padded_v(int vdim) { return (vdim + 15) & ~15; }
+int padded_v(int vdim) { return (vdim + 63) & ~63; }
 int64_t image_size(int dim, int vdim) {
-    const int64_t u = static_cast<int64_t>(padded_v(vdim)) * Image<64>::SU * 4;
+    const int64_t u = static_cast<int64_t>(padded_v(vdim) / 64) * C * Image<64>::SU * 4;
     return (dim <= 64 ? Image<64>::kU : Image<128>::kU) + u;
 }
 
-template <int DP, int NW>
+template <int DP>
 int launch_chain(const spk_delta_args& a, int64_t image, int vp, float* outputs, cudaStream_t s) {
-    constexpr int bytes = Chain<DP, NW>::kBytes;
-    const cudaError_t e = cudaFuncSetAttribute(delta_chain_kernel<DP, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    constexpr int bytes = Chain<DP>::kBytes;
+    const cudaError_t e = cudaFuncSetAttribute(delta_chain_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) return spk_set_cuda_error(e);
-    delta_chain_kernel<DP, NW><<<dim3((vp + NW * 16 - 1) / (NW * 16), a.heads, a.n_portions), 32 * NW + 32, bytes, s>>>(a, image, vp, outputs);
+    delta_chain_kernel<DP><<<dim3((vp + NW * 16 - 1) / (NW * 16), a.heads, a.n_portions), 32 * NW + 32, bytes, s>>>(a, image, outputs);
     SPK_CHECK_LAUNCH();
     return SPK_OK;
 }
@@ -495,13 +532,13 @@ template <int DP>
 int launch(const spk_delta_args& a, float* outputs, cudaStream_t s) {
     const int vp = padded_v(a.vdim);
     const int64_t image = image_size(a.dim, a.vdim);
-    const size_t bytes = sizeof(float) * C * (4 * DP + static_cast<size_t>(vp));
+    const size_t bytes = sizeof(float) * C * (4 * (DP + 8) + static_cast<size_t>(vp));
     auto* fn = a.taps == 4 ? delta_chunk_kernel<DP, 4> : delta_chunk_kernel<DP, 0>;
     const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
     if (e != cudaSuccess) return spk_set_cuda_error(e);
     fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, image, vp);
     SPK_CHECK_LAUNCH();
-    return launch_chain<DP, 4>(a, image, vp, outputs, s);  // a warp per scheduler: the chain is bound by its MMAs
+    return launch_chain<DP>(a, image, vp, outputs, s);
 }
 
 }  // namespace

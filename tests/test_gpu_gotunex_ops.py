@@ -493,10 +493,11 @@ def test_delta_prefill_portions_and_decode(dev, status, heads, kv_heads, dim, vd
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("decay", [(20.0, 60.0), (-30.0, -20.0), (-8.0, 12.0)])
+@pytest.mark.parametrize("decay", [(20.0, 60.0), (-30.0, -20.0), (-8.0, 12.0), (1.0, 3.0), (3.0, 5.0)])
 @pytest.mark.parametrize("dim,vdim", [(64, 64), (128, 128), (40, 24)])
 def test_delta_with_extreme_decays(dev, status, decay, dim, vdim, dtype):
-    """Decays that wipe the state in one step, that keep it for good, and both side by side."""
+    """Decays that wipe the state in one step, that keep it for good, both side by side, and strong ones a chunk just can or cannot
+    divide by."""
     n = 150
     case = DeltaCase(dev, dtype, n, 2, 1, dim, vdim, 4, 11, decay=decay)
     want, state = case.want()
