@@ -306,7 +306,7 @@ constexpr int kScanCols = 32;
 template <typename T, int NR>
 __global__ void __launch_bounds__(4 * kScanCols)
 delta_scan_kernel(const spk_delta_args a) {
-    constexpr int D = 16 * NR, kScanTokens = NR > 8 ? 4 : 8;  // tokens staged at a time
+    constexpr int D = 16 * NR, kScanTokens = NR > 16 ? 2 : NR > 8 ? 4 : 8;  // tokens staged at a time
     __shared__ __align__(16) float gs[2][kScanTokens][D], ks[2][kScanTokens][D], gk[2][kScanTokens][D], gq[2][kScanTokens][D];
     __shared__ float qk[2][kScanTokens], bs[2][kScanTokens], vs[2][kScanTokens][kScanCols];
     const int4 po = reinterpret_cast<const int4*>(a.portions)[blockIdx.z];
@@ -512,7 +512,7 @@ int launch_out(const spk_delta_args& a, const float* outputs, cudaStream_t s) {
 
 template <typename T>
 int launch_prefill(const spk_delta_args& a, cudaStream_t s) {
-    if (a.dim > 256) return SPK_ERR_UNSUPPORTED;
+    if (a.dim > 512) return SPK_ERR_UNSUPPORTED;
     delta_prepare_kernel<T><<<a.n_chunks, kThreads, 0, s>>>(a);
     SPK_CHECK_LAUNCH();
     const dim3 grid((a.vdim + kScanCols - 1) / kScanCols, a.heads, a.n_portions);
@@ -520,7 +520,8 @@ int launch_prefill(const spk_delta_args& a, cudaStream_t s) {
     if (a.dim <= 32) delta_scan_kernel<T, 2><<<grid, threads, 0, s>>>(a);
     else if (a.dim <= 64) delta_scan_kernel<T, 4><<<grid, threads, 0, s>>>(a);
     else if (a.dim <= 128) delta_scan_kernel<T, 8><<<grid, threads, 0, s>>>(a);
-    else delta_scan_kernel<T, 16><<<grid, threads, 0, s>>>(a);
+    else if (a.dim <= 256) delta_scan_kernel<T, 16><<<grid, threads, 0, s>>>(a);
+    else delta_scan_kernel<T, 32><<<grid, threads, 0, s>>>(a);
     SPK_CHECK_LAUNCH();
     return launch_out<T>(a, carve(a).o, s);
 }

@@ -74,15 +74,70 @@ __device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4
             float y = 0.0f;
 #pragma unroll
             for (int i = 0; i < TAPS; ++i) y = fmaf(win[i], f[i], y);
-            dst[t * stride] = t < len ? y * rcp(1.0f + ex2(-1.4426950408889634f * y)) : 0.0f;
+            dst[t * stride] = t < len ? y * sigmoid_fast(y) : 0.0f;
         }
     } else {
         for (int t = 0; t < C; ++t) {
             float y = 0.0f;
             if (t < len)
                 for (int i = 0; i < taps; ++i) y = fmaf(raw(t - (taps - 1 - i)), w[c * taps + i], y);
-            dst[t * stride] = t < len ? y * rcp(1.0f + ex2(-1.4426950408889634f * y)) : 0.0f;
+            dst[t * stride] = t < len ? y * sigmoid_fast(y) : 0.0f;
         }
+    }
+}
+
+// The same for channels c and c + 1 over half a chunk (eight tokens from `first`), two channels per access; every pair of channels aligned.
+template <int TAPS>
+__device__ __forceinline__ void conv_pair(const spk_delta_args& a, const int4& po, int64_t t0, int len, int first, const void* src, int64_t c, const float* ring,
+                                          int channels, int at, const float* w, float* dst, int stride) {
+    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(src) + (t0 + first) * a.ld + c;
+    const int before = static_cast<int>(t0 - po.x) + first;  // tokens of the portion ahead of the half
+    uint32_t x[C / 2];
+    float f0[TAPS], f1[TAPS], w0[TAPS], w1[TAPS];
+#pragma unroll
+    for (int t = 0; t < C / 2; ++t) x[t] = first + t < len ? *reinterpret_cast<const uint32_t*>(p + t * a.ld) : 0u;
+    if (TAPS == 4) {  // two channels' filters are two 16-byte loads
+        const float4 u0 = *reinterpret_cast<const float4*>(w + c * 4), u1 = *reinterpret_cast<const float4*>(w + c * 4 + 4);
+        f0[0] = u0.x; f0[1 % TAPS] = u0.y; f0[2 % TAPS] = u0.z; f0[3 % TAPS] = u0.w;
+        f1[0] = u1.x; f1[1 % TAPS] = u1.y; f1[2 % TAPS] = u1.z; f1[3 % TAPS] = u1.w;
+    } else {
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) {
+            f0[i] = w[c * TAPS + i];
+            f1[i] = w[(c + 1) * TAPS + i];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) {
+        const int j = i - (TAPS - 1), pos = po.w + before + j;
+        float y0 = 0.0f, y1 = 0.0f;
+        if (before + j >= 0) {
+            const uint32_t u = *reinterpret_cast<const uint32_t*>(p + j * a.ld);
+            y0 = __uint_as_float(u << 16);
+            y1 = __uint_as_float(u & 0xffff0000u);
+        } else if (pos >= 0) {
+            y0 = ring[(pos % TAPS) * channels + at];
+            y1 = ring[(pos % TAPS) * channels + at + 1];
+        }
+        w0[i + 1] = y0;
+        w1[i + 1] = y1;
+    }
+#pragma unroll
+    for (int t = 0; t < C / 2; ++t) {
+        float y0 = 0.0f, y1 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i) {
+            w0[i] = w0[i + 1];
+            w1[i] = w1[i + 1];
+            y0 = fmaf(w0[i], f0[i], y0);
+            y1 = fmaf(w1[i], f1[i], y1);
+        }
+        w0[TAPS - 1] = __uint_as_float(x[t] << 16);
+        w1[TAPS - 1] = __uint_as_float(x[t] & 0xffff0000u);
+        y0 = fmaf(w0[TAPS - 1], f0[TAPS - 1], y0);
+        y1 = fmaf(w1[TAPS - 1], f1[TAPS - 1], y1);
+        const bool in = first + t < len;
+        *reinterpret_cast<float2*>(dst + (first + t) * stride) = make_float2(in ? y0 * sigmoid_fast(y0) : 0.0f, in ? y1 * sigmoid_fast(y1) : 0.0f);
     }
 }
 
@@ -145,7 +200,7 @@ __device__ __noinline__ void pair_products(const float* q, const float* k, const
 // CTA = (chunk, head).
 template <int DP, int TAPS>
 __global__ void __launch_bounds__(kThreads, 4)
-delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp) {
+delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int vp, const bool pairs) {
     using I = Image<DP>;
     constexpr int SQ = DP + 8;   // row stride: MMA fragments read without bank conflicts
     constexpr float kSmallest = 1e-30f;
@@ -178,7 +233,23 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
     }
     const int my_d = threadIdx.x % DP;  // kThreads is a multiple of DP: one channel for all of a thread's values
     const float bias = my_d < dim ? a.dt_bias[static_cast<int64_t>(h) * dim + my_d] : 0.0f, rate = expf(a.a_log[h]);
-    for (int i = threadIdx.x; i < 2 * DP + vp; i += kThreads) {
+    const bool paired = TAPS > 0 && pairs;
+    if constexpr (TAPS > 0) {  // two channels and half the tokens per thread and turn
+        for (int i = paired ? threadIdx.x : 2 * DP + vp; i < 2 * DP + vp; i += kThreads) {
+            const int kind = i < DP ? 0 : i < 2 * DP ? 1 : 2;  // k, q, v: uniform over a warp
+            const int j = i - kind * DP, half = kind == 2 ? vp / 2 : DP / 2, c = 2 * (j % half), first = j / half * (C / 2);
+            const int width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : SQ, head = kind == 2 ? h : grp;
+            float* dst = (kind == 0 ? k : kind == 1 ? q : v) + c;
+            if (c < width) {
+                conv_pair<TAPS>(a, po, t0, len, first, kind == 0 ? a.k : kind == 1 ? a.q : a.v, static_cast<int64_t>(head) * width + c, ring, sh.channels,
+                                (kind == 0 ? sh.qk : kind == 1 ? 0 : 2 * sh.qk) + head * width + c, kind == 0 ? a.conv_k : kind == 1 ? a.conv_q : a.conv_v, dst, stride);
+            } else {
+#pragma unroll
+                for (int t = 0; t < C / 2; ++t) *reinterpret_cast<float2*>(dst + (first + t) * stride) = make_float2(0.0f, 0.0f);
+            }
+        }
+    }
+    for (int i = paired ? 2 * DP + vp : threadIdx.x; i < 2 * DP + vp; i += kThreads) {
         const int kind = i < DP ? 0 : i < 2 * DP ? 1 : 2;  // k, q, v: uniform over a warp
         const int c = i - kind * DP, width = kind == 2 ? vdim : dim, stride = kind == 2 ? vp : SQ;
         float* dst = (kind == 0 ? k : kind == 1 ? q : v) + c;
@@ -194,7 +265,7 @@ delta_chunk_kernel(const spk_delta_args a, const int64_t image_bytes, const int 
 #pragma unroll
     for (int j = 0; j < RAW; ++j) {
         const int t = (threadIdx.x + j * kThreads) / DP;
-        g[t * SQ + my_d] = my_d < dim && t < len ? expf(spk_log_decay(raw_a[j] + bias, rate)) : 1.0f;
+        g[t * SQ + my_d] = my_d < dim && t < len ? spk_decay_series(raw_a[j] + bias, rate) : 1.0f;
     }
     if (threadIdx.x < C)
         beta[threadIdx.x] = static_cast<int>(threadIdx.x) < len ? spk_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(a.b)[(t0 + threadIdx.x) * a.ld + h])) : 0.0f;
@@ -536,7 +607,10 @@ int launch(const spk_delta_args& a, float* outputs, cudaStream_t s) {
     auto* fn = a.taps == 4 ? delta_chunk_kernel<DP, 4> : delta_chunk_kernel<DP, 0>;
     const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
     if (e != cudaSuccess) return spk_set_cuda_error(e);
-    fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, image, vp);
+    auto even = [&](const void* p) { return reinterpret_cast<uintptr_t>(p) % 4 == 0; };
+    auto wide = [&](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool pairs = a.ld % 2 == 0 && a.dim % 2 == 0 && a.vdim % 2 == 0 && even(a.q) && even(a.k) && even(a.v) && wide(a.conv_q) && wide(a.conv_k) && wide(a.conv_v);
+    fn<<<dim3(a.n_chunks, a.heads), kThreads, bytes, s>>>(a, image, vp, pairs);
     SPK_CHECK_LAUNCH();
     return launch_chain<DP>(a, image, vp, outputs, s);
 }

@@ -63,23 +63,16 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
     const int width = part == 0 ? a.q_rank : a.rank;
     const T* src = part == 0 ? static_cast<const T*>(a.cq) + t * a.ld : static_cast<const T*>(a.kv) + t * a.ld;
     const float* w = part == 0 ? a.w_q : a.w_kv;
-    constexpr int KEEP = VEC ? 12 : 1;  // groups of four a lane keeps between the two passes
-    float4 keep[KEEP];
     float ss = 0.0f;
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        keep[i] = spk_load4<T, VEC>(src + c, width - c);
-    }
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i) ss += (keep[i].x * keep[i].x + keep[i].y * keep[i].y) + (keep[i].z * keep[i].z + keep[i].w * keep[i].w);
-    for (int c = 4 * (lane + 32 * KEEP); c < width; c += 128) {
+#pragma unroll 4
+    for (int c = 4 * lane; c < width; c += 128) {
         const float4 x = spk_load4<T, VEC>(src + c, width - c);
         ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
     }
     const float inv = 1.0f / sqrtf(spk_warp_sum(ss) / static_cast<float>(width) + a.eps);
-    auto put = [&](int c, const float4& x) {
-        const float4 m = spk_load4<float, VEC>(w + c, width - c);
+#pragma unroll 4
+    for (int c = 4 * lane; c < width; c += 128) {
+        const float4 x = spk_load4<T, VEC>(src + c, width - c), m = spk_load4<float, VEC>(w + c, width - c);
         const float4 y = make_float4(x.x * inv * m.x, x.y * inv * m.y, x.z * inv * m.z, x.w * inv * m.w);
         if (part == 0) {
             spk_store4<T, VEC>(static_cast<T*>(a.cq_out) + t * width + c, y, width - c);
@@ -91,11 +84,7 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
             for (int k = 0; k < 4; ++k)
                 if (c + k < width) page[spk_latent_channel(lay, r, c + k)] = spk_from_float<T>(e[k]);
         }
-    };
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i)
-        if (4 * (lane + 32 * i) < width) put(4 * (lane + 32 * i), keep[i]);
-    for (int c = 4 * (lane + 32 * KEEP); c < width; c += 128) put(c, spk_load4<T, VEC>(src + c, width - c));
+    }
 }
 
 // ---- queries ---------------------------------------------------------------------------------------------------------

@@ -467,7 +467,7 @@ class DeltaCase:
 
 
 DELTA_SIZES = [(4, 2, 24, 40, 4), (3, 1, 10, 7, 1), (2, 2, 13, 21, 6), (4, 2, 64, 64, 4), (2, 1, 128, 128, 4), (2, 1, 160, 144, 2), (3, 3, 32, 130, 3),
-               (2, 2, 100, 36, 4)]
+               (2, 2, 100, 36, 4), (1, 1, 300, 20, 3)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
