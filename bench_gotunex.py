@@ -95,9 +95,9 @@ def gotunex_kernels(shape: str, device, repeats: int, pk: dict, only=()) -> dict
     ones = torch.ones(max(width, Q, K, ff), device=device)
     out = {}
 
-    def add(name, make, nbytes, flops=0):
+    def add(name, make, nbytes, flops=0, at_least=0):
         if not only or any(name.startswith(o) for o in only):
-            out[name] = entry(timed_sets(make, nbytes, repeats), nbytes, flops, pk)
+            out[name] = entry(timed_sets(make, max(nbytes, at_least), repeats), nbytes, flops, pk)
 
     table = torch.rand(4096, E, device=device).topk(top).indices.to(torch.int32)
     part = lambda o, i: [rnd(o, i) * i ** -0.5 for _ in range(E)]
@@ -178,9 +178,7 @@ def gotunex_kernels(shape: str, device, repeats: int, pk: dict, only=()) -> dict
             q, g, o = rnd(rows, H, pool.pad), rnd(rows, H * V), rnd(rows, H * V)
             return lambda: latent.latent_attention(q, pool, tables, sink, w_uv, g, o, vdim=V, scale=0.02, seq_lens=lens)
         nbytes = rows * keys * (K + R) * 2 + rows * H * (K + R + 2 * V) * 2 + H * V * K * 2
-        if not only or any("latent_attention decode".startswith(x) or x.startswith("latent_attention decode") for x in only):
-            out[f"latent_attention decode {rows}x{keys}"] = entry(timed_sets(mk_dec, max(rows * keys * (K + R) * 2, 5 << 20), repeats), nbytes,
-                                                                  rows * keys * H * (4 * K + 2 * R), pk)
+        add(f"latent_attention decode {rows}x{keys}", mk_dec, nbytes, rows * keys * H * (4 * K + 2 * R), 5 << 20)
     for seqs, n in ((16, 512), (2, 4096)):
         nb = seqs * n // 16
         pool = PagedLatentPool(nb, 16, K, R, BF, device)

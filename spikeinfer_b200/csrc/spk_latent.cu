@@ -26,13 +26,16 @@ __device__ __forceinline__ float2 rot_factor(const float* table, int64_t positio
 }
 
 // ---- norms, rotation, page write -----------------------------------------------------------------------------------
-// One warp per (token, part): the query latent, the cached latent, the rotated key part.
-template <typename T, bool VEC>
+// WPI warps per (token, part): the query latent, the cached latent, the rotated key part.  One warp for many tokens, a CTA for few.
+template <typename T, bool VEC, int WPI>
 __global__ void __launch_bounds__(kThreads)
 latent_prepare_kernel(const spk_latent_prepare_args a) {
-    const int lane = threadIdx.x & 31;
+    constexpr int L = 32 * WPI;
+    static_assert(WPI == 1 || WPI == kWarps, "a warp or a CTA per item");
+    __shared__ float sums[32];
+    const int lane = threadIdx.x % L;
     const int parts = a.kv != nullptr ? 3 : 1;
-    const int64_t item = static_cast<int64_t>(blockIdx.x) * kWarps + (threadIdx.x >> 5);
+    const int64_t item = static_cast<int64_t>(blockIdx.x) * (kWarps / WPI) + threadIdx.x / L;
     const int64_t t = item / parts;
     if (t >= a.n) return;
     const int part = static_cast<int>(item % parts);
@@ -52,7 +55,7 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
         const T* src = static_cast<const T*>(a.kv) + t * a.ld + a.rank;
         const int half = a.rot_dim / 2;
         const int64_t pos = a.positions[t];
-        for (int i = lane; i < half; i += 32) {
+        for (int i = lane; i < half; i += L) {
             const float2 f = rot_factor(a.rot_table, a.rot_positions, half, pos, i, a.status);
             const float u = spk_to_float<T>(src[i]), v = spk_to_float<T>(src[i + half]);
             page[spk_latent_channel(lay, r, a.rank_pad + i)] = spk_from_float<T>(u * f.x - v * f.y);
@@ -63,15 +66,17 @@ latent_prepare_kernel(const spk_latent_prepare_args a) {
     const int width = part == 0 ? a.q_rank : a.rank;
     const T* src = part == 0 ? static_cast<const T*>(a.cq) + t * a.ld : static_cast<const T*>(a.kv) + t * a.ld;
     const float* w = part == 0 ? a.w_q : a.w_kv;
-    float ss = 0.0f;
+    float ss[1] = {0.0f};
 #pragma unroll 4
-    for (int c = 4 * lane; c < width; c += 128) {
+    for (int c = 4 * lane; c < width; c += 4 * L) {
         const float4 x = spk_load4<T, VEC>(src + c, width - c);
-        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+        ss[0] += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
     }
-    const float inv = 1.0f / sqrtf(spk_warp_sum(ss) / static_cast<float>(width) + a.eps);
+    if (WPI == 1) ss[0] = spk_warp_sum(ss[0]);
+    else spk_block_sum<1>(ss, sums);
+    const float inv = 1.0f / sqrtf(ss[0] / static_cast<float>(width) + a.eps);
 #pragma unroll 4
-    for (int c = 4 * lane; c < width; c += 128) {
+    for (int c = 4 * lane; c < width; c += 4 * L) {
         const float4 x = spk_load4<T, VEC>(src + c, width - c), m = spk_load4<float, VEC>(w + c, width - c);
         const float4 y = make_float4(x.x * inv * m.x, x.y * inv * m.y, x.z * inv * m.z, x.w * inv * m.w);
         if (part == 0) {
@@ -412,35 +417,40 @@ latent_out_mma_kernel(const spk_latent_out_args a, const bool vec_w) {
     };
     for (int c = 0; c < kOutStages - 1; ++c) fetch(c);
     spk_grid_wait();
-    range_weights(a, h, t0, rows, wts);
-    __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3, m = lane >> 3, mr = lane & 7;
     const int cw = (warp & 3) * 16, kw = (warp >> 2) * 64;
-    {
-        constexpr int U = 8, K = 64;
-        const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
-        const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank + c4;
-        const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
-        for (int g = 0; g < 2 * chunks; g += U) {
-            float4 y[U];
+    constexpr int U = 8, K = 64;
+    const int r = threadIdx.x >> 4, c4 = (threadIdx.x & 15) * 4;
+    const float* part = a.partials + ((t0 + r) * a.splits * a.heads + h) * a.rank + c4;
+    const int64_t step = static_cast<int64_t>(a.heads) * a.rank;
+    auto sums_of = [&](float4 (&x)[U], int s, int g) {  // a range's sums at 8 x 64 latent channels
 #pragma unroll
-            for (int u = 0; u < U; ++u) y[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < rows) {
-                for (int s = 0; s < a.splits; ++s) {
-                    const float f = wts[r * a.splits + s];
-                    if (f == 0.0f) continue;
+        for (int u = 0; u < U; ++u) x[u] = spk_load4<float, VEC>(part + s * step + (g + u) * K, r < rows ? a.rank - (g + u) * K - c4 : 0);
+    };
+    float4 head_sums[U];  // of the first range, on their way while the weights are made
+    sums_of(head_sums, 0, 0);
+    range_weights(a, h, t0, rows, wts);
+    __syncthreads();
+    for (int g = 0; g < 2 * chunks; g += U) {
+        float4 y[U];
 #pragma unroll
-                    for (int u = 0; u < U; ++u) {
-                        const float4 x = spk_load4<float, VEC>(part + s * step + (g + u) * K, a.rank - (g + u) * K - c4);
-                        y[u] = make_float4(fmaf(f, x.x, y[u].x), fmaf(f, x.y, y[u].y), fmaf(f, x.z, y[u].z), fmaf(f, x.w, y[u].w));
-                    }
+        for (int u = 0; u < U; ++u) y[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < rows) {
+            for (int s = 0; s < a.splits; ++s) {
+                const float f = wts[r * a.splits + s];
+                if (f == 0.0f) continue;  // a range without keys was never written
+                if (s > 0 || g > 0) sums_of(head_sums, s, g);
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    const float4 x = head_sums[u];
+                    y[u] = make_float4(fmaf(f, x.x, y[u].x), fmaf(f, x.y, y[u].y), fmaf(f, x.z, y[u].z), fmaf(f, x.w, y[u].w));
                 }
             }
-#pragma unroll
-            for (int u = 0; u < U; ++u)
-                if (g + u < 2 * chunks)
-                    *reinterpret_cast<uint2*>(os + r * SO + (g + u) * K + c4) = make_uint2(pack_bf16(y[u].x, y[u].y), pack_bf16(y[u].z, y[u].w));
         }
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+            if (g + u < 2 * chunks)
+                *reinterpret_cast<uint2*>(os + r * SO + (g + u) * K + c4) = make_uint2(pack_bf16(y[u].x, y[u].y), pack_bf16(y[u].z, y[u].w));
     }
     float acc[2][4] = {};
     for (int c = 0; c < chunks; ++c) {
@@ -492,17 +502,24 @@ int with_smem(const void* fn, size_t bytes) {
     return SPK_OK;
 }
 
+template <typename T, bool VEC>
+int launch_prepare_form(const spk_latent_prepare_args& a, cudaStream_t s) {
+    const int64_t items = a.n * (a.kv != nullptr ? 3 : 1);
+    const bool few = items <= 4 * 148;
+    const int64_t grid = few ? items : (items + kWarps - 1) / kWarps;
+    if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
+    if (few) latent_prepare_kernel<T, VEC, kWarps><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a);
+    else latent_prepare_kernel<T, VEC, 1><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a);
+    SPK_CHECK_LAUNCH();
+    return SPK_OK;
+}
+
 template <typename T>
 int launch_prepare(const spk_latent_prepare_args& a, cudaStream_t s) {
-    const int64_t items = a.n * (a.kv != nullptr ? 3 : 1), grid = (items + kWarps - 1) / kWarps;
-    if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
     auto at = [](const void* p, size_t b) { return reinterpret_cast<uintptr_t>(p) % b == 0; };
     const bool vec = a.ld % 4 == 0 && a.q_rank % 4 == 0 && a.rank % 4 == 0 && (a.rank_pad + a.rot_pad) % 4 == 0 && at(a.cq, 4 * sizeof(T)) &&
                      at(a.kv, 4 * sizeof(T)) && at(a.cq_out, 4 * sizeof(T)) && at(a.pool, 16) && at(a.w_q, 16) && at(a.w_kv, 16);
-    if (vec) latent_prepare_kernel<T, true><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a);
-    else latent_prepare_kernel<T, false><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return vec ? launch_prepare_form<T, true>(a, s) : launch_prepare_form<T, false>(a, s);
 }
 
 template <typename T>
