@@ -23,7 +23,7 @@ constexpr int kPTile = kKeys * 128;        // a step's weights: 64 keys x (32 hi
 constexpr int kHeads = 32;                 // heads of a CTA
 constexpr int kQTile = kHeads * 128;
 constexpr int kSoftThreads = 128;
-constexpr int kThreads = kSoftThreads + 96;
+constexpr int kThreads = kSoftThreads + 128;  // warp 7 only helps to write the sums
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kSlack = 8.0f;             // a score may exceed the reference by 2^8
 
@@ -101,6 +101,16 @@ latent_decode_kernel(const spk_latent_attn_args a) {
         bars->abort = 0;
     }
     if (warp == 0) tmem_alloc(smem_u32(&bars->tmem), Sh::kColumns);
+    // a step's pages, one block-table entry per lane of the copying warp, the first on its way during the set-up
+    const int gran = a.block_size < kKeys ? a.block_size : kKeys;  // rows per copy
+    const int pages = kKeys / gran;                                // per step, at most 4
+    const int bs_log2 = 31 - __clz(a.block_size);
+    const int32_t* table = a.tables + row * a.table_stride;
+    auto entry = [&](int s) {
+        const int j = lo + s * kKeys + lane * gran;
+        return lane < pages && s < tiles && j < hi ? table[j >> bs_log2] : 0;
+    };
+    int next = warp == 4 ? entry(0) : 0;
     fence_async_shared();
     tc_fence_before();
     __syncthreads();
@@ -112,17 +122,9 @@ latent_decode_kernel(const spk_latent_attn_args a) {
     spk_grid_release();
 
     if (warp == 4) {  // ---- cache rows
-        const int gran = a.block_size < kKeys ? a.block_size : kKeys;  // rows per copy
-        const int pages = kKeys / gran;                                // per step, at most 4
-        const int bs_log2 = 31 - __clz(a.block_size);
-        const int32_t* table = a.tables + row * a.table_stride;
         const SpkPageLayout lay = spk_latent_layout(a.block_size, a.rank_pad, a.rot_pad, 1);
         const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a.pool);
-        auto entry = [&](int s) {
-            const int j = lo + s * kKeys + lane * gran;
-            return lane < pages && s < tiles && j < hi ? table[j >> bs_log2] : 0;
-        };
-        int next = entry(0), issued = 0;
+        int issued = 0;
         for (int s = 0; s < tiles; ++s) {
             const int mine = next;
             next = entry(s + 1);
@@ -193,7 +195,7 @@ latent_decode_kernel(const spk_latent_attn_args a) {
         }
         if (who) mma_commit(smem_u32(&bars->o_full));
         mbar_wait(smem_u32(&bars->o_full), 0);
-    } else {  // ---- scores to weights
+    } else if (warp < 4) {  // ---- scores to weights
         // query rows into the operand layout, zeros beyond the heads
         const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + (t * a.heads + h0) * (CT * 64);
 #pragma unroll 6
@@ -310,9 +312,6 @@ latent_decode_kernel(const spk_latent_attn_args a) {
             tc_fence_before();
             mbar_arrive(smem_u32(&bars->p_full[buf]));
         }
-        const bool ok = __all_sync(~0u, mbar_wait(smem_u32(&bars->o_full), 0, abort) && *abort == 0);
-        tc_fence_after();
-        const int64_t rec = (t * a.splits + blockIdx.z) * a.heads + h0;
         // denominators: over this warp's keys, then over the warps
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -328,11 +327,19 @@ latent_decode_kernel(const spk_latent_attn_args a) {
         soft_barrier();
         if (warp == 0 && lane < nh) {
             const float total = (bars->top[0][0][lane] + bars->top[0][1][lane]) + (bars->top[0][2][lane] + bars->top[0][3][lane]);
-            *reinterpret_cast<float2*>(a.stats + 2 * (rec + lane)) = make_float2(ref_own / kLog2e, ok ? total : 0.0f);
+            *reinterpret_cast<float2*>(a.stats + 2 * ((t * a.splits + blockIdx.z) * a.heads + h0 + lane)) = make_float2(ref_own / kLog2e, total);
         }
+    }
+    __syncwarp();
+    __syncthreads();  // every part has ended; the last one waited for the sums
+    {  // ---- all warps write the sums: a warp reaches the lanes of its quarter, the two halves of the CTA take turns at the blocks
+        const bool ok = *abort == 0;
+        tc_fence_after();
+        const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
+        const int64_t rec = (t * a.splits + blockIdx.z) * a.heads + h0;
 #pragma unroll 1
-        for (int b = 0; b < MB; ++b) {
-            const int c = b * 128 + warp * 32 + lane;
+        for (int b = warp >> 2; b < MB; b += 2) {
+            const int c = b * 128 + (warp & 3) * 32 + lane;
             uint32_t x[32], y[32];
             tmem_ld32(tmem + lanes + kTmemO + b * 2 * kHeads, x);
             tmem_ld32(tmem + lanes + kTmemO + b * 2 * kHeads + kHeads, y);
