@@ -441,6 +441,7 @@ delta_out_vec_kernel(const spk_delta_args a, const float* __restrict__ outputs) 
     const int c = 4 * (threadIdx.x % L);
     const int64_t t = item / a.heads;
     const int64_t at = (item % a.heads) * V + c;
+    spk_grid_wait();  // launched to overlap the end of the recurrence
     const float4 o = in ? __ldcs(reinterpret_cast<const float4*>(outputs + item * V + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
     const float4 g = spk_load4<T, true>(static_cast<const T*>(a.gate) + (in ? t * a.ld2 + at : 0), 4);
     const float4 w = *reinterpret_cast<const float4*>(a.w_norm + c);
@@ -498,10 +499,8 @@ int launch_out(const spk_delta_args& a, const float* outputs, cudaStream_t s) {
         const int per = kThreads / (a.vdim / 4);
         const int64_t grid = (a.n * a.heads + per - 1) / per;
         if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;
-        if (a.vdim == 64) delta_out_vec_kernel<T, 64><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);
-        else delta_out_vec_kernel<T, 128><<<static_cast<unsigned>(grid), kThreads, 0, s>>>(a, outputs);
-        SPK_CHECK_LAUNCH();
-        return SPK_OK;
+        return spk_launch(a.vdim == 64 ? delta_out_vec_kernel<T, 64> : delta_out_vec_kernel<T, 128>, dim3(static_cast<unsigned>(grid)), kThreads, 0, s, true, a,
+                          outputs);
     }
     const int64_t grid = (a.n * a.heads + kThreads / 32 - 1) / (kThreads / 32);
     if (grid > 0x7fffffffLL) return SPK_ERR_TOO_LARGE;

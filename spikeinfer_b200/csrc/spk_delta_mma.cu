@@ -428,7 +428,10 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, float* __r
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int4 po = reinterpret_cast<const int4*>(a.portions)[blockIdx.z];  // first token, tokens, row, tokens before
     const int4 sq = reinterpret_cast<const int4*>(a.seqs)[blockIdx.z];      // first chunk, chunks, row, tokens before
-    if (po.z < 0 || po.z >= a.state_rows) return;                            // flagged by the chunks
+    if (po.z < 0 || po.z >= a.state_rows) {  // flagged by the chunks
+        spk_grid_wait();
+        return;
+    }
     const int v0 = blockIdx.x * NW * 16;
     const int columns = min(NW * 16, a.vdim - v0);
     if (threadIdx.x == 0) {
@@ -441,6 +444,7 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, float* __r
     fence_async_shared();
     __syncthreads();
     if (warp == NW) {
+        spk_grid_wait();  // placed ahead of the chunks' end: their operands are complete from here on
         if (lane == 0) {
             int issued = 0;
             for (int c = 0; c < sq.y; ++c) {
@@ -472,6 +476,7 @@ delta_chain_kernel(const spk_delta_args a, const int64_t image_bytes, float* __r
                 const int d = n * 8 + tig * 2 + (i & 1), e = v1 + (i >> 1) * 8;
                 S[n][i] = live && po.w > 0 && d < dim && e < vdim ? state[static_cast<int64_t>(d) * vdim + e] : 0.0f;
             }
+        spk_grid_wait();  // and the convolutions' past has been read
         for (int c = 0; c < sq.y; ++c) {
             const int st = c % NS;
             if (!__all_sync(~0u, mbar_wait(smem_u32(full + st), (c / NS) & 1, abort))) break;
@@ -594,9 +599,7 @@ int launch_chain(const spk_delta_args& a, int64_t image, int vp, float* outputs,
     constexpr int bytes = Chain<DP>::kBytes;
     const cudaError_t e = cudaFuncSetAttribute(delta_chain_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) return spk_set_cuda_error(e);
-    delta_chain_kernel<DP><<<dim3((vp + NW * 16 - 1) / (NW * 16), a.heads, a.n_portions), 32 * NW + 32, bytes, s>>>(a, image, outputs);
-    SPK_CHECK_LAUNCH();
-    return SPK_OK;
+    return spk_launch(delta_chain_kernel<DP>, dim3((vp + NW * 16 - 1) / (NW * 16), a.heads, a.n_portions), 32 * NW + 32, bytes, s, true, a, image, outputs);
 }
 
 template <int DP>
