@@ -90,6 +90,11 @@ __device__ __forceinline__ void conv_channel(const spk_delta_args& a, const int4
 template <int TAPS>
 __device__ __forceinline__ void conv_pair(const spk_delta_args& a, const int4& po, int64_t t0, int len, int first, const void* src, int64_t c, const float* ring,
                                           int channels, int at, const float* w, float* dst, int stride) {
+    if (first >= len) {  // no token of this half, and none between it and the last one to look back at
+#pragma unroll
+        for (int t = 0; t < C / 2; ++t) *reinterpret_cast<float2*>(dst + (first + t) * stride) = make_float2(0.0f, 0.0f);
+        return;
+    }
     const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(src) + (t0 + first) * a.ld + c;
     const int before = static_cast<int>(t0 - po.x) + first;  // tokens of the portion ahead of the half
     uint32_t x[C / 2];
