@@ -241,6 +241,19 @@ def test_snapshot_restores_the_recurrent_state(dev):
     assert torch.equal(eng.decode_steps(6), first)
 
 
+def test_feed_forward_beside_the_mixer_changes_nothing(dev):
+    tokens = prompt("mixed", 60, 9)
+    out = []
+    for side in (0, 1 << 20):
+        eng = engine("mixed", torch.bfloat16, dev)
+        eng.model.side_tokens = side
+        row = eng.open_request()
+        logits = [run(eng, row, tokens[:41]), run(eng, row, tokens[41:43])]
+        logits += [run(eng, row, [t]).clone() for t in tokens[43:]]
+        out.append(torch.cat(logits))
+    assert torch.equal(*out)
+
+
 def test_a_shared_cache_is_stored_once(dev):
     eng = engine("mixed", torch.bfloat16, dev)
     layers = eng.cache.layers

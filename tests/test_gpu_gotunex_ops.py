@@ -120,7 +120,7 @@ def run_experts(dev, status, weights, ids, x, active=None):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("n,width,experts,top,ff", [(1, 45, 2, 2, 9), (5, 88, 7, 3, 40), (130, 72, 5, 1, 200), (300, 130, 3, 2, 136),
-                                                    (700, 64, 4, 2, 64), (33, 320, 64, 4, 257)])
+                                                    (700, 64, 4, 2, 64), (33, 320, 64, 4, 257), (250, 72, 4, 1, 96)])
 def test_experts(dev, status, n, width, experts, top, ff, dtype):
     w, weights, ids, x, cfg = expert_case(dev, dtype, n, width, experts, top, ff, n + ff)
     x = go.rms(x.double(), 0.0)
